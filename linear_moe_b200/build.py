@@ -22,6 +22,10 @@ OBJ = os.path.join(ROOT, "build")
 
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "--use_fast_math",
               "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden"]
+# sources whose fp32 instantiations serve models in true 32-bit: IEEE division and the accurate exp / tanh
+PRECISE = {"chunk_attn.cu", "parallel_block.cu"}
+# what serving a model of the listed kind needs (``build_serving``); everything else is training, communication and fp8
+SERVING = {"parallel_block": ("chunk_attn.cu", "chunk_attn_tc.cu", "parallel_block.cu", "gemm_dense.cu", "gemm_skinny.cu")}
 
 
 def _nvcc() -> str:
@@ -45,10 +49,15 @@ def _run(cmd):
     return r.stdout + r.stderr
 
 
-def build_cuda(verbose: bool = False, extra_flags=()) -> str:
+def _flags(src: str):
+    return [f for f in NVCC_FLAGS if not (f == "--use_fast_math" and os.path.basename(src) in PRECISE)]
+
+
+def build_cuda(verbose: bool = False, extra_flags=(), sources=None, name: str = "liblmoe.so") -> str:
+    """``lib/<name>`` from ``sources`` (file names in ``csrc``; default: all of them)."""
     os.makedirs(LIB, exist_ok=True)
     os.makedirs(OBJ, exist_ok=True)
-    srcs = sorted(glob.glob(os.path.join(CSRC, "*.cu")))
+    srcs = sorted(glob.glob(os.path.join(CSRC, "*.cu"))) if sources is None else [os.path.join(CSRC, s) for s in sources]
     hdrs = glob.glob(os.path.join(CSRC, "*.cuh")) + glob.glob(os.path.join(CSRC, "*.h"))
     nvcc = _nvcc()
     objs, jobs = [], []
@@ -56,15 +65,30 @@ def build_cuda(verbose: bool = False, extra_flags=()) -> str:
         o = os.path.join(OBJ, os.path.basename(s)[:-3] + ".o")
         objs.append(o)
         if _newer(o, [s] + hdrs):
-            jobs.append([nvcc, *NVCC_FLAGS, *extra_flags, "-I", CSRC, "-c", s, "-o", o])
+            jobs.append([nvcc, *_flags(s), *extra_flags, "-I", CSRC, "-c", s, "-o", o])
     with ThreadPoolExecutor(max_workers=min(8, max(len(jobs), 1))) as ex:
         for out in ex.map(_run, jobs):
             if verbose and out.strip():
                 print(out)
-    so = os.path.join(LIB, "liblmoe.so")
+    so = os.path.join(LIB, name)
     if jobs or _newer(so, objs):
         _run([nvcc, "-shared", "-o", so, *objs, "-lcudart"])
     return so
+
+
+def build_serving(kind: str) -> str:
+    """The kernel library for serving one kind of model (a key of ``SERVING``): the full ``liblmoe.so`` when it is there and
+    newer than its sources, else a library of the sources that kind needs, compiled on the first call.  Processes that start
+    together build once (a lock file), and a finished library replaces the old one in one step."""
+    import fcntl
+    full = os.path.join(LIB, "liblmoe.so")
+    srcs = glob.glob(os.path.join(CSRC, "*.cu")) + glob.glob(os.path.join(CSRC, "*.cuh")) + glob.glob(os.path.join(CSRC, "*.h"))
+    if not _newer(full, srcs):
+        return full
+    os.makedirs(LIB, exist_ok=True)
+    with open(os.path.join(LIB, ".build.lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return build_cuda(sources=SERVING[kind], name=f"liblmoe_{kind}.so")
 
 
 def build_host(verbose: bool = False, sanitize: bool = False, out_dir: str = None) -> str:

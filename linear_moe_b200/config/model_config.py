@@ -20,7 +20,7 @@ LA_MODULES = (
     "gated_deltanet", "gsa", "based", "rebased", "hgrn2", "rwkv6", "rwkv7",
     "mamba2", "lasp2", "mom_gla", "mom_gated_deltanet", "mom_linear_attention",
 )
-BASE_MODELS = ("qwen2", "llama3", "mixtral", "deepseek_v2")
+BASE_MODELS = ("qwen2", "llama3", "mixtral", "deepseek_v2", "lagisun")
 
 
 @dataclass
@@ -47,7 +47,7 @@ class ModelConfig:
     qk_layernorm: bool = False
     sliding_window: Optional[int] = None
     # ---- positional -----------------------------------------------------
-    position_embedding_type: str = "rope"         # rope | none
+    position_embedding_type: str = "rope"         # rope | none | learned (layer-list designs: table of max_position_embeddings rows)
     rotary_base: float = 10000.0
     rotary_percent: float = 1.0
     rotary_interleaved: bool = False
@@ -132,6 +132,10 @@ class ModelConfig:
     qk_nope_head_dim: int = 128
     qk_rope_head_dim: int = 64
     v_head_dim: int = 128
+    # ---- layer list (designs whose layers have sizes of their own; parallel mixer + feed-forward blocks) ----
+    # one entry per layer: {"attn": ops.chunk_attn.ChunkAttnSpec, "bias_rows": rows of the distance table, "ff": width or None}
+    layers: Optional[Tuple[dict, ...]] = None
+    residual_multiplier: float = 1.0              # factor of every block's output before it joins the residual stream
     # ---- precision / memory --------------------------------------------
     params_dtype: torch.dtype = torch.float32
     fp8: Optional[str] = None                     # None | "rowwise": e4m3 GEMMs, one current-amax scale per operand row (ops/fp8.py)
@@ -148,6 +152,10 @@ class ModelConfig:
             self.kv_channels = self.hidden_size // self.num_attention_heads
         if self.num_query_groups is None:
             self.num_query_groups = self.num_attention_heads
+        if (self.base_model == "lagisun") != (self.layers is not None):
+            raise ValueError("a lagisun model is described by its layer list (and no other family has one)")
+        if self.layers is not None:
+            self.num_layers = len(self.layers)
         if self.base_model not in BASE_MODELS:
             raise ValueError(f"unknown base model {self.base_model!r}")
         if self.la_module is not None and self.la_module not in LA_MODULES:

@@ -36,9 +36,18 @@ __device__ __forceinline__ void st_cluster_f32(float* p, uint32_t rank, float v)
 
 // NTILES 1: M <= 8, 2: M <= 16.  KS: CTAs of a cluster that split K between them (for matrices with few rows, so that
 // every SM streams a piece of W); their partial tiles meet in the shared memory of the cluster's first CTA.
-template <int NTILES, int KS>
+// OUT: bf16 result, fp32 result, or fp32 added to what y holds (the residual stream of a decode step).
+enum { OUT_BF16 = 0, OUT_F32 = 1, OUT_F32_ADD = 2 };
+template <int OUT>
+__device__ __forceinline__ void put(void* y, long long i, float v) {
+    if (OUT == OUT_BF16) reinterpret_cast<bf16*>(y)[i] = __float2bfloat16(v);
+    else if (OUT == OUT_F32) reinterpret_cast<float*>(y)[i] = v;
+    else reinterpret_cast<float*>(y)[i] += v;
+}
+
+template <int NTILES, int KS, int OUT>
 __global__ void __launch_bounds__(256) gemm_skinny_kernel(const bf16* __restrict__ x, long long ldx, const bf16* __restrict__ W,
-                                                          long long ldw, bf16* __restrict__ y, long long ldy, int M, int N, int K) {
+                                                          long long ldw, void* y, long long ldy, int M, int N, int K) {
     __shared__ float red[8][NTILES][32][4];
     __shared__ float cred[KS][NTILES][32][4];
     const int w = threadIdx.x >> 5, l = threadIdx.x & 31;
@@ -132,18 +141,18 @@ __global__ void __launch_bounds__(256) gemm_skinny_kernel(const bf16* __restrict
     if (w < NTILES) {
         const int n0 = 8 * w + 2 * q;                                   // batch rows n0, n0 + 1
         if (n0 < M) {
-            if (lo_ok) y[(long long)n0 * ldy + row_lo] = __float2bfloat16(s[0]);
-            if (hi_ok) y[(long long)n0 * ldy + row_hi] = __float2bfloat16(s[2]);
+            if (lo_ok) put<OUT>(y, (long long)n0 * ldy + row_lo, s[0]);
+            if (hi_ok) put<OUT>(y, (long long)n0 * ldy + row_hi, s[2]);
         }
         if (n0 + 1 < M) {
-            if (lo_ok) y[(long long)(n0 + 1) * ldy + row_lo] = __float2bfloat16(s[1]);
-            if (hi_ok) y[(long long)(n0 + 1) * ldy + row_hi] = __float2bfloat16(s[3]);
+            if (lo_ok) put<OUT>(y, (long long)(n0 + 1) * ldy + row_lo, s[1]);
+            if (hi_ok) put<OUT>(y, (long long)(n0 + 1) * ldy + row_hi, s[3]);
         }
     }
 }
 
-template <int NTILES, int KS>
-static int launch_skinny(const bf16* x, long long ldx, const bf16* W, long long ldw, bf16* y, long long ldy, int M, int N, int K,
+template <int NTILES, int KS, int OUT>
+static int launch_skinny(const bf16* x, long long ldx, const bf16* W, long long ldw, void* y, long long ldy, int M, int N, int K,
                          cudaStream_t st) {
     const int blocks = ((N + 15) / 16) * KS;
     cudaLaunchConfig_t cfg = {};
@@ -169,21 +178,12 @@ static int launch_skinny(const bf16* x, long long ldx, const bf16* W, long long 
     }
     cfg.attrs = attr;
     cfg.numAttrs = na;
-    return (int)cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<NTILES, KS>, x, ldx, W, ldw, y, ldy, M, N, K);
+    return (int)cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<NTILES, KS, OUT>, x, ldx, W, ldw, y, ldy, M, N, K);
 }
 
-}  // namespace sk
-}  // namespace lmoe
-
-// x [M, K] (row pitch ldx), W [N, K] (row pitch ldw), y [M, N] (row pitch ldy), all bf16; M <= 16, K a multiple of 32,
-// pitches multiples of 8 elements and bases 16-byte aligned.  Returns -1 for shapes it does not take.
-LMOE_API int lmoe_gemm_skinny(const void* x, long long ldx, const void* W, long long ldw, void* y, long long ldy, int M, int N,
-                              int K, cudaStream_t st) {
-    using namespace lmoe;
-    if (M <= 0 || M > 16 || N <= 0 || K <= 0 || K % 32 != 0 || ldx % 8 != 0 || ldw % 8 != 0) return -1;
-    if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(W)) & 15) return -1;
-    const bf16 *xb = (const bf16*)x, *Wb = (const bf16*)W;
-    bf16* yb = (bf16*)y;
+template <int OUT>
+static int dispatch(const bf16* x, long long ldx, const bf16* W, long long ldw, void* y, long long ldy, int M, int N, int K,
+                    cudaStream_t st) {
     // few row blocks: four CTAs of a cluster split K so that the whole GPU streams W
     static int sms = 0;
     if (sms == 0) {
@@ -191,8 +191,34 @@ LMOE_API int lmoe_gemm_skinny(const void* x, long long ldx, const void* W, long 
         if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess) sms = 148;
     }
     const bool split = (N + 15) / 16 < 2 * sms && K % 128 == 0;
-    if (M <= 8) return split ? sk::launch_skinny<1, 4>(xb, ldx, Wb, ldw, yb, ldy, M, N, K, st)
-                             : sk::launch_skinny<1, 1>(xb, ldx, Wb, ldw, yb, ldy, M, N, K, st);
-    return split ? sk::launch_skinny<2, 4>(xb, ldx, Wb, ldw, yb, ldy, M, N, K, st)
-                 : sk::launch_skinny<2, 1>(xb, ldx, Wb, ldw, yb, ldy, M, N, K, st);
+    if (M <= 8) return split ? launch_skinny<1, 4, OUT>(x, ldx, W, ldw, y, ldy, M, N, K, st)
+                             : launch_skinny<1, 1, OUT>(x, ldx, W, ldw, y, ldy, M, N, K, st);
+    return split ? launch_skinny<2, 4, OUT>(x, ldx, W, ldw, y, ldy, M, N, K, st)
+                 : launch_skinny<2, 1, OUT>(x, ldx, W, ldw, y, ldy, M, N, K, st);
+}
+
+}  // namespace sk
+}  // namespace lmoe
+
+static int skinny_shape_ok(const void* x, long long ldx, const void* W, long long ldw, int M, int N, int K) {
+    if (M <= 0 || M > 16 || N <= 0 || K <= 0 || K % 32 != 0 || ldx % 8 != 0 || ldw % 8 != 0) return 0;
+    return ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(W)) & 15) == 0;
+}
+
+// x [M, K] (row pitch ldx), W [N, K] (row pitch ldw), y [M, N] (row pitch ldy), all bf16; M <= 16, K a multiple of 32,
+// pitches multiples of 8 elements and bases 16-byte aligned.  Returns -1 for shapes it does not take.
+LMOE_API int lmoe_gemm_skinny(const void* x, long long ldx, const void* W, long long ldw, void* y, long long ldy, int M, int N,
+                              int K, cudaStream_t st) {
+    using namespace lmoe;
+    if (!skinny_shape_ok(x, ldx, W, ldw, M, N, K)) return -1;
+    return sk::dispatch<sk::OUT_BF16>((const bf16*)x, ldx, (const bf16*)W, ldw, y, ldy, M, N, K, st);
+}
+
+// The same product in fp32: y [M, N] floats, overwritten or (accumulate != 0) added to.
+LMOE_API int lmoe_gemm_skinny_f32(const void* x, long long ldx, const void* W, long long ldw, float* y, long long ldy, int M, int N,
+                                  int K, int accumulate, cudaStream_t st) {
+    using namespace lmoe;
+    if (!skinny_shape_ok(x, ldx, W, ldw, M, N, K)) return -1;
+    return accumulate ? sk::dispatch<sk::OUT_F32_ADD>((const bf16*)x, ldx, (const bf16*)W, ldw, y, ldy, M, N, K, st)
+                      : sk::dispatch<sk::OUT_F32>((const bf16*)x, ldx, (const bf16*)W, ldw, y, ldy, M, N, K, st);
 }

@@ -1,0 +1,171 @@
+// Row kernels of blocks whose mixer and feed-forward read the same fp32 residual stream and add into it together:
+//   stream_norm        y = x / rms(x) [* gain]: the fp32 stream -> the input of the block's fused projection (bf16 or fp32).  A
+//                      one-number norm gain is a scalar on the projection's outputs, so two norms of the same stream
+//                      need one pass and one matrix product; the consumers of the projection apply their gain.
+//   embed_norm         x = embedding[token] + position table[position], in fp32, together with the first block's norm
+//   poly_norm          sum over p = 1, 2, 3 of w_p u^p / rms(u^p), plus w_4 (element-wise powers, rms over the row)
+// Rows are padded (stream and activations to a multiple of 32 elements, pad = 0), so that every product is aligned for TMA.
+// Compiled without fast-math: the same code serves the fp32 model.
+#include "common.cuh"
+
+namespace lmoe {
+namespace pb {
+
+constexpr int THREADS = 256;
+
+// stores 4 values at y[c .. c + 3] (c a multiple of 4)
+__device__ __forceinline__ void store4(float* y, float4 v) { *reinterpret_cast<float4*>(y) = v; }
+__device__ __forceinline__ void store4(bf16* y, float4 v) {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    uint2 r;
+    r.x = *reinterpret_cast<uint32_t*>(&lo);
+    r.y = *reinterpret_cast<uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(y) = r;
+}
+
+// x [rows, ldx] fp32, y [rows, ldy]; columns width .. pad of x hold zeros, and y gets zeros there
+template <typename T>
+__global__ void __launch_bounds__(THREADS) stream_norm_kernel(const float* __restrict__ x, long long ldx, T* __restrict__ y,
+                                                              long long ldy, int width, int pad, float eps, const float* gain) {
+    pdl_trigger();
+    __shared__ float red[32];
+    const float* xr = x + (long long)blockIdx.x * ldx;
+    T* yr = y + (long long)blockIdx.x * ldy;
+    constexpr int NV = 4;                                   // float4s a thread keeps in registers (rows up to 4096 wide)
+    float4 v[NV];
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = (threadIdx.x + i * THREADS) * 4;
+        v[i] = c < pad ? *reinterpret_cast<const float4*>(xr + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        s += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    }
+    for (int c = (threadIdx.x + NV * THREADS) * 4; c < pad; c += THREADS * 4) {
+        const float4 t = *reinterpret_cast<const float4*>(xr + c);
+        s += t.x * t.x + t.y * t.y + t.z * t.z + t.w * t.w;
+    }
+    const float r = (gain == nullptr ? 1.f : *gain) / sqrtf(block_sum(s, red) / width + eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = (threadIdx.x + i * THREADS) * 4;
+        if (c < pad) store4(yr + c, make_float4(v[i].x * r, v[i].y * r, v[i].z * r, v[i].w * r));
+    }
+    for (int c = (threadIdx.x + NV * THREADS) * 4; c < pad; c += THREADS * 4) {
+        const float4 t = *reinterpret_cast<const float4*>(xr + c);
+        store4(yr + c, make_float4(t.x * r, t.y * r, t.z * r, t.w * r));
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(THREADS) embed_norm_kernel(const long long* __restrict__ ids, const int* __restrict__ pos,
+                                                             const T* __restrict__ emb, const T* __restrict__ ptab, float* __restrict__ x,
+                                                             long long ldx, T* __restrict__ y, long long ldy, int width, int pad,
+                                                             int vocab, int npos, float eps) {
+    pdl_trigger();
+    __shared__ float red[32];
+    // ids and positions are checked on the host; the clamp keeps a bad one from becoming a bad address
+    const long long id = min(max(ids[blockIdx.x], 0LL), (long long)vocab - 1);
+    const T* er = emb + id * width;
+    const T* pr = ptab == nullptr ? nullptr : ptab + (long long)min(max(pos[blockIdx.x], 0), npos - 1) * width;
+    float* xr = x + (long long)blockIdx.x * ldx;
+    T* yr = y + (long long)blockIdx.x * ldy;
+    float s = 0.f;
+    for (int c = threadIdx.x; c < pad; c += THREADS) {
+        float v = 0.f;
+        if (c < width) v = to_f(er[c]) + (pr == nullptr ? 0.f : to_f(pr[c]));
+        xr[c] = v;
+        s += v * v;
+    }
+    const float r = 1.f / sqrtf(block_sum(s, red) / width + eps);
+    for (int c = threadIdx.x; c < pad; c += THREADS) yr[c] = from_f<T>(xr[c] * r);
+}
+
+// z [rows, ldz] -> out [rows, ldo]; gain: the norm gain of the projection's input; act = {w_1, w_2, w_3, w_4}; out *= mul.
+// Columns ff .. ff_pad of out get zeros.
+template <typename T>
+__global__ void __launch_bounds__(THREADS) poly_norm_kernel(const T* __restrict__ z, long long ldz, T* __restrict__ out, long long ldo,
+                                                            int ff, int ff_pad, const float* __restrict__ gain,
+                                                            const float* __restrict__ act, float eps, float mul, int vec) {
+    pdl_trigger();
+    __shared__ float red[32];
+    const T* zr = z + (long long)blockIdx.x * ldz;
+    T* orow = out + (long long)blockIdx.x * ldo;
+    const float g = *gain;
+    constexpr int W = Vec<T>::N;
+    float s1 = 0.f, s2 = 0.f, s3 = 0.f;
+    auto add = [&](float u) {
+        u *= g;
+        const float u2 = u * u, u3 = u2 * u;
+        s1 += u2;
+        s2 += u2 * u2;
+        s3 += u3 * u3;
+    };
+    if (vec) {
+        for (int c = threadIdx.x * W; c < ff; c += THREADS * W) {
+            Vec<T> v;
+            v.load(zr + c);
+#pragma unroll
+            for (int i = 0; i < W; ++i) add(v.get(i));
+        }
+    } else {
+        for (int c = threadIdx.x; c < ff; c += THREADS) add(to_f(zr[c]));
+    }
+    const float inv = 1.f / ff;
+    const float r1 = act[0] / sqrtf(block_sum(s1, red) * inv + eps);
+    const float r2 = act[1] / sqrtf(block_sum(s2, red) * inv + eps);
+    const float r3 = act[2] / sqrtf(block_sum(s3, red) * inv + eps);
+    const float e = act[3];
+    auto f = [&](float u) {
+        u *= g;
+        return mul * (((r3 * u + r2) * u + r1) * u + e);
+    };
+    if (vec) {
+        for (int c = threadIdx.x * W; c < ff; c += THREADS * W) {
+            Vec<T> v, o;
+            v.load(zr + c);
+#pragma unroll
+            for (int i = 0; i < W; ++i) o.set(i, f(v.get(i)));
+            o.store(orow + c);
+        }
+    } else {
+        for (int c = threadIdx.x; c < ff; c += THREADS) orow[c] = from_f<T>(f(to_f(zr[c])));
+    }
+    for (int c = ff + threadIdx.x; c < ff_pad; c += THREADS) orow[c] = from_f<T>(0.f);
+}
+
+}  // namespace pb
+}  // namespace lmoe
+
+using namespace lmoe;
+
+// x [rows, ldx] fp32 with zeros in columns width .. pad; y bf16 (dt 1) or fp32 (dt 0); pad a multiple of 4, 16-byte rows; gain: one
+// float or null
+LMOE_API int lmoe_stream_norm(const float* x, long long ldx, void* y, long long ldy, int rows, int width, int pad, float eps,
+                              const float* gain, int dt, cudaStream_t st) {
+    if (rows <= 0 || width <= 0 || pad < width || pad % 4 || ldx % 4 || ldy % 4) return -1;
+    if (dt) pb::stream_norm_kernel<bf16><<<rows, pb::THREADS, 0, st>>>(x, ldx, (bf16*)y, ldy, width, pad, eps, gain);
+    else pb::stream_norm_kernel<float><<<rows, pb::THREADS, 0, st>>>(x, ldx, (float*)y, ldy, width, pad, eps, gain);
+    return (int)cudaGetLastError();
+}
+
+// emb [vocab, width], ptab [npos, width] or null, in the model's dtype; ids int64, pos int32
+LMOE_API int lmoe_embed_norm(const long long* ids, const int* pos, const void* emb, const void* ptab, float* x, long long ldx, void* y,
+                             long long ldy, int rows, int width, int pad, int vocab, int npos, float eps, int dt, cudaStream_t st) {
+    if (rows <= 0 || width <= 0 || pad < width || vocab <= 0 || (ptab != nullptr && npos <= 0)) return -1;
+    if (dt) pb::embed_norm_kernel<bf16><<<rows, pb::THREADS, 0, st>>>(ids, pos, (const bf16*)emb, (const bf16*)ptab, x, ldx, (bf16*)y,
+                                                                      ldy, width, pad, vocab, npos, eps);
+    else pb::embed_norm_kernel<float><<<rows, pb::THREADS, 0, st>>>(ids, pos, (const float*)emb, (const float*)ptab, x, ldx, (float*)y,
+                                                                    ldy, width, pad, vocab, npos, eps);
+    return (int)cudaGetLastError();
+}
+
+LMOE_API int lmoe_poly_norm(const void* z, long long ldz, void* out, long long ldo, int rows, int ff, int ff_pad, const float* gain,
+                            const float* act, float eps, float mul, int dt, cudaStream_t st) {
+    if (rows <= 0 || ff <= 0 || ff_pad < ff) return -1;
+    const int w = dt ? 8 : 4;
+    const int vec = ff % w == 0 && ldz % w == 0 && ldo % w == 0 &&
+                    ((reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+    if (dt) pb::poly_norm_kernel<bf16><<<rows, pb::THREADS, 0, st>>>((const bf16*)z, ldz, (bf16*)out, ldo, ff, ff_pad, gain, act, eps, mul, vec);
+    else pb::poly_norm_kernel<float><<<rows, pb::THREADS, 0, st>>>((const float*)z, ldz, (float*)out, ldo, ff, ff_pad, gain, act, eps, mul, vec);
+    return (int)cudaGetLastError();
+}

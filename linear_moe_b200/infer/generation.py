@@ -116,16 +116,23 @@ class GraphedDecodeStep:
     def supported(model, caches: List[dict], device) -> bool:
         if device.type != "cuda" or model.mesh.world_size != 1 or not caches:     # graph replay is a one-process path
             return False
+        if getattr(model, "packed_rows", False):
+            return True
         if any(s.mixer in ("attn", "mla") for s in model.specs):              # KV caches grow with every token
             return False
         return all(all(torch.is_tensor(v) for v in c.values()) for c in caches)   # nested caches (MoM) decode eagerly
 
+    def _forward(self, tok):
+        if self.rows is not None:
+            return self.model(tok, caches=self.caches, batch=self.rows)
+        return self.model(tok, caches=self.caches, position_offset=0)
+
     def _capture(self) -> bool:
-        static = [dict(c) for c in self.caches]                # the state tensors the graph will read and update
+        static = [] if self.rows is not None else [dict(c) for c in self.caches]                # the state tensors the graph will read and update
         graph = torch.cuda.CUDAGraph()
         try:
             with torch.cuda.graph(graph):
-                self.logits = self.model(self.tok, caches=self.caches, position_offset=0)
+                self.logits = self._forward(self.tok)
                 for c, st in zip(self.caches, static):        # forward rebinds every entry to a new tensor
                     for k, v in st.items():
                         v.copy_(c[k])
@@ -147,7 +154,7 @@ class GraphedDecodeStep:
             self.tok.copy_(tok)
             self._capture()                                    # capturing records the step without running it
         if self.failed:
-            return self.model(tok, caches=self.caches, position_offset=0)
+            return self._forward(tok)
         self.tok.copy_(tok)
         self.graph.replay()
         return self.logits
@@ -163,6 +170,10 @@ def generate_tokens(model, tokens: torch.Tensor, lengths: torch.Tensor, *, eod: 
     ``cuda_graph``: replay the one-token steps from a CUDA graph (``GraphedDecodeStep``) when the model allows it; the
     prefill and the first two one-token steps run eagerly (they also serve as the warm-up before the capture)."""
     model.eval()
+    if getattr(model, "packed_rows", False):
+        return _generate_packed(model, tokens, lengths, eod if use_eod_for_early_termination else None,
+                                lambda lg: sample(lg, top_k, top_p, temperature, model.cfg.vocab_size, generator),
+                                repetition_penalty, return_log_probs, cuda_graph)
     B, L = tokens.shape
     min_len = int(lengths.min())
     caches = model.new_cache()
@@ -207,6 +218,64 @@ def generate_tokens(model, tokens: torch.Tensor, lengths: torch.Tensor, *, eod: 
     if return_log_probs:
         logps = PF.broadcast_from_last_stage(model, logps, tuple(logps.shape), torch.float32, tokens.device)
     return tokens, gen_len, logps
+
+
+def _generate_packed(model, tokens, lengths, eod: Optional[int], draw, repetition_penalty: float, return_log_probs: bool,
+                     cuda_graph: bool):
+    """``generate_tokens`` for models that run packed rows: every prompt is processed whole, then each request goes on from
+    its own position, and one that has reached its end leaves the batch and gives its slot back."""
+    from .session import InferenceSession
+    B, L = tokens.shape
+    dev = tokens.device
+    at = [min(int(n), L) for n in lengths]                             # next position of every request
+    gen_len = [L] * B
+    logps = torch.zeros(B, L - 1, dtype=torch.float32, device=dev) if return_log_probs else None
+    ses = InferenceSession(model, slots=B, cuda_graph=cuda_graph)
+    prompts = [tokens[b, :at[b]] for b in range(B)]
+    slots, logits = ses.start(prompts, [list(range(n)) for n in at] if return_log_probs else None)
+    if return_log_probs:                                               # scores inside the prompts
+        lp, row = F.log_softmax(logits, -1), 0
+        for b, n in enumerate(at):
+            logps[b, :n - 1] = lp[row:row + n - 1].gather(1, prompts[b][1:, None]).squeeze(1)
+            row += n
+        ends = torch.tensor(at, device=dev).cumsum(0) - 1
+        logits = logits.index_select(0, ends)
+    live = list(range(B))
+    while live:
+        keep = [k for k, b in enumerate(live) if at[b] < L]
+        if len(keep) < len(live):
+            ses.finish([slots[b] for b in live if at[b] >= L])
+            live, logits = [live[k] for k in keep], logits[keep]
+            if not live:
+                break
+        idx, pos = torch.tensor(live, device=dev), torch.tensor([at[b] for b in live], device=dev)
+        if repetition_penalty != 1.0:
+            upto = torch.arange(L, device=dev)[None, :] < pos[:, None]
+            seen = torch.where(upto, tokens[idx], tokens[idx, :1])     # columns not reached yet repeat the first token
+            logits = apply_repetition_penalty(logits, seen, repetition_penalty)
+        new = draw(logits)
+        tokens[idx, pos] = new
+        if return_log_probs:
+            logps[idx, pos - 1] = F.log_softmax(logits, -1).gather(1, new[:, None]).squeeze(1)
+        hit = (new == eod).tolist() if eod is not None else [False] * len(live)
+        for k, b in enumerate(live):
+            at[b] += 1
+            if hit[k]:
+                gen_len[b] = at[b]
+        if any(hit):
+            ses.finish([slots[b] for k, b in enumerate(live) if hit[k]])
+            on = [k for k in range(len(live)) if not hit[k]]
+            live, new = [live[k] for k in on], new[on]
+        go = [k for k, b in enumerate(live) if at[b] < L]
+        if not go:
+            ses.finish([slots[b] for b in live])
+            break
+        if len(go) < len(live):
+            ses.finish([slots[b] for b in live if at[b] >= L])
+            live, new = [live[k] for k in go], new[go]
+        logits = ses.step([slots[b] for b in live], new)
+    end = max(at)
+    return tokens[:, :end], torch.tensor(gen_len, device=dev), (None if logps is None else logps)
 
 
 @dataclass

@@ -24,8 +24,8 @@ from typing import List, Optional, Tuple
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: Optional[str]      # 'lsm' | 'attn' | 'mla' | 'mamba' | None
-    ffn: Optional[str]        # 'mlp' | 'moe' | None
+    mixer: Optional[str]      # 'lsm' | 'attn' | 'mla' | 'mamba' | 'chunk_attn' | None
+    ffn: Optional[str]        # 'mlp' | 'moe' | 'poly_mlp' | None
     symbol: str               # source symbol, for logs and checkpoints
     index: int                # global index in the expanded list
 
@@ -85,6 +85,8 @@ def _ffn_kind(cfg, layer_idx: int) -> str:
 
 
 def expand_layer_pattern(cfg) -> List[LayerSpec]:
+    if cfg.layers is not None:
+        return [LayerSpec("chunk_attn", "poly_mlp" if l["ff"] else None, "C", i) for i, l in enumerate(cfg.layers)]
     attn_kind = "mla" if cfg.base_model == "deepseek_v2" else "attn"
     specs: List[Tuple[Optional[str], Optional[str], str]] = []
     if cfg.use_la_module and cfg.la_module == "mamba2":

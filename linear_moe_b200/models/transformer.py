@@ -5,7 +5,8 @@ One model class serves every family of the reference: ``GPTModel`` (softmax atte
 ``MambaStack`` (``M``/``*``/``-`` patterns) — model/qwen2/model.py, model/qwen2/hybrid/
 hybrid_model.py:28-248, hybrid_transformer_block.py:87-474, sequence_modeling/ssm.py:73-250,
 mamba2/mamba_model.py:16-209 — for the four backbones (qwen2, llama3, mixtral, deepseek_v2), which
-differ only in configuration (attention kind, router order, shared expert, biases).
+differ only in configuration (attention kind, router order, shared expert, biases).  Layer-list designs (``ModelConfig.layers``)
+build ``ParallelBlock`` (models/parallel_block.py) instead of ``Block``.
 
 A ``Block`` is one pre-norm residual layer: optional token mixer, optional FFN
 (transformer_layer.py:179-273, mamba_layer.py:27-80).  Module names follow the Megatron-Core
@@ -28,13 +29,14 @@ import torch.utils.checkpoint as ckpt
 from .. import ops
 from ..config.model_config import ModelConfig
 from ..dist.mesh import Mesh, single_process_mesh
-from ..parallel.tensor_parallel import LMHead, VocabParallelEmbedding
+from ..parallel.tensor_parallel import LMHead, VocabParallelEmbedding, init_normal
 from .attention import MLASelfAttention, SelfAttention
 from .layout import LayerSpec, split_for_pipeline
 from .lsm_layers import LinearAttention, LinearRNN
 from .mamba2 import MambaMixer
 from .moe import MLP, MoELayer
 from .mom import MomLinearAttention
+from .parallel_block import ParallelBlock, forward_rows, new_slot_cache
 
 
 class Norm(nn.Module):
@@ -150,16 +152,27 @@ class CausalLM(nn.Module):
         vpp = mesh.par.virtual_pipeline_model_parallel_size
         self.specs: List[LayerSpec] = split_for_pipeline(all_specs, mesh.pp, pp_rank, vpp, vpp_rank)
         dt, sp = cfg.params_dtype, self.sequence_parallel
+        if cfg.layers is not None and mesh.world_size > 1:
+            raise ValueError("layer-list models (parallel blocks) run on one rank")
         if pre_process:
             self.embedding = nn.Module()
             self.embedding.word_embeddings = VocabParallelEmbedding(cfg.vocab_size, cfg.hidden_size, mesh=mesh,
                                                                     std=cfg.init_method_std, sequence_parallel=sp,
                                                                     dtype=dt, device=device)
+            if cfg.position_embedding_type == "learned":
+                self.embedding.position_embeddings = nn.Module()
+                self.embedding.position_embeddings.weight = nn.Parameter(
+                    init_normal((cfg.max_position_embeddings, cfg.hidden_size), cfg.init_method_std,
+                                "embedding.position_embeddings.weight", device).to(dt))
         self.decoder = nn.Module()
         self.decoder.layers = nn.ModuleList(
-            [Block(cfg, s, mesh, f"decoder.layers.{s.index}", sp, device) for s in self.specs])
+            [ParallelBlock(cfg, s, f"decoder.layers.{s.index}", device) if s.mixer == "chunk_attn" else Block(cfg, s, mesh, f"decoder.layers.{s.index}", sp, device) for s in self.specs])
         if post_process:
-            self.decoder.final_layernorm = Norm(cfg, device)
+            if cfg.layers is not None:
+                self.decoder.final_layernorm = nn.Module()         # one number for all coordinates
+                self.decoder.final_layernorm.weight = nn.Parameter(torch.ones((), device=device))
+            else:
+                self.decoder.final_layernorm = Norm(cfg, device)
             tied = self.embedding.word_embeddings.weight if (cfg.tie_embeddings and pre_process) else None
             # tied weights with the embedding on another pipeline stage: this stage holds a copy drawn from the same key
             # (equal values); the optimizer sums the two copies' gradients, so both receive the same update
@@ -182,9 +195,20 @@ class CausalLM(nn.Module):
                 # holds the whole table and contributes the gradient of its own layers
                 self.lower_bounds.pp_shared_grad = "all"
 
+        if cfg.layers is not None:
+            self.requires_grad_(False)                             # serving only: the block's kernels have no backward pass
+
     # ------------------------------------------------------------------
-    def new_cache(self) -> List[dict]:
-        """One dict per local block: recurrent states / KV caches for decoding."""
+    @property
+    def packed_rows(self) -> bool:
+        """Does the model run batches of requests at different positions (packed rows and a slot cache)?"""
+        return self.cfg.layers is not None
+
+    def new_cache(self, slots: int = 1):
+        """One dict per local block: recurrent states / KV caches for decoding.  Models that run packed rows get a
+        ``SlotCache`` (a list of such dicts with buffers for ``slots`` requests)."""
+        if self.packed_rows:
+            return new_slot_cache(self, slots)
         return [dict() for _ in self.decoder.layers]
 
     def _run_blocks(self, x, residual, caches, position_offset):
@@ -222,7 +246,12 @@ class CausalLM(nn.Module):
 
     def forward(self, input_ids: Optional[torch.Tensor] = None, labels: Optional[torch.Tensor] = None, *,
                 hidden_in: Optional[torch.Tensor] = None, caches: Optional[List[dict]] = None,
-                position_offset: int = 0, parallel_output: bool = False, return_hidden: bool = False):
+                position_offset: int = 0, parallel_output: bool = False, return_hidden: bool = False, batch=None,
+                logit_rows: Optional[torch.Tensor] = None):
+        """``batch`` (``ops.chunk_attn.RowBatch``; models that run packed rows): ``input_ids`` are the packed tokens of its
+        requests and the result has one row per token, or per entry of ``logit_rows``."""
+        if self.packed_rows:
+            return forward_rows(self, input_ids, labels, caches, position_offset, batch, logit_rows, return_hidden)
         if self.pre_process:
             x = self.embedding.word_embeddings(input_ids)
         else:

@@ -33,6 +33,20 @@ def linear(x, weight, bias=None):
     return F.linear(x, weight.to(x.dtype), None if bias is None else bias.to(x.dtype))
 
 
+def linear_f32(x, weight):
+    """``x W^T`` for 2-D ``x`` with the fp32 accumulators as the result (logits)."""
+    if _cuda(x):
+        return _K().linear_f32(x, weight)
+    return F.linear(x.float(), weight.float())
+
+
+def linear_add_(acc, x, weight):
+    """``acc += x W^T`` for an fp32 ``acc`` (a residual stream); in place, without a rounded intermediate."""
+    if _cuda(x):
+        return _K().linear_add_(acc, x, weight)
+    return acc.add_(F.linear(x.float(), weight.float()))
+
+
 def linear_swiglu(x, weight, bias=None):
     """``swiglu(x W^T)`` with W = [gate; up]; on CUDA the activation runs in the GEMM epilogue."""
     if _cuda(x) and x.dtype == torch.bfloat16 and bias is None:
@@ -305,6 +319,10 @@ def softmax_attention(q, k, v, scale=None, causal=True, q_offset: int = 0, windo
     if _cuda(q):
         return _K().flash_attention(q, k, v, scale, causal, q_offset, window)
     return R.softmax_attention(q, k, v, scale, causal, q_offset, window)
+
+
+# ---- packed-row operators of parallel blocks (serving only) ---------------------------------------
+from .chunk_attn import chunk_attention, embed_norm, poly_norm, stream_norm   # noqa: E402,F401
 
 
 # ---- linear sequence models -----------------------------------------------

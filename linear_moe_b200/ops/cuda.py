@@ -42,6 +42,15 @@ def lib_path() -> str:
     return os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "lib", "liblmoe.so")
 
 
+def use_library(path: str):
+    """Take the kernels from ``path`` (``build.build_serving``) instead of ``lib/liblmoe.so``; before the first kernel call."""
+    global _LIB
+    if _LIB is None:
+        _LIB = ctypes.CDLL(path)
+    elif _LIB._name != path and _LIB._name != lib_path():
+        raise RuntimeError(f"the kernel library {_LIB._name} is already loaded")
+
+
 def lib() -> ctypes.CDLL:
     global _LIB
     if _LIB is None:
@@ -207,6 +216,40 @@ def linear_skinny(x, weight):
     _check(lib().lmoe_gemm_skinny(_p(x2), ll(x2.stride(0)), _p(weight), ll(weight.stride(0)), _p(y), ll(N), _i32(M), _i32(N),
                                   _i32(K), _st()), "gemm_skinny")
     return y
+
+
+def _skinny_f32(x, weight, y, accumulate: bool):
+    ll = ctypes.c_longlong
+    _check(lib().lmoe_gemm_skinny_f32(_p(x), ll(x.stride(0)), _p(weight), ll(weight.stride(0)), _p(y), ll(y.stride(0)), _i32(x.shape[0]),
+                                      _i32(weight.shape[0]), _i32(x.shape[1]), _i32(int(accumulate)), _st()), "gemm_skinny_f32")
+
+
+def linear_f32(x, weight):
+    """``x [M, K] W^T`` with an fp32 result: weight streaming for up to 16 rows, else the dense tcgen05 kernel; fp32 operands
+    (and bf16 shapes outside the kernels' alignment rules) take the library product."""
+    from . import gemm
+    if x.dtype == torch.float32:
+        return F.linear(x, weight)
+    if _skinny_ok(x, weight) and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0:
+        y = torch.empty(x.shape[0], weight.shape[0], dtype=torch.float32, device=x.device)
+        _skinny_f32(x, weight, y, False)
+        return y
+    if gemm.dense_ok(x, weight) and weight.shape[0] % 8 == 0:
+        return gemm.dense(x, weight, out_dtype=torch.float32)
+    return torch.mm(x, weight.t(), out_dtype=torch.float32)
+
+
+def linear_add_(acc, x, weight):
+    """``acc [M, N] += x W^T`` in fp32 (weight streaming for up to 16 rows, TMA reduce-add epilogue of the dense kernel else)."""
+    from . import gemm
+    if x.dtype == torch.float32:
+        return acc.addmm_(x, weight.t())
+    if _skinny_ok(x, weight) and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0:
+        _skinny_f32(x, weight, acc, True)
+        return acc
+    if gemm.dense_ok(x, weight) and weight.shape[0] % 8 == 0 and acc.stride(0) % 4 == 0 and acc.data_ptr() % 16 == 0:
+        return gemm.dense(x, weight, out=acc, accumulate=True)
+    return acc.add_(torch.mm(x, weight.t(), out_dtype=torch.float32))
 
 
 def linear(x, weight, bias=None):
