@@ -71,6 +71,9 @@ def parse():
     p.add_argument("--tokens-per-gpu", type=int, default=TOKENS_PER_GPU)
     p.add_argument("--layers", type=int, default=None, help="debug only: fewer layers (marks the result invalid)")
     p.add_argument("--no-e2e", action="store_true")
+    p.add_argument("--serve", action="store_true", help="instead of the training benchmark: prefill / decode throughput and kernel "
+                   "times of the Lagisun design beside the Llama3-shaped transformer at equal size (one GPU)")
+    p.add_argument("--serve-sizes", type=str, default="1b,8b", help="sizes of --serve")
     p.add_argument("--overlap-grad-reduce", action=argparse.BooleanOptionalAction, default=False,
                    help="reduce-scatter the gradients of a block while the backward pass of the blocks before it runs "
                         "(bitwise the same result; measured 2 - 3 ms per step slower than one reduce after backward at N = 2, "
@@ -95,6 +98,9 @@ def main():
     args = parse()
     if args.impl == "reference":
         return reference_arm()
+    if args.serve:
+        from linear_moe_b200.bench.serve import main as serve
+        return serve(args.serve_sizes.split(","))
     import torch
     import torch.distributed as dist
     from linear_moe_b200.config.model_config import ParallelConfig, TrainConfig

@@ -5,6 +5,7 @@ samples and every stage receives the sampled tokens; rank 0 prints the completio
 
   python examples/generate.py --load /path/to/ckpt --text-generate-input-file prompts.jsonl <model flags>
   torchrun --nproc-per-node 2 --master-addr 127.0.0.1 examples/generate.py --pipeline-model-parallel-size 2 ...
+  python examples/generate.py --model-dir /path/to/folder --text-generate-input-file prompts.jsonl --cuda-graph-decode
   LMOE_SERVE_PORT=5000 python examples/generate.py --load /path/to/ckpt <model flags>     # serve PUT /api instead
 """
 import os
@@ -19,6 +20,7 @@ from linear_moe_b200.config.arguments import parse_args                         
 from linear_moe_b200.data.tokenizer import build_tokenizer                        # noqa: E402
 from linear_moe_b200.dist.mesh import init_distributed, single_process_mesh       # noqa: E402
 from linear_moe_b200.infer.generation import GPTPredictor                         # noqa: E402
+from linear_moe_b200.models.registry import load_model                           # noqa: E402
 from linear_moe_b200.models.transformer import CausalLM                           # noqa: E402
 
 if __name__ == "__main__":
@@ -32,9 +34,15 @@ if __name__ == "__main__":
     else:
         mesh = single_process_mesh()
     dev = torch.device("cuda", torch.cuda.current_device()) if torch.cuda.is_available() else torch.device("cpu")
+    if args.model_dir:
+        if distributed:
+            raise SystemExit("--model-dir runs in one process")
+        model = load_model(args.model_dir, getattr(torch, args.model_dtype), dev)
+        cfg = model.cfg
+    else:
+        model = CausalLM(cfg, mesh, pre_process=mesh.is_first_stage, post_process=mesh.is_last_stage, device=dev).to(dev)
     tok, _ = build_tokenizer(args.patch_tokenizer_type, args.tokenizer_model, cfg.vocab_size, args.extra_vocab_size)
-    model = CausalLM(cfg, mesh, pre_process=mesh.is_first_stage, post_process=mesh.is_last_stage, device=dev).to(dev)
-    if tc.load:
+    if tc.load and not args.model_dir:
         if tc.use_dist_ckpt:
             from linear_moe_b200.ckpt.sharded import load_sharded
             per = cfg.num_layers // mesh.pp

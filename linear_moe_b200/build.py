@@ -25,7 +25,7 @@ NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", 
 # sources whose fp32 instantiations serve models in true 32-bit: IEEE division and the accurate exp / tanh
 PRECISE = {"chunk_attn.cu", "parallel_block.cu"}
 # what serving a model of the listed kind needs (``build_serving``); everything else is training, communication and fp8
-SERVING = {"parallel_block": ("chunk_attn.cu", "chunk_attn_tc.cu", "parallel_block.cu", "gemm_dense.cu", "gemm_skinny.cu")}
+SERVING = {"parallel_block": ("chunk_attn.cu", "chunk_attn_step.cu", "chunk_attn_tc.cu", "parallel_block.cu", "gemm_dense.cu", "gemm_skinny.cu")}
 
 
 def _nvcc() -> str:

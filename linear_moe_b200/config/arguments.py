@@ -353,6 +353,10 @@ def build_parser() -> argparse.ArgumentParser:
     _flag(g, "--text-generate-input-file", type=str, default="")
     _flag(g, "--text-generate-output-file", type=str, default="")
     _flag(g, "--text-generate-gt-file", type=str, default="")
+    _flag(g, "--model-dir", type=str, default=None,
+          help="generation / serving: folder with config.json (of a registered architecture) and model.safetensors, instead of "
+               "--load and the model flags")
+    _flag(g, "--model-dtype", type=str, default="bfloat16", choices=["bfloat16", "float32"], help="precision of --model-dir")
     _flag(g, "--time", action="store_true")
     _flag(g, "--input-len", type=int, default=1)
     _flag(g, "--eval-dev", action="store_true")

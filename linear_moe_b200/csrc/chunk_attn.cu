@@ -11,7 +11,7 @@
 //   chunk_attn_rows_kernel   prompts, any head sizes, bf16 or fp32 (all arithmetic fp32): tiles of 32 queries x 32 keys,
 //                            online softmax.  Keys of the chunk that precede this call come from the cache.  The bf16 fast path for
 //                            prompts is chunk_attn_tc.cu.
-//   chunk_attn_step_kernel   one token per request: a cluster of CTAs splits the keys of (request, kv head), the partial
+//   chunk_attn_step_kernel   one token per request, any head sizes, bf16 or fp32 (bf16 fast path: chunk_attn_step.cu): a cluster of CTAs splits the keys of (request, kv head), the partial
 //                            softmaxes meet in distributed shared memory; the new key and value are read from the projection and
 //                            stored into the cache on the way; the gate is applied in the same kernel
 //   chunk_store_kernel       keys / values of a prompt's last chunk -> cache
@@ -25,24 +25,6 @@
 namespace lmoe {
 namespace ca {
 namespace cg = cooperative_groups;
-
-struct Args {
-    const void* z;            // [rows, ldz] projection output
-    void* out;                // [rows, ldo]
-    void *kc, *vc;            // cache [slots, cap_rows, G, dkp] / [slots, cap_rows, G, dvp]
-    const float* lut;         // [H, nlut] bias by distance (the last entry holds for everything beyond)
-    const float* gain;        // 1 float
-    const int* items;         // rows kernel: [n, 8] work items
-    const int* slots;         // step: [B]; store: [rows]
-    const int* pos;           // step: [B]; store: [rows] position of the token
-    const int* ends;          // store: [rows] length of the token's request after this call
-    long long ldz, ldo;
-    int zq, zk, zv, zg;       // first columns
-    int H, G, dk, dv, dkp, dvp;
-    int cap_rows, size, nlut;
-    int n;                    // work items / requests / rows
-    float scale, cap, mul;
-};
 
 __device__ __forceinline__ float capped(float s, float cap) { return cap > 0.f ? cap * tanhf(s / cap) : s; }
 

@@ -102,11 +102,12 @@ class GraphedDecodeStep:
     updates) that the host cannot issue as fast as the GPU runs them.  Models whose every cache entry has a fixed size
     (all mixers linear sequence models or Mamba2: O(1) recurrent state, no growing KV cache) make the step static, so it
     is captured once and replayed: the token is copied into a static buffer, the graph runs the whole forward, and the
-    new states are copied back over the state buffers the graph reads.  Softmax-attention layers (KV cache grows by one
-    row per token) are not supported and fall back to eager decoding."""
+    new states are copied back over the state buffers the graph reads.  Softmax-attention layers whose KV cache grows by one
+    row per token are not supported and fall back to eager decoding.  A ``SlotCache`` is updated in place by the step, so
+    nothing is copied back; ``rows`` then holds the requests' positions and slots in device tensors that the caller fills."""
 
-    def __init__(self, model, caches: List[dict], batch: int, device):
-        self.model, self.caches = model, caches
+    def __init__(self, model, caches: List[dict], batch: int, device, rows=None):
+        self.model, self.caches, self.rows = model, caches, rows
         self.tok = torch.zeros(batch, 1, dtype=torch.long, device=device)
         self.graph: Optional["torch.cuda.CUDAGraph"] = None
         self.logits: Optional[torch.Tensor] = None

@@ -199,14 +199,18 @@ def chunk_attention(z: torch.Tensor, out: torch.Tensor, spec: ChunkAttnSpec, lay
         assert k.dtype == v.dtype == z.dtype and k.shape[1] == v.shape[1]
         a.kc, a.vc, a.cap_rows, a.dkp, a.dvp = k.data_ptr(), v.data_ptr(), k.shape[1], k.shape[3], v.shape[3]
     dt = K._dt(z)
+    fast = dt == 1 and spec.tensor_core() and spec.softcap + table.peak <= SCORE_BOUND
     if batch.decode:
         assert cache is not None
         a.n = batch.requests
-        K._check(K.lib().lmoe_chunk_attn_step(ctypes.byref(a), _splits(spec, batch.requests, K.num_sms()), dt, K._st()), "chunk_attn_step")
+        splits = _splits(spec, batch.requests, K.num_sms())
+        if fast:
+            K._check(K.lib().lmoe_chunk_attn_step_mma(ctypes.byref(a), splits, K._st()), "chunk_attn_step_mma")
+        else:
+            K._check(K.lib().lmoe_chunk_attn_step(ctypes.byref(a), splits, dt, K._st()), "chunk_attn_step")
         return
     inside = batch.continues_inside_chunk(spec.chunk)
-    if (dt == 1 and spec.tensor_core() and not inside and spec.softcap + table.peak <= SCORE_BOUND
-            and table.lut.shape[1] <= LUT_ENTRIES_TC):
+    if fast and not inside and table.lut.shape[1] <= LUT_ENTRIES_TC:
         from . import gemm
         t = _TcArgs()
         items = batch.items(spec.chunk, 128)
