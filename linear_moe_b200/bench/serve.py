@@ -91,7 +91,7 @@ def whole_model(size: str) -> list:
     lla = CausalLM(llama_config(**kw), device=dev).eval()
     row("llama3-shaped", f"prefill {B}x{T}", _events(lambda: lla(ids, caches=lla.new_cache()), 5), B * T)
     for n in (8, 64):
-        caches = [lla.new_cache() for _ in range(1)][0]
+        caches = lla.new_cache()
         ctx = torch.randint(0, VOCAB, (n, CTX), device=dev)
         for c in range(0, CTX, 512):
             lla(ctx[:, c:c + 512], caches=caches, position_offset=c)

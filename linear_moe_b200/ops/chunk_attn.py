@@ -2,7 +2,7 @@
 
 All operators work on packed rows: the tokens of a batch's requests, one after the other (:class:`RowBatch` says which row
 belongs to which request and position).  CUDA tensors (bf16 or fp32) take the kernels of ``csrc/chunk_attn.cu``,
-``csrc/chunk_attn_tc.cu`` and ``csrc/parallel_block.cu``; CPU tensors take the eager definitions of
+``csrc/chunk_attn_tc.cu``, ``csrc/chunk_attn_step.cu`` and ``csrc/parallel_block.cu``; CPU tensors take the eager definitions of
 :mod:`linear_moe_b200.ref.chunk_attn`.  These operators serve (no backward pass).
 """
 from __future__ import annotations
@@ -167,10 +167,12 @@ def _no_grad(*ts):
 
 
 def _splits(spec: ChunkAttnSpec, requests: int, sms: int) -> int:
-    """CTAs that share the keys of one (request, kv head): as many as fill the GPU, at least 64 keys of a full chunk each."""
+    """CTAs (1 - 8, one cluster) that share the keys of one (request, kv head): as many as stay resident together (four of
+    the step kernel per SM, three with head sizes over 64), with at least 64 keys of a full chunk each."""
     ctas = requests * spec.kv_heads * ((spec.heads // spec.kv_heads + 7) // 8)
+    room = sms * (3 if max(spec.dim, spec.vdim) > 64 else 4)
     s = 1
-    while s < 8 and ctas * s < 2 * sms and spec.chunk >= 128 * s:
+    while s < 8 and ctas * s * 2 <= room and spec.chunk >= 128 * s:
         s *= 2
     return s
 
