@@ -20,7 +20,8 @@ LA_MODULES = (
     "gated_deltanet", "gsa", "based", "rebased", "hgrn2", "rwkv6", "rwkv7",
     "mamba2", "lasp2", "mom_gla", "mom_gated_deltanet", "mom_linear_attention",
 )
-BASE_MODELS = ("qwen2", "llama3", "mixtral", "deepseek_v2", "lagisun")
+BASE_MODELS = ("qwen2", "llama3", "mixtral", "deepseek_v2", "lagisun", "sonodra")
+LAYER_LIST_MODELS = ("lagisun", "sonodra")        # described by ModelConfig.layers; run packed rows, serve only
 
 
 @dataclass
@@ -35,7 +36,7 @@ class ModelConfig:
     ffn_hidden_size: int = 1024
     vocab_size: int = 32000                       # already padded
     max_position_embeddings: int = 4096
-    normalization: str = "RMSNorm"                # RMSNorm | LayerNorm
+    normalization: str = "RMSNorm"                # RMSNorm | LayerNorm | ScalarRMSNorm (one number per norm)
     norm_eps: float = 1e-6
     swiglu: bool = True
     add_bias_linear: bool = False
@@ -132,8 +133,11 @@ class ModelConfig:
     qk_nope_head_dim: int = 128
     qk_rope_head_dim: int = 64
     v_head_dim: int = 128
-    # ---- layer list (designs whose layers have sizes of their own; parallel mixer + feed-forward blocks) ----
-    # one entry per layer: {"attn": ops.chunk_attn.ChunkAttnSpec, "bias_rows": rows of the distance table, "ff": width or None}
+    # ---- layer list (designs whose layers have sizes of their own) ----
+    # lagisun: parallel mixer + feed-forward blocks, one entry per layer
+    #   {"attn": ops.chunk_attn.ChunkAttnSpec, "bias_rows": rows of the distance table, "ff": width or None}
+    # sonodra: sequential blocks with a norm at both ends of a sublayer, one entry per layer
+    #   {"mixer": ops.packed_attn.AttentionSpec or LatentSpec, "ff": width (gated), ops.moe_rows.ExpertsSpec, or None}
     layers: Optional[Tuple[dict, ...]] = None
     residual_multiplier: float = 1.0              # factor of every block's output before it joins the residual stream
     # ---- precision / memory --------------------------------------------
@@ -152,8 +156,8 @@ class ModelConfig:
             self.kv_channels = self.hidden_size // self.num_attention_heads
         if self.num_query_groups is None:
             self.num_query_groups = self.num_attention_heads
-        if (self.base_model == "lagisun") != (self.layers is not None):
-            raise ValueError("a lagisun model is described by its layer list (and no other family has one)")
+        if (self.base_model in LAYER_LIST_MODELS) != (self.layers is not None):
+            raise ValueError(f"{', '.join(LAYER_LIST_MODELS)} models are described by their layer list (and no other family has one)")
         if self.layers is not None:
             self.num_layers = len(self.layers)
         if self.base_model not in BASE_MODELS:

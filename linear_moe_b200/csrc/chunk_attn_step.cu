@@ -13,6 +13,7 @@
 // While the kernel before it (the projection) still runs, it fetches the first cached keys and values.
 #include <cooperative_groups.h>
 
+#include "attn_math.cuh"
 #include "chunk_attn.cuh"
 #include "common.cuh"
 #include "mma_utils.cuh"
@@ -24,16 +25,6 @@ namespace cg = cooperative_groups;
 constexpr int WARPS = 4, HEADS = 8;
 constexpr float LOG2E = 1.4426950408889634f;
 
-__device__ __forceinline__ float ex2(float x) {
-    float r;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
-    return r;
-}
-__device__ __forceinline__ float rcp(float x) {
-    float r;
-    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
-    return r;
-}
 __device__ __forceinline__ uint32_t pack2(float lo, float hi) {
     __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<uint32_t*>(&h);

@@ -16,6 +16,7 @@
 // The bias table of the head sits in shared memory, shifted and padded so that a tile needs no clamping of its index; tiles
 // entirely beyond the table's end use its last value.
 // Every mbarrier wait is bounded; on expiry the error word is set and the CTA drains and frees its tensor memory.
+#include "attn_math.cuh"
 #include "chunk_attn.cuh"
 #include "flash_tc_utils.cuh"
 
@@ -49,17 +50,6 @@ struct __align__(1024) Smem {
     uint32_t tmem_base;
     int abort_flag;
 };
-
-__device__ __forceinline__ float ex2(float x) {
-    float r;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
-    return r;
-}
-__device__ __forceinline__ float rcp(float x) {
-    float r;
-    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
-    return r;
-}
 
 template <int DQ, int DV>
 __global__ void __launch_bounds__(THREADS, 1)

@@ -45,7 +45,17 @@ struct Params {
     int* err;
     int out_f32;              // pair kernel: C is fp32 (weight gradients straight into the fp32 accumulators)
     int accumulate;           // with out_f32: C += result instead of C = result
+    const float* row_scale;   // mode 1, bf16 output: C = (row_scale[row] * relu(result))^2 (null: C = result)
 };
+
+// the squared-relu epilogue on a thread's 32 columns of one row
+__device__ __forceinline__ void relu2(uint32_t (&v)[32], float scale) {
+#pragma unroll
+    for (int i = 0; i < 32; ++i) {
+        const float t = scale * fmaxf(__uint_as_float(v[i]), 0.f);
+        v[i] = __float_as_uint(t * t);
+    }
+}
 
 
 // One output tile of the (possibly grouped) problem.
@@ -207,11 +217,13 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
             const uint32_t taddr = tmem_base + ((uint32_t)(q * 32) << 16) + buf * BN;
             bf16* crow = C + t.c_off + (long long)r * p.ldc;
             const bool zero = t.kblocks == 0;            // an expert without tokens: its weight gradient is zero
+            const float scale = p.row_scale != nullptr ? p.row_scale[t.a_row + r] : 0.f;
 #pragma unroll 1
             for (int c = 0; c < BN; c += 32) {
                 uint32_t v[32];
                 tmem_ld32(taddr + c, v);
                 tmem_ld_wait();
+                if (p.row_scale != nullptr) relu2(v, scale);
                 if (r < t.rows_valid) {
 #pragma unroll
                     for (int g = 0; g < 4; ++g) {
@@ -372,6 +384,7 @@ gemm_grouped_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_c
             const uint32_t taddr = tmem_base + ((uint32_t)(q * 32) << 16) + buf * BN;
             const bool zero = t.kblocks == 0;                        // an expert without tokens: its weight gradient is zero
             uint8_t* stg = sm.stage_out[warp - 2];                   // 32 rows x 128 bytes, 16-byte chunks xor-swizzled
+            const float scale = p.row_scale != nullptr ? p.row_scale[t.a_row + r0 + lane] : 0.f;
             if (p.out_f32) {
                 // fp32 output (optionally accumulating): 32 columns = 128 bytes per row and pass through the staging buffer
                 float* C32 = reinterpret_cast<float*>(C);
@@ -408,6 +421,7 @@ gemm_grouped_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_c
                     uint32_t v[32];
                     tmem_ld32(taddr + c + hc * 32, v);
                     tmem_ld_wait();
+                    if (p.row_scale != nullptr) relu2(v, scale);
 #pragma unroll
                     for (int g = 0; g < 4; ++g) {
                         uint4 o;
@@ -467,10 +481,10 @@ using namespace lmoe::gg;
 // mode 0: dense (M, N, K).  mode 1: grouped along M by offs (A rows), B holds num_groups matrices stacked along its rows.
 // mode 2: grouped along K by offs (rows of A and B), C holds num_groups outputs c_group_stride elements apart.
 // pairs != 0: CTA-pair kernel (256-row tiles; in mode 1 every offset must be a multiple of 256).
-LMOE_API int lmoe_gemm_grouped(const void* A, int a_rows, int a_cols, int lda, int a_mn, const void* B, int b_rows, int b_cols,
-                               int ldb, int b_mn, void* C, int ldc, int mode, int M, int N, int K, int num_groups,
-                               const int* offs, long long c_group_stride, int* err, int num_sms, int pairs, int out_f32, int accumulate,
-                               cudaStream_t st) {
+static int gemm_grouped_impl(const void* A, int a_rows, int a_cols, int lda, int a_mn, const void* B, int b_rows, int b_cols,
+                             int ldb, int b_mn, void* C, int ldc, int mode, int M, int N, int K, int num_groups,
+                             const int* offs, long long c_group_stride, int* err, int num_sms, int pairs, int out_f32, int accumulate,
+                             const float* row_scale, cudaStream_t st) {
     if (lda % 8 || ldb % 8 || ldc % 8 || a_cols % 8 || b_cols % 8 || N % 8) return -1;
     CUtensorMap ma, mb;
     int rc = make_map(&ma, A, (uint64_t)a_rows, (uint64_t)a_cols, (uint64_t)lda, a_mn ? 64 : BM);
@@ -480,7 +494,7 @@ LMOE_API int lmoe_gemm_grouped(const void* A, int a_rows, int a_cols, int lda, i
     Params p;
     p.mode = mode; p.M = M; p.N = N; p.K = K; p.ldc = ldc; p.num_groups = num_groups; p.offs = offs;
     p.c_group_stride = c_group_stride; p.b_group_rows = b_mn ? K : N; p.err = err;
-    p.out_f32 = out_f32; p.accumulate = accumulate;
+    p.out_f32 = out_f32; p.accumulate = accumulate; p.row_scale = row_scale;
     if (out_f32 && !pairs) return -3;
     if (pairs) {
         if (!a_mn && !b_mn) return launch_pair<false, false>(ma, mb, (bf16*)C, p, num_sms, st);
@@ -492,4 +506,22 @@ LMOE_API int lmoe_gemm_grouped(const void* A, int a_rows, int a_cols, int lda, i
     if (!a_mn && b_mn) return launch<false, true>(ma, mb, (bf16*)C, p, num_sms, st);
     if (a_mn && b_mn) return launch<true, true>(ma, mb, (bf16*)C, p, num_sms, st);
     return launch<true, false>(ma, mb, (bf16*)C, p, num_sms, st);
+}
+
+LMOE_API int lmoe_gemm_grouped(const void* A, int a_rows, int a_cols, int lda, int a_mn, const void* B, int b_rows, int b_cols,
+                               int ldb, int b_mn, void* C, int ldc, int mode, int M, int N, int K, int num_groups,
+                               const int* offs, long long c_group_stride, int* err, int num_sms, int pairs, int out_f32, int accumulate,
+                               cudaStream_t st) {
+    return gemm_grouped_impl(A, a_rows, a_cols, lda, a_mn, B, b_rows, b_cols, ldb, b_mn, C, ldc, mode, M, N, K, num_groups, offs,
+                             c_group_stride, err, num_sms, pairs, out_f32, accumulate, nullptr, st);
+}
+
+// C[rows_e, N] = (row_scale[row] * relu(A[rows_e, K] * W[e][N, K]^T))^2 with A [a_rows, lda], W [num_groups * N, ldb], bf16; offsets multiples
+// of 128 (pairs: 256), row_scale [a_rows].
+LMOE_API int lmoe_gemm_grouped_relu2(const void* A, int a_rows, int lda, const void* W, int ldb, void* C, int ldc, int N, int K,
+                                     int num_groups, const int* offs, const float* row_scale, int* err, int num_sms, int pairs,
+                                     cudaStream_t st) {
+    if (row_scale == nullptr) return -1;
+    return gemm_grouped_impl(A, a_rows, K, lda, 0, W, num_groups * N, K, ldb, 0, C, ldc, 1, 0, N, K, num_groups, offs, 0, err, num_sms, pairs,
+                             0, 0, row_scale, st);
 }

@@ -1,0 +1,385 @@
+// Packed-row softmax attention for any head size, bf16 or fp32 (arithmetic in fp32), and the row kernels around it:
+//   packed_attn_rows_kernel   prompts (mathematics and work items: packed_attn_tc.cu, the bf16 fast path): tiles of TQ queries x TQ
+//                             keys, online softmax
+//   packed_attn_step_kernel   one token per request from the cache (bf16 fast path: packed_attn_step.cu)
+//   qk_norm_rope_kernel       RMS norm of all query rows of a projection and of all key rows, before the heads are split, then
+//                             interleaved rotary positions, in place; the new keys and values enter the cache
+//   latent_norm_kernel        RMS norm of a latent projection into a matrix of its own and into the cache
+//   gather_rows_kernel        rows of a matrix and of a cache -> rows of a buffer (a prompt that goes on from a cache)
+//   gate_rows_kernel          o *= sigmoid(g)
+// Compiled without fast-math: the fp32 instantiations serve models in true 32-bit.
+#include "common.cuh"
+#include "packed_attn.cuh"
+
+namespace lmoe {
+namespace pag {
+using pa::Cache;
+using pa::Prompt;
+using pa::Step;
+
+// ------------------------------------------------------------------------------------------------------------------ prompts
+// TQ queries (32 or 16), four threads per query
+template <typename T, int TQ>
+__global__ void __launch_bounds__(TQ * 4) packed_attn_rows_kernel(Prompt a) {
+    constexpr int TK = TQ, NT = TQ * 4, KP = TK / 4;
+    extern __shared__ float sm[];
+    const int dk = a.dk, dv = a.dv, ldk = dk + 1;
+    float* Q = sm;                       // [TQ][dk + 1]
+    float* K = Q + TQ * ldk;             // [TK][dk + 1]
+    float* V = K + TK * ldk;             // [TK][dv]
+    float* O = V + TK * dv;              // [TQ][dv]
+    float* S = O + TQ * dv;              // [TQ][TK + 1]
+    const int* it = a.items + (long long)blockIdx.x * pa::I_N;
+    const int row0 = it[pa::I_ROW], nq = it[pa::I_NQ], c0 = it[pa::I_C0], krow = it[pa::I_KROW];
+    const int h = blockIdx.y, hk = h / (a.H / a.G);
+    for (int i = threadIdx.x; i < TQ * dk; i += NT) {
+        const int r = i / dk, d = i % dk;
+        Q[r * ldk + d] = r < nq ? to_f(((const T*)a.q)[(row0 + r) * a.ldq + h * dk + d]) : 0.f;
+    }
+    for (int i = threadIdx.x; i < TQ * dv; i += NT) O[i] = 0.f;
+    const int r = threadIdx.x >> 2, part = threadIdx.x & 3;
+    const int qi = c0 + min(r, nq - 1);  // rows beyond the item repeat its last query
+    float m = -INFINITY, l = 0.f;
+    const int k_beg = a.window > 0 ? max(0, c0 - a.window + 1) : 0, k_end = c0 + nq;
+    for (int k0 = k_beg; k0 < k_end; k0 += TK) {
+        __syncthreads();
+        for (int i = threadIdx.x; i < TK * dk; i += NT) {
+            const int j = i / dk, d = i % dk;
+            K[j * ldk + d] = k0 + j < k_end ? to_f(((const T*)a.k)[(long long)(krow + k0 + j) * a.ldk + hk * dk + d]) : 0.f;
+        }
+        for (int i = threadIdx.x; i < TK * dv; i += NT) {
+            const int j = i / dv, d = i % dv;
+            V[i] = k0 + j < k_end ? to_f(((const T*)a.v)[(long long)(krow + k0 + j) * a.ldv + hk * dv + d]) : 0.f;
+        }
+        __syncthreads();
+        float s[KP];
+#pragma unroll
+        for (int e = 0; e < KP; ++e) s[e] = 0.f;
+        for (int d = 0; d < dk; ++d) {
+            const float q = Q[r * ldk + d];
+#pragma unroll
+            for (int e = 0; e < KP; ++e) s[e] += q * K[(part + 4 * e) * ldk + d];
+        }
+        float mx = m;
+#pragma unroll
+        for (int e = 0; e < KP; ++e) {
+            const int key = k0 + part + 4 * e;
+            s[e] = key <= qi && (a.window <= 0 || key > qi - a.window) ? s[e] * a.scale : -INFINITY;
+            mx = fmaxf(mx, s[e]);
+        }
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+        const float corr = m == -INFINITY ? 0.f : expf(m - mx);
+        float ps = 0.f;
+#pragma unroll
+        for (int e = 0; e < KP; ++e) {
+            const float p = mx == -INFINITY ? 0.f : expf(s[e] - mx);   // no visible key yet
+            S[r * (TK + 1) + part + 4 * e] = p;
+            ps += p;
+        }
+        ps += __shfl_xor_sync(0xffffffffu, ps, 1);
+        ps += __shfl_xor_sync(0xffffffffu, ps, 2);
+        l = l * corr + ps;
+        m = mx;
+        __syncwarp();
+        for (int d = part; d < dv; d += 4) {
+            float o = O[r * dv + d] * corr;
+            for (int j = 0; j < TK; ++j) o += S[r * (TK + 1) + j] * V[j * dv + d];
+            O[r * dv + d] = o;
+        }
+        __syncwarp();
+    }
+    if (r < nq) {
+        T* out = (T*)a.out + (row0 + r) * a.ldo + h * dv;
+        const T* g = a.gate == nullptr ? nullptr : (const T*)a.gate + (row0 + r) * a.ldg + h * dv;
+        for (int d = part; d < dv; d += 4) {
+            const float o = O[r * dv + d] / l;
+            out[d] = from_f<T>(g == nullptr ? o : o / (1.f + expf(-to_f(g[d]))));
+        }
+    }
+}
+
+template <typename T, int TQ>
+static int launch_rows(const Prompt& a, cudaStream_t st) {
+    const size_t smem = sizeof(float) * (2 * TQ * (size_t)(a.dk + 1) + 2 * TQ * (size_t)a.dv + TQ * (TQ + 1));
+    if (smem > 227 * 1024) return -2;
+    cudaError_t e = cudaFuncSetAttribute(packed_attn_rows_kernel<T, TQ>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    packed_attn_rows_kernel<T, TQ><<<dim3(a.n, a.H), TQ * 4, smem, st>>>(a);
+    return (int)cudaGetLastError();
+}
+
+// ---------------------------------------------------------------------------------------------------------------- one token
+constexpr int ST = 256, SK = 64;         // threads, keys per tile
+
+// grid (H, n)
+template <typename T>
+__global__ void __launch_bounds__(ST) packed_attn_step_kernel(Step a) {
+    extern __shared__ float sm[];
+    float* Q = sm;                       // [dk]
+    float* O = Q + a.dk;                 // [dv]
+    float* P = O + a.dv;                 // [SK]
+    __shared__ long long rows[SK];
+    __shared__ float red[32];
+    const int h = blockIdx.x, b = blockIdx.y, hk = h / (a.H / a.G);
+    const int w = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int slot = a.slots[b], pos = a.pos[b];
+    const int first = a.c.table == nullptr ? max(0, pos + 1 - a.c.cap) : a.window > 0 ? max(0, pos + 1 - a.window) : 0;
+    const T* q = (const T*)a.q + (long long)b * a.ldq + (long long)h * a.dk;
+    for (int d = threadIdx.x; d < a.dk; d += ST) Q[d] = to_f(q[d]);
+    for (int d = threadIdx.x; d < a.dv; d += ST) O[d] = 0.f;
+    float m = -INFINITY, l = 0.f;
+    for (int k0 = first; k0 <= pos; k0 += SK) {
+        const int nt = min(SK, pos + 1 - k0);
+        __syncthreads();
+        if (threadIdx.x < nt) rows[threadIdx.x] = a.c.row(slot, k0 + threadIdx.x) * a.G + hk;
+        __syncthreads();
+        for (int j = w; j < nt; j += ST / 32) {
+            const T* k = (const T*)a.c.k + rows[j] * a.dk;
+            float s = 0.f;
+            for (int d = lane; d < a.dk; d += 32) s += Q[d] * to_f(k[d]);
+            s = warp_sum(s);
+            if (lane == 0) P[j] = s * a.scale;
+        }
+        __syncthreads();
+        const float x = threadIdx.x < nt ? P[threadIdx.x] : -INFINITY;
+        const float mx = fmaxf(m, block_max(x, red));
+        const float p = threadIdx.x < nt ? expf(x - mx) : 0.f;
+        if (threadIdx.x < nt) P[threadIdx.x] = p;
+        const float ps = block_sum(p, red);                  // also orders the writes of P
+        const float corr = m == -INFINITY ? 0.f : expf(m - mx);
+        l = l * corr + ps;
+        m = mx;
+        for (int d = threadIdx.x; d < a.dv; d += ST) {
+            float o = O[d] * corr;
+            for (int j = 0; j < nt; ++j) o += P[j] * to_f(((const T*)a.c.v)[rows[j] * a.dv + d]);
+            O[d] = o;
+        }
+    }
+    T* out = (T*)a.out + (long long)b * a.ldo + (long long)h * a.dv;
+    for (int d = threadIdx.x; d < a.dv; d += ST) out[d] = from_f<T>(O[d] / l);
+}
+
+template <typename T>
+static int launch_step(const Step& a, cudaStream_t st) {
+    const size_t smem = sizeof(float) * (a.dk + a.dv + SK);
+    if (smem > 200 * 1024) return -2;
+    cudaError_t e = cudaFuncSetAttribute(packed_attn_step_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    packed_attn_step_kernel<T><<<dim3(a.H, a.n), ST, smem, st>>>(a);
+    return (int)cudaGetLastError();
+}
+
+// --------------------------------------------------------------------------------------------------------------- row kernels
+constexpr int THREADS = 256;
+
+struct QkNorm {
+    void* z;                             // [rows, ldz]: queries (H x dk), keys (G x dk), values (G x dv) from columns zq, zk, zv
+    const float *wq, *wk;                // norm weights [H * dk], [G * dk] (null: no norm)
+    const double* freq;                  // [rot / 2] rotation per position (null: no rotation)
+    Cache c;                             // k null: nothing is stored
+    const int *pos, *slots, *ends;       // [rows]; ends: length of the request after this call, null: store every row
+    long long ldz;
+    int zq, zk, zv, H, G, dk, dv;        // dk, dv as laid out (padded with zero columns)
+    int nq, nk;                          // numbers in a norm (H, G x the unpadded size)
+    int rot;
+    float eps;
+    int rows;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(THREADS) qk_norm_rope_kernel(QkNorm a) {
+    pdl_trigger();
+    constexpr int W = Vec<T>::N;
+    extern __shared__ float2 turn[];     // [rot / 2] (cos, sin)
+    __shared__ float red[32];
+    const int row = blockIdx.x, pos = a.pos[row];
+    T* z = (T*)a.z + (long long)row * a.ldz;
+    for (int i = threadIdx.x; i < a.rot / 2; i += THREADS) {
+        // range reduction in double: the angle is exact to fp32 at any position
+        constexpr double TWO_PI = 6.283185307179586476925286766559;
+        const double angle = (double)pos * a.freq[i];
+        const float r = (float)(angle - TWO_PI * rint(angle / TWO_PI));
+        turn[i] = make_float2(cosf(r), sinf(r));
+    }
+    float rq = 1.f, rk = 1.f;
+    auto square_sum = [&](const T* p, int n) {
+        float s = 0.f;
+        for (int i = threadIdx.x * W; i < n; i += THREADS * W) {
+            Vec<T> v;
+            v.load(p + i);
+#pragma unroll
+            for (int e = 0; e < W; ++e) s += v.get(e) * v.get(e);
+        }
+        return s;
+    };
+    if (a.wq != nullptr) rq = 1.f / sqrtf(block_sum(square_sum(z + a.zq, a.H * a.dk), red) / a.nq + a.eps);
+    if (a.wk != nullptr) rk = 1.f / sqrtf(block_sum(square_sum(z + a.zk, a.G * a.dk), red) / a.nk + a.eps);
+    __syncthreads();
+    T* kd = nullptr;
+    T* vd = nullptr;
+    // a ring keeps the request's last `cap` positions: of the rows that share a place only the last one is stored
+    if (a.c.k != nullptr && (a.ends == nullptr || a.c.table != nullptr || pos >= a.ends[row] - a.c.cap)) {
+        const long long r = a.c.row(a.slots[row], pos) * a.G;
+        kd = (T*)a.c.k + r * a.dk;
+        vd = (T*)a.c.v + r * a.dv;
+    }
+    auto finish = [&](T* p, int n, const float* weight, float r, T* dst) {
+        for (int i = threadIdx.x * W; i < n; i += THREADS * W) {
+            Vec<T> v;
+            v.load(p + i);
+            const int d = i % a.dk;
+            float x[W];
+#pragma unroll
+            for (int e = 0; e < W; ++e) x[e] = weight == nullptr ? v.get(e) : v.get(e) * r * weight[i + e];
+#pragma unroll
+            for (int e = 0; e < W; e += 2) {
+                if (d + e < a.rot) {
+                    const float2 cs = turn[(d + e) / 2];
+                    const float u = x[e], t = x[e + 1];
+                    x[e] = u * cs.x - t * cs.y;
+                    x[e + 1] = t * cs.x + u * cs.y;
+                }
+            }
+#pragma unroll
+            for (int e = 0; e < W; ++e) v.set(e, x[e]);
+            v.store(p + i);
+            if (dst != nullptr) v.store(dst + i);
+        }
+    };
+    finish(z + a.zq, a.H * a.dk, a.wq, rq, nullptr);
+    finish(z + a.zk, a.G * a.dk, a.wk, rk, kd);
+    if (vd != nullptr)
+        for (int i = threadIdx.x * W; i < a.G * a.dv; i += THREADS * W) {
+            Vec<T> v;
+            v.load(z + a.zv + i);
+            v.store(vd + i);
+        }
+}
+
+struct LatentNorm {
+    const void* z;                       // [rows, ldz], latent projection from column 0 (pitch ldz)
+    void* c;                             // [rows, ldc] normed rows
+    const float* weight;                 // [rank]
+    Cache cache;                         // k null: nothing is stored
+    const int *pos, *slots;
+    long long ldz, ldc;
+    int width, rank;                     // columns as laid out (padded with zeros), numbers in the norm
+    float eps;
+    int rows;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(THREADS) latent_norm_kernel(LatentNorm a) {
+    pdl_trigger();
+    __shared__ float red[32];
+    constexpr int W = Vec<T>::N;
+    const int row = blockIdx.x;
+    const T* z = (const T*)a.z + (long long)row * a.ldz;
+    T* c = (T*)a.c + (long long)row * a.ldc;
+    T* dst = a.cache.k == nullptr ? nullptr : (T*)a.cache.k + a.cache.row(a.slots[row], a.pos[row]) * a.width;
+    float s = 0.f;
+    for (int i = threadIdx.x * W; i < a.width; i += blockDim.x * W) {
+        Vec<T> v;
+        v.load(z + i);
+#pragma unroll
+        for (int e = 0; e < W; ++e) s += v.get(e) * v.get(e);
+    }
+    const float r = 1.f / sqrtf(block_sum(s, red) / a.rank + a.eps);
+    for (int i = threadIdx.x * W; i < a.width; i += blockDim.x * W) {
+        Vec<T> v;
+        v.load(z + i);
+#pragma unroll
+        for (int e = 0; e < W; ++e) v.set(e, v.get(e) * r * a.weight[i + e]);
+        v.store(c + i);
+        if (dst != nullptr) v.store(dst + i);
+    }
+}
+
+// meta [n, 4]: {destination row, source row of `src` or -1, slot, position}
+template <typename T>
+__global__ void __launch_bounds__(128) gather_rows_kernel(T* dst, long long ldd, const T* src, long long lds, Cache c, int cols,
+                                                          const int4* __restrict__ meta) {
+    constexpr int W = Vec<T>::N;
+    const int4 e = meta[blockIdx.x];
+    const T* s = e.y >= 0 ? src + e.y * lds : (const T*)c.k + c.row(e.z, e.w) * cols;
+    T* d = dst + e.x * ldd;
+    for (int i = threadIdx.x * W; i < cols; i += 128 * W) {
+        Vec<T> v;
+        v.load(s + i);
+        v.store(d + i);
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(THREADS) gate_rows_kernel(T* o, long long ldo, const T* g, long long ldg, int cols) {
+    T* orow = o + (long long)blockIdx.x * ldo;
+    const T* grow = g + (long long)blockIdx.x * ldg;
+    for (int i = threadIdx.x; i < cols; i += THREADS) orow[i] = from_f<T>(to_f(orow[i]) / (1.f + expf(-to_f(grow[i]))));
+}
+
+static bool aligned(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
+
+}  // namespace pag
+}  // namespace lmoe
+
+using namespace lmoe;
+
+// dt: 1 bf16, 0 fp32.  Work items of `tile` (32 or 16) queries at most; scale of any sign.
+LMOE_API int lmoe_packed_attn_rows(const pa::Prompt* ap, int tile, int dt, cudaStream_t st) {
+    const pa::Prompt& a = *ap;
+    if (a.n <= 0 || a.H <= 0 || a.G <= 0 || a.H % a.G || a.dk <= 0 || a.dv <= 0) return -1;
+    if (tile == 32) return dt ? pag::launch_rows<bf16, 32>(a, st) : pag::launch_rows<float, 32>(a, st);
+    if (tile == 16) return dt ? pag::launch_rows<bf16, 16>(a, st) : pag::launch_rows<float, 16>(a, st);
+    return -1;
+}
+
+LMOE_API int lmoe_packed_attn_step_any(const pa::Step* ap, int dt, cudaStream_t st) {
+    const pa::Step& a = *ap;
+    if (a.n <= 0 || a.H <= 0 || a.G <= 0 || a.H % a.G || a.dk <= 0 || a.dv <= 0 || (a.c.table == nullptr && a.c.cap <= 0)) return -1;
+    return dt ? pag::launch_step<bf16>(a, st) : pag::launch_step<float>(a, st);
+}
+
+// dk, dv, ldz and the first columns multiples of 8 (bf16) or 4 (fp32), rot even
+LMOE_API int lmoe_qk_norm_rope(const pag::QkNorm* ap, int dt, cudaStream_t st) {
+    const pag::QkNorm& a = *ap;
+    const int w = dt ? 8 : 4;
+    if (a.rows <= 0 || a.H <= 0 || a.G <= 0 || a.dk % w || a.dv % w || a.ldz % w || a.zq % w || a.zk % w || a.zv % w || a.rot % 2 || a.rot < 0 ||
+        a.rot > a.dk || a.nq <= 0 || a.nk <= 0 || !pag::aligned(a.z) || !pag::aligned(a.c.k) || !pag::aligned(a.c.v) ||
+        (a.c.k != nullptr && a.c.table == nullptr && a.c.cap <= 0) || (a.rot > 0 && a.freq == nullptr))
+        return -1;
+    const size_t smem = sizeof(float2) * (a.rot / 2);
+    if (smem > 40 * 1024) return -2;
+    if (dt) pag::qk_norm_rope_kernel<bf16><<<a.rows, pag::THREADS, smem, st>>>(a);
+    else pag::qk_norm_rope_kernel<float><<<a.rows, pag::THREADS, smem, st>>>(a);
+    return (int)cudaGetLastError();
+}
+
+LMOE_API int lmoe_latent_norm(const pag::LatentNorm* ap, int dt, cudaStream_t st) {
+    const pag::LatentNorm& a = *ap;
+    const int w = dt ? 8 : 4;
+    if (a.rows <= 0 || a.width <= 0 || a.rank <= 0 || a.width % w || a.ldz % w || a.ldc % w || !pag::aligned(a.z) || !pag::aligned(a.c) ||
+        !pag::aligned(a.cache.k) || (a.cache.k != nullptr && a.cache.table == nullptr && a.cache.cap <= 0))
+        return -1;
+    const int threads = a.width > 128 * w ? 256 : 128;
+    if (dt) pag::latent_norm_kernel<bf16><<<a.rows, threads, 0, st>>>(a);
+    else pag::latent_norm_kernel<float><<<a.rows, threads, 0, st>>>(a);
+    return (int)cudaGetLastError();
+}
+
+// cols: row length in both places; the cache rows are the request's whole rows (all kv heads)
+LMOE_API int lmoe_gather_rows(void* dst, long long ldd, const void* src, long long lds, const pa::Cache* c, int cols, const int* meta, int n,
+                              int dt, cudaStream_t st) {
+    const int w = dt ? 8 : 4;
+    if (n <= 0 || cols <= 0 || cols % w || ldd % w || lds % w || !pag::aligned(dst) || !pag::aligned(src) || !pag::aligned(meta)) return -1;
+    if (dt) pag::gather_rows_kernel<bf16><<<n, 128, 0, st>>>((bf16*)dst, ldd, (const bf16*)src, lds, *c, cols, (const int4*)meta);
+    else pag::gather_rows_kernel<float><<<n, 128, 0, st>>>((float*)dst, ldd, (const float*)src, lds, *c, cols, (const int4*)meta);
+    return (int)cudaGetLastError();
+}
+
+LMOE_API int lmoe_gate_rows(void* o, long long ldo, const void* g, long long ldg, int rows, int cols, int dt, cudaStream_t st) {
+    if (rows <= 0 || cols <= 0) return -1;
+    if (dt) pag::gate_rows_kernel<bf16><<<rows, pag::THREADS, 0, st>>>((bf16*)o, ldo, (const bf16*)g, ldg, cols);
+    else pag::gate_rows_kernel<float><<<rows, pag::THREADS, 0, st>>>((float*)o, ldo, (const float*)g, ldg, cols);
+    return (int)cudaGetLastError();
+}

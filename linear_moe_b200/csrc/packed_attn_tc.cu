@@ -1,0 +1,293 @@
+// Causal softmax attention over packed prompts on the 5th-generation tensor cores (bf16, head sizes up to 128 in multiples of 8),
+// with an optional sliding window and an optional output gate:
+//     o = sigmoid(gate) * softmax(q . k * scale) v          key j visible to query i when 0 <= i - j (< window)
+// Queries, keys and values are rows of separate matrices (packed_attn.cuh); a work item is up to 128 queries of one request.
+//
+// One CTA = one work item of one head, warp roles as in flash_attn_tc.cu and chunk_attn_tc.cu:
+//   warp 0      TMA producer: Q once, then K_j / V_j tiles of 128 keys through two 2-stage rings; only tiles inside the window
+//   warp 1      MMA issuer: S_{j+1} = Q K_{j+1}^T before O += P_j V_j
+//   warps 4..19 four warps per 32 query rows split the columns: one tensor-memory read of the scores, row maximum over the parts
+//               (shared memory and a named barrier), P = exp2(S - m), bf16 pack into the 128-byte-swizzled P tile
+// O accumulates in tensor memory over all key tiles.  The maximum a row is scaled by may lag behind the true one by LAG (in
+// units of log2), so that P stays below 2^LAG; only when a row runs ahead of that is O multiplied in tensor memory.
+// Every mbarrier wait is bounded; on expiry the error word is set and the CTA drains and frees its tensor memory.
+#include "attn_math.cuh"
+#include "flash_tc_utils.cuh"
+#include "packed_attn.cuh"
+
+namespace lmoe {
+namespace patc {
+using namespace lmoe::fatc;
+using pa::Prompt;
+
+constexpr float LAG = 8.f;
+
+template <int DQ, int DV>
+struct __align__(1024) Smem {
+    uint8_t q[BM * DQ * 2];
+    uint8_t k[2][BN * DQ * 2];
+    uint8_t v[2][BN * DV * 2];
+    uint8_t p[BM * BN * 2];
+    float mx[2][SPLIT][BM], ls[SPLIT][BM];
+    uint64_t q_full, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[2], pv_done, p_ready;
+    uint32_t tmem_base;
+    int abort_flag;
+};
+
+__device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t (&r)[16]) {
+    asm volatile("tcgen05.st.sync.aligned.32x32b.x16.b32 [%16], {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15};"
+                 :: "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]),
+                    "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(taddr) : "memory");
+}
+__device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
+
+template <int DQ, int DV>
+__global__ void __launch_bounds__(THREADS, 1)
+packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
+                      const __grid_constant__ CUtensorMap tmV, Prompt a) {
+    extern __shared__ uint8_t smem_raw[];
+    Smem<DQ, DV>& sm = *reinterpret_cast<Smem<DQ, DV>*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+    constexpr int KQ = DQ / 64, KV = DV / 64;               // 64-element blocks along the head dimensions
+    constexpr uint32_t TMEM_COLS = 512, O_COL = 2 * BN;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int* it = a.items + (long long)blockIdx.x * pa::I_N;
+    const int row0 = it[pa::I_ROW], nq = it[pa::I_NQ], c0 = it[pa::I_C0], krow = it[pa::I_KROW];
+    const int h = blockIdx.y, hk = h / (a.H / a.G);
+    const int nb_lo = a.window > 0 ? max(0, c0 - a.window + 1) / BN : 0;
+    const int n_it = (c0 + nq + BN - 1) / BN - nb_lo;       // at least 1: a query sees its own key
+    volatile int* abort_flag = &sm.abort_flag;
+    int* err = a.err;
+
+    if (threadIdx.x == 0) {
+        mbar_init(&sm.q_full, 1);
+        for (int s = 0; s < 2; ++s) {
+            mbar_init(&sm.k_full[s], 1); mbar_init(&sm.k_empty[s], 1);
+            mbar_init(&sm.v_full[s], 1); mbar_init(&sm.v_empty[s], 1);
+            mbar_init(&sm.s_full[s], 1);
+        }
+        mbar_init(&sm.pv_done, 1);
+        mbar_init(&sm.p_ready, 4 * SPLIT);
+        sm.abort_flag = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    if (warp == 1) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" :: "r"(s32(&sm.tmem_base)), "r"(TMEM_COLS) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem_base = sm.tmem_base;
+
+    if (warp == 0) {
+        if (lane == 0) {
+            mbar_expect_tx(&sm.q_full, BM * DQ * 2);
+#pragma unroll
+            for (int kb = 0; kb < KQ; ++kb) tma_load_4d(sm.q + kb * BM * 128, &tmQ, &sm.q_full, kb * 64, h, row0, 0);
+            for (int j = 0; j < n_it; ++j) {
+                const int s = j & 1;
+                const uint32_t ph = (j >> 1) & 1;
+                const int key0 = krow + (nb_lo + j) * BN;
+                if (!mbar_wait_suspend(&sm.k_empty[s], ph ^ 1, abort_flag, err, 0x7100 | s)) break;
+                mbar_expect_tx(&sm.k_full[s], BN * DQ * 2);
+#pragma unroll
+                for (int kb = 0; kb < KQ; ++kb) tma_load_4d(sm.k[s] + kb * BN * 128, &tmK, &sm.k_full[s], kb * 64, hk, key0, 0);
+                if (!mbar_wait_suspend(&sm.v_empty[s], ph ^ 1, abort_flag, err, 0x7200 | s)) break;
+                mbar_expect_tx(&sm.v_full[s], BN * DV * 2);
+#pragma unroll
+                for (int kk = 0; kk < BN / 64; ++kk)        // MN-major operand: per 64 keys, DV/64 boxes of {64 d, 64 keys}
+#pragma unroll
+                    for (int nb = 0; nb < KV; ++nb)
+                        tma_load_4d(sm.v[s] + (kk * KV + nb) * 8192, &tmV, &sm.v_full[s], nb * 64, hk, key0 + kk * 64, 0);
+            }
+        }
+    } else if (warp == 1) {
+        const uint32_t issue = lane == 0 ? 1u : 0u;
+        constexpr uint32_t idesc_s = idesc_bf16<false, BN>();
+        constexpr uint32_t idesc_o = idesc_bf16<true, DV>();
+        bool ok = mbar_wait_suspend(&sm.q_full, 0, abort_flag, err, 0x8000);
+        auto issue_s = [&](int j) -> bool {
+            const int s = j & 1;
+            if (!mbar_wait_suspend(&sm.k_full[s], (j >> 1) & 1, abort_flag, err, 0x8100 | s)) return false;
+            tc_fence_after();
+            const uint32_t ql = desc_lo<false>(s32(sm.q)), kl = desc_lo<false>(s32(sm.k[s]));
+#pragma unroll
+            for (int kk = 0; kk < DQ / UMMA_K; ++kk) {
+                const uint32_t off = ((kk / 4) * (BM * 128) + (kk % 4) * 32) >> 4;
+                umma_lo(tmem_base + s * BN, ql + off, kl + off, idesc_s, kk > 0 ? 1u : 0u, issue);
+            }
+            umma_commit_if(&sm.k_empty[s], issue);
+            umma_commit_if(&sm.s_full[s], issue);
+            return true;
+        };
+        if (ok) ok = issue_s(0);
+        for (int j = 0; ok && j < n_it; ++j) {
+            // score buffer (j + 1) & 1 was last read for P_{j-1}, whose p_ready was waited for in the previous iteration
+            if (j + 1 < n_it) { ok = issue_s(j + 1); if (!ok) break; }
+            const int s = j & 1;
+            if (!mbar_wait_suspend(&sm.v_full[s], (j >> 1) & 1, abort_flag, err, 0x8200 | s)) break;
+            if (!mbar_wait_suspend(&sm.p_ready, j & 1, abort_flag, err, 0x8300)) break;
+            tc_fence_after();
+            const uint32_t pl = desc_lo<false>(s32(sm.p)), vl = desc_lo<true>(s32(sm.v[s]));
+#pragma unroll
+            for (int kk = 0; kk < BN / UMMA_K; ++kk) {
+                const uint32_t aoff = ((kk / 4) * (BM * 128) + (kk % 4) * 32) >> 4;
+                const uint32_t boff = ((kk / 4) * (KV * 8192) + (kk % 4) * 2048) >> 4;
+                umma_lo(tmem_base + O_COL, pl + aoff, vl + boff, idesc_o, (j > 0 || kk > 0) ? 1u : 0u, issue);
+            }
+            umma_commit_if(&sm.v_empty[s], issue);
+            umma_commit_if(&sm.pv_done, issue);
+        }
+    } else if (warp >= 4) {
+        const int qd = warp & 3, part = (warp - 4) >> 2;
+        const int r = qd * 32 + lane;                         // query row inside the tile
+        const uint32_t lane_addr = tmem_base + ((uint32_t)(qd * 32) << 16);
+        constexpr int CW = BN / SPLIT, OW = DV / SPLIT;       // score / output columns of this thread
+        static_assert(CW == 32 && OW % 16 == 0, "tensor-memory load widths");
+        const float sc = a.scale * LOG2E, lag = LAG / sc;
+        uint8_t* prow = sm.p + ((part * CW) >> 6) * (BM * 128) + (r >> 3) * 1024 + (r & 7) * 128;
+        const int ch0 = ((part * CW) & 63) >> 3;
+        float m = -INFINITY, l = 0.f;
+        bool alive = true;
+        for (int j = 0; j < n_it; ++j) {
+            const int s = j & 1, tile0 = (nb_lo + j) * BN;
+            if (!mbar_wait_suspend(&sm.s_full[s], (j >> 1) & 1, abort_flag, err, 0x9100 | s)) { alive = false; break; }
+            tc_fence_after();
+            uint32_t v[CW];
+            tmem_ld32(lane_addr + s * BN + part * CW, v);
+            tmem_ld_wait();
+            if (tile0 + BN - 1 > c0 || (a.window > 0 && tile0 <= c0 + BM - 1 - a.window)) {
+                const int hi = c0 + r - (tile0 + part * CW);  // columns up to hi are not in the future
+                const int lo = a.window > 0 ? hi - a.window : -1;
+#pragma unroll
+                for (int c = 0; c < CW; ++c)
+                    if (c > hi || c <= lo) v[c] = 0xff800000u;                  // -inf
+            }
+            float mx4[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                mx4[e] = fmaxf(__uint_as_float(v[e]), __uint_as_float(v[e + 4]));
+#pragma unroll
+                for (int c = 8; c < CW; c += 8) mx4[e] = max3(mx4[e], __uint_as_float(v[c + e]), __uint_as_float(v[c + e + 4]));
+            }
+            sm.mx[s][part][r] = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
+            asm volatile("bar.sync %0, %1;" :: "r"(1 + qd), "n"(32 * SPLIT) : "memory");
+            float mx = sm.mx[s][0][r];
+#pragma unroll
+            for (int p = 1; p < SPLIT; ++p) mx = fmaxf(mx, sm.mx[s][p][r]);
+            // the four parts of a row see the same numbers and decide alike
+            const bool grow = mx > m + lag;                   // also the first visible key of the row (m = -inf)
+            const bool scaled = grow && m != -INFINITY;
+            const float corr = scaled ? ex2((m - mx) * sc) : 1.f;
+            if (grow) m = mx;
+            l *= corr;
+            if (__any_sync(0xffffffffu, scaled)) {            // not before tile 1: O holds something
+                if (!mbar_wait_suspend(&sm.pv_done, (j - 1) & 1, abort_flag, err, 0x9200)) { alive = false; break; }
+                tc_fence_after();
+#pragma unroll
+                for (int c = 0; c < OW; c += 16) {
+                    uint32_t o[16];
+                    tmem_ld16(lane_addr + O_COL + part * OW + c, o);
+                    tmem_ld_wait();
+#pragma unroll
+                    for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * corr);
+                    tmem_st16(lane_addr + O_COL + part * OW + c, o);
+                }
+                tmem_st_wait();
+            }
+            const float nm = m == -INFINITY ? 0.f : -m * sc;
+            const float2 sc2 = make_float2(sc, sc), nm2 = make_float2(nm, nm);
+            float2 sum0 = make_float2(0.f, 0.f), sum1 = make_float2(0.f, 0.f);
+#pragma unroll
+            for (int c = 0; c < CW; c += 4) {
+                const float2 x01 = __ffma2_rn(make_float2(__uint_as_float(v[c]), __uint_as_float(v[c + 1])), sc2, nm2);
+                const float2 x23 = __ffma2_rn(make_float2(__uint_as_float(v[c + 2]), __uint_as_float(v[c + 3])), sc2, nm2);
+                const float p0 = ex2(x01.x), p1 = ex2(x01.y), p2 = ex2(x23.x), p3 = ex2(x23.y);
+                sum0 = __fadd2_rn(sum0, make_float2(p0, p1));
+                sum1 = __fadd2_rn(sum1, make_float2(p2, p3));
+                v[c >> 1] = pack_bf16(p0, p1);
+                v[(c >> 1) + 1] = pack_bf16(p2, p3);
+            }
+            l += (sum0.x + sum0.y) + (sum1.x + sum1.y);
+            // the P tile is free once O += P_{j-1} V_{j-1} has completed
+            if (j > 0 && !mbar_wait_suspend(&sm.pv_done, (j - 1) & 1, abort_flag, err, 0x9300)) { alive = false; break; }
+#pragma unroll
+            for (int c = 0; c < 4; ++c)
+                *reinterpret_cast<uint4*>(prow + (((ch0 + c) ^ (r & 7)) << 4)) = make_uint4(v[4 * c], v[4 * c + 1], v[4 * c + 2], v[4 * c + 3]);
+            tc_fence_before();
+            asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&sm.p_ready);
+        }
+        if (alive) alive = mbar_wait_suspend(&sm.pv_done, (n_it - 1) & 1, abort_flag, err, 0x9400);
+        tc_fence_after();
+        sm.ls[part][r] = l;
+        asm volatile("bar.sync %0, %1;" :: "r"(1 + qd), "n"(32 * SPLIT) : "memory");
+        l = 0.f;
+#pragma unroll
+        for (int p = 0; p < SPLIT; ++p) l += sm.ls[p][r];
+        uint32_t o[OW];
+        tmem_ld<OW>(lane_addr + O_COL + part * OW, o);
+        tmem_ld_wait();
+        if (alive && r < nq) {
+            const float w = 1.f / l;
+            const long long row = row0 + r;
+            const bf16* gp = a.gate == nullptr ? nullptr : (const bf16*)a.gate + row * a.ldg + h * a.dv;
+            bf16* op = (bf16*)a.out + row * a.ldo + h * a.dv;
+#pragma unroll
+            for (int c = 0; c < OW; c += 8) {
+                const int col = part * OW + c;
+                if (col < a.dv) {
+                    Vec<bf16> g, y;
+                    if (gp != nullptr) g.load(gp + col);
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) {
+                        const float x = __uint_as_float(o[c + i]) * w;
+                        y.set(i, gp != nullptr ? x * rcp(1.f + ex2(-LOG2E * g.get(i))) : x);
+                    }
+                    y.store(op + col);
+                }
+            }
+        }
+    }
+    tc_fence_before();
+    __syncthreads();
+    if (warp == 1) {
+        tc_fence_after();
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" :: "r"(tmem_base), "r"(TMEM_COLS) : "memory");
+    }
+}
+
+template <int DQ, int DV>
+static int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const Prompt& a, cudaStream_t st) {
+    const size_t smem = sizeof(Smem<DQ, DV>) + 1024;
+    static_assert(sizeof(Smem<DQ, DV>) + 1024 <= 227 * 1024, "shared memory of one CTA");
+    cudaError_t e = cudaFuncSetAttribute(packed_attn_tc_kernel<DQ, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    packed_attn_tc_kernel<DQ, DV><<<dim3(a.n, a.H), THREADS, smem, st>>>(mq, mk, mv, a);
+    return (int)cudaGetLastError();
+}
+
+}  // namespace patc
+}  // namespace lmoe
+
+using namespace lmoe;
+
+// bf16; q [q_rows, ldq], k / v [k_rows, ldk / ldv], gate [q_rows, ldg] or null: bases 16-byte aligned, pitches and head sizes
+// multiples of 8, head sizes up to 128, scale > 0.  items: up to 128 queries each; every row they name lies inside the matrices.
+LMOE_API int lmoe_packed_attn_tc(const pa::Prompt* ap, cudaStream_t st) {
+    using namespace lmoe::patc;
+    const Prompt& a = *ap;
+    if (a.n <= 0 || a.q_rows <= 0 || a.k_rows <= 0 || a.H <= 0 || a.G <= 0 || a.H % a.G || a.dk <= 0 || a.dk > 128 || a.dv <= 0 || a.dv > 128 ||
+        a.dk % 8 || a.dv % 8 || a.ldq % 8 || a.ldk % 8 || a.ldv % 8 || a.ldo % 8 || (a.gate != nullptr && a.ldg % 8) || !(a.scale > 0.f) ||
+        ((reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.k) | reinterpret_cast<uintptr_t>(a.v) |
+          reinterpret_cast<uintptr_t>(a.gate) | reinterpret_cast<uintptr_t>(a.out)) & 15))
+        return -1;
+    CUtensorMap mq, mk, mv;
+    int rc = make_map_4d(&mq, a.q, 1, a.q_rows, a.H, a.dk, (long long)a.q_rows * a.ldq, a.ldq, a.dk, BM);
+    if (rc == 0) rc = make_map_4d(&mk, a.k, 1, a.k_rows, a.G, a.dk, (long long)a.k_rows * a.ldk, a.ldk, a.dk, BN);
+    if (rc == 0) rc = make_map_4d(&mv, a.v, 1, a.k_rows, a.G, a.dv, (long long)a.k_rows * a.ldv, a.ldv, a.dv, 64);
+    if (rc) return rc;
+    if (a.dk <= 64) return a.dv <= 64 ? launch<64, 64>(mq, mk, mv, a, st) : launch<64, 128>(mq, mk, mv, a, st);
+    return a.dv <= 64 ? launch<128, 64>(mq, mk, mv, a, st) : launch<128, 128>(mq, mk, mv, a, st);
+}

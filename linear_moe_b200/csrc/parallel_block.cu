@@ -1,8 +1,9 @@
 // Row kernels of blocks whose mixer and feed-forward read the same fp32 residual stream and add into it together:
 //   stream_norm        y = x / rms(x) [* gain]: the fp32 stream -> the input of the block's fused projection (bf16 or fp32).  A
 //                      one-number norm gain is a scalar on the projection's outputs, so two norms of the same stream
-//                      need one pass and one matrix product; the consumers of the projection apply their gain.
-//   embed_norm         x = embedding[token] + position table[position], in fp32, together with the first block's norm
+//                      need one pass and one matrix product; the consumers of the projection apply their gain.  A gain with
+//                      one number per column (gain_n > 1, padded like x) is applied here.
+//   embed_norm         x = embedding[token] [+ position table[position]], in fp32, together with the first block's norm
 //   poly_norm          sum over p = 1, 2, 3 of w_p u^p / rms(u^p), plus w_4 (element-wise powers, rms over the row)
 // Rows are padded (stream and activations to a multiple of 32 elements, pad = 0), so that every product is aligned for TMA.
 // Compiled without fast-math: the same code serves the fp32 model.
@@ -26,7 +27,7 @@ __device__ __forceinline__ void store4(bf16* y, float4 v) {
 // x [rows, ldx] fp32, y [rows, ldy]; columns width .. pad of x hold zeros, and y gets zeros there
 template <typename T>
 __global__ void __launch_bounds__(THREADS) stream_norm_kernel(const float* __restrict__ x, long long ldx, T* __restrict__ y,
-                                                              long long ldy, int width, int pad, float eps, const float* gain) {
+                                                              long long ldy, int width, int pad, float eps, const float* gain, int gain_n) {
     pdl_trigger();
     __shared__ float red[32];
     const float* xr = x + (long long)blockIdx.x * ldx;
@@ -44,23 +45,24 @@ __global__ void __launch_bounds__(THREADS) stream_norm_kernel(const float* __res
         const float4 t = *reinterpret_cast<const float4*>(xr + c);
         s += t.x * t.x + t.y * t.y + t.z * t.z + t.w * t.w;
     }
-    const float r = (gain == nullptr ? 1.f : *gain) / sqrtf(block_sum(s, red) / width + eps);
+    const float r = (gain_n == 1 ? *gain : 1.f) / sqrtf(block_sum(s, red) / width + eps);
+    auto put = [&](int c, float4 t) {
+        const float4 g = gain_n > 1 ? *reinterpret_cast<const float4*>(gain + c) : make_float4(1.f, 1.f, 1.f, 1.f);
+        store4(yr + c, make_float4(t.x * r * g.x, t.y * r * g.y, t.z * r * g.z, t.w * r * g.w));
+    };
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
         const int c = (threadIdx.x + i * THREADS) * 4;
-        if (c < pad) store4(yr + c, make_float4(v[i].x * r, v[i].y * r, v[i].z * r, v[i].w * r));
+        if (c < pad) put(c, v[i]);
     }
-    for (int c = (threadIdx.x + NV * THREADS) * 4; c < pad; c += THREADS * 4) {
-        const float4 t = *reinterpret_cast<const float4*>(xr + c);
-        store4(yr + c, make_float4(t.x * r, t.y * r, t.z * r, t.w * r));
-    }
+    for (int c = (threadIdx.x + NV * THREADS) * 4; c < pad; c += THREADS * 4) put(c, *reinterpret_cast<const float4*>(xr + c));
 }
 
 template <typename T>
 __global__ void __launch_bounds__(THREADS) embed_norm_kernel(const long long* __restrict__ ids, const int* __restrict__ pos,
                                                              const T* __restrict__ emb, const T* __restrict__ ptab, float* __restrict__ x,
                                                              long long ldx, T* __restrict__ y, long long ldy, int width, int pad,
-                                                             int vocab, int npos, float eps) {
+                                                             int vocab, int npos, float eps, const float* gain) {
     pdl_trigger();
     __shared__ float red[32];
     // ids and positions are checked on the host; the clamp keeps a bad one from becoming a bad address
@@ -77,7 +79,7 @@ __global__ void __launch_bounds__(THREADS) embed_norm_kernel(const long long* __
         s += v * v;
     }
     const float r = 1.f / sqrtf(block_sum(s, red) / width + eps);
-    for (int c = threadIdx.x; c < pad; c += THREADS) yr[c] = from_f<T>(xr[c] * r);
+    for (int c = threadIdx.x; c < pad; c += THREADS) yr[c] = from_f<T>(gain == nullptr ? xr[c] * r : xr[c] * r * gain[c]);
 }
 
 // z [rows, ldz] -> out [rows, ldo]; gain: the norm gain of the projection's input; act = {w_1, w_2, w_3, w_4}; out *= mul.
@@ -138,24 +140,27 @@ __global__ void __launch_bounds__(THREADS) poly_norm_kernel(const T* __restrict_
 
 using namespace lmoe;
 
-// x [rows, ldx] fp32 with zeros in columns width .. pad; y bf16 (dt 1) or fp32 (dt 0); pad a multiple of 4, 16-byte rows; gain: one
-// float or null
+// x [rows, ldx] fp32 with zeros in columns width .. pad; y bf16 (dt 1) or fp32 (dt 0); pad a multiple of 4, 16-byte rows; gain: null
+// (gain_n 0), one float (gain_n 1) or pad floats (gain_n pad)
 LMOE_API int lmoe_stream_norm(const float* x, long long ldx, void* y, long long ldy, int rows, int width, int pad, float eps,
-                              const float* gain, int dt, cudaStream_t st) {
-    if (rows <= 0 || width <= 0 || pad < width || pad % 4 || ldx % 4 || ldy % 4) return -1;
-    if (dt) pb::stream_norm_kernel<bf16><<<rows, pb::THREADS, 0, st>>>(x, ldx, (bf16*)y, ldy, width, pad, eps, gain);
-    else pb::stream_norm_kernel<float><<<rows, pb::THREADS, 0, st>>>(x, ldx, (float*)y, ldy, width, pad, eps, gain);
+                              const float* gain, int gain_n, int dt, cudaStream_t st) {
+    if (rows <= 0 || width <= 0 || pad < width || pad % 4 || ldx % 4 || ldy % 4 || (gain_n != 0 && gain_n != 1 && gain_n != pad) ||
+        (gain_n != 0) != (gain != nullptr) || (gain_n > 1 && (reinterpret_cast<uintptr_t>(gain) & 15)))
+        return -1;
+    if (dt) pb::stream_norm_kernel<bf16><<<rows, pb::THREADS, 0, st>>>(x, ldx, (bf16*)y, ldy, width, pad, eps, gain, gain_n);
+    else pb::stream_norm_kernel<float><<<rows, pb::THREADS, 0, st>>>(x, ldx, (float*)y, ldy, width, pad, eps, gain, gain_n);
     return (int)cudaGetLastError();
 }
 
-// emb [vocab, width], ptab [npos, width] or null, in the model's dtype; ids int64, pos int32
+// emb [vocab, width], ptab [npos, width] or null, in the model's dtype; ids int64, pos int32; gain [pad] or null
 LMOE_API int lmoe_embed_norm(const long long* ids, const int* pos, const void* emb, const void* ptab, float* x, long long ldx, void* y,
-                             long long ldy, int rows, int width, int pad, int vocab, int npos, float eps, int dt, cudaStream_t st) {
+                             long long ldy, int rows, int width, int pad, int vocab, int npos, float eps, const float* gain, int dt,
+                             cudaStream_t st) {
     if (rows <= 0 || width <= 0 || pad < width || vocab <= 0 || (ptab != nullptr && npos <= 0)) return -1;
     if (dt) pb::embed_norm_kernel<bf16><<<rows, pb::THREADS, 0, st>>>(ids, pos, (const bf16*)emb, (const bf16*)ptab, x, ldx, (bf16*)y,
-                                                                      ldy, width, pad, vocab, npos, eps);
+                                                                      ldy, width, pad, vocab, npos, eps, gain);
     else pb::embed_norm_kernel<float><<<rows, pb::THREADS, 0, st>>>(ids, pos, (const float*)emb, (const float*)ptab, x, ldx, (float*)y,
-                                                                    ldy, width, pad, vocab, npos, eps);
+                                                                    ldy, width, pad, vocab, npos, eps, gain);
     return (int)cudaGetLastError();
 }
 

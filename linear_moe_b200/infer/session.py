@@ -1,5 +1,5 @@
 """The step function of models that run packed rows: requests start together from whole prompts, then go on one token at a
-time, each from its own position, with their keys and values in a ``SlotCache``.  Generation (``generation.generate_tokens``)
+time, each from its own position, with what the layers keep of them in a ``SlotCache``.  Generation (``generation.generate_tokens``)
 and trace replay (``infer/trace.py``) both drive this class."""
 from __future__ import annotations
 
@@ -7,19 +7,19 @@ from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
 
-from ..ops.chunk_attn import RowBatch
+from ..ops.row_batch import RowBatch
 from .generation import GraphedDecodeStep
 
 
 class InferenceSession:
     """``cuda_graph``: replay one-token steps from a CUDA graph per batch size (the first two steps of a size run eagerly and
-    warm up the kernels)."""
+    warm up the kernels).  ``slots`` / ``tokens``: requests and tokens to make room for from the start (the cache grows)."""
 
-    def __init__(self, model, slots: int = 1, cuda_graph: bool = False):
+    def __init__(self, model, slots: int = 1, cuda_graph: bool = False, tokens: int = 0):
         assert getattr(model, "packed_rows", False), "this model has no packed-row step"
         self.model = model.eval()
         self.device = next(model.parameters()).device
-        self.cache = model.new_cache(slots)
+        self.cache = model.new_cache(slots, tokens)
         self.limit = model.cfg.max_position_embeddings
         self.cuda_graph = cuda_graph and GraphedDecodeStep.supported(model, self.cache, self.device)
         self._graphs: Dict[int, GraphedDecodeStep] = {}
@@ -42,12 +42,13 @@ class InferenceSession:
         starts = [self.cache.lengths[s] for s in slots]
         counts = [int(t.numel()) for t in tokens]
         self._check(tokens, [s + c for s, c in zip(starts, counts)])
-        batch = RowBatch(starts, counts, slots, self.device)
         if want is None:
             want = [[c - 1] for c in counts]
         for w, c in zip(want, counts):
             if any(not 0 <= i < c for i in w):
                 raise ValueError("a wanted place is outside the request's new tokens")
+        batch = RowBatch(starts, counts, slots, self.device)
+        self.cache.reserve(slots, [s + c for s, c in zip(starts, counts)])
         rows = [batch.row0[r] + i for r, w in enumerate(want) for i in w]
         ids = torch.cat([t.reshape(-1) for t in tokens]).to(device=self.device, dtype=torch.long)
         pick = torch.tensor(rows or [0], device=self.device)           # the head runs on the wanted rows only
@@ -74,6 +75,7 @@ class InferenceSession:
         if len(set(slots)) != B or int(tokens.numel()) != B:
             raise ValueError("one token per slot, each slot once")
         if self.cuda_graph:
+            self.cache.reserve(slots, [self.cache.lengths[s] + 1 for s in slots])
             if self._graph_generation != self.cache.generation:        # the buffers have moved
                 self._graphs, self._seen, self._graph_generation, self._loaded = {}, {}, self.cache.generation, None
             self._seen[B] = self._seen.get(B, 0) + 1

@@ -52,7 +52,7 @@ def main(argv=None) -> int:
     ap.add_argument("--model", required=True, help="folder with config.json and model.safetensors")
     ap.add_argument("--dtype", required=True, choices=["bfloat16", "float32"])
     ap.add_argument("--out", required=True, help="where the logits go")
-    ap.add_argument("--max-tokens", type=int, default=0, help="upper bound of the tokens in the cache (accepted; slots grow on demand)")
+    ap.add_argument("--max-tokens", type=int, default=0, help="the most tokens that live requests hold (sizes the cache, which grows on demand)")
     ap.add_argument("--cuda-graph", action="store_true", help="replay one-token steps from CUDA graphs")
     a = ap.parse_args(argv)
     import torch
@@ -63,8 +63,7 @@ def main(argv=None) -> int:
     from ..ops import gemm
     from .session import InferenceSession
     model = load_model(a.model, getattr(torch, a.dtype), torch.device("cuda", 0))
-    # slots are sized by the layers' chunks, not by the context, and grow with the number of live requests
-    session = InferenceSession(model, slots=4, cuda_graph=a.cuda_graph)
+    session = InferenceSession(model, slots=4, cuda_graph=a.cuda_graph, tokens=min(max(a.max_tokens, 0), 1 << 20))
 
     def done(text):
         gemm.check_error()

@@ -1,0 +1,94 @@
+"""Forward pass and cache of models that run packed rows: the tokens of a batch's requests are consecutive rows of an fp32 residual
+stream, and every block works on all of them (``ops.row_batch.RowBatch`` says which row is which request and position).
+
+A block of such a model has
+
+    input_gain()                     weight of the norm in front of it (``None``: plain unit-RMS rows)
+    cache_spec(limit)                what it keeps per request (``infer.kv_cache``), for positions below ``limit``
+    forward(x, h, step, nxt)         ``x`` the stream, updated in place; ``h`` its normed rows; returns the normed rows for the
+                                     block ``nxt`` (``None`` behind the last one)
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass, field
+from typing import Callable, Dict, Optional, Tuple
+
+import torch
+import torch.nn as nn
+
+from .. import ops
+from ..infer.kv_cache import SlotCache
+from ..ops.row_batch import RowBatch, round_up
+
+ROW_PAD = 32                  # stream and activation rows are padded to this many elements (weight-streaming and TMA alignment)
+
+
+@dataclass
+class RowStep:
+    """What the blocks share during one call."""
+    batch: RowBatch
+    caches: Optional[SlotCache]
+    latents: Dict[int, torch.Tensor] = field(default_factory=dict)    # layer -> latent rows, for the layers that borrow them
+
+    def cache(self, layer: int) -> Optional[dict]:
+        return None if self.caches is None else self.caches[layer]
+
+
+class RowBlock(nn.Module):
+    """A block of such a model.  ``places()`` maps the checkpoint's tensor names (without the layer) to views inside the block's
+    parameters and the tensors' shapes; weights may be stored fused and padded."""
+
+    def places(self) -> Dict[str, Tuple[torch.Tensor, Tuple[int, ...]]]:
+        raise NotImplementedError
+
+    @torch.no_grad()
+    def load(self, get: Callable[[str], torch.Tensor]):
+        for name, (view, shape) in self.places().items():
+            t = get(name)
+            if tuple(t.shape) != tuple(shape):
+                raise ValueError(f"{name}: shape {tuple(t.shape)}, the configuration asks for {tuple(shape)}")
+            view.copy_(t.reshape(view.shape))
+
+
+def new_slot_cache(model, slots: int = 1, tokens: int = 0) -> SlotCache:
+    limit = model.cfg.max_position_embeddings
+    p = model.embedding.word_embeddings.weight
+    return SlotCache([b.cache_spec(limit) for b in model.decoder.layers], slots, p.device, p.dtype, tokens)
+
+
+def forward_rows(model, input_ids, labels, caches, position_offset: int, batch: Optional[RowBatch], logit_rows, return_hidden: bool):
+    """With ``batch``: packed tokens in, one row per token (or per entry of ``logit_rows``) out.  Without: ``input_ids [B, T]``, all
+    rows at ``position_offset``, ``[B, T, ...]`` out."""
+    cfg, rect = model.cfg, None
+    if batch is None:
+        rect = B, T = input_ids.shape
+        slots = None
+        if caches is not None:                                      # request b in slot b
+            missing = [s for s in range(B) if s not in caches.lengths]
+            if missing:
+                caches.acquire(len(missing))
+            slots = list(range(B))
+            caches.reserve(slots, [position_offset + T] * B)
+        batch = RowBatch([position_offset] * B, [T] * B, slots, input_ids.device)
+    if batch.reach() > cfg.max_position_embeddings:
+        raise ValueError(f"position {batch.reach() - 1} is beyond the model's table of {cfg.max_position_embeddings} positions")
+    emb, w, blocks = model.embedding, cfg.hidden_size, model.decoder.layers
+    pos = getattr(emb, "position_embeddings", None)
+    x, h = ops.embed_norm(input_ids.reshape(-1), batch.pos, emb.word_embeddings.weight, None if pos is None else pos.weight,
+                          round_up(w, ROW_PAD), cfg.norm_eps, blocks[0].input_gain())
+    taps = getattr(model, "residual_taps", None)                    # a list here receives the stream after every layer
+    step, dtype = RowStep(batch, caches), h.dtype
+    for blk, nxt in zip(blocks, [*blocks[1:], None]):
+        h = blk(x, h, step, nxt)
+        if taps is not None:
+            taps.append(x[:, :w].clone())
+    if logit_rows is not None:
+        x = x.index_select(0, logit_rows)
+    h = ops.stream_norm(x, w, cfg.norm_eps, dtype, model.decoder.final_layernorm.weight)[:, :w]
+    shape = rect if (rect is not None and logit_rows is None) else (h.shape[0],)
+    if return_hidden:
+        return h.reshape(*shape, w)
+    if labels is not None:
+        return model.output_layer(h.reshape(*shape, w), labels)
+    out = model.output_layer.weight
+    return ops.linear_f32(h, out).reshape(*shape, out.shape[0])

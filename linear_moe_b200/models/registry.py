@@ -15,7 +15,11 @@ import torch
 from ..ckpt.safetensors_io import read_header, read_tensors
 from ..config.model_config import ModelConfig
 from ..ops.chunk_attn import ChunkAttnSpec
+from ..ops.moe_rows import ExpertsSpec
+from ..ops.packed_attn import AttentionSpec, LatentSpec
 from .transformer import CausalLM
+
+UNBOUNDED = 1 << 30           # positions of a model without a position table
 
 
 @dataclass(frozen=True)
@@ -85,18 +89,66 @@ def _lagisun_config(raw: dict, shapes: Dict[str, Tuple[int, ...]]) -> ModelConfi
                        ffn_hidden_size=first["ff"] or 0)
 
 
-@torch.no_grad()
 def _lagisun_load(model: CausalLM, tensors: Dict[str, torch.Tensor]):
-    whole = {"embed": model.embedding.word_embeddings.weight, "pos": model.embedding.position_embeddings.weight,
-             "final.norm": model.decoder.final_layernorm.weight, "head": model.output_layer.weight}
+    _load_rows(model, tensors, {"pos": model.embedding.position_embeddings.weight})
+
+
+register(Architecture("Lagisun", _lagisun_config, _lagisun_load, "parallel_block"))
+
+
+# ---------------------------------------------------------------------------------------------------------------- Sonodra
+def _sonodra_mixer(i: int, layers: list):
+    kind, m = layers[i]["type"], layers[i]["mixer"]
+    if kind == "attention":
+        rot, mask = m.get("rot"), m.get("mask")
+        return AttentionSpec(heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"], scale=m["scale"], qk_norm=True,
+                             window=None if mask is None else mask["size"], rot_dims=0 if rot is None else rot["dims"],
+                             rot_base=1.0 if rot is None else rot["base"])
+    if kind == "latent_attention":
+        j = m.get("kv_from")
+        if j is not None:
+            lender = layers[j] if 0 <= j < i else {"type": None}
+            if lender["type"] != kind or lender["mixer"].get("kv_from") is not None or lender["mixer"]["kv_rank"] != m["kv_rank"]:
+                raise ValueError(f"layer {i}: takes the latents of layer {j}, which is no earlier layer with latents of its own and the same kv_rank")
+        return LatentSpec(heads=m["heads"], dim=m["dim"], vdim=m["vdim"], rank=m["kv_rank"], scale=m["scale"], source=j)
+    raise ValueError(f"layer {i}: unknown mixer {kind!r}")
+
+
+def _sonodra_config(raw: dict, shapes: Dict[str, Tuple[int, ...]]) -> ModelConfig:
+    layers = []
+    for i, l in enumerate(raw["layers"]):
+        mlp, ff = l.get("mlp"), None
+        if mlp is not None and mlp["kind"] == "dense":
+            ff = mlp["ff"]
+        elif mlp is not None and mlp["kind"] == "moe":
+            ff = ExpertsSpec(mlp["router"]["experts"], mlp["router"]["top"], mlp["expert"]["ff"])
+        elif mlp is not None:
+            raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+        layers.append({"mixer": _sonodra_mixer(i, raw["layers"]), "ff": ff})
+    first = layers[0]["mixer"]
+    return ModelConfig(base_model="sonodra", layers=tuple(layers), hidden_size=raw["width"], vocab_size=raw["vocab"], norm_eps=raw["norm"]["eps"],
+                       max_position_embeddings=UNBOUNDED, num_attention_heads=first.heads, kv_channels=first.dim)
+
+
+def _sonodra_load(model: CausalLM, tensors: Dict[str, torch.Tensor]):
+    _load_rows(model, tensors, {})
+
+
+@torch.no_grad()
+def _load_rows(model: CausalLM, tensors: Dict[str, torch.Tensor], more: Dict[str, torch.Tensor]):
+    """Tensors of a packed-row model: ``embed``, ``final.norm``, ``head``, those in ``more``, and every layer's under ``l<i>.``."""
+    norm = model.decoder.final_layernorm.weight
+    if norm.dim():                                                  # padded rows: nothing behind the width
+        norm.zero_()
+        norm = norm[:model.cfg.hidden_size]
+    whole = {"embed": model.embedding.word_embeddings.weight, "final.norm": norm, "head": model.output_layer.weight, **more}
     for name, dst in whole.items():
         t = tensors[name]
         if t.shape != dst.shape:
             raise ValueError(f"{name}: shape {tuple(t.shape)}, the configuration asks for {tuple(dst.shape)}")
         dst.copy_(t)
     for i, blk in enumerate(model.decoder.layers):
-        for part in blk.parts():
-            blk.load_part(part, tensors[f"l{i}.{part}"])
+        blk.load(lambda name: tensors[f"l{i}.{name}"])
 
 
-register(Architecture("Lagisun", _lagisun_config, _lagisun_load, "parallel_block"))
+register(Architecture("Sonodra", _sonodra_config, _sonodra_load, "sandwich_block"))

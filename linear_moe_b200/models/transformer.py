@@ -6,7 +6,7 @@ One model class serves every family of the reference: ``GPTModel`` (softmax atte
 hybrid_model.py:28-248, hybrid_transformer_block.py:87-474, sequence_modeling/ssm.py:73-250,
 mamba2/mamba_model.py:16-209 — for the four backbones (qwen2, llama3, mixtral, deepseek_v2), which
 differ only in configuration (attention kind, router order, shared expert, biases).  Layer-list designs (``ModelConfig.layers``)
-build ``ParallelBlock`` (models/parallel_block.py) instead of ``Block``.
+build ``ParallelBlock`` (models/parallel_block.py) or ``SandwichBlock`` (models/sandwich_block.py) instead of ``Block``.
 
 A ``Block`` is one pre-norm residual layer: optional token mixer, optional FFN
 (transformer_layer.py:179-273, mamba_layer.py:27-80).  Module names follow the Megatron-Core
@@ -36,7 +36,9 @@ from .lsm_layers import LinearAttention, LinearRNN
 from .mamba2 import MambaMixer
 from .moe import MLP, MoELayer
 from .mom import MomLinearAttention
-from .parallel_block import ParallelBlock, forward_rows, new_slot_cache
+from .packed_rows import ROW_PAD, forward_rows, new_slot_cache
+from .parallel_block import ParallelBlock
+from .sandwich_block import SandwichBlock
 
 
 class Norm(nn.Module):
@@ -78,6 +80,14 @@ def build_mixer(cfg: ModelConfig, spec: LayerSpec, mesh: Mesh, key: str, sp: boo
             return MomLinearAttention(cfg, mesh, n, key, sp, device)
         return LinearAttention(cfg, mesh, n, key, sp, device)
     raise ValueError(spec.mixer)
+
+
+def build_block(cfg: ModelConfig, spec: LayerSpec, mesh: Mesh, key: str, sp: bool, device):
+    if spec.symbol == "C":
+        return ParallelBlock(cfg, spec, key, device)
+    if spec.symbol == "S":
+        return SandwichBlock(cfg, spec, key, device)
+    return Block(cfg, spec, mesh, key, sp, device)
 
 
 class Block(nn.Module):
@@ -153,7 +163,7 @@ class CausalLM(nn.Module):
         self.specs: List[LayerSpec] = split_for_pipeline(all_specs, mesh.pp, pp_rank, vpp, vpp_rank)
         dt, sp = cfg.params_dtype, self.sequence_parallel
         if cfg.layers is not None and mesh.world_size > 1:
-            raise ValueError("layer-list models (parallel blocks) run on one rank")
+            raise ValueError("layer-list models (packed rows) run on one rank")
         if pre_process:
             self.embedding = nn.Module()
             self.embedding.word_embeddings = VocabParallelEmbedding(cfg.vocab_size, cfg.hidden_size, mesh=mesh,
@@ -165,12 +175,12 @@ class CausalLM(nn.Module):
                     init_normal((cfg.max_position_embeddings, cfg.hidden_size), cfg.init_method_std,
                                 "embedding.position_embeddings.weight", device).to(dt))
         self.decoder = nn.Module()
-        self.decoder.layers = nn.ModuleList(
-            [ParallelBlock(cfg, s, f"decoder.layers.{s.index}", device) if s.mixer == "chunk_attn" else Block(cfg, s, mesh, f"decoder.layers.{s.index}", sp, device) for s in self.specs])
+        self.decoder.layers = nn.ModuleList([build_block(cfg, s, mesh, f"decoder.layers.{s.index}", sp, device) for s in self.specs])
         if post_process:
             if cfg.layers is not None:
-                self.decoder.final_layernorm = nn.Module()         # one number for all coordinates
-                self.decoder.final_layernorm.weight = nn.Parameter(torch.ones((), device=device))
+                self.decoder.final_layernorm = nn.Module()         # one number, or one per column of the padded rows
+                shape = () if cfg.normalization == "ScalarRMSNorm" else (-(-cfg.hidden_size // ROW_PAD) * ROW_PAD,)
+                self.decoder.final_layernorm.weight = nn.Parameter(torch.ones(shape, device=device))
             else:
                 self.decoder.final_layernorm = Norm(cfg, device)
             tied = self.embedding.word_embeddings.weight if (cfg.tie_embeddings and pre_process) else None
@@ -196,7 +206,7 @@ class CausalLM(nn.Module):
                 self.lower_bounds.pp_shared_grad = "all"
 
         if cfg.layers is not None:
-            self.requires_grad_(False)                             # serving only: the block's kernels have no backward pass
+            self.requires_grad_(False)                             # serving only: the blocks' kernels have no backward pass
 
     # ------------------------------------------------------------------
     @property
@@ -204,11 +214,11 @@ class CausalLM(nn.Module):
         """Does the model run batches of requests at different positions (packed rows and a slot cache)?"""
         return self.cfg.layers is not None
 
-    def new_cache(self, slots: int = 1):
+    def new_cache(self, slots: int = 1, tokens: int = 0):
         """One dict per local block: recurrent states / KV caches for decoding.  Models that run packed rows get a
-        ``SlotCache`` (a list of such dicts with buffers for ``slots`` requests)."""
+        ``SlotCache`` (a list of such dicts with buffers for ``slots`` requests and ``tokens`` tokens; it grows)."""
         if self.packed_rows:
-            return new_slot_cache(self, slots)
+            return new_slot_cache(self, slots, tokens)
         return [dict() for _ in self.decoder.layers]
 
     def _run_blocks(self, x, residual, caches, position_offset):
@@ -248,7 +258,7 @@ class CausalLM(nn.Module):
                 hidden_in: Optional[torch.Tensor] = None, caches: Optional[List[dict]] = None,
                 position_offset: int = 0, parallel_output: bool = False, return_hidden: bool = False, batch=None,
                 logit_rows: Optional[torch.Tensor] = None):
-        """``batch`` (``ops.chunk_attn.RowBatch``; models that run packed rows): ``input_ids`` are the packed tokens of its
+        """``batch`` (``ops.row_batch.RowBatch``; models that run packed rows): ``input_ids`` are the packed tokens of its
         requests and the result has one row per token, or per entry of ``logit_rows``."""
         if self.packed_rows:
             return forward_rows(self, input_ids, labels, caches, position_offset, batch, logit_rows, return_hidden)

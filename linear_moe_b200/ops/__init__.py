@@ -321,8 +321,11 @@ def softmax_attention(q, k, v, scale=None, causal=True, q_offset: int = 0, windo
     return R.softmax_attention(q, k, v, scale, causal, q_offset, window)
 
 
-# ---- packed-row operators of parallel blocks (serving only) ---------------------------------------
+# ---- packed-row operators (serving only) -----------------------------------------------------------
 from .chunk_attn import chunk_attention, embed_norm, poly_norm, stream_norm   # noqa: E402,F401
+from .moe_rows import experts_relu2   # noqa: E402,F401
+from .packed_attn import (causal_attention, gather_rows, latent_absorb, latent_norm, latent_up, qk_norm_rope_,   # noqa: E402,F401
+                          residual_norm, step_attention, sublayer_out, swiglu_in)
 
 
 # ---- linear sequence models -----------------------------------------------

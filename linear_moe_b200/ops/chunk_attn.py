@@ -1,26 +1,23 @@
 """Chunked, soft-capped, distance-biased, gated attention and the other row operators of a parallel block.
 
-All operators work on packed rows: the tokens of a batch's requests, one after the other (:class:`RowBatch` says which row
-belongs to which request and position).  CUDA tensors (bf16 or fp32) take the kernels of ``csrc/chunk_attn.cu``,
-``csrc/chunk_attn_tc.cu``, ``csrc/chunk_attn_step.cu`` and ``csrc/parallel_block.cu``; CPU tensors take the eager definitions of
-:mod:`linear_moe_b200.ref.chunk_attn`.  These operators serve (no backward pass).
+All operators work on packed rows: the tokens of a batch's requests, one after the other
+(:class:`~linear_moe_b200.ops.row_batch.RowBatch` says which row belongs to which request and position).  CUDA tensors (bf16 or
+fp32) take the kernels of ``csrc/chunk_attn.cu``, ``csrc/chunk_attn_tc.cu``, ``csrc/chunk_attn_step.cu`` and
+``csrc/parallel_block.cu``; CPU tensors take the eager definitions of :mod:`linear_moe_b200.ref.chunk_attn`.  These operators serve (no backward pass).
 """
 from __future__ import annotations
 
 import ctypes
 from dataclasses import dataclass
-from typing import Dict, List, Optional, Sequence, Tuple
+from typing import Optional
 
 import torch
 
 from ..ref import chunk_attn as RC
+from .row_batch import RowBatch, round_up
 
 SCORE_BOUND = 60.0            # exp of a score within +-60 stays far inside fp32: no running maximum needed
 LUT_ENTRIES_TC = 4096 - 512   # distances the tensor-core kernel keeps in shared memory
-
-
-def round_up(n: int, m: int) -> int:
-    return (n + m - 1) // m * m
 
 
 @dataclass(frozen=True)
@@ -63,72 +60,6 @@ class RowLayout:
             out.append(at)
             at += round_up(n, 8)
         return RowLayout(*out, at)
-
-
-class RowBatch:
-    """Which request and which position every packed row is.
-
-    ``starts[r]``: tokens of request r that earlier calls have processed; ``counts[r]``: its tokens in this call; ``slots[r]``:
-    its place in the cache (``None`` without a cache).  ``decode`` batches (one token each, from the cache) take their
-    positions and slots from device tensors, so that a captured graph can be replayed with other values in them."""
-
-    def __init__(self, starts: Sequence[int], counts: Sequence[int], slots: Optional[Sequence[int]], device):
-        assert len(starts) == len(counts) and all(c > 0 for c in counts) and all(s >= 0 for s in starts)
-        assert slots is not None or not any(starts), "a request can only go on from a cache"
-        self.starts, self.counts, self.device = list(starts), list(counts), torch.device(device)
-        self.slots = None if slots is None else list(slots)
-        self.requests, self.rows = len(self.counts), sum(self.counts)
-        self.decode = self.slots is not None and all(c == 1 for c in self.counts) and any(self.starts)
-        self.row0 = [0]
-        for c in self.counts:
-            self.row0.append(self.row0[-1] + c)
-        cnt = torch.tensor(self.counts)
-        first = torch.repeat_interleave(torch.tensor(self.row0[:-1]), cnt)
-        pos = torch.arange(self.rows) - first + torch.repeat_interleave(torch.tensor(self.starts), cnt)
-        end = torch.repeat_interleave(torch.tensor(self.starts) + cnt, cnt)
-        slot = torch.repeat_interleave(torch.tensor(self.slots if self.slots is not None else [0] * self.requests), cnt)
-        packed = torch.stack([pos, end, slot]).to(torch.int32)
-        if self.device.type == "cuda":
-            packed = packed.pin_memory().to(self.device, non_blocking=True)
-        self.pos, self.end, self.slot = packed[0], packed[1], packed[2]
-        self._items: Dict[Tuple[int, int], torch.Tensor] = {}
-
-    @classmethod
-    def one_token(cls, pos: torch.Tensor, slot: torch.Tensor) -> "RowBatch":
-        """One token per request, positions and slots (int32) only known on the device."""
-        b = cls.__new__(cls)
-        b.requests = b.rows = int(pos.numel())
-        b.starts = b.slots = None
-        b.counts, b.row0 = [1] * b.rows, list(range(b.rows + 1))
-        b.pos, b.slot, b.end, b.device, b.decode = pos, slot, None, pos.device, True
-        b._items = {}
-        return b
-
-    def reach(self) -> int:
-        """One more than the largest position in the batch (0 if only the device knows)."""
-        return 0 if self.starts is None else max(s + c for s, c in zip(self.starts, self.counts))
-
-    def continues_inside_chunk(self, chunk: int) -> bool:
-        """Does any request need keys of its chunk that an earlier call has processed?"""
-        return any(s % chunk for s in self.starts)
-
-    def items(self, chunk: int, tile: int) -> torch.Tensor:
-        """Work items ``[n, 8]`` int32 (``csrc/chunk_attn.cuh``): every chunk's queries in tiles, those with most keys first."""
-        key = (chunk, tile)
-        if key not in self._items:
-            out: List[Tuple[int, ...]] = []
-            for r in range(self.requests):
-                lo, hi, slot = self.starts[r], self.starts[r] + self.counts[r], 0 if self.slots is None else self.slots[r]
-                p = lo
-                while p < hi:
-                    c_beg = p // chunk * chunk                       # chunk of position p
-                    stop = min(hi, c_beg + chunk, p + tile)
-                    out.append((self.row0[r] + p - lo, stop - p, p - c_beg, max(lo - c_beg, 0), slot, 0, 0, 0))
-                    p = stop
-            out.sort(key=lambda t: -(t[2] + t[1]))
-            t = torch.tensor(out, dtype=torch.int32)
-            self._items[key] = t.pin_memory().to(self.device, non_blocking=True) if self.device.type == "cuda" else t
-        return self._items[key]
 
 
 @dataclass
@@ -233,8 +164,8 @@ def chunk_attention(z: torch.Tensor, out: torch.Tensor, spec: ChunkAttnSpec, lay
 
 
 def stream_norm(x: torch.Tensor, width: int, eps: float, dtype, gain: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """fp32 residual stream ``[rows, pad]`` (zeros behind ``width``) -> ``x / rms(x)`` (times the one number ``gain``) in
-    ``dtype``, same padding."""
+    """fp32 residual stream ``[rows, pad]`` (zeros behind ``width``) -> ``x / rms(x)`` in ``dtype``, same padding, times ``gain``:
+    one number, or one per column (``[pad]``)."""
     if not x.is_cuda:
         y = RC.unit_norm(x[:, :width], eps, x.shape[1])
         return (y if gain is None else y * gain).to(dtype)
@@ -242,17 +173,20 @@ def stream_norm(x: torch.Tensor, width: int, eps: float, dtype, gain: Optional[t
     _no_grad(x)
     y = torch.empty(x.shape, dtype=dtype, device=x.device)
     K._check(K.lib().lmoe_stream_norm(K._p(x), ctypes.c_longlong(x.stride(0)), K._p(y), ctypes.c_longlong(y.stride(0)), x.shape[0], width,
-                                      x.shape[1], ctypes.c_float(eps), K._p(gain), K._dt(y), K._st()), "stream_norm")
+                                      x.shape[1], ctypes.c_float(eps), K._p(gain), 0 if gain is None else gain.numel(), K._dt(y), K._st()), "stream_norm")
     return y
 
 
-def embed_norm(ids: torch.Tensor, pos: torch.Tensor, emb: torch.Tensor, ptab: Optional[torch.Tensor], pad: int, eps: float):
-    """``x = emb[ids] + ptab[pos]`` as fp32 rows padded to ``pad`` columns, and ``x / rms(x)`` in the table's dtype."""
+def embed_norm(ids: torch.Tensor, pos: torch.Tensor, emb: torch.Tensor, ptab: Optional[torch.Tensor], pad: int, eps: float,
+               gain: Optional[torch.Tensor] = None):
+    """``x = emb[ids] (+ ptab[pos])`` as fp32 rows padded to ``pad`` columns, and ``x / rms(x)`` (times ``gain [pad]``) in the
+    table's dtype."""
     width = emb.shape[1]
     if not emb.is_cuda:
         x = torch.zeros(ids.numel(), pad)
         x[:, :width] = emb[ids].float() + (0 if ptab is None else ptab[pos.long()].float())
-        return x, RC.unit_norm(x[:, :width], eps, pad).to(emb.dtype)
+        y = RC.unit_norm(x[:, :width], eps, pad)
+        return x, (y if gain is None else y * gain).to(emb.dtype)
     from . import cuda as K
     _no_grad(emb)
     ids = ids.contiguous()
@@ -260,7 +194,7 @@ def embed_norm(ids: torch.Tensor, pos: torch.Tensor, emb: torch.Tensor, ptab: Op
     y = torch.empty(ids.numel(), pad, dtype=emb.dtype, device=emb.device)
     K._check(K.lib().lmoe_embed_norm(K._p(ids), K._p(pos), K._p(emb), K._p(ptab), K._p(x), ctypes.c_longlong(pad), K._p(y),
                                      ctypes.c_longlong(pad), ids.numel(), width, pad, emb.shape[0], 0 if ptab is None else ptab.shape[0],
-                                     ctypes.c_float(eps), K._dt(emb), K._st()), "embed_norm")
+                                     ctypes.c_float(eps), K._p(gain), K._dt(emb), K._st()), "embed_norm")
     return x, y
 
 

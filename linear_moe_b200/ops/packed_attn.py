@@ -1,0 +1,344 @@
+"""Softmax attention over packed rows with a cache, and the row operators of blocks that norm both ends of a sublayer.
+
+Two kinds of attention share the kernels: grouped-query attention (optional norm over the whole query and key projections, optional
+interleaved rotary positions, optional sliding window) and latent attention (keys and values are products of one cached latent row
+per token).  Operators work on packed rows (:class:`~linear_moe_b200.ops.row_batch.RowBatch`).  CUDA tensors (bf16 or fp32) take the kernels of
+``csrc/packed_attn*.cu``, ``csrc/latent_step.cu`` and ``csrc/sandwich_block.cu``; CPU tensors take the eager definitions of
+:mod:`linear_moe_b200.ref.packed_attn`.  These operators serve (no backward pass).
+
+Head sizes and latents are laid out in multiples of 16 and 32 (zero weight rows), so every size meets the kernels' alignment.
+"""
+from __future__ import annotations
+
+import ctypes
+from dataclasses import dataclass
+from typing import Optional
+
+import torch
+
+from ..ref import packed_attn as RP
+from .row_batch import RowBatch, round_up
+
+ROWS_SMEM = 227 * 1024 // 4   # floats of shared memory a prompt kernel for any head size may use
+
+
+@dataclass(frozen=True)
+class AttentionSpec:
+    """Grouped-query attention: sizes and constants of one layer."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    window: Optional[int] = None      # position i sees the `window` positions up to and including i
+    rot_dims: int = 0                 # leading dimensions of a head that are rotated, in neighbouring pairs
+    rot_base: float = 10000.0
+    qk_norm: bool = False             # RMS norm over the whole query (key) projection, before the heads are split
+
+    def __post_init__(self):
+        if min(self.heads, self.kv_heads, self.dim, self.vdim) < 1 or (self.window is not None and self.window < 1):
+            raise ValueError("attention sizes must be positive")
+        if self.heads % self.kv_heads:
+            raise ValueError(f"{self.heads} query heads do not share {self.kv_heads} key/value heads evenly")
+        if self.rot_dims % 2 or not 0 <= self.rot_dims <= self.dim:
+            raise ValueError(f"{self.rot_dims} rotated dimensions in a head of {self.dim}")
+        _check_scale(self.scale)
+
+    @property
+    def dk(self) -> int:              # as laid out
+        return round_up(self.dim, 16)
+
+    @property
+    def dv(self) -> int:
+        return round_up(self.vdim, 16)
+
+    def frequencies(self, device) -> Optional[torch.Tensor]:
+        if not self.rot_dims:
+            return None
+        i = torch.arange(self.rot_dims // 2, dtype=torch.float64)
+        return (float(self.rot_base) ** (-2.0 * i / self.rot_dims)).to(device)
+
+
+@dataclass(frozen=True)
+class LatentSpec:
+    """Latent attention without positions: sizes and constants of one layer."""
+    heads: int
+    dim: int
+    vdim: int
+    rank: int
+    scale: float
+    source: Optional[int] = None      # layer whose latents this one uses (None: its own)
+
+    def __post_init__(self):
+        if min(self.heads, self.dim, self.vdim, self.rank) < 1:
+            raise ValueError("attention sizes must be positive")
+        _check_scale(self.scale)
+
+    @property
+    def dk(self) -> int:
+        return round_up(self.dim, 16)
+
+    @property
+    def dv(self) -> int:
+        return round_up(self.vdim, 16)
+
+    @property
+    def width(self) -> int:           # latent row as laid out
+        return round_up(self.rank, 32)
+
+
+def _check_scale(scale: float):
+    if not scale > 0:
+        raise ValueError(f"score scale {scale}: the online softmax needs a positive one")
+
+
+@dataclass(frozen=True)
+class QkvLayout:
+    """First columns of queries, keys and values in a projection's output."""
+    q: int
+    k: int
+    v: int
+    width: int
+
+    @staticmethod
+    def of(s: AttentionSpec) -> "QkvLayout":
+        k = s.heads * s.dk
+        v = k + s.kv_heads * s.dk
+        return QkvLayout(0, k, v, v + s.kv_heads * s.dv)
+
+
+# ------------------------------------------------------------------------------------------------------- kernel arguments
+_P, _LL, _I, _F = ctypes.c_void_p, ctypes.c_longlong, ctypes.c_int, ctypes.c_float
+
+
+def _fields(**groups):
+    return [(n, t) for t, names in groups.values() for n in names.split()]
+
+
+class _Prompt(ctypes.Structure):
+    _fields_ = _fields(a=(_P, "q k v gate out items err"), b=(_LL, "ldq ldk ldv ldg ldo"), c=(_I, "H G dk dv window n q_rows k_rows"), d=(_F, "scale"))
+
+
+class _Cache(ctypes.Structure):
+    _fields_ = _fields(a=(_P, "k v table"), b=(_I, "table_ld cap"))
+
+
+class _Step(ctypes.Structure):
+    _fields_ = _fields(a=(_P, "q out"), b=(_Cache, "c"), c=(_P, "pos slots"), d=(_LL, "ldq ldo"), e=(_I, "H G dk dv window n"), f=(_F, "scale"))
+
+
+class _QkNorm(ctypes.Structure):
+    _fields_ = _fields(a=(_P, "z wq wk freq"), b=(_Cache, "c"), c=(_P, "pos slots ends"), d=(_LL, "ldz"),
+                       e=(_I, "zq zk zv H G dk dv nq nk rot"), f=(_F, "eps"), g=(_I, "rows"))
+
+
+class _LatentNorm(ctypes.Structure):
+    _fields_ = _fields(a=(_P, "z c weight"), b=(_Cache, "cache"), c=(_P, "pos slots"), d=(_LL, "ldz ldc"), e=(_I, "width rank"), f=(_F, "eps"),
+                       g=(_I, "rows"))
+
+
+def _cache_args(cache: Optional[dict], name: Optional[str] = None) -> _Cache:
+    """``name``: address only this buffer (as the key buffer)."""
+    c = _Cache()
+    if cache is None:
+        return c
+    k = cache[name or "k"]
+    assert k.is_contiguous() and cache["v"].is_contiguous()
+    c.k, c.v = k.data_ptr(), cache["v"].data_ptr()
+    if "table" in cache:
+        c.table, c.table_ld = cache["table"].data_ptr(), cache["table"].stride(0)
+    c.cap = k.shape[1]
+    return c
+
+
+def _no_grad(*ts):
+    if torch.is_grad_enabled() and any(t is not None and t.requires_grad for t in ts):
+        raise RuntimeError("the packed-row kernels have no backward pass: run under torch.no_grad()")
+
+
+def _ptr(t: Optional[torch.Tensor]) -> int:
+    return 0 if t is None else t.data_ptr()
+
+
+# --------------------------------------------------------------------------------------------------------------- attention
+def causal_attention(q, k, v, out, heads: int, kv_heads: int, dk: int, dv: int, scale: float, window: Optional[int], batch: RowBatch,
+                     gate: Optional[torch.Tensor] = None):
+    """Prompts: ``out [rows, heads * dv] = softmax(q . k * scale) v`` (times ``sigmoid(gate)``), ``q [rows, heads * dk]``; ``k``, ``v``
+    ``[key rows, kv_heads * d]`` in the order of ``batch.key_sources`` (the rows themselves when no request goes on from a cache)."""
+    if not q.is_cuda:
+        return RP.causal_attention(q, k, v, out, heads, kv_heads, dk, dv, scale, window, batch, gate)
+    from . import cuda as K
+    from . import gemm
+    _no_grad(q, k, v, gate)
+    assert q.dtype == k.dtype == v.dtype == out.dtype and all(t.stride(1) == 1 for t in (q, k, v, out)) and q.shape[0] == batch.rows
+    assert k.shape[0] == v.shape[0] == batch.key_rows(window) and (gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1))
+    a = _Prompt()
+    a.q, a.k, a.v, a.gate, a.out = q.data_ptr(), k.data_ptr(), v.data_ptr(), _ptr(gate), out.data_ptr()
+    a.ldq, a.ldk, a.ldv, a.ldg, a.ldo = q.stride(0), k.stride(0), v.stride(0), 0 if gate is None else gate.stride(0), out.stride(0)
+    a.H, a.G, a.dk, a.dv, a.window, a.scale = heads, kv_heads, dk, dv, window or 0, scale
+    a.q_rows, a.k_rows = q.shape[0], k.shape[0]
+    dt = K._dt(q)
+    fast = dt == 1 and dk <= 128 and dv <= 128
+    tile = 128 if fast else 32 if 64 * (dk + 1) + 64 * dv + 32 * 33 <= ROWS_SMEM else 16
+    items = batch.causal_items(window, tile)
+    a.items, a.n = items.data_ptr(), items.shape[0]
+    if fast:
+        a.err = gemm._err(q.device).data_ptr()
+        K._check(K.lib().lmoe_packed_attn_tc(ctypes.byref(a), K._st()), "packed_attn_tc")
+    else:
+        K._check(K.lib().lmoe_packed_attn_rows(ctypes.byref(a), tile, dt, K._st()), "packed_attn_rows")
+
+
+def step_splits(requests: int, heads: int, kv_heads: int, dk: int, dv: int, shared: bool, rows: Optional[int], sms: int) -> int:
+    """CTAs (1 - 8, one cluster) that share the keys of one (request, kv head): as many as stay resident together.  ``rows``: the
+    most keys there can be, where that is known."""
+    per_group = heads // kv_heads
+    tile = 32 if per_group > 16 else 16
+    ctas = requests * kv_heads * -(-per_group // tile)
+    smem = 256 * (dk + (0 if shared else dv)) + tile * (2 * dk + 512)
+    room = sms * max(1, min(2 if tile == 32 or dv > 256 else 4, 220 * 1024 // smem))
+    s = 1
+    while s < 8 and ctas * s * 2 <= room and (rows is None or rows > 64 * s):
+        s *= 2
+    return s
+
+
+def step_attention(q, out, heads: int, kv_heads: int, dk: int, dv: int, scale: float, window: Optional[int], cache: dict, batch: RowBatch):
+    """One token per request, whose key and value are in the cache already: ``q [n, heads * dk]`` -> ``out [n, heads * dv]``."""
+    if not q.is_cuda:
+        return RP.step_attention(q, out, heads, kv_heads, dk, dv, scale, window, cache, batch)
+    from . import cuda as K
+    _no_grad(q)
+    assert q.dtype == out.dtype == cache["k"].dtype and q.stride(1) == 1 and out.stride(1) == 1 and q.shape[0] == batch.rows
+    a = _Step()
+    a.q, a.out, a.c, a.pos, a.slots = q.data_ptr(), out.data_ptr(), _cache_args(cache), batch.pos.data_ptr(), batch.slot.data_ptr()
+    a.ldq, a.ldo, a.H, a.G, a.dk, a.dv, a.window, a.n, a.scale = q.stride(0), out.stride(0), heads, kv_heads, dk, dv, window or 0, q.shape[0], scale
+    dt, shared = K._dt(q), cache["v"].data_ptr() == cache["k"].data_ptr()
+    tile = 32 if heads // kv_heads > 16 else 16
+    stages = max(256 * (dk + 8 + (0 if shared else dv + 8)), tile * (dv + 4) * 4)
+    if dt == 1 and dk % 16 == 0 and dv % 16 == 0 and dv <= 512 and stages + tile * (2 * dk + 600) < 226 * 1024:
+        splits = step_splits(q.shape[0], heads, kv_heads, dk, dv, shared, None if "table" in cache else cache["k"].shape[1], K.num_sms())
+        K._check(K.lib().lmoe_packed_attn_step(ctypes.byref(a), splits, K._st()), "packed_attn_step")
+    else:
+        K._check(K.lib().lmoe_packed_attn_step_any(ctypes.byref(a), dt, K._st()), "packed_attn_step_any")
+
+
+def gather_rows(dst, src: Optional[torch.Tensor], cache: Optional[dict], name: str, meta: torch.Tensor):
+    """``dst[meta[:, 0]]`` = rows ``meta[:, 1]`` of ``src``, or (-1) the cached row of slot ``meta[:, 2]``, position ``meta[:, 3]``."""
+    if not meta.shape[0]:
+        return
+    if not dst.is_cuda:
+        return RP.gather_rows(dst, src, name, cache, meta)
+    from . import cuda as K
+    ld = ctypes.c_longlong
+    assert dst.stride(1) == 1 and (src is None or (src.stride(1) == 1 and src.dtype == dst.dtype))
+    c = _cache_args(cache, name)
+    K._check(K.lib().lmoe_gather_rows(K._p(dst), ld(dst.stride(0)), K._p(src), ld(0 if src is None else src.stride(0)), ctypes.byref(c), dst.shape[1],
+                                      K._p(meta), meta.shape[0], K._dt(dst), K._st()), "gather_rows")
+
+
+# ------------------------------------------------------------------------------------------------------------ row operators
+def qk_norm_rope_(z, lay: QkvLayout, spec: AttentionSpec, wq, wk, freq, eps: float, batch: RowBatch, cache: Optional[dict]):
+    """Norm and rotate the queries and keys of a projection's output in place; the keys and values enter the cache."""
+    nq, nk = spec.heads * spec.dim, spec.kv_heads * spec.dim
+    if not z.is_cuda:
+        return RP.qk_norm_rope_(z, lay, spec.heads, spec.kv_heads, spec.dk, spec.dv, nq, nk, wq, wk, freq, eps, batch, cache)
+    from . import cuda as K
+    _no_grad(z)
+    a = _QkNorm()
+    a.z, a.wq, a.wk, a.freq, a.c = z.data_ptr(), _ptr(wq), _ptr(wk), _ptr(freq), _cache_args(cache)
+    a.pos, a.slots, a.ends = batch.pos.data_ptr(), batch.slot.data_ptr(), _ptr(batch.end)
+    a.ldz, a.zq, a.zk, a.zv = z.stride(0), lay.q, lay.k, lay.v
+    a.H, a.G, a.dk, a.dv, a.nq, a.nk, a.rot, a.eps, a.rows = spec.heads, spec.kv_heads, spec.dk, spec.dv, nq, nk, spec.rot_dims, eps, z.shape[0]
+    K._check(K.lib().lmoe_qk_norm_rope(ctypes.byref(a), K._dt(z), K._st()), "qk_norm_rope")
+
+
+def latent_norm(z, weight, rank: int, eps: float, batch: RowBatch, cache: Optional[dict]) -> torch.Tensor:
+    """Latent rows ``[rows, width]`` from their projection; they enter the cache."""
+    if not z.is_cuda:
+        return RP.latent_norm(z, weight, rank, eps, batch, cache)
+    from . import cuda as K
+    _no_grad(z)
+    c = torch.empty(z.shape, dtype=z.dtype, device=z.device)
+    a = _LatentNorm()
+    a.z, a.c, a.weight, a.cache, a.pos, a.slots = z.data_ptr(), c.data_ptr(), weight.data_ptr(), _cache_args(cache), batch.pos.data_ptr(), batch.slot.data_ptr()
+    a.ldz, a.ldc, a.width, a.rank, a.eps, a.rows = z.stride(0), c.stride(0), z.shape[1], rank, eps, z.shape[0]
+    K._check(K.lib().lmoe_latent_norm(ctypes.byref(a), K._dt(z), K._st()), "latent_norm")
+    return c
+
+
+def latent_absorb(q, w_uk, heads: int, dk: int) -> torch.Tensor:
+    """``q [n, heads * dk]`` -> ``[n, heads * width]``: every head's query in terms of the latent, ``w_uk [heads * dk, width]``."""
+    n, width = q.shape[0], w_uk.shape[1]
+    if q.is_cuda and q.dtype == torch.bfloat16:
+        from . import cuda as K
+        _no_grad(q, w_uk)
+        out, ld = torch.empty(n, heads * width, dtype=q.dtype, device=q.device), ctypes.c_longlong
+        K._check(K.lib().lmoe_latent_absorb(K._p(q), ld(q.stride(0)), K._p(w_uk), K._p(out), ld(out.stride(0)), n, heads, dk, width, K._st()),
+                 "latent_absorb")
+        return out
+    return torch.matmul(q.reshape(n, heads, dk).transpose(0, 1), w_uk.reshape(heads, dk, width)).transpose(0, 1).reshape(n, -1)
+
+
+def latent_up(x, w_uv, gate, heads: int, dv: int) -> torch.Tensor:
+    """``x [n, heads * width]`` (mixed latents) -> ``[n, heads * dv]`` values times ``sigmoid(gate)``; ``w_uv [heads * dv, width]``."""
+    n, width = x.shape[0], w_uv.shape[1]
+    if x.is_cuda:
+        from . import cuda as K
+        _no_grad(x, w_uv, gate)
+        ld = ctypes.c_longlong
+        if x.dtype == torch.bfloat16:
+            out = torch.empty(n, heads * dv, dtype=x.dtype, device=x.device)
+            K._check(K.lib().lmoe_latent_up(K._p(x), ld(x.stride(0)), K._p(w_uv), K._p(gate), ld(gate.stride(0)), K._p(out), ld(out.stride(0)), n,
+                                            heads, dv, width, K._st()), "latent_up")
+            return out
+    out = torch.matmul(x.reshape(n, heads, width).transpose(0, 1), w_uv.reshape(heads, dv, width).transpose(1, 2))
+    out = out.transpose(0, 1).reshape(n, heads * dv)
+    if not x.is_cuda:
+        return (out.float() * torch.sigmoid(gate.float())).to(x.dtype)
+    out = out.contiguous()
+    K._check(K.lib().lmoe_gate_rows(K._p(out), ld(out.stride(0)), K._p(gate), ld(gate.stride(0)), n, heads * dv, K._dt(out), K._st()), "gate_rows")
+    return out
+
+
+def residual_norm(x, y, width: int, post, pre: Optional[torch.Tensor], eps: float, dtype, dest: Optional[torch.Tensor] = None, top: int = 0):
+    """``x += y / rms(y) * post`` on the fp32 stream, in place; returns ``x / rms(x) * pre`` in ``dtype`` (``pre`` ``None``: nothing).
+    With ``top``, token t's y is the sum of rows ``dest[t * top + k]`` (``dest`` ``None``: of rows ``t * top + k``)."""
+    if not x.is_cuda:
+        return RP.residual_norm(x, y, width, post, pre, eps, dtype, dest, top)
+    from . import cuda as K
+    _no_grad(x, y)
+    ld = ctypes.c_longlong
+    h = None if pre is None else torch.empty(x.shape, dtype=dtype, device=x.device)
+    assert y.shape[1] >= x.shape[1] and y.stride(1) == 1 and (top or y.shape[0] == x.shape[0])
+    K._check(K.lib().lmoe_residual_norm(K._p(x), ld(x.stride(0)), K._p(y), ld(y.stride(0)), K._dt(y), K._p(dest), top, K._p(post), K._p(pre), K._p(h),
+                                        ld(0 if h is None else h.stride(0)), x.shape[0], width, x.shape[1], ctypes.c_float(eps),
+                                        1 if dtype == torch.bfloat16 else 0, K._st()), "residual_norm")
+    return h
+
+
+FEW_ROWS = 256                # products of this few rows keep their fp32 result (their cost is reading the weights)
+
+
+def sublayer_out(x, weight) -> torch.Tensor:
+    """The last product of a sublayer, in fp32 for few rows."""
+    from . import linear, linear_f32
+    return linear_f32(x, weight) if x.shape[0] <= FEW_ROWS else linear(x, weight)
+
+
+def swiglu_in(h, w1) -> torch.Tensor:
+    """``silu(h Wg^T) * (h Wu^T)`` for ``w1 = [Wg; Wu]``: in the epilogue of the product for many bf16 rows, else a kernel after it."""
+    from . import linear
+    if not h.is_cuda:
+        g, u = linear(h, w1).float().chunk(2, -1)
+        return (torch.nn.functional.silu(g) * u).to(h.dtype)
+    from . import cuda as K
+    from . import gemm
+    _no_grad(h, w1)
+    if h.shape[0] > 16 and gemm.dense_ok(h, w1) and w1.shape[0] % 16 == 0:
+        return gemm.dense_swiglu(h, w1, want_pre=False)[0]
+    z = linear(h, w1)
+    ff, ld = w1.shape[0] // 2, ctypes.c_longlong
+    out = torch.empty(z.shape[0], ff, dtype=z.dtype, device=z.device)
+    K._check(K.lib().lmoe_swiglu_rows(K._p(z), ld(z.stride(0)), K._p(out), ld(ff), z.shape[0], ff, K._dt(z), K._st()), "swiglu_rows")
+    return out

@@ -1,0 +1,116 @@
+"""Eager definitions of the row operators of :mod:`linear_moe_b200.ops.packed_attn` and :mod:`linear_moe_b200.ops.moe_rows` (what
+CPU tensors run).  Rows are laid out as for the kernels: head sizes and latents padded with zero columns."""
+from __future__ import annotations
+
+from typing import Optional
+
+import torch
+
+PAGE = 64
+
+
+def cache_rows(cache: dict, name: str, slot: int, positions: torch.Tensor) -> torch.Tensor:
+    """Rows ``[n, heads, dim]`` of a slot, as a copy."""
+    buf, at = cache[name], _places(cache, slot, positions)
+    return buf.reshape(-1, *buf.shape[2:])[at]
+
+
+def _places(cache: dict, slot: int, positions: torch.Tensor) -> torch.Tensor:
+    if "table" in cache:
+        return cache["table"][slot].long()[positions // PAGE] * PAGE + positions % PAGE
+    rows = cache["k"].shape[1]
+    return slot * rows + positions % rows
+
+
+def store(cache: dict, name: str, slot: int, positions: torch.Tensor, rows: torch.Tensor):
+    buf = cache[name]
+    buf.view(-1, *buf.shape[2:])[_places(cache, slot, positions)] = rows.to(buf.dtype)
+
+
+def mix(q, k, v, scale: float, first_query: int, window: Optional[int]):
+    """``q [n, H, d]`` at key indices ``first_query ..``, ``k [m, G, d]``, ``v [m, G, e]`` -> ``[n, H, e]`` (fp32)."""
+    n, H, G = q.shape[0], q.shape[1], k.shape[1]
+    i, j = torch.arange(first_query, first_query + n)[:, None], torch.arange(k.shape[0])[None, :]
+    hidden = j > i if window is None else (j > i) | (j <= i - window)
+    s = torch.einsum("ihd,jhd->hij", q.float(), k.float().repeat_interleave(H // G, 1)) * scale
+    return torch.einsum("hij,jhd->ihd", s.masked_fill(hidden, float("-inf")).softmax(-1), v.float().repeat_interleave(H // G, 1))
+
+
+def causal_attention(q, k, v, out, H, G, dk, dv, scale, window, batch, gate):
+    krow = 0
+    for r, (past, n) in enumerate(zip(batch.past(window), batch.counts)):
+        a, b = batch.row0[r], batch.row0[r + 1]
+        ks = slice(krow, krow + past + n)
+        o = mix(q[a:b].reshape(n, H, dk), k[ks].reshape(-1, G, dk), v[ks].reshape(-1, G, dv), scale, past, window).reshape(n, H * dv)
+        out[a:b] = (o if gate is None else o * torch.sigmoid(gate[a:b].float())).to(out.dtype)
+        krow += past + n
+
+
+def step_attention(q, out, H, G, dk, dv, scale, window, cache, batch):
+    for r, (p, slot) in enumerate(zip(batch.pos.tolist(), batch.slot.tolist())):
+        span = window if "table" in cache else cache["k"].shape[1]
+        at = torch.arange(0 if span is None else max(0, p + 1 - span), p + 1)
+        k, v = cache_rows(cache, "k", slot, at), cache_rows(cache, "v", slot, at)
+        out[r] = mix(q[r:r + 1].reshape(1, H, dk), k, v, scale, len(at) - 1, None).reshape(-1).to(out.dtype)
+
+
+def rotate_pairs(x, pos, freq):
+    """``x [n, heads, d]``: neighbouring pairs of the first ``2 len(freq)`` dimensions turn by ``pos * freq``."""
+    angle = pos.double()[:, None] * freq[None, :]
+    c, s = torch.cos(angle).float()[:, None], torch.sin(angle).float()[:, None]
+    y, rot = x.clone(), 2 * len(freq)
+    u, v = x[..., 0:rot:2], x[..., 1:rot:2]
+    y[..., 0:rot:2], y[..., 1:rot:2] = u * c - v * s, v * c + u * s
+    return y
+
+
+def qk_norm_rope_(z, lay, H, G, dk, dv, nq, nk, wq, wk, freq, eps, batch, cache):
+    for at, heads, numbers, w in ((lay.q, H, nq, wq), (lay.k, G, nk, wk)):
+        x = z[:, at:at + heads * dk].float()
+        if w is not None:
+            x = x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) / numbers + eps) * w
+        x = x.reshape(-1, heads, dk)
+        z[:, at:at + heads * dk] = (x if freq is None else rotate_pairs(x, batch.pos, freq)).reshape(-1, heads * dk).to(z.dtype)
+    if cache is None:
+        return
+    for r, slot in enumerate(batch.slot.tolist()):
+        p = batch.pos[r:r + 1].long()
+        store(cache, "k", slot, p, z[r:r + 1, lay.k:lay.k + G * dk].reshape(1, G, dk))
+        store(cache, "v", slot, p, z[r:r + 1, lay.v:lay.v + G * dv].reshape(1, G, dv))
+
+
+def latent_norm(z, weight, rank, eps, batch, cache):
+    x = z.float()
+    c = (x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) / rank + eps) * weight).to(z.dtype)
+    if cache is not None:
+        for r, slot in enumerate(batch.slot.tolist()):
+            store(cache, "k", slot, batch.pos[r:r + 1].long(), c[r:r + 1, None])
+    return c
+
+
+def gather_rows(dst, src, name, cache, meta):
+    for d, s, slot, pos in meta.tolist():
+        dst[d] = src[s] if s >= 0 else cache_rows(cache, name, slot, torch.tensor([pos]))[0].reshape(-1)
+
+
+def residual_norm(x, y, width, post, pre, eps, dtype, dest, top):
+    if top:
+        y = y.float()[torch.arange(x.shape[0] * top) if dest is None else dest.long()].reshape(x.shape[0], top, -1).sum(1)
+    y = y[:, :x.shape[1]].float()
+    x.add_(y * torch.rsqrt(y.pow(2).sum(-1, keepdim=True) / width + eps) * post)
+    return None if pre is None else (x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) / width + eps) * pre).to(dtype)
+
+
+def route(logits, top):
+    z, idx = torch.topk(logits, top, -1)
+    return torch.sigmoid(z), idx
+
+
+def experts_relu2(h, logits, up, down, top):
+    """Rows ``[n * top, width]``: expert(weight * h) of every (token, expert)."""
+    w, idx = route(logits, top)
+    y = torch.zeros(h.shape[0] * top, down.shape[1])
+    for p, (wt, e) in enumerate(zip(w.flatten().tolist(), idx.flatten().tolist())):
+        a = (wt * torch.relu(up[e].float() @ h[p // top].float())).pow(2).to(h.dtype)
+        y[p] = down[e].float() @ a.float()
+    return y

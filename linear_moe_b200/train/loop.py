@@ -79,7 +79,7 @@ class Trainer:
                  device: Optional[torch.device] = None, dataset=None, valid_dataset=None,
                  model_provider: Optional[Callable] = None, forward_step: Optional[Callable] = None):
         if cfg.layers is not None:
-            raise ValueError("layer-list models (parallel blocks) serve only: their kernels have no backward pass")
+            raise ValueError("layer-list models (packed rows) serve only: their kernels have no backward pass")
         self.cfg, self.par, self.tc = cfg, par, tc
         self.mesh = mesh or single_process_mesh()
         self.device = device or (torch.device("cuda", torch.cuda.current_device()) if torch.cuda.is_available()
