@@ -144,7 +144,10 @@ def greedy(w, cfg, prompt, steps):
 
 def random_model(cfg, seed=0, gain=1.0):
     """Random weights for ``cfg`` under the checkpoint's names, rounded to bf16.  ``gain`` sharpens the attention (scales the
-    latent layers' query weights and the others' query norm)."""
+    latent layers' query weights and the others' query norm).
+
+    The routers decide clearly: the first columns of the stream hold a random order of the experts for each token (no sublayer adds
+    to them) and the routers read mostly these, so that rounding does not send a token to another expert."""
     g = torch.Generator().manual_seed(seed)
 
     def rnd(*shape, std):
@@ -155,10 +158,13 @@ def random_model(cfg, seed=0, gain=1.0):
 
     d, V = cfg["width"], cfg["vocab"]
     w = {"embed": rnd(V, d, std=1.0), "head": rnd(V, d, std=d ** -0.5), "final.norm": weight(d, 0.9)}
+    E = max([l["mlp"]["router"]["experts"] for l in cfg["layers"] if l.get("mlp") and l["mlp"]["kind"] == "moe"], default=0)
+    w["embed"][:, :E] = torch.stack([torch.randperm(E, generator=g) for _ in range(V)]).bfloat16() * (3.0 / max(E, 1)) - 1.5
     for n, layer in enumerate(cfg["layers"]):
         m, l, x = layer["mixer"], f"l{n}.", f"l{n}.mix."
         H, dk, dv = m["heads"], m["dim"], m["vdim"]
         w[l + "norm1"], w[l + "norm1b"] = weight(d, 1.1), weight(d, 0.7)
+        w[l + "norm1b"][:E] = 0
         if layer["type"] == "latent_attention":
             r = m["kv_rank"]
             w[x + "q"] = rnd(H * dk, d, std=gain * d ** -0.5)
@@ -176,12 +182,15 @@ def random_model(cfg, seed=0, gain=1.0):
         if ff is None:
             continue
         w[l + "norm2"], w[l + "norm2b"], x = weight(d, 0.9), weight(d, 0.8), l + "mlp."
+        w[l + "norm2b"][:E] = 0
         if ff["kind"] == "dense":
             f = ff["ff"]
             w[x + "gate"], w[x + "up"], w[x + "down"] = rnd(f, d, std=d ** -0.5), rnd(f, d, std=d ** -0.5), rnd(d, f, std=f ** -0.5)
         else:
-            f, E = ff["expert"]["ff"], ff["router"]["experts"]
-            w[x + "router"] = rnd(E, d, std=1.5 * d ** -0.5)
-            for e in range(E):
+            f, n_e = ff["expert"]["ff"], ff["router"]["experts"]
+            w[x + "router"] = rnd(n_e, d, std=0.1 * d ** -0.5)
+            w[x + "router"][torch.arange(n_e), torch.randperm(E, generator=g)[:n_e]] = 1.5
+            w[l + "norm2"][:E] = 1.0
+            for e in range(n_e):
                 w[f"{x}e{e}.up"], w[f"{x}e{e}.down"] = rnd(f, d, std=2 * d ** -0.5), rnd(d, f, std=f ** -0.5)
     return w

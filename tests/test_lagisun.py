@@ -5,7 +5,6 @@ import io
 import json
 import math
 import os
-import struct
 import subprocess
 import sys
 
@@ -17,22 +16,9 @@ from linear_moe_b200.infer.generation import generate_tokens
 from linear_moe_b200.infer.session import InferenceSession
 from linear_moe_b200.models.registry import load_model
 from linear_moe_b200.ops import chunk_attn as CA
+from linear_moe_b200.ops.row_batch import RowBatch, round_up
 from linear_moe_b200.ref.chunk_attn import distance_bucket
-
-ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
-GPU = pytest.mark.gpu
-WHERE = [("cpu", "float32"), pytest.param(("cuda", "float32"), marks=GPU), pytest.param(("cuda", "bfloat16"), marks=GPU)]
-where = pytest.mark.parametrize("where", WHERE, ids=["cpu", "cuda-fp32", "cuda-bf16"])
-
-
-def tol(where):
-    """Allowed root-mean-square error relative to that of the expected values."""
-    return 0.02 if where[1] == "bfloat16" else 2e-5
-
-
-def rel(got, want):
-    got, want = got.detach().double().cpu(), want.double()
-    return float((got - want).pow(2).mean().sqrt() / want.pow(2).mean().sqrt())
+from serving_utils import GPU, ROOT, folder, padded, prompt, rel, tol, where
 
 
 def mixer(heads, kv_heads, dim, vdim, size, cap=25.0, far=40, scale=None):
@@ -61,26 +47,6 @@ CONFIGS = {
 }
 
 
-def write_safetensors(path, tensors):
-    head, at, blobs = {"__metadata__": {"origin": "test"}}, 0, []
-    for name, t in tensors.items():
-        raw = t.contiguous().view(torch.uint8).numpy().tobytes() if t.dim() else t.reshape(1).view(torch.uint8).numpy().tobytes()
-        head[name] = {"dtype": {torch.bfloat16: "BF16", torch.float32: "F32"}[t.dtype], "shape": list(t.shape), "data_offsets": [at, at + len(raw)]}
-        blobs.append(raw)
-        at += len(raw)
-    h = json.dumps(head).encode()
-    with open(path, "wb") as f:
-        f.write(struct.pack("<Q", len(h)) + h + b"".join(blobs))
-
-
-def folder(path, cfg, w):
-    os.makedirs(path, exist_ok=True)
-    with open(os.path.join(path, "config.json"), "w") as f:
-        json.dump(cfg, f)
-    write_safetensors(os.path.join(path, "model.safetensors"), w)
-    return str(path)
-
-
 @pytest.fixture(scope="module")
 def build(tmp_path_factory):
     """``build(name, where) -> (model, weights, config)``; a model is made once per module."""
@@ -100,10 +66,6 @@ def build(tmp_path_factory):
     return get
 
 
-def prompt(cfg, n, seed=0):
-    return torch.randint(0, cfg["vocab"], (n,), generator=torch.Generator().manual_seed(seed * 1000 + n))
-
-
 # ------------------------------------------------------------------------------------------------------- single mechanisms
 def test_distance_buckets():
     for rows, far in ((4, 10), (8, 9), (12, 50), (16, 1000), (32, 128)):
@@ -121,7 +83,7 @@ def test_distance_buckets():
 @where
 @pytest.mark.parametrize("rows,width", [(1, 32), (5, 50), (3, 96), (2, 5000)])
 def test_stream_norm(where, rows, width):
-    x = torch.zeros(rows, CA.round_up(width, 32))
+    x = torch.zeros(rows, round_up(width, 32))
     x[:, :width] = torch.randn(rows, width) * torch.tensor([10.0 ** -k for k in range(rows)])[:, None]
     gain = torch.tensor(1.7)
     for g in (None, gain):
@@ -136,7 +98,7 @@ def test_poly_norm(where, ff):
     dev, dt = where[0], getattr(torch, where[1])
     z = (torch.randn(3, ff + 11) * torch.tensor([0.01, 1.0, 30.0])[:, None]).to(dt)
     act, gain = torch.tensor([0.7, -0.5, 0.4, 0.1]), torch.tensor(0.8)
-    out = torch.full((3, CA.round_up(ff, 32) + 32), float("nan"), dtype=dt).to(dev)
+    out = torch.full((3, round_up(ff, 32) + 32), float("nan"), dtype=dt).to(dev)
     CA.poly_norm(z.to(dev)[:, 8:8 + ff], out[:, 32:], ff, gain.to(dev), act.to(dev), 1e-3, 0.6)
     want = 0.6 * O.poly_norm(z[:, 8:8 + ff].double() * 0.8, act, 1e-3)
     for r in range(3):
@@ -172,8 +134,8 @@ def run_attention(where, c, T, starts, counts, slots=None, sharp=None, rows=14, 
     z = z.to(dt)
     tab = torch.randn(rows, H, generator=g)
     table = CA.build_bias_table(tab.to(dev), spec)
-    gain, out = torch.tensor(0.9, device=dev), torch.full((T, CA.round_up(H * dv, 32)), 7.0, dtype=dt, device=dev)
-    batch = CA.RowBatch(starts, counts, slots, dev)
+    gain, out = torch.tensor(0.9, device=dev), torch.full((T, round_up(H * dv, 32)), 7.0, dtype=dt, device=dev)
+    batch = RowBatch(starts, counts, slots, dev)
     CA.chunk_attention(z.to(dev), out, spec, lay, table, gain, batch, cache, 0.5)
     zd = z.double() * 0.9
     return out[:, :H * dv], (spec, lay, zd, tab, c)
@@ -235,8 +197,8 @@ def test_attention_one_token_steps(where, c):
     """Prompts stored into scattered slots, then single tokens that cross a chunk border, requests at different positions."""
     dev, dt = where[0], getattr(torch, where[1])
     size, H, G = c["mask"]["size"], c["heads"], c["kv_heads"]
-    cache = {"k": torch.full((9, size, G, CA.round_up(c["dim"], 8)), 1e3, dtype=dt, device=dev),
-             "v": torch.full((9, size, G, CA.round_up(c["vdim"], 8)), 1e3, dtype=dt, device=dev)}
+    cache = {"k": torch.full((9, size, G, round_up(c["dim"], 8)), 1e3, dtype=dt, device=dev),
+             "v": torch.full((9, size, G, round_up(c["vdim"], 8)), 1e3, dtype=dt, device=dev)}
     starts, slots = [size - 2, 2 * size - 1, 1, size], [7, 0, 3, 8]
     rows = [[], [], [], []]                                             # (rows of all z so far) of every request
     zs, at = [], 0
@@ -400,14 +362,6 @@ def test_limits_are_refused(build):
 
 
 # --------------------------------------------------------------------------------------- generation, folders, command line
-def padded(prompts, extra):
-    L = max(map(len, prompts)) + extra
-    t = torch.zeros(len(prompts), L, dtype=torch.long)
-    for b, p in enumerate(prompts):
-        t[b, :len(p)] = p
-    return t, torch.tensor([len(p) for p in prompts])
-
-
 @where
 @pytest.mark.parametrize("graph", [False, True])
 def test_greedy_generation(build, where, graph):
