@@ -72,7 +72,8 @@ def parse():
     p.add_argument("--layers", type=int, default=None, help="debug only: fewer layers (marks the result invalid)")
     p.add_argument("--no-e2e", action="store_true")
     p.add_argument("--serve", action="store_true", help="instead of the training benchmark: prefill / decode throughput and kernel "
-                   "times of the Lagisun design beside the Llama3-shaped transformer at equal size (one GPU)")
+                   "times of a served design beside the framework's closest other model at equal size (one GPU)")
+    p.add_argument("--serve-model", choices=["lagisun", "sonodra"], default="lagisun", help="design of --serve")
     p.add_argument("--serve-sizes", type=str, default="1b,8b", help="sizes of --serve")
     p.add_argument("--overlap-grad-reduce", action=argparse.BooleanOptionalAction, default=False,
                    help="reduce-scatter the gradients of a block while the backward pass of the blocks before it runs "
@@ -99,7 +100,10 @@ def main():
     if args.impl == "reference":
         return reference_arm()
     if args.serve:
-        from linear_moe_b200.bench.serve import main as serve
+        if args.serve_model == "sonodra":
+            from linear_moe_b200.bench.serve_sonodra import main as serve
+        else:
+            from linear_moe_b200.bench.serve import main as serve
         return serve(args.serve_sizes.split(","))
     import torch
     import torch.distributed as dist

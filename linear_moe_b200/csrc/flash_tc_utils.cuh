@@ -88,13 +88,17 @@ __device__ __forceinline__ float max3(float a, float b, float c) {
 }
 // Bounded wait that lets the hardware suspend the warp (try_wait with a time hint) instead of spinning on test_wait:
 // the 16 softmax warps share 4 schedulers, a spinning warp takes issue slots from the others.
+__device__ __forceinline__ bool mbar_try_suspend(uint64_t* bar, uint32_t parity) {
+    uint32_t ok;
+    asm volatile("{\n.reg .pred p;\nmbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2, %3;\nselp.u32 %0, 1, 0, p;\n}"
+                 : "=r"(ok) : "r"(s32(bar)), "r"(parity), "r"(20000u) : "memory");
+    return ok != 0;
+}
 __device__ __forceinline__ bool mbar_wait_suspend(uint64_t* bar, uint32_t parity, volatile int* abort_flag, int* err, int code) {
+    if (mbar_try_suspend(bar, parity)) return true;
     const long long t0 = clock64();
     for (;;) {
-        uint32_t ok;
-        asm volatile("{\n.reg .pred p;\nmbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2, %3;\nselp.u32 %0, 1, 0, p;\n}"
-                     : "=r"(ok) : "r"(s32(bar)), "r"(parity), "r"(20000u) : "memory");
-        if (ok) return true;
+        if (mbar_try_suspend(bar, parity)) return true;
         if (*abort_flag) return false;
         if (clock64() - t0 > WAIT_CYCLES) break;
     }

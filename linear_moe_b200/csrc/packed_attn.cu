@@ -187,35 +187,63 @@ struct QkNorm {
     int rows;
 };
 
+// sums of two numbers per thread over the block; red: 16 float2
+__device__ __forceinline__ float2 block_sum2(float2 v, float2* red) {
+    v.x = warp_sum(v.x);
+    v.y = warp_sum(v.y);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    __syncthreads();
+    v = make_float2(0.f, 0.f);
+    for (int i = 0; i < THREADS / 32; ++i) {
+        v.x += red[i].x;
+        v.y += red[i].y;
+    }
+    return v;
+}
+
 template <typename T>
 __global__ void __launch_bounds__(THREADS) qk_norm_rope_kernel(QkNorm a) {
     pdl_trigger();
-    constexpr int W = Vec<T>::N;
+    constexpr int W = Vec<T>::N, NV = sizeof(T) == 2 ? 3 : 2;           // pieces a thread keeps in registers
     extern __shared__ float2 turn[];     // [rot / 2] (cos, sin)
-    __shared__ float red[32];
+    __shared__ float2 red[THREADS / 32];
     const int row = blockIdx.x, pos = a.pos[row];
+    const int nq = a.H * a.dk, n = nq + a.G * a.dk;                     // queries, then keys
     T* z = (T*)a.z + (long long)row * a.ldz;
+    auto at = [&](int i) { return z + (i < nq ? a.zq + i : a.zk + i - nq); };
+    Vec<T> v[NV];
+#pragma unroll
+    for (int t = 0; t < NV; ++t) {
+        const int i = (threadIdx.x + t * THREADS) * W;
+        if (i < n) v[t].load(at(i));
+    }
     for (int i = threadIdx.x; i < a.rot / 2; i += THREADS) {
         // range reduction in double: the angle is exact to fp32 at any position
-        constexpr double TWO_PI = 6.283185307179586476925286766559;
+        constexpr double TWO_PI = 6.283185307179586476925286766559, INV = 0.15915494309189533576888376337251;
         const double angle = (double)pos * a.freq[i];
-        const float r = (float)(angle - TWO_PI * rint(angle / TWO_PI));
+        const float r = (float)(angle - TWO_PI * rint(angle * INV));
         turn[i] = make_float2(cosf(r), sinf(r));
     }
-    float rq = 1.f, rk = 1.f;
-    auto square_sum = [&](const T* p, int n) {
+    float2 sum = make_float2(0.f, 0.f);
+    auto square = [&](const Vec<T>& x, int i) {
         float s = 0.f;
-        for (int i = threadIdx.x * W; i < n; i += THREADS * W) {
-            Vec<T> v;
-            v.load(p + i);
 #pragma unroll
-            for (int e = 0; e < W; ++e) s += v.get(e) * v.get(e);
-        }
-        return s;
+        for (int e = 0; e < W; ++e) s += x.get(e) * x.get(e);
+        if (i < nq) sum.x += s;
+        else sum.y += s;
     };
-    if (a.wq != nullptr) rq = 1.f / sqrtf(block_sum(square_sum(z + a.zq, a.H * a.dk), red) / a.nq + a.eps);
-    if (a.wk != nullptr) rk = 1.f / sqrtf(block_sum(square_sum(z + a.zk, a.G * a.dk), red) / a.nk + a.eps);
-    __syncthreads();
+#pragma unroll
+    for (int t = 0; t < NV; ++t) {
+        const int i = (threadIdx.x + t * THREADS) * W;
+        if (i < n) square(v[t], i);
+    }
+    for (int i = (threadIdx.x + NV * THREADS) * W; i < n; i += THREADS * W) {
+        Vec<T> x;
+        x.load(at(i));
+        square(x, i);
+    }
+    sum = block_sum2(sum, red);                                         // its barrier also covers `turn`
+    const float rq = 1.f / sqrtf(sum.x / a.nq + a.eps), rk = 1.f / sqrtf(sum.y / a.nk + a.eps);
     T* kd = nullptr;
     T* vd = nullptr;
     // a ring keeps the request's last `cap` positions: of the rows that share a place only the last one is stored
@@ -224,36 +252,43 @@ __global__ void __launch_bounds__(THREADS) qk_norm_rope_kernel(QkNorm a) {
         kd = (T*)a.c.k + r * a.dk;
         vd = (T*)a.c.v + r * a.dv;
     }
-    auto finish = [&](T* p, int n, const float* weight, float r, T* dst) {
-        for (int i = threadIdx.x * W; i < n; i += THREADS * W) {
-            Vec<T> v;
-            v.load(p + i);
-            const int d = i % a.dk;
-            float x[W];
+    auto finish = [&](Vec<T>& x, int i) {
+        const bool is_q = i < nq;
+        const int c = is_q ? i : i - nq, d = c % a.dk;
+        const float* weight = is_q ? a.wq : a.wk;
+        const float r = is_q ? rq : rk;
+        float f[W];
 #pragma unroll
-            for (int e = 0; e < W; ++e) x[e] = weight == nullptr ? v.get(e) : v.get(e) * r * weight[i + e];
+        for (int e = 0; e < W; ++e) f[e] = weight == nullptr ? x.get(e) : x.get(e) * r * weight[c + e];
 #pragma unroll
-            for (int e = 0; e < W; e += 2) {
-                if (d + e < a.rot) {
-                    const float2 cs = turn[(d + e) / 2];
-                    const float u = x[e], t = x[e + 1];
-                    x[e] = u * cs.x - t * cs.y;
-                    x[e + 1] = t * cs.x + u * cs.y;
-                }
+        for (int e = 0; e < W; e += 2) {
+            if (d + e < a.rot) {
+                const float2 cs = turn[(d + e) / 2];
+                const float u = f[e], t = f[e + 1];
+                f[e] = u * cs.x - t * cs.y;
+                f[e + 1] = t * cs.x + u * cs.y;
             }
-#pragma unroll
-            for (int e = 0; e < W; ++e) v.set(e, x[e]);
-            v.store(p + i);
-            if (dst != nullptr) v.store(dst + i);
         }
+#pragma unroll
+        for (int e = 0; e < W; ++e) x.set(e, f[e]);
+        x.store(at(i));
+        if (!is_q && kd != nullptr) x.store(kd + c);
     };
-    finish(z + a.zq, a.H * a.dk, a.wq, rq, nullptr);
-    finish(z + a.zk, a.G * a.dk, a.wk, rk, kd);
+#pragma unroll
+    for (int t = 0; t < NV; ++t) {
+        const int i = (threadIdx.x + t * THREADS) * W;
+        if (i < n) finish(v[t], i);
+    }
+    for (int i = (threadIdx.x + NV * THREADS) * W; i < n; i += THREADS * W) {
+        Vec<T> x;
+        x.load(at(i));
+        finish(x, i);
+    }
     if (vd != nullptr)
         for (int i = threadIdx.x * W; i < a.G * a.dv; i += THREADS * W) {
-            Vec<T> v;
-            v.load(z + a.zv + i);
-            v.store(vd + i);
+            Vec<T> x;
+            x.load(z + a.zv + i);
+            x.store(vd + i);
         }
 }
 
@@ -269,30 +304,51 @@ struct LatentNorm {
     int rows;
 };
 
+// one warp per row
 template <typename T>
-__global__ void __launch_bounds__(THREADS) latent_norm_kernel(LatentNorm a) {
+__global__ void __launch_bounds__(128) latent_norm_kernel(LatentNorm a) {
     pdl_trigger();
-    __shared__ float red[32];
-    constexpr int W = Vec<T>::N;
-    const int row = blockIdx.x;
+    constexpr int W = Vec<T>::N, NV = 16 / W * 2;            // pieces a lane keeps in registers (rows up to 1024 wide)
+    const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (row >= a.rows) return;
     const T* z = (const T*)a.z + (long long)row * a.ldz;
     T* c = (T*)a.c + (long long)row * a.ldc;
     T* dst = a.cache.k == nullptr ? nullptr : (T*)a.cache.k + a.cache.row(a.slots[row], a.pos[row]) * a.width;
+    Vec<T> v[NV];
     float s = 0.f;
-    for (int i = threadIdx.x * W; i < a.width; i += blockDim.x * W) {
-        Vec<T> v;
-        v.load(z + i);
+    auto square = [&](const Vec<T>& x) {
 #pragma unroll
-        for (int e = 0; e < W; ++e) s += v.get(e) * v.get(e);
+        for (int e = 0; e < W; ++e) s += x.get(e) * x.get(e);
+    };
+#pragma unroll
+    for (int t = 0; t < NV; ++t) {
+        const int i = (lane + t * 32) * W;
+        if (i < a.width) v[t].load(z + i);
     }
-    const float r = 1.f / sqrtf(block_sum(s, red) / a.rank + a.eps);
-    for (int i = threadIdx.x * W; i < a.width; i += blockDim.x * W) {
-        Vec<T> v;
-        v.load(z + i);
 #pragma unroll
-        for (int e = 0; e < W; ++e) v.set(e, v.get(e) * r * a.weight[i + e]);
-        v.store(c + i);
-        if (dst != nullptr) v.store(dst + i);
+    for (int t = 0; t < NV; ++t)
+        if ((lane + t * 32) * W < a.width) square(v[t]);
+    for (int i = (lane + NV * 32) * W; i < a.width; i += 32 * W) {
+        Vec<T> x;
+        x.load(z + i);
+        square(x);
+    }
+    const float r = 1.f / sqrtf(warp_sum(s) / a.rank + a.eps);
+    auto finish = [&](Vec<T>& x, int i) {
+#pragma unroll
+        for (int e = 0; e < W; ++e) x.set(e, x.get(e) * r * a.weight[i + e]);
+        x.store(c + i);
+        if (dst != nullptr) x.store(dst + i);
+    };
+#pragma unroll
+    for (int t = 0; t < NV; ++t) {
+        const int i = (lane + t * 32) * W;
+        if (i < a.width) finish(v[t], i);
+    }
+    for (int i = (lane + NV * 32) * W; i < a.width; i += 32 * W) {
+        Vec<T> x;
+        x.load(z + i);
+        finish(x, i);
     }
 }
 
@@ -361,9 +417,8 @@ LMOE_API int lmoe_latent_norm(const pag::LatentNorm* ap, int dt, cudaStream_t st
     if (a.rows <= 0 || a.width <= 0 || a.rank <= 0 || a.width % w || a.ldz % w || a.ldc % w || !pag::aligned(a.z) || !pag::aligned(a.c) ||
         !pag::aligned(a.cache.k) || (a.cache.k != nullptr && a.cache.table == nullptr && a.cache.cap <= 0))
         return -1;
-    const int threads = a.width > 128 * w ? 256 : 128;
-    if (dt) pag::latent_norm_kernel<bf16><<<a.rows, threads, 0, st>>>(a);
-    else pag::latent_norm_kernel<float><<<a.rows, threads, 0, st>>>(a);
+    if (dt) pag::latent_norm_kernel<bf16><<<(a.rows + 3) / 4, 128, 0, st>>>(a);
+    else pag::latent_norm_kernel<float><<<(a.rows + 3) / 4, 128, 0, st>>>(a);
     return (int)cudaGetLastError();
 }
 

@@ -190,17 +190,21 @@ def causal_attention(q, k, v, out, heads: int, kv_heads: int, dk: int, dv: int, 
 
 
 def step_splits(requests: int, heads: int, kv_heads: int, dk: int, dv: int, shared: bool, rows: Optional[int], sms: int) -> int:
-    """CTAs (1 - 8, one cluster) that share the keys of one (request, kv head): as many as stay resident together.  ``rows``: the
-    most keys there can be, where that is known."""
-    per_group = heads // kv_heads
-    tile = 32 if per_group > 16 else 16
-    ctas = requests * kv_heads * -(-per_group // tile)
-    smem = 256 * (dk + (0 if shared else dv)) + tile * (2 * dk + 512)
-    room = sms * max(1, min(2 if tile == 32 or dv > 256 else 4, 220 * 1024 // smem))
+    """CTAs (1 - 8, one cluster) that share the keys of one (request, 16 heads of a kv head): as many as stay resident together, two
+    per SM while their stages of keys fit.  ``rows``: the most keys there can be, where that is known."""
+    ctas = requests * kv_heads * -(-(heads // kv_heads) // 16)
+    room = sms * (2 if _step_bytes(dk, dv, shared) <= 110 * 1024 else 1)
     s = 1
     while s < 8 and ctas * s * 2 <= room and (rows is None or rows > 64 * s):
         s *= 2
     return s
+
+
+def _step_bytes(dk: int, dv: int, shared: bool) -> int:
+    """Shared memory of the one-token kernel with two stages (csrc/packed_attn_step.cu)."""
+    keys = 64 if max(dk, dv) <= 128 else 32
+    blocks = -(-dk // 64) + (0 if shared else -(-dv // 64))
+    return max(2 * blocks * keys * 128, 64 * (dv + 4)) + 32 * (dk + 8) + 512 * (keys + 4) + 32 * (keys + 8) + 192 + 1024
 
 
 def step_attention(q, out, heads: int, kv_heads: int, dk: int, dv: int, scale: float, window: Optional[int], cache: dict, batch: RowBatch):
@@ -208,17 +212,17 @@ def step_attention(q, out, heads: int, kv_heads: int, dk: int, dv: int, scale: f
     if not q.is_cuda:
         return RP.step_attention(q, out, heads, kv_heads, dk, dv, scale, window, cache, batch)
     from . import cuda as K
+    from . import gemm
     _no_grad(q)
     assert q.dtype == out.dtype == cache["k"].dtype and q.stride(1) == 1 and out.stride(1) == 1 and q.shape[0] == batch.rows
     a = _Step()
     a.q, a.out, a.c, a.pos, a.slots = q.data_ptr(), out.data_ptr(), _cache_args(cache), batch.pos.data_ptr(), batch.slot.data_ptr()
     a.ldq, a.ldo, a.H, a.G, a.dk, a.dv, a.window, a.n, a.scale = q.stride(0), out.stride(0), heads, kv_heads, dk, dv, window or 0, q.shape[0], scale
     dt, shared = K._dt(q), cache["v"].data_ptr() == cache["k"].data_ptr()
-    tile = 32 if heads // kv_heads > 16 else 16
-    stages = max(256 * (dk + 8 + (0 if shared else dv + 8)), tile * (dv + 4) * 4)
-    if dt == 1 and dk % 16 == 0 and dv % 16 == 0 and dv <= 512 and stages + tile * (2 * dk + 600) < 226 * 1024:
+    if dt == 1 and dk % 16 == 0 and dv % 16 == 0 and max(dk, dv) <= 512 and _step_bytes(dk, dv, shared) < 224 * 1024:
+        rows = cache["k"].shape[0] * cache["k"].shape[1]
         splits = step_splits(q.shape[0], heads, kv_heads, dk, dv, shared, None if "table" in cache else cache["k"].shape[1], K.num_sms())
-        K._check(K.lib().lmoe_packed_attn_step(ctypes.byref(a), splits, K._st()), "packed_attn_step")
+        K._check(K.lib().lmoe_packed_attn_step(ctypes.byref(a), rows, splits, K._p(gemm._err(q.device)), K._st()), "packed_attn_step")
     else:
         K._check(K.lib().lmoe_packed_attn_step_any(ctypes.byref(a), dt, K._st()), "packed_attn_step_any")
 

@@ -49,8 +49,9 @@ CONFIGS = {
     # every branch, sizes that differ by layer, two layers that borrow the same latents, windows shorter and longer than a page
     "mixed": config((grouped(6, 3, 24, 40, 21, 16), moe(6, 2, 40)), (latent(5, 32, 24, 48), dense(112)), (latent(3, 16, 40, 48, source=1), None),
                     (grouped(4, 1, 64, 32, 70, 64, base=500.0), moe(4, 1, 72)), (latent(2, 48, 16, 48, source=1, scale=0.3), moe(5, 3, 16)), width=96),
-    # nothing divides by 8
-    "odd": config((latent(3, 10, 6, 19), moe(7, 3, 13)), (grouped(5, 5, 10, 7, 23, 6), dense(45)), (latent(2, 7, 5, 19, source=0), None), width=50, vocab=77),
+    # nothing divides by 8; two layers with latents of their own, the last one borrows the first one's
+    "odd": config((latent(3, 10, 6, 19), moe(7, 3, 13)), (grouped(5, 5, 10, 7, 23, 6), dense(45)), (latent(1, 9, 9, 19), dense(10)),
+                  (latent(2, 7, 5, 19, source=0), None), width=50, vocab=77),
     # full tensor-core tiles, more than 16 and more than 32 heads on one key, windows over one 128-query tile
     "wide": config((latent(40, 64, 128, 160), dense(256)), (grouped(24, 1, 128, 64, 150, 32), moe(12, 4, 96)), (grouped(4, 2, 128, 128, 300, 128), dense(64)),
                    width=128),
