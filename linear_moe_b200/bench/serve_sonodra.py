@@ -11,6 +11,7 @@ between the iterations; decode kernels are captured in a CUDA graph that loops o
 from __future__ import annotations
 
 import json
+import time
 
 import torch
 
@@ -168,8 +169,10 @@ def kernels(size: str) -> list:
     row("rms_norm (qwen2), heads of the queries", "norm + rotary", timeit(lambda: ops.rms_norm(qf, torch.ones(aD, device=dev, dtype=bf))), bytes_=rows * aH * aD * 4)
     del qf, kf, vf, z
     zc, wc = rnd(rows, R + H * D), torch.ones(R, device=dev)
-    row("latent_norm", "norm", timeit(lambda: PA.latent_norm(zc[:, H * D:], wc, R, 1e-5, batch, None)), bytes_=rows * R * 4)
-    del zc
+    row("latent_norm", "latent norm", timeit(lambda: PA.latent_norm(zc[:, H * D:], wc, R, 1e-5, batch, None)), bytes_=rows * R * 4)
+    zr, wr = zc[:, H * D:].contiguous(), torch.ones(R, device=dev, dtype=bf)
+    row("rms_norm (qwen2) on rows of that size", "latent norm", timeit(lambda: ops.rms_norm(zr, wr)), bytes_=rows * R * 4)
+    del zc, zr
     x, y, h, one, oneb = torch.randn(rows, w, device=dev), rnd(rows, w), rnd(rows, w), torch.ones(w, device=dev), torch.ones(w, device=dev, dtype=bf)
     row("residual_norm", "norm", timeit(lambda: PA.residual_norm(x, y, w, one, one, 1e-5, bf)), bytes_=rows * w * 12)
     row("add_rms_norm (qwen2)", "norm", timeit(lambda: ops.add_rms_norm(h, y, oneb)), bytes_=rows * w * 8)
@@ -206,7 +209,9 @@ def kernels(size: str) -> list:
     del xs, a, y2, x, y, h, o, c
     gemm.check_error()
 
-    # ---- one-token steps
+    # ---- one-token steps (after a pause: the products above run at the power limit, and the clock recovers slowly)
+    torch.cuda.synchronize()
+    time.sleep(3)
     for n in (8, 64):
         one_tok = RowBatch.one_token(torch.full((n,), CTX - 1, dtype=torch.int32, device=dev), torch.arange(n, dtype=torch.int32, device=dev))
 
