@@ -55,7 +55,7 @@ __global__ void __launch_bounds__(RT) route_rows_kernel(const float* __restrict_
 
 __global__ void place_offsets_kernel(const int* __restrict__ counts, int* __restrict__ offs, int E, int align) {
     __shared__ int part[1024];
-    int base = 0;                                            // padded rows of the experts before this round's
+    int base = 0;                                            // padded rows of the experts before this pass
     for (int e0 = 0; e0 < E; e0 += blockDim.x) {
         const int e = e0 + threadIdx.x;
         int v = e < E ? (counts[e] + align - 1) / align * align : 0;
