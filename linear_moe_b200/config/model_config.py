@@ -20,8 +20,8 @@ LA_MODULES = (
     "gated_deltanet", "gsa", "based", "rebased", "hgrn2", "rwkv6", "rwkv7",
     "mamba2", "lasp2", "mom_gla", "mom_gated_deltanet", "mom_linear_attention",
 )
-BASE_MODELS = ("qwen2", "llama3", "mixtral", "deepseek_v2", "lagisun", "sonodra")
-LAYER_LIST_MODELS = ("lagisun", "sonodra")        # described by ModelConfig.layers; run packed rows, serve only
+BASE_MODELS = ("qwen2", "llama3", "mixtral", "deepseek_v2", "lagisun", "sonodra", "gafonex")
+LAYER_LIST_MODELS = ("lagisun", "sonodra", "gafonex")        # described by ModelConfig.layers; run packed rows, serve only
 
 
 @dataclass
@@ -138,7 +138,11 @@ class ModelConfig:
     #   {"attn": ops.chunk_attn.ChunkAttnSpec, "bias_rows": rows of the distance table, "ff": width or None}
     # sonodra: sequential blocks with a norm at both ends of a sublayer, one entry per layer
     #   {"mixer": ops.packed_attn.AttentionSpec or LatentSpec, "ff": width (gated), ops.moe_rows.ExpertsSpec, or None}
+    # gafonex: sequential blocks with a norm behind a sublayer only, one entry per layer
+    #   {"mixer": ops.packed_attn.AttentionSpec or ops.retention.RetentionSpec, "ff": width (gated, ReLU) or None}
     layers: Optional[Tuple[dict, ...]] = None
+    norm_groups: int = 1                          # layer-list designs: parts of a row that are normed by themselves
+    logit_softcap: Optional[float] = None         # layer-list designs: logits become cap * tanh(logits / cap)
     residual_multiplier: float = 1.0              # factor of every block's output before it joins the residual stream
     # ---- precision / memory --------------------------------------------
     params_dtype: torch.dtype = torch.float32
@@ -160,6 +164,10 @@ class ModelConfig:
             raise ValueError(f"{', '.join(LAYER_LIST_MODELS)} models are described by their layer list (and no other family has one)")
         if self.layers is not None:
             self.num_layers = len(self.layers)
+        if self.norm_groups < 1 or self.hidden_size % self.norm_groups:
+            raise ValueError(f"a width of {self.hidden_size} has no {self.norm_groups} equal parts")
+        if self.logit_softcap is not None and not self.logit_softcap > 0:
+            raise ValueError(f"soft cap {self.logit_softcap}")
         if self.base_model not in BASE_MODELS:
             raise ValueError(f"unknown base model {self.base_model!r}")
         if self.la_module is not None and self.la_module not in LA_MODULES:

@@ -8,7 +8,7 @@
 //   out_mode 0: C bf16 = result      1: C fp32 = result      2: C fp32 += result (cp.reduce.async.bulk .add, done in L2)
 //   epi 1 (K-major operands, bf16 out): B = [gate rows ; up rows] of a SwiGLU fc1 weight ([2F, K]).  CTA 0 of the pair
 //          stages 128 gate rows, CTA 1 the matching 128 up rows, so accumulator columns [0,128) / [128,256) are gate / up
-//          of the same 128 outputs; the epilogue writes silu(gate) * up to C [M,F] and, if Y != null, the
+//          of the same 128 outputs; the epilogue writes silu(gate) * up (or relu(gate) * up) to C [M,F] and, if Y != null, the
 //          pre-activations to Y [M,2F] (what the backward pass needs).  No re-tiling of the weight.
 //   epi 2 (A K-major, B MN-major, bf16 out): the data-gradient GEMM of fc2, dAct = dY W2, with the SwiGLU backward in
 //          the epilogue: the tile of dAct never leaves the SM; the matching gate / up pre-activations are fetched by TMA
@@ -50,6 +50,7 @@ struct Params {
     int f_half;        // epi 1: F (rows of the gate block of B)
     int* err;
     const bf16* bias;  // out mode 0 without epilogue function: [N] added to every row, or null
+    int relu = 0;      // epi 1: relu(gate) * up instead of silu(gate) * up
 };
 
 __device__ __forceinline__ void tma_store_2d(const CUtensorMap* map, const void* src, int c0, int c1) {
@@ -243,8 +244,9 @@ gemm_dense_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant
                     }
 #pragma unroll
                     for (int i = 0; i < 32; ++i) {
-                        g0[i] = __float_as_uint(silu_f(__uint_as_float(g0[i])) * __uint_as_float(u0[i]));
-                        g1[i] = __float_as_uint(silu_f(__uint_as_float(g1[i])) * __uint_as_float(u1[i]));
+                        const float a0 = __uint_as_float(g0[i]), a1 = __uint_as_float(g1[i]);
+                        g0[i] = __float_as_uint((p.relu ? fmaxf(a0, 0.f) : silu_f(a0)) * __uint_as_float(u0[i]));
+                        g1[i] = __float_as_uint((p.relu ? fmaxf(a1, 0.f) : silu_f(a1)) * __uint_as_float(u1[i]));
                     }
                     uint8_t* s = stg0 + (nst & 1) * OUT_BYTES;
                     if (lane == 0) bulk_wait_read<1>();
@@ -468,11 +470,11 @@ LMOE_API int lmoe_gemm_dense_bias(const void* A, int lda, int a_mn, const void* 
     return gemm_dense_impl(A, lda, a_mn, B, ldb, b_mn, C, ldc, 0, M, N, K, band, err, num_sms, st, bias);
 }
 
-// act[M,F] = silu(x Wg^T) * (x Wu^T) with W = [Wg ; Wu] of shape [2F, K] (pitch ldw); if Y != null the pre-activations
+// act[M,F] = silu(x Wg^T) * (x Wu^T) (kind 1: relu in place of silu) with W = [Wg ; Wu] of shape [2F, K] (pitch ldw); if Y != null the pre-activations
 // x W^T go to Y [M, 2F] (pitch ldy).  F % 8 == 0, K % 8 == 0.
 LMOE_API int lmoe_gemm_dense_swiglu(const void* X, int ldx, const void* W, int ldw, void* act, int ldact, void* Y, int ldy,
-                                    int M, int F, int K, int band, int* err, int num_sms, cudaStream_t st) {
-    if (M <= 0 || F <= 0 || K <= 0) return -1;
+                                    int M, int F, int K, int band, int kind, int* err, int num_sms, cudaStream_t st) {
+    if (M <= 0 || F <= 0 || K <= 0 || kind < 0 || kind > 1) return -1;
     if (ldx % 8 || ldw % 8 || K % 8 || F % 8 || ldact % 8 || (Y != nullptr && ldy % 8)) return -1;
     if (((uintptr_t)X | (uintptr_t)W | (uintptr_t)act | (uintptr_t)Y) & 15) return -2;
     CUtensorMap ma, mb, mc, my;
@@ -488,7 +490,7 @@ LMOE_API int lmoe_gemm_dense_swiglu(const void* X, int ldx, const void* W, int l
         if (rc) return rc;
     }
     Params p;
-    p.M = M; p.N = F; p.K = K; p.band = band > 0 ? band : 8; p.f_half = F; p.err = err; p.bias = nullptr;
+    p.M = M; p.N = F; p.K = K; p.band = band > 0 ? band : 8; p.f_half = F; p.err = err; p.bias = nullptr; p.relu = kind;
     return launch<false, false, 0, 1>(ma, mb, mc, my, Y != nullptr ? 1 : 0, p, num_sms, st);
 }
 

@@ -1,7 +1,7 @@
 // Row kernels of blocks that norm both ends of a sublayer, x += post(f(pre(x))), around an fp32 residual stream:
 //   residual_norm   y = the sublayer's output rows (or the sum of a token's expert rows);  x += y / rms(y) * post;
 //                   h = x / rms(x) * pre, the input of the next sublayer: one pass over the stream per sublayer
-//   swiglu_rows     silu(gate) * up
+//   glu_rows        silu(gate) * up, or relu(gate) * up
 // Rows are padded to a multiple of 4 elements (pad = 0).  Compiled without fast-math: the same code serves the fp32 model.
 #include "common.cuh"
 
@@ -86,7 +86,7 @@ __global__ void __launch_bounds__(THREADS) residual_norm_kernel(float* __restric
 
 // z [rows, ldz]: gate in columns 0 .. ff, up in ff .. 2 ff
 template <typename T>
-__global__ void __launch_bounds__(THREADS) swiglu_rows_kernel(const T* __restrict__ z, long long ldz, T* __restrict__ out, long long ldo, int ff) {
+__global__ void __launch_bounds__(THREADS) glu_rows_kernel(const T* __restrict__ z, long long ldz, T* __restrict__ out, long long ldo, int ff, int relu) {
     pdl_trigger();
     constexpr int W = Vec<T>::N;
     const T* zr = z + (long long)blockIdx.x * ldz;
@@ -98,7 +98,7 @@ __global__ void __launch_bounds__(THREADS) swiglu_rows_kernel(const T* __restric
 #pragma unroll
         for (int i = 0; i < W; ++i) {
             const float t = g.get(i);
-            g.set(i, t / (1.f + expf(-t)) * u.get(i));
+            g.set(i, (relu ? fmaxf(t, 0.f) : t / (1.f + expf(-t))) * u.get(i));
         }
         g.store(o + c);
     }
@@ -127,12 +127,13 @@ LMOE_API int lmoe_residual_norm(float* x, long long ldx, const void* y, long lon
               : sb::launch<float, float>(x, ldx, y, ldy, dest, top, post, pre, h, ldh, rows, width, pad, eps, st);
 }
 
-LMOE_API int lmoe_swiglu_rows(const void* z, long long ldz, void* out, long long ldo, int rows, int ff, int dt, cudaStream_t st) {
+// kind: 0 silu, 1 relu
+LMOE_API int lmoe_glu_rows(const void* z, long long ldz, void* out, long long ldo, int rows, int ff, int kind, int dt, cudaStream_t st) {
     const int w = dt ? 8 : 4;
-    if (rows <= 0 || ff <= 0 || ff % w || ldz % w || ldo % w || ((reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(out)) & 15)) return -1;
+    if (kind < 0 || kind > 1 || rows <= 0 || ff <= 0 || ff % w || ldz % w || ldo % w || ((reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(out)) & 15)) return -1;
     int cols = (ff + sb::THREADS * w - 1) / (sb::THREADS * w);
     if (rows > 1024) cols = 1;
-    if (dt) sb::swiglu_rows_kernel<bf16><<<dim3(rows, cols), sb::THREADS, 0, st>>>((const bf16*)z, ldz, (bf16*)out, ldo, ff);
-    else sb::swiglu_rows_kernel<float><<<dim3(rows, cols), sb::THREADS, 0, st>>>((const float*)z, ldz, (float*)out, ldo, ff);
+    if (dt) sb::glu_rows_kernel<bf16><<<dim3(rows, cols), sb::THREADS, 0, st>>>((const bf16*)z, ldz, (bf16*)out, ldo, ff, kind);
+    else sb::glu_rows_kernel<float><<<dim3(rows, cols), sb::THREADS, 0, st>>>((const float*)z, ldz, (float*)out, ldo, ff, kind);
     return (int)cudaGetLastError();
 }

@@ -9,6 +9,8 @@ token until it is released; each layer says what it needs (``None``: nothing of 
 * :class:`LayerPages`  one row per token, in pages of :data:`PAGE` rows taken from a pool as a request grows.  Page numbers hold for
   all paged layers alike, so one table ``[slots, pages]`` (int32, on the device) serves the model.  A row is a key and a value
   (``[pages, PAGE, heads, dim]``) or, with ``v_dim = 0``, one vector that is both (a latent).
+* :class:`LayerState`  one fp32 matrix per head, ``[slots, heads, k_dim, v_dim]``: the state of a recurrence, whatever the context.  It is not
+  cleared when a slot is handed out; a request's first call starts from zero instead of reading it.
 
 Because the buffers never move while a request lives (unless they have to grow, which changes ``generation``), one-token steps
 can be captured in a CUDA graph.
@@ -40,8 +42,16 @@ class LayerPages:
     v_dim: int = 0            # 0: the key row is the value too
 
 
+@dataclass(frozen=True)
+class LayerState:
+    """A recurrent state."""
+    heads: int
+    k_dim: int
+    v_dim: int
+
+
 class SlotCache:
-    def __init__(self, layers: Sequence[Optional[Union[LayerRows, LayerPages]]], slots: int, device, dtype, tokens: int = 0):
+    def __init__(self, layers: Sequence[Optional[Union[LayerRows, LayerPages, LayerState]]], slots: int, device, dtype, tokens: int = 0):
         """``tokens``: live tokens to make room for from the start (paged layers; the pool grows when there are more)."""
         self.spec, self.device, self.dtype = list(layers), torch.device(device), dtype
         self.layers: List[Dict[str, torch.Tensor]] = [{} for _ in self.spec]
@@ -65,8 +75,8 @@ class SlotCache:
     def __getitem__(self, i: int) -> Dict[str, torch.Tensor]:
         return self.layers[i]
 
-    def _buffer(self, c: dict, name: str, shape, keep: int):
-        t = torch.zeros(shape, dtype=self.dtype, device=self.device)
+    def _buffer(self, c: dict, name: str, shape, keep: int, dtype=None):
+        t = torch.zeros(shape, dtype=dtype or self.dtype, device=self.device)
         if name in c:
             t[:keep] = c[name]
         c[name] = t
@@ -76,6 +86,8 @@ class SlotCache:
             if isinstance(s, LayerRows):
                 for name, dim in (("k", s.k_dim), ("v", s.v_dim)):
                     self._buffer(c, name, (slots, s.rows, s.heads, dim), self.slots)
+            elif isinstance(s, LayerState):
+                self._buffer(c, "s", (slots, s.heads, s.k_dim, s.v_dim), self.slots, torch.float32)
         if self.paged:
             self._resize_table(slots, max(self._table_host.shape[1], 16))
         self.free += range(self.slots, slots)

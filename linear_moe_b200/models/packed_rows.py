@@ -3,10 +3,11 @@ stream, and every block works on all of them (``ops.row_batch.RowBatch`` says wh
 
 A block of such a model has
 
-    input_gain()                     weight of the norm in front of it (``None``: plain unit-RMS rows)
+    reads_stream                     it takes the stream's rows as they are (no norm in front of it)
+    input_gain()                     else: weight of the norm in front of it (``None``: plain unit-RMS rows)
     cache_spec(limit)                what it keeps per request (``infer.kv_cache``), for positions below ``limit``
-    forward(x, h, step, nxt)         ``x`` the stream, updated in place; ``h`` its normed rows; returns the normed rows for the
-                                     block ``nxt`` (``None`` behind the last one)
+    forward(x, h, step, nxt)         ``x`` the stream, updated in place; ``h`` its normed (plain) rows; returns those for the block
+                                     ``nxt`` (``None`` behind the last one)
 """
 from __future__ import annotations
 
@@ -15,6 +16,7 @@ from typing import Callable, Dict, Optional, Tuple
 
 import torch
 import torch.nn as nn
+import torch.nn.functional as F
 
 from .. import ops
 from ..infer.kv_cache import SlotCache
@@ -29,6 +31,7 @@ class RowStep:
     batch: RowBatch
     caches: Optional[SlotCache]
     latents: Dict[int, torch.Tensor] = field(default_factory=dict)    # layer -> latent rows, for the layers that borrow them
+    values: Dict[int, torch.Tensor] = field(default_factory=dict)     # layer -> value rows, for the layers that mix them into theirs
 
     def cache(self, layer: int) -> Optional[dict]:
         return None if self.caches is None else self.caches[layer]
@@ -37,6 +40,7 @@ class RowStep:
 class RowBlock(nn.Module):
     """A block of such a model.  ``places()`` maps the checkpoint's tensor names (without the layer) to views inside the block's
     parameters and the tensors' shapes; weights may be stored fused and padded."""
+    reads_stream = False
 
     def places(self) -> Dict[str, Tuple[torch.Tensor, Tuple[int, ...]]]:
         raise NotImplementedError
@@ -74,8 +78,11 @@ def forward_rows(model, input_ids, labels, caches, position_offset: int, batch: 
         raise ValueError(f"position {batch.reach() - 1} is beyond the model's table of {cfg.max_position_embeddings} positions")
     emb, w, blocks = model.embedding, cfg.hidden_size, model.decoder.layers
     pos = getattr(emb, "position_embeddings", None)
-    x, h = ops.embed_norm(input_ids.reshape(-1), batch.pos, emb.word_embeddings.weight, None if pos is None else pos.weight,
-                          round_up(w, ROW_PAD), cfg.norm_eps, blocks[0].input_gain())
+    if blocks[0].reads_stream:
+        x, h = ops.embed_rows(input_ids.reshape(-1), emb.word_embeddings.weight, round_up(w, ROW_PAD))
+    else:
+        x, h = ops.embed_norm(input_ids.reshape(-1), batch.pos, emb.word_embeddings.weight, None if pos is None else pos.weight,
+                              round_up(w, ROW_PAD), cfg.norm_eps, blocks[0].input_gain())
     taps = getattr(model, "residual_taps", None)                    # a list here receives the stream after every layer
     step, dtype = RowStep(batch, caches), h.dtype
     for blk, nxt in zip(blocks, [*blocks[1:], None]):
@@ -84,11 +91,18 @@ def forward_rows(model, input_ids, labels, caches, position_offset: int, batch: 
             taps.append(x[:, :w].clone())
     if logit_rows is not None:
         x = x.index_select(0, logit_rows)
-    h = ops.stream_norm(x, w, cfg.norm_eps, dtype, model.decoder.final_layernorm.weight)[:, :w]
+    gain = model.decoder.final_layernorm.weight
+    h = ops.stream_norm(x, w, cfg.norm_eps, dtype, gain) if cfg.norm_groups == 1 else ops.group_norm(x, w, cfg.norm_groups, gain, cfg.norm_eps, dtype)
+    h = h[:, :w]
     shape = rect if (rect is not None and logit_rows is None) else (h.shape[0],)
     if return_hidden:
         return h.reshape(*shape, w)
-    if labels is not None:
+    if labels is not None and not cfg.logit_softcap:
         return model.output_layer(h.reshape(*shape, w), labels)
     out = model.output_layer.weight
-    return ops.linear_f32(h, out).reshape(*shape, out.shape[0])
+    logits = ops.linear_f32(h, out)
+    if cfg.logit_softcap:
+        ops.softcap_(logits, cfg.logit_softcap)
+    if labels is not None:
+        return F.cross_entropy(logits, labels.reshape(-1), reduction="none").reshape(shape)
+    return logits.reshape(*shape, out.shape[0])

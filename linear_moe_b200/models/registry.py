@@ -16,7 +16,8 @@ from ..ckpt.safetensors_io import read_header, read_tensors
 from ..config.model_config import ModelConfig
 from ..ops.chunk_attn import ChunkAttnSpec
 from ..ops.moe_rows import ExpertsSpec
-from ..ops.packed_attn import AttentionSpec, LatentSpec
+from ..ops.packed_attn import AttentionSpec, LatentSpec, RotaryScaling
+from ..ops.retention import RetentionSpec
 from .transformer import CausalLM
 
 UNBOUNDED = 1 << 30           # positions of a model without a position table
@@ -152,3 +153,45 @@ def _load_rows(model: CausalLM, tensors: Dict[str, torch.Tensor], more: Dict[str
 
 
 register(Architecture("Sonodra", _sonodra_config, _sonodra_load, "sandwich_block"))
+
+
+# ---------------------------------------------------------------------------------------------------------------- Gafonex
+def _gafonex_mixer(i: int, layers: list, lender: Optional[int]):
+    """``lender``: the first layer whose values are shared."""
+    kind, m = layers[i]["type"], layers[i]["mixer"]
+    rot = m.get("rot") or {"dims": 0, "base": 1.0}
+    scaling = rot.get("scaling")
+    if kind == "retention":
+        if scaling is not None:
+            raise ValueError(f"layer {i}: retention has no rotary scaling")
+        return RetentionSpec(heads=m["heads"], dim=m["dim"], vdim=m["vdim"], decay=tuple(m["decay"]), rot_dims=rot["dims"], rot_base=rot["base"])
+    if kind == "attention":
+        shares = bool(m.get("v_mix", False))
+        if shares and any(m[n] != layers[lender]["mixer"][n] for n in ("kv_heads", "vdim")):
+            raise ValueError(f"layer {i}: its values do not have the shape of those of layer {lender}")
+        return AttentionSpec(heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"], scale=m["scale"], head_norm=True,
+                             rot_dims=rot["dims"], rot_base=rot["base"], rot_halves=True, value_norm=True, talk=True,
+                             rot_scaling=None if scaling is None else RotaryScaling(**{n: scaling[n] for n in ("factor", "original", "fast", "slow")}),
+                             value_source=lender if shares else None)
+    raise ValueError(f"layer {i}: unknown mixer {kind!r}")
+
+
+def _gafonex_config(raw: dict, shapes: Dict[str, Tuple[int, ...]]) -> ModelConfig:
+    layers = []
+    lender = next((i for i, l in enumerate(raw["layers"]) if l["type"] == "attention" and l["mixer"].get("v_mix", False)), None)
+    for i, l in enumerate(raw["layers"]):
+        mlp = l.get("mlp")
+        if mlp is not None and mlp.get("kind", "dense") != "dense":
+            raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+        layers.append({"mixer": _gafonex_mixer(i, raw["layers"], lender), "ff": None if mlp is None else mlp["ff"]})
+    first = layers[0]["mixer"]
+    return ModelConfig(base_model="gafonex", layers=tuple(layers), hidden_size=raw["width"], vocab_size=raw["vocab"], norm_eps=raw["norm"]["eps"],
+                       norm_groups=raw["norm"]["groups"], logit_softcap=raw.get("logit_softcap"), max_position_embeddings=UNBOUNDED,
+                       num_attention_heads=first.heads, kv_channels=first.dim)
+
+
+def _gafonex_load(model: CausalLM, tensors: Dict[str, torch.Tensor]):
+    _load_rows(model, tensors, {})
+
+
+register(Architecture("Gafonex", _gafonex_config, _gafonex_load, "post_norm_block"))

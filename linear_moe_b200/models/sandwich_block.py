@@ -29,7 +29,7 @@ from .packed_rows import ROW_PAD, RowBlock, RowStep
 RING_MAX = 16384              # windows over this many tokens take pages
 
 
-def _blank(shape, cfg, device) -> nn.Parameter:
+def blank(shape, cfg, device) -> nn.Parameter:
     return nn.Parameter(torch.zeros(shape, dtype=cfg.params_dtype, device=device), requires_grad=False)
 
 
@@ -39,12 +39,12 @@ def _norm(width: int, device, pad: Optional[int] = None) -> nn.Parameter:
     return nn.Parameter(w, requires_grad=False)
 
 
-def _heads(m: torch.Tensor, at: int, heads: int, laid_out: int, size: int, cols: int) -> torch.Tensor:
+def head_rows(m: torch.Tensor, at: int, heads: int, laid_out: int, size: int, cols: int) -> torch.Tensor:
     """Rows of ``heads`` heads of ``size`` numbers, laid out ``laid_out`` apart from row ``at``, as a view ``[heads, size, cols]``."""
     return m[at:at + heads * laid_out].view(heads, laid_out, m.shape[1])[:, :size, :cols]
 
 
-class _Part(nn.Module):
+class Part(nn.Module):
     """``places()``: as ``RowBlock.places``."""
 
     def places(self) -> Dict[str, Tuple[torch.Tensor, Tuple[int, ...]]]:
@@ -57,30 +57,46 @@ class _Part(nn.Module):
                     view.copy_(init_normal(shape, std, f"{key}.{name}", view.device).reshape(view.shape))
 
 
-class GroupedAttention(_Part):
+class GroupedAttention(Part):
     def __init__(self, cfg, s: AttentionSpec, device):
         super().__init__()
         self.s, self.lay, self.width, self.eps = s, QkvLayout.of(s), cfg.hidden_size, cfg.norm_eps
         pad = round_up(cfg.hidden_size, ROW_PAD)
-        self.linear_in = _blank((self.lay.width, pad), cfg, device)
-        self.linear_out = _blank((pad, round_up(s.heads * s.dv, ROW_PAD)), cfg, device)
-        if s.qk_norm:
-            self.q_norm, self.k_norm = (_norm(s.dk * n, device) for n in (s.heads, s.kv_heads))
+        self.linear_in = blank((self.lay.width, pad), cfg, device)
+        self.linear_out = blank((pad, round_up(s.heads * s.dv, ROW_PAD)), cfg, device)
+        if s.qk_norm or s.head_norm:
+            self.q_norm, self.k_norm = (_norm(s.dk * (n if s.qk_norm else 1), device) for n in (s.heads, s.kv_heads))
             with torch.no_grad():
                 for w in (self.q_norm, self.k_norm):
                     w.view(-1, s.dk)[:, s.dim:] = 0
+        if s.talk:
+            self.talk = nn.Parameter(torch.eye(s.heads, device=device), requires_grad=False)
+        if s.value_source is not None:
+            self.vmix = nn.Parameter(torch.full((), 0.5, device=device), requires_grad=False)
         self.register_buffer("freq", s.frequencies(device), persistent=False)
 
     def places(self):
         s, l, d = self.s, self.lay, self.width
-        out = {"q": (_heads(self.linear_in, l.q, s.heads, s.dk, s.dim, d), (s.heads * s.dim, d)),
-               "k": (_heads(self.linear_in, l.k, s.kv_heads, s.dk, s.dim, d), (s.kv_heads * s.dim, d)),
-               "v": (_heads(self.linear_in, l.v, s.kv_heads, s.dv, s.vdim, d), (s.kv_heads * s.vdim, d)),
+        out = {"q": (head_rows(self.linear_in, l.q, s.heads, s.dk, s.dim, d), (s.heads * s.dim, d)),
+               "k": (head_rows(self.linear_in, l.k, s.kv_heads, s.dk, s.dim, d), (s.kv_heads * s.dim, d)),
+               "v": (head_rows(self.linear_in, l.v, s.kv_heads, s.dv, s.vdim, d), (s.kv_heads * s.vdim, d)),
                "o": (self.linear_out[:d, :s.heads * s.dv].view(d, s.heads, s.dv)[..., :s.vdim], (d, s.heads * s.vdim))}
         if s.qk_norm:
             out["q.norm"] = (self.q_norm.view(-1, s.dk)[:, :s.dim], (s.heads * s.dim,))
             out["k.norm"] = (self.k_norm.view(-1, s.dk)[:, :s.dim], (s.kv_heads * s.dim,))
+        elif s.head_norm:
+            out["q.norm"], out["k.norm"] = (self.q_norm[:s.dim], (s.dim,)), (self.k_norm[:s.dim], (s.dim,))
+        if s.talk:
+            out["talk"] = (self.talk, (s.heads, s.heads))
+        if s.value_source is not None:
+            out["vmix"] = (self.vmix, ())
         return out
+
+    def randomise(self, std: float, key: str):
+        super().randomise(std, key)
+        if self.s.talk:
+            with torch.no_grad():
+                self.talk.add_(torch.eye(self.s.heads, device=self.talk.device))
 
     def cache_spec(self, limit: int):
         s = self.s
@@ -91,17 +107,24 @@ class GroupedAttention(_Part):
     def forward(self, h, step: RowStep, layer: int) -> torch.Tensor:
         s, l, batch, cache = self.s, self.lay, step.batch, step.cache(layer)
         z = ops.linear(h, self.linear_in)
-        out = _out(h, self.linear_out, s.heads * s.dv)
+        out = activation_rows(h, self.linear_out, s.heads * s.dv)
         o, sizes = out[:, :s.heads * s.dv], (s.heads, s.kv_heads, s.dk, s.dv, s.scale, s.window)
-        norms = (self.q_norm, self.k_norm) if s.qk_norm else (None, None)
+        norms = (self.q_norm, self.k_norm) if s.qk_norm or s.head_norm else (None, None)
+        talk = self.talk if s.talk else None
         grown = not batch.decode and batch.key_rows(s.window) > batch.rows
         if grown:                          # a prompt goes on: its cached keys leave the ring before the new ones enter it
             k, v = (torch.empty(batch.key_rows(s.window), s.kv_heads * d, dtype=z.dtype, device=z.device) for d in (s.dk, s.dv))
             for t, name in ((k, "k"), (v, "v")):
                 ops.gather_rows(t, None, cache, name, batch.key_sources(s.window, True))
-        ops.qk_norm_rope_(z, l, s, *norms, self.freq, self.eps, batch, cache)
+        if s.head_norm:
+            borrows = s.value_source is not None and s.value_source != layer
+            ops.head_norm_rope_(z, l, s, *norms, self.freq, self.eps, batch, cache, *((step.values[s.value_source], self.vmix) if borrows else ()))
+            if s.value_source == layer:
+                step.values[layer] = z[:, l.v:]
+        else:
+            ops.qk_norm_rope_(z, l, s, *norms, self.freq, self.eps, batch, cache)
         if batch.decode:
-            ops.step_attention(z[:, :l.k], o, *sizes, cache, batch)
+            ops.step_attention(z[:, :l.k], o, *sizes, cache, batch, talk)
         else:
             zk, zv = z[:, l.k:l.v], z[:, l.v:]
             if grown:
@@ -109,11 +132,11 @@ class GroupedAttention(_Part):
                     ops.gather_rows(t, src, cache, name, batch.key_sources(s.window, False))
             else:
                 k, v = zk, zv
-            ops.causal_attention(z[:, :l.k], k, v, o, *sizes, batch)
+            ops.causal_attention(z[:, :l.k], k, v, o, *sizes, batch, None, talk)
         return ops.sublayer_out(out, self.linear_out)
 
 
-class LatentAttention(_Part):
+class LatentAttention(Part):
     """Queries ``W_q h``; keys and values of a head are ``W_uk c`` and ``W_uv c`` of the cached latent ``c = norm(W_dkv h)``, which a
     layer with ``source`` takes from that layer.  A prompt expands the latents and runs ordinary attention; a one-token step moves
     ``W_uk`` to the query and ``W_uv`` behind the mix, so that it reads every cached latent once."""
@@ -124,18 +147,18 @@ class LatentAttention(_Part):
         pad, own = round_up(cfg.hidden_size, ROW_PAD), s.source is None
         self.at_c = s.heads * s.dk                                            # columns of the projection: queries | latent | gate
         self.at_g = self.at_c + (s.width if own else 0)
-        self.linear_in = _blank((self.at_g + s.heads * s.dv, pad), cfg, device)
-        self.linear_kv = _blank((s.heads * (s.dk + s.dv), s.width), cfg, device)
-        self.linear_out = _blank((pad, round_up(s.heads * s.dv, ROW_PAD)), cfg, device)
+        self.linear_in = blank((self.at_g + s.heads * s.dv, pad), cfg, device)
+        self.linear_kv = blank((s.heads * (s.dk + s.dv), s.width), cfg, device)
+        self.linear_out = blank((pad, round_up(s.heads * s.dv, ROW_PAD)), cfg, device)
         if own:
             self.c_norm = _norm(s.rank, device, s.width)
 
     def places(self):
         s, d, n = self.s, self.width, self.s.heads * self.s.dk
-        out = {"q": (_heads(self.linear_in, 0, s.heads, s.dk, s.dim, d), (s.heads * s.dim, d)),
-               "g": (_heads(self.linear_in, self.at_g, s.heads, s.dv, s.vdim, d), (s.heads * s.vdim, d)),
-               "uk": (_heads(self.linear_kv, 0, s.heads, s.dk, s.dim, s.rank), (s.heads * s.dim, s.rank)),
-               "uv": (_heads(self.linear_kv, n, s.heads, s.dv, s.vdim, s.rank), (s.heads * s.vdim, s.rank)),
+        out = {"q": (head_rows(self.linear_in, 0, s.heads, s.dk, s.dim, d), (s.heads * s.dim, d)),
+               "g": (head_rows(self.linear_in, self.at_g, s.heads, s.dv, s.vdim, d), (s.heads * s.vdim, d)),
+               "uk": (head_rows(self.linear_kv, 0, s.heads, s.dk, s.dim, s.rank), (s.heads * s.dim, s.rank)),
+               "uv": (head_rows(self.linear_kv, n, s.heads, s.dv, s.vdim, s.rank), (s.heads * s.vdim, s.rank)),
                "o": (self.linear_out[:d, :s.heads * s.dv].view(d, s.heads, s.dv)[..., :s.vdim], (d, s.heads * s.vdim))}
         if s.source is None:
             out["dkv"] = (self.linear_in[self.at_c:self.at_c + s.rank, :d], (s.rank, d))
@@ -158,7 +181,7 @@ class LatentAttention(_Part):
                 ops.gather_rows(c, new, cache, "k", batch.key_sources(None, False))
             step.latents[layer] = c
         gate, n = z[:, self.at_g:], s.heads * s.dk
-        out = _out(h, self.linear_out, s.heads * s.dv)
+        out = activation_rows(h, self.linear_out, s.heads * s.dv)
         o = out[:, :s.heads * s.dv]
         if batch.decode:
             q = ops.latent_absorb(z[:, :n], self.linear_kv[:n], s.heads, s.dk)
@@ -175,21 +198,22 @@ class LatentAttention(_Part):
         return ops.sublayer_out(out, self.linear_out)
 
 
-def _out(h, weight, used: int) -> torch.Tensor:
+def activation_rows(h, weight, used: int) -> torch.Tensor:
     """Input of the output projection; columns that nothing writes are zero."""
     return (torch.empty if weight.shape[1] == used else torch.zeros)(h.shape[0], weight.shape[1], dtype=h.dtype, device=h.device)
 
 
-class GatedMLP(_Part):
-    """``W_down (silu(W_gate h) * (W_up h))``."""
+class GatedMLP(Part):
+    """``W_down (act(W_gate h) * (W_up h))``, SiLU or ReLU."""
     top = 0
 
-    def __init__(self, cfg, ff: int, device):
+    def __init__(self, cfg, ff: int, device, act: str = "silu"):
         super().__init__()
+        self.act = act
         self.ff, self.ffp, self.width = ff, round_up(ff, ROW_PAD), cfg.hidden_size
         pad = round_up(cfg.hidden_size, ROW_PAD)
-        self.linear_fc1 = _blank((2 * self.ffp, pad), cfg, device)
-        self.linear_fc2 = _blank((pad, self.ffp), cfg, device)
+        self.linear_fc1 = blank((2 * self.ffp, pad), cfg, device)
+        self.linear_fc2 = blank((pad, self.ffp), cfg, device)
 
     def places(self):
         d, f = self.width, self.ff
@@ -197,19 +221,19 @@ class GatedMLP(_Part):
                 "down": (self.linear_fc2[:d, :f], (d, f))}
 
     def forward(self, h):
-        return ops.sublayer_out(ops.swiglu_in(h, self.linear_fc1), self.linear_fc2), None
+        return ops.sublayer_out(ops.glu_in(h, self.linear_fc1, self.act), self.linear_fc2), None
 
 
-class SquaredReluExperts(_Part):
+class SquaredReluExperts(Part):
     """Every token's ``top`` experts ``W_down relu(W_up (s h))^2`` with the largest sigmoid scores s, summed."""
 
     def __init__(self, cfg, e: ExpertsSpec, device):
         super().__init__()
         self.e, self.top, self.width = e, e.top, cfg.hidden_size
         pad, ffp = round_up(cfg.hidden_size, ROW_PAD), round_up(e.ff, ROW_PAD)
-        self.router = _blank((round_up(e.experts, 8), pad), cfg, device)
-        self.linear_fc1 = _blank((e.experts, ffp, pad), cfg, device)
-        self.linear_fc2 = _blank((e.experts, pad, ffp), cfg, device)
+        self.router = blank((round_up(e.experts, 8), pad), cfg, device)
+        self.linear_fc1 = blank((e.experts, ffp, pad), cfg, device)
+        self.linear_fc2 = blank((e.experts, pad, ffp), cfg, device)
 
     def places(self):
         d, e = self.width, self.e
@@ -233,7 +257,7 @@ class SandwichBlock(RowBlock):
         self.mix = LatentAttention(cfg, mixer, device) if isinstance(mixer, LatentSpec) else GroupedAttention(cfg, mixer, device)
         self.mix.randomise(cfg.init_method_std, key + ".mix")
         self.norm1, self.norm1b = (_norm(self.width, device, pad) for _ in range(2))
-        self.mlp: Optional[_Part] = None
+        self.mlp: Optional[Part] = None
         if ff is not None:
             self.mlp = GatedMLP(cfg, ff, device) if isinstance(ff, int) else SquaredReluExperts(cfg, ff, device)
             self.mlp.randomise(cfg.init_method_std, key + ".mlp")

@@ -6,7 +6,8 @@ One model class serves every family of the reference: ``GPTModel`` (softmax atte
 hybrid_model.py:28-248, hybrid_transformer_block.py:87-474, sequence_modeling/ssm.py:73-250,
 mamba2/mamba_model.py:16-209 — for the four backbones (qwen2, llama3, mixtral, deepseek_v2), which
 differ only in configuration (attention kind, router order, shared expert, biases).  Layer-list designs (``ModelConfig.layers``)
-build ``ParallelBlock`` (models/parallel_block.py) or ``SandwichBlock`` (models/sandwich_block.py) instead of ``Block``.
+build ``ParallelBlock`` (models/parallel_block.py), ``SandwichBlock`` (models/sandwich_block.py) or ``PostNormBlock``
+(models/post_norm_block.py) instead of ``Block``.
 
 A ``Block`` is one pre-norm residual layer: optional token mixer, optional FFN
 (transformer_layer.py:179-273, mamba_layer.py:27-80).  Module names follow the Megatron-Core
@@ -38,6 +39,7 @@ from .moe import MLP, MoELayer
 from .mom import MomLinearAttention
 from .packed_rows import ROW_PAD, forward_rows, new_slot_cache
 from .parallel_block import ParallelBlock
+from .post_norm_block import PostNormBlock
 from .sandwich_block import SandwichBlock
 
 
@@ -87,6 +89,8 @@ def build_block(cfg: ModelConfig, spec: LayerSpec, mesh: Mesh, key: str, sp: boo
         return ParallelBlock(cfg, spec, key, device)
     if spec.symbol == "S":
         return SandwichBlock(cfg, spec, key, device)
+    if spec.symbol == "P":
+        return PostNormBlock(cfg, spec, key, device)
     return Block(cfg, spec, mesh, key, sp, device)
 
 

@@ -323,9 +323,11 @@ def softmax_attention(q, k, v, scale=None, causal=True, q_offset: int = 0, windo
 
 # ---- packed-row operators (serving only) -----------------------------------------------------------
 from .chunk_attn import chunk_attention, embed_norm, poly_norm, stream_norm   # noqa: E402,F401
+from .group_norm import embed_rows, group_norm, residual_group_norm, softcap_   # noqa: E402,F401
 from .moe_rows import experts_relu2   # noqa: E402,F401
-from .packed_attn import (causal_attention, gather_rows, latent_absorb, latent_norm, latent_up, qk_norm_rope_,   # noqa: E402,F401
-                          residual_norm, step_attention, sublayer_out, swiglu_in)
+from .packed_attn import (causal_attention, gather_rows, glu_in, head_norm_rope_, latent_absorb, latent_norm, latent_up,   # noqa: E402,F401
+                          qk_norm_rope_, residual_norm, rotate_heads_, step_attention, sublayer_out)
+from .retention import retention   # noqa: E402,F401
 
 
 # ---- linear sequence models -----------------------------------------------

@@ -138,8 +138,9 @@ def dense(a: torch.Tensor, b: torch.Tensor, a_mn: bool = False, b_mn: bool = Fal
     return out
 
 
-def dense_swiglu(x: torch.Tensor, w: torch.Tensor, want_pre: bool = True, band: Optional[int] = None, out_shape=None):
-    """``silu(x Wg^T) * (x Wu^T)`` for ``w = [Wg ; Wu]`` (``[2F, K]``, the ordinary fc1 layout) with the activation in
+def dense_swiglu(x: torch.Tensor, w: torch.Tensor, want_pre: bool = True, band: Optional[int] = None, out_shape=None,
+                 relu: bool = False):
+    """``silu(x Wg^T) * (x Wu^T)`` (``relu``: ReLU in place of SiLU) for ``w = [Wg ; Wu]`` (``[2F, K]``, the ordinary fc1 layout) with the activation in
     the GEMM epilogue.  Returns ``(act [M,F], pre [M,2F] or None)``; ``pre`` is what the backward pass needs."""
     from . import cuda as K
     M, Kd = x.shape
@@ -150,7 +151,7 @@ def dense_swiglu(x: torch.Tensor, w: torch.Tensor, want_pre: bool = True, band: 
     rc = K.lib().lmoe_gemm_dense_swiglu(K._p(x), ctypes.c_int(x.stride(0)), K._p(w), ctypes.c_int(w.stride(0)), K._p(act),
                                         ctypes.c_int(Fh), K._p(pre), ctypes.c_int(F2), ctypes.c_int(M),
                                         ctypes.c_int(Fh), ctypes.c_int(Kd), ctypes.c_int(BAND if band is None else band),
-                                        K._p(_err(x.device)), ctypes.c_int(K.NUM_SMS), K._st())
+                                        ctypes.c_int(int(relu)), K._p(_err(x.device)), ctypes.c_int(K.NUM_SMS), K._st())
     K._check(rc, "gemm_dense_swiglu")
     return act, pre
 

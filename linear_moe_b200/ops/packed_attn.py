@@ -1,9 +1,9 @@
 """Softmax attention over packed rows with a cache, and the row operators of blocks that norm both ends of a sublayer.
 
-Two kinds of attention share the kernels: grouped-query attention (optional norm over the whole query and key projections, optional
-interleaved rotary positions, optional sliding window) and latent attention (keys and values are products of one cached latent row
-per token).  Operators work on packed rows (:class:`~linear_moe_b200.ops.row_batch.RowBatch`).  CUDA tensors (bf16 or fp32) take the kernels of
-``csrc/packed_attn*.cu``, ``csrc/latent_step.cu`` and ``csrc/sandwich_block.cu``; CPU tensors take the eager definitions of
+Two kinds of attention share the kernels: grouped-query attention (optional norm over the whole query and key projections or over every
+head, optional rotary positions in either pairing, optional sliding window, optional talking heads, optional norm and mixing of the values)
+and latent attention (keys and values are products of one cached latent row per token).  Operators work on packed rows (:class:`~linear_moe_b200.ops.row_batch.RowBatch`).  CUDA tensors (bf16 or fp32) take the kernels of
+``csrc/packed_attn*.cu``, ``csrc/talk_step.cu``, ``csrc/latent_step.cu`` and ``csrc/sandwich_block.cu``; CPU tensors take the eager definitions of
 :mod:`linear_moe_b200.ref.packed_attn`.  These operators serve (no backward pass).
 
 Head sizes and latents are laid out in multiples of 16 and 32 (zero weight rows), so every size meets the kernels' alignment.
@@ -11,6 +11,7 @@ Head sizes and latents are laid out in multiples of 16 and 32 (zero weight rows)
 from __future__ import annotations
 
 import ctypes
+import math
 from dataclasses import dataclass
 from typing import Optional
 
@@ -20,6 +21,39 @@ from ..ref import packed_attn as RP
 from .row_batch import RowBatch, round_up
 
 ROWS_SMEM = 227 * 1024 // 4   # floats of shared memory a prompt kernel for any head size may use
+
+
+@dataclass(frozen=True)
+class RotaryScaling:
+    """YaRN: pairs that turn less than ``slow`` times over ``original`` positions are slowed down by ``factor``, those that turn more than
+    ``fast`` times are not, and the ones between are blended; queries and keys grow a little with ``factor`` (Peng et al., "YaRN:
+    Efficient Context Window Extension of Large Language Models")."""
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+    def __post_init__(self):
+        if not min(self.factor, self.original, self.fast, self.slow) > 0:
+            raise ValueError("rotary scaling needs positive numbers")
+
+    @property
+    def size(self) -> float:
+        return 0.1 * math.log(self.factor) + 1.0
+
+
+def rotary_frequencies(dims: int, base: float, scaling: Optional[RotaryScaling] = None) -> torch.Tensor:
+    """Angle per position of every pair, fp64 ``[dims / 2]``."""
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    f = float(base) ** (-2.0 * i / max(dims, 1))
+    if scaling is None or not dims:
+        return f
+
+    def pair(turns: float) -> float:                                  # number of the pair that turns so often over `original`
+        return dims * math.log(scaling.original / (2 * math.pi * turns)) / (2 * math.log(base))
+    lo, hi = max(math.floor(pair(scaling.fast)), 0), min(math.ceil(pair(scaling.slow)), dims - 1)
+    ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0, 1)
+    return f / scaling.factor * ramp + f * (1 - ramp)
 
 
 @dataclass(frozen=True)
@@ -34,6 +68,12 @@ class AttentionSpec:
     rot_dims: int = 0                 # leading dimensions of a head that are rotated, in neighbouring pairs
     rot_base: float = 10000.0
     qk_norm: bool = False             # RMS norm over the whole query (key) projection, before the heads are split
+    head_norm: bool = False           # RMS norm of every query and key head, with one weight per dimension for all heads
+    rot_halves: bool = False          # pairs (i, i + rot_dims / 2) instead of neighbours (with head_norm)
+    rot_scaling: Optional[RotaryScaling] = None
+    value_norm: bool = False          # every value head over its root mean square (with head_norm)
+    talk: bool = False                # the softmax weights of the heads are mixed by a [heads, heads] table
+    value_source: Optional[int] = None    # layer whose values are mixed into this one's (its own number: it only lends them)
 
     def __post_init__(self):
         if min(self.heads, self.kv_heads, self.dim, self.vdim) < 1 or (self.window is not None and self.window < 1):
@@ -42,6 +82,10 @@ class AttentionSpec:
             raise ValueError(f"{self.heads} query heads do not share {self.kv_heads} key/value heads evenly")
         if self.rot_dims % 2 or not 0 <= self.rot_dims <= self.dim:
             raise ValueError(f"{self.rot_dims} rotated dimensions in a head of {self.dim}")
+        if self.qk_norm and self.head_norm:
+            raise ValueError("queries and keys are normed as a whole or by head")
+        if not self.head_norm and (self.rot_halves or self.value_norm or self.rot_scaling or self.value_source is not None):
+            raise ValueError("rotation of halves, rotary scaling and operations on values come with the norm by head")
         _check_scale(self.scale)
 
     @property
@@ -53,10 +97,11 @@ class AttentionSpec:
         return round_up(self.vdim, 16)
 
     def frequencies(self, device) -> Optional[torch.Tensor]:
-        if not self.rot_dims:
-            return None
-        i = torch.arange(self.rot_dims // 2, dtype=torch.float64)
-        return (float(self.rot_base) ** (-2.0 * i / self.rot_dims)).to(device)
+        return rotary_frequencies(self.rot_dims, self.rot_base, self.rot_scaling).to(device) if self.rot_dims else None
+
+    @property
+    def rot_size(self) -> float:
+        return 1.0 if self.rot_scaling is None else self.rot_scaling.size
 
 
 @dataclass(frozen=True)
@@ -116,7 +161,8 @@ def _fields(**groups):
 
 
 class _Prompt(ctypes.Structure):
-    _fields_ = _fields(a=(_P, "q k v gate out items err"), b=(_LL, "ldq ldk ldv ldg ldo"), c=(_I, "H G dk dv window n q_rows k_rows"), d=(_F, "scale"))
+    _fields_ = _fields(a=(_P, "q k v gate out items err"), b=(_LL, "ldq ldk ldv ldg ldo"), c=(_I, "H G dk dv window n q_rows k_rows"), d=(_F, "scale"),
+                       e=(_I, "cross"))
 
 
 class _Cache(ctypes.Structure):
@@ -124,12 +170,22 @@ class _Cache(ctypes.Structure):
 
 
 class _Step(ctypes.Structure):
-    _fields_ = _fields(a=(_P, "q out"), b=(_Cache, "c"), c=(_P, "pos slots"), d=(_LL, "ldq ldo"), e=(_I, "H G dk dv window n"), f=(_F, "scale"))
+    _fields_ = _fields(a=(_P, "q out"), b=(_Cache, "c"), c=(_P, "pos slots"), d=(_LL, "ldq ldo"), e=(_I, "H G dk dv window n"), f=(_F, "scale"),
+                       g=(_I, "cross"))
 
 
 class _QkNorm(ctypes.Structure):
     _fields_ = _fields(a=(_P, "z wq wk freq"), b=(_Cache, "c"), c=(_P, "pos slots ends"), d=(_LL, "ldz"),
                        e=(_I, "zq zk zv H G dk dv nq nk rot"), f=(_F, "eps"), g=(_I, "rows"))
+
+
+class _HeadNorm(ctypes.Structure):
+    _fields_ = _fields(a=(_P, "z wq wk freq first mix"), b=(_Cache, "c"), c=(_P, "pos slots ends"), d=(_LL, "ldz ldf"),
+                       e=(_I, "zq zk zv H G V dk dv nk nv rot halves norm_v"), f=(_F, "size eps"), g=(_I, "rows"))
+
+
+class _TalkStep(ctypes.Structure):
+    _fields_ = _fields(a=(_Step, "s"), b=(_P, "table scores parts"), c=(_LL, "lds"))
 
 
 class _LatentNorm(ctypes.Structure):
@@ -162,11 +218,12 @@ def _ptr(t: Optional[torch.Tensor]) -> int:
 
 # --------------------------------------------------------------------------------------------------------------- attention
 def causal_attention(q, k, v, out, heads: int, kv_heads: int, dk: int, dv: int, scale: float, window: Optional[int], batch: RowBatch,
-                     gate: Optional[torch.Tensor] = None):
+                     gate: Optional[torch.Tensor] = None, talk: Optional[torch.Tensor] = None):
     """Prompts: ``out [rows, heads * dv] = softmax(q . k * scale) v`` (times ``sigmoid(gate)``), ``q [rows, heads * dk]``; ``k``, ``v``
-    ``[key rows, kv_heads * d]`` in the order of ``batch.key_sources`` (the rows themselves when no request goes on from a cache)."""
+    ``[key rows, kv_heads * d]`` in the order of ``batch.key_sources`` (the rows themselves when no request goes on from a cache).
+    ``talk [heads, heads]`` (fp32): head h mixes its values with ``sum_g talk[h, g] softmax_g``."""
     if not q.is_cuda:
-        return RP.causal_attention(q, k, v, out, heads, kv_heads, dk, dv, scale, window, batch, gate)
+        return RP.causal_attention(q, k, v, out, heads, kv_heads, dk, dv, scale, window, batch, gate, talk)
     from . import cuda as K
     from . import gemm
     _no_grad(q, k, v, gate)
@@ -179,6 +236,8 @@ def causal_attention(q, k, v, out, heads: int, kv_heads: int, dk: int, dv: int, 
     a.q_rows, a.k_rows = q.shape[0], k.shape[0]
     dt = K._dt(q)
     fast = dt == 1 and dk <= 128 and dv <= 128
+    if talk is not None:
+        return _talk_prompt(a, q, out, talk, window, batch, fast)
     tile = 128 if fast else 32 if 64 * (dk + 1) + 64 * dv + 32 * 33 <= ROWS_SMEM else 16
     items = batch.causal_items(window, tile)
     a.items, a.n = items.data_ptr(), items.shape[0]
@@ -187,6 +246,38 @@ def causal_attention(q, k, v, out, heads: int, kv_heads: int, dk: int, dv: int, 
         K._check(K.lib().lmoe_packed_attn_tc(ctypes.byref(a), K._st()), "packed_attn_tc")
     else:
         K._check(K.lib().lmoe_packed_attn_rows(ctypes.byref(a), tile, dt, K._st()), "packed_attn_rows")
+
+
+TALK_BYTES = 1 << 30          # room for the softmax outputs of all heads over all value heads; longer prompts go in parts
+
+
+def _talk_prompt(a: _Prompt, q, out, talk, window: Optional[int], batch: RowBatch, fast: bool):
+    """Mixing the weights and then applying them to the values is, the sums exchanged, applying every head's weights to every value head
+    and mixing the results: the softmax stays online and no weight leaves the tensor core."""
+    from . import cuda as K
+    from . import gemm
+    assert not a.gate and talk.shape == (a.H, a.H) and talk.dtype == torch.float32 and talk.is_contiguous()
+    dt, width = K._dt(q), a.H * a.G * a.dv
+    tile = 128 if fast else 32 if 64 * (a.dk + 1) + 64 * a.dv + 32 * 33 <= ROWS_SMEM else 16
+    many = max(TALK_BYTES // (width * q.element_size()) // tile * tile, tile)
+    for r0, r1, items in batch.causal_parts(window, tile, many):
+        each = torch.empty(r1 - r0, width, dtype=q.dtype, device=q.device)
+        a.items, a.n, a.cross = items.data_ptr(), items.shape[0], 1
+        a.out, a.ldo = each.data_ptr() - r0 * width * q.element_size(), width          # row r0 is the buffer's first
+        if fast:
+            a.err = gemm._err(q.device).data_ptr()
+            K._check(K.lib().lmoe_packed_attn_tc(ctypes.byref(a), K._st()), "packed_attn_tc")
+        else:
+            K._check(K.lib().lmoe_packed_attn_rows(ctypes.byref(a), tile, dt, K._st()), "packed_attn_rows")
+        head_mix(each, talk, out[r0:r1], a.H, a.G, a.dv)
+
+
+def head_mix(x, talk, out, heads: int, kv_heads: int, dv: int):
+    """``x [n, heads, kv_heads, dv]`` (a head's weights over every value head) -> ``out[n, h] = sum_g talk[h, g] x[n, g, value head of h]``."""
+    from . import cuda as K
+    ld = ctypes.c_longlong
+    K._check(K.lib().lmoe_head_mix(K._p(x), ld(x.stride(0)), K._p(talk), K._p(out), ld(out.stride(0)), x.shape[0], heads, kv_heads, dv, K._dt(x), K._st()),
+             "head_mix")
 
 
 def step_splits(requests: int, heads: int, kv_heads: int, dk: int, dv: int, shared: bool, rows: Optional[int], sms: int) -> int:
@@ -207,10 +298,12 @@ def _step_bytes(dk: int, dv: int, shared: bool) -> int:
     return max(2 * blocks * keys * 128, 64 * (dv + 4)) + 32 * (dk + 8) + 512 * (keys + 4) + 32 * (keys + 8) + 192 + 1024
 
 
-def step_attention(q, out, heads: int, kv_heads: int, dk: int, dv: int, scale: float, window: Optional[int], cache: dict, batch: RowBatch):
-    """One token per request, whose key and value are in the cache already: ``q [n, heads * dk]`` -> ``out [n, heads * dv]``."""
+def step_attention(q, out, heads: int, kv_heads: int, dk: int, dv: int, scale: float, window: Optional[int], cache: dict, batch: RowBatch,
+                   talk: Optional[torch.Tensor] = None):
+    """One token per request, whose key and value are in the cache already: ``q [n, heads * dk]`` -> ``out [n, heads * dv]``; ``talk`` as
+    in ``causal_attention``."""
     if not q.is_cuda:
-        return RP.step_attention(q, out, heads, kv_heads, dk, dv, scale, window, cache, batch)
+        return RP.step_attention(q, out, heads, kv_heads, dk, dv, scale, window, cache, batch, talk)
     from . import cuda as K
     from . import gemm
     _no_grad(q)
@@ -219,12 +312,47 @@ def step_attention(q, out, heads: int, kv_heads: int, dk: int, dv: int, scale: f
     a.q, a.out, a.c, a.pos, a.slots = q.data_ptr(), out.data_ptr(), _cache_args(cache), batch.pos.data_ptr(), batch.slot.data_ptr()
     a.ldq, a.ldo, a.H, a.G, a.dk, a.dv, a.window, a.n, a.scale = q.stride(0), out.stride(0), heads, kv_heads, dk, dv, window or 0, q.shape[0], scale
     dt, shared = K._dt(q), cache["v"].data_ptr() == cache["k"].data_ptr()
+    if talk is not None:
+        return _talk_step(a, q, out, talk, cache)
     if dt == 1 and dk % 16 == 0 and dv % 16 == 0 and max(dk, dv) <= 512 and _step_bytes(dk, dv, shared) < 224 * 1024:
         rows = cache["k"].shape[0] * cache["k"].shape[1]
         splits = step_splits(q.shape[0], heads, kv_heads, dk, dv, shared, None if "table" in cache else cache["k"].shape[1], K.num_sms())
         K._check(K.lib().lmoe_packed_attn_step(ctypes.byref(a), rows, splits, K._p(gemm._err(q.device)), K._st()), "packed_attn_step")
     else:
         K._check(K.lib().lmoe_packed_attn_step_any(ctypes.byref(a), dt, K._st()), "packed_attn_step_any")
+
+
+TALK_HEADS = 256              # heads whose mixing table the one-token kernel keeps in shared memory (8 rows of it)
+
+
+def talk_splits(requests: int, heads: int, kv_heads: int, rows: int, sms: int) -> int:
+    """CTAs (1 - 8, one cluster) that share the keys of a (request, kv head, 8 heads): about four per SM, with at least 64 keys each when
+    the ``rows`` cached ones are all in use."""
+    ctas = requests * kv_heads * -(-(heads // kv_heads) // 8)
+    s = 1
+    while s < 8 and ctas * s * 2 <= 4 * sms and rows >= 128 * s:
+        s *= 2
+    return s
+
+
+def _talk_step(a: _Step, q, out, talk, cache: dict):
+    """Scores of all heads first, then every value head's mix of them: two passes, each of which reads its half of the cache once."""
+    from . import cuda as K
+    assert talk.shape == (a.H, a.H) and talk.dtype == torch.float32 and talk.is_contiguous()
+    n, dev, dt = q.shape[0], q.device, K._dt(q)
+    rows = cache["table"].stride(0) * cache["k"].shape[1] if "table" in cache else cache["k"].shape[1]      # of one request
+    if dt == 1 and a.dk % 16 == 0 and a.dv % 16 == 0 and max(a.dk, a.dv) <= 128 and a.H <= TALK_HEADS:
+        splits, t = talk_splits(n, a.H, a.G, rows, K.num_sms()), _TalkStep()
+        ld = round_up(rows, 64)
+        scores = torch.empty(n, a.H, ld, dtype=torch.float32, device=dev)
+        parts = torch.empty(n, a.H, splits, 2, dtype=torch.float32, device=dev)
+        t.s, t.table, t.scores, t.parts, t.lds = a, talk.data_ptr(), scores.data_ptr(), parts.data_ptr(), ld
+        K._check(K.lib().lmoe_talk_step(ctypes.byref(t), splits, K._st()), "talk_step", 2)
+        return
+    each = torch.empty(n, a.H * a.G * a.dv, dtype=q.dtype, device=dev)
+    a.out, a.ldo, a.cross = each.data_ptr(), each.stride(0), 1
+    K._check(K.lib().lmoe_packed_attn_step_any(ctypes.byref(a), dt, K._st()), "packed_attn_step_any")
+    head_mix(each, talk, out, a.H, a.G, a.dv)
 
 
 def gather_rows(dst, src: Optional[torch.Tensor], cache: Optional[dict], name: str, meta: torch.Tensor):
@@ -255,6 +383,43 @@ def qk_norm_rope_(z, lay: QkvLayout, spec: AttentionSpec, wq, wk, freq, eps: flo
     a.ldz, a.zq, a.zk, a.zv = z.stride(0), lay.q, lay.k, lay.v
     a.H, a.G, a.dk, a.dv, a.nq, a.nk, a.rot, a.eps, a.rows = spec.heads, spec.kv_heads, spec.dk, spec.dv, nq, nk, spec.rot_dims, eps, z.shape[0]
     K._check(K.lib().lmoe_qk_norm_rope(ctypes.byref(a), K._dt(z), K._st()), "qk_norm_rope")
+
+
+def head_norm_rope_(z, lay: QkvLayout, spec: AttentionSpec, wq, wk, freq, eps: float, batch: RowBatch, cache: Optional[dict],
+                    first: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None):
+    """Norm every query, key and value head of a projection's output and rotate queries and keys, in place; keys and values enter the
+    cache.  ``first``, ``mix``: values become ``(1 - mix) v + mix first`` behind their norm (``mix`` one fp32 number)."""
+    if not z.is_cuda:
+        return RP.head_norm_rope_(z, lay, spec, wq, wk, freq, eps, batch, cache, first, mix)
+    a = _head_args(z, lay.q, lay.k, spec.heads, spec.kv_heads, spec.dk, spec.rot_dims, spec.rot_halves, freq, spec.rot_size, batch)
+    a.wq, a.wk, a.c, a.ends = _ptr(wq), _ptr(wk), _cache_args(cache), _ptr(batch.end)
+    a.zv, a.V, a.dv, a.nk, a.nv, a.norm_v, a.eps = lay.v, spec.kv_heads, spec.dv, spec.dim, spec.vdim, int(spec.value_norm), eps
+    if first is not None:
+        assert first.dtype == z.dtype and first.shape == (z.shape[0], spec.kv_heads * spec.dv) and first.stride(1) == 1
+        a.first, a.ldf, a.mix = first.data_ptr(), first.stride(0), mix.data_ptr()
+    _head_launch(a, z)
+
+
+def rotate_heads_(z, at_q: int, at_k: int, heads: int, kv_heads: int, dk: int, dims: int, halves: bool, freq, size: float, batch: RowBatch):
+    """Rotate the first ``dims`` dimensions of every query and key head in place."""
+    if not dims:
+        return
+    if not z.is_cuda:
+        return RP.rotate_heads_(z, at_q, at_k, heads, kv_heads, dk, halves, freq, size, batch)
+    _head_launch(_head_args(z, at_q, at_k, heads, kv_heads, dk, dims, halves, freq, size, batch), z)
+
+
+def _head_args(z, at_q, at_k, heads, kv_heads, dk, dims, halves, freq, size, batch) -> _HeadNorm:
+    _no_grad(z)
+    a = _HeadNorm()
+    a.z, a.freq, a.pos, a.slots, a.ldz, a.zq, a.zk = z.data_ptr(), _ptr(freq), batch.pos.data_ptr(), batch.slot.data_ptr(), z.stride(0), at_q, at_k
+    a.H, a.G, a.dk, a.nk, a.rot, a.halves, a.size, a.rows = heads, kv_heads, dk, dk, dims, int(halves), size, z.shape[0]
+    return a
+
+
+def _head_launch(a: _HeadNorm, z):
+    from . import cuda as K
+    K._check(K.lib().lmoe_head_norm_rope(ctypes.byref(a), K._dt(z), K._st()), "head_norm_rope")
 
 
 def latent_norm(z, weight, rank: int, eps: float, batch: RowBatch, cache: Optional[dict]) -> torch.Tensor:
@@ -330,19 +495,22 @@ def sublayer_out(x, weight) -> torch.Tensor:
     return linear_f32(x, weight) if x.shape[0] <= FEW_ROWS else linear(x, weight)
 
 
-def swiglu_in(h, w1) -> torch.Tensor:
-    """``silu(h Wg^T) * (h Wu^T)`` for ``w1 = [Wg; Wu]``: in the epilogue of the product for many bf16 rows, else a kernel after it."""
+ACTIVATIONS = ("silu", "relu")            # as numbered in csrc/gemm_dense.cu and csrc/sandwich_block.cu
+
+
+def glu_in(h, w1, act: str = "silu") -> torch.Tensor:
+    """``act(h Wg^T) * (h Wu^T)`` for ``w1 = [Wg; Wu]``: in the epilogue of the product for many bf16 rows, else a kernel after it."""
     from . import linear
     if not h.is_cuda:
         g, u = linear(h, w1).float().chunk(2, -1)
-        return (torch.nn.functional.silu(g) * u).to(h.dtype)
+        return (getattr(torch.nn.functional, act)(g) * u).to(h.dtype)
     from . import cuda as K
     from . import gemm
     _no_grad(h, w1)
     if h.shape[0] > 16 and gemm.dense_ok(h, w1) and w1.shape[0] % 16 == 0:
-        return gemm.dense_swiglu(h, w1, want_pre=False)[0]
+        return gemm.dense_swiglu(h, w1, want_pre=False, relu=act == "relu")[0]
     z = linear(h, w1)
     ff, ld = w1.shape[0] // 2, ctypes.c_longlong
     out = torch.empty(z.shape[0], ff, dtype=z.dtype, device=z.device)
-    K._check(K.lib().lmoe_swiglu_rows(K._p(z), ld(z.stride(0)), K._p(out), ld(ff), z.shape[0], ff, K._dt(z), K._st()), "swiglu_rows")
+    K._check(K.lib().lmoe_glu_rows(K._p(z), ld(z.stride(0)), K._p(out), ld(ff), z.shape[0], ff, ACTIVATIONS.index(act), K._dt(z), K._st()), "glu_rows")
     return out

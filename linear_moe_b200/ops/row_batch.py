@@ -100,6 +100,45 @@ class RowBatch:
             return self._table(key, out)
         return self._items[key]
 
+    def causal_parts(self, window: Optional[int], tile: int, rows: int) -> list:
+        """``(first row, end, work items)`` of consecutive parts of at most ``rows`` rows each (``rows`` at least ``tile``)."""
+        key = ("parts", window, tile, rows)
+        if key not in self._items:
+            whole = self.causal_items(window, tile)
+            if self.rows <= rows:
+                self._items[key] = [(0, self.rows, whole)]
+            else:
+                table, parts, i = sorted(whole.tolist()), [], 0
+                while i < len(table):
+                    first, j = table[i][0], i + 1
+                    while j < len(table) and table[j][0] + table[j][1] - first <= rows:
+                        j += 1
+                    part = sorted(table[i:j], key=lambda t: -(t[2] + t[1] if window is None else min(t[2] + t[1], window + tile)))
+                    parts.append((first, table[j - 1][0] + table[j - 1][1], self._table(key + (first,), part)))
+                    i = j
+                self._items[key] = parts
+        return self._items[key]
+
+    def recurrent_groups(self, tokens: int):
+        """Every request's new tokens in groups of at most ``tokens``: ``(groups, states, requests)`` as int32 tables (``csrc/retention.cuh``).
+        A group is (first row, tokens, slot, flags, state in front, state behind): flag 1: the request's first group, flag 2: its last one,
+        flag 4: the request has a past; the states are places in a buffer of ``states`` (-1: none).  Requests of more than one group are
+        listed as (slot, flags, first state, groups, tokens of a group); ``None`` when there are none."""
+        key = ("recurrent", tokens)
+        if key not in self._items:
+            groups, many, states = [], [], 0
+            for r, n in enumerate(self.counts):
+                slot, past, count = 0 if self.slots is None else self.slots[r], 4 if self.starts[r] else 0, -(-n // tokens)
+                if count > 1:
+                    many.append((slot, past, states, count, tokens, 0, 0, 0))
+                for i in range(count):
+                    last = i == count - 1
+                    groups.append((self.row0[r] + i * tokens, n - i * tokens if last else tokens, slot, past + (i == 0) + 2 * last,
+                                   states + i - 1 if i else -1, -1 if last else states + i, 0, 0))
+                states += count - 1
+            self._items[key] = (self._table(key + (0,), groups), states, self._table(key + (1,), many) if many else None)
+        return self._items[key]
+
     def key_sources(self, window: Optional[int], cached: bool) -> torch.Tensor:
         """Where rows of the key matrix come from, ``[n, 4]`` int32 (destination, new row or -1, slot, position): the cached
         ones, or the new ones."""

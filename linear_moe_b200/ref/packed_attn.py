@@ -27,31 +27,35 @@ def store(cache: dict, name: str, slot: int, positions: torch.Tensor, rows: torc
     buf.view(-1, *buf.shape[2:])[_places(cache, slot, positions)] = rows.to(buf.dtype)
 
 
-def mix(q, k, v, scale: float, first_query: int, window: Optional[int]):
-    """``q [n, H, d]`` at key indices ``first_query ..``, ``k [m, G, d]``, ``v [m, G, e]`` -> ``[n, H, e]`` (fp32)."""
+def mix(q, k, v, scale: float, first_query: int, window: Optional[int], talk=None):
+    """``q [n, H, d]`` at key indices ``first_query ..``, ``k [m, G, d]``, ``v [m, G, e]`` -> ``[n, H, e]`` (fp32).  ``talk [H, H]`` mixes
+    the heads' weights."""
     n, H, G = q.shape[0], q.shape[1], k.shape[1]
     i, j = torch.arange(first_query, first_query + n)[:, None], torch.arange(k.shape[0])[None, :]
     hidden = j > i if window is None else (j > i) | (j <= i - window)
     s = torch.einsum("ihd,jhd->hij", q.float(), k.float().repeat_interleave(H // G, 1)) * scale
-    return torch.einsum("hij,jhd->ihd", s.masked_fill(hidden, float("-inf")).softmax(-1), v.float().repeat_interleave(H // G, 1))
+    w = s.masked_fill(hidden, float("-inf")).softmax(-1)
+    if talk is not None:
+        w = torch.einsum("hg,gij->hij", talk.float(), w)
+    return torch.einsum("hij,jhd->ihd", w, v.float().repeat_interleave(H // G, 1))
 
 
-def causal_attention(q, k, v, out, H, G, dk, dv, scale, window, batch, gate):
+def causal_attention(q, k, v, out, H, G, dk, dv, scale, window, batch, gate, talk=None):
     krow = 0
     for r, (past, n) in enumerate(zip(batch.past(window), batch.counts)):
         a, b = batch.row0[r], batch.row0[r + 1]
         ks = slice(krow, krow + past + n)
-        o = mix(q[a:b].reshape(n, H, dk), k[ks].reshape(-1, G, dk), v[ks].reshape(-1, G, dv), scale, past, window).reshape(n, H * dv)
+        o = mix(q[a:b].reshape(n, H, dk), k[ks].reshape(-1, G, dk), v[ks].reshape(-1, G, dv), scale, past, window, talk).reshape(n, H * dv)
         out[a:b] = (o if gate is None else o * torch.sigmoid(gate[a:b].float())).to(out.dtype)
         krow += past + n
 
 
-def step_attention(q, out, H, G, dk, dv, scale, window, cache, batch):
+def step_attention(q, out, H, G, dk, dv, scale, window, cache, batch, talk=None):
     for r, (p, slot) in enumerate(zip(batch.pos.tolist(), batch.slot.tolist())):
         span = window if "table" in cache else cache["k"].shape[1]
         at = torch.arange(0 if span is None else max(0, p + 1 - span), p + 1)
         k, v = cache_rows(cache, "k", slot, at), cache_rows(cache, "v", slot, at)
-        out[r] = mix(q[r:r + 1].reshape(1, H, dk), k, v, scale, len(at) - 1, None).reshape(-1).to(out.dtype)
+        out[r] = mix(q[r:r + 1].reshape(1, H, dk), k, v, scale, len(at) - 1, None, talk).reshape(-1).to(out.dtype)
 
 
 def rotate_pairs(x, pos, freq):
@@ -71,12 +75,57 @@ def qk_norm_rope_(z, lay, H, G, dk, dv, nq, nk, wq, wk, freq, eps, batch, cache)
             x = x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) / numbers + eps) * w
         x = x.reshape(-1, heads, dk)
         z[:, at:at + heads * dk] = (x if freq is None else rotate_pairs(x, batch.pos, freq)).reshape(-1, heads * dk).to(z.dtype)
+    _store_rows(z, lay, G, dk, dv, batch, cache)
+
+
+def _store_rows(z, lay, G, dk, dv, batch, cache):
     if cache is None:
         return
     for r, slot in enumerate(batch.slot.tolist()):
         p = batch.pos[r:r + 1].long()
         store(cache, "k", slot, p, z[r:r + 1, lay.k:lay.k + G * dk].reshape(1, G, dk))
         store(cache, "v", slot, p, z[r:r + 1, lay.v:lay.v + G * dv].reshape(1, G, dv))
+
+
+def rotate_halves(x, pos, freq, size):
+    """``x [n, heads, d]``: dimensions i and i + len(freq) turn by ``pos * freq[i]`` and grow by ``size``."""
+    angle, half = pos.double()[:, None] * freq[None, :], len(freq)
+    c, s = (size * torch.cos(angle)).float()[:, None], (size * torch.sin(angle)).float()[:, None]
+    y, u, v = x.clone(), x[..., :half], x[..., half:2 * half]
+    y[..., :half], y[..., half:2 * half] = u * c - v * s, v * c + u * s
+    return y
+
+
+def _turn(x, pos, halves, freq, size):
+    if freq is None:
+        return x
+    if halves:
+        return rotate_halves(x, pos, freq, size)
+    y = rotate_pairs(x, pos, freq)
+    y[..., :2 * len(freq)] *= size
+    return y
+
+
+def rotate_heads_(z, at_q, at_k, heads, kv_heads, dk, halves, freq, size, batch):
+    for at, n in ((at_q, heads), (at_k, kv_heads)):
+        x = z[:, at:at + n * dk].float().reshape(-1, n, dk)
+        z[:, at:at + n * dk] = _turn(x, batch.pos, halves, freq, size).reshape(-1, n * dk).to(z.dtype)
+
+
+def head_norm_rope_(z, lay, s, wq, wk, freq, eps, batch, cache, first, mix):
+    for at, n, w in ((lay.q, s.heads, wq), (lay.k, s.kv_heads, wk)):
+        x = z[:, at:at + n * s.dk].float().reshape(-1, n, s.dk)
+        x = x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) / s.dim + eps) * w
+        z[:, at:at + n * s.dk] = _turn(x, batch.pos, s.rot_halves, freq, s.rot_size).reshape(-1, n * s.dk).to(z.dtype)
+    at = slice(lay.v, lay.v + s.kv_heads * s.dv)
+    v = z[:, at].float().reshape(-1, s.kv_heads, s.dv)
+    if s.value_norm:
+        v = v * torch.rsqrt(v.pow(2).sum(-1, keepdim=True) / s.vdim + eps)
+    v = v.reshape(-1, s.kv_heads * s.dv)
+    if first is not None:
+        v = (1 - mix) * v + mix * first.float()
+    z[:, at] = v.to(z.dtype)
+    _store_rows(z, lay, s.kv_heads, s.dk, s.dv, batch, cache)
 
 
 def latent_norm(z, weight, rank, eps, batch, cache):

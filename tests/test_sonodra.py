@@ -184,7 +184,7 @@ def test_norms_with_a_weight_per_column(where):
 def test_gated_feed_forward(where, rows):
     dev, dt = where[0], getattr(torch, where[1])
     h, w1, w2 = torch.randn(rows, 64).to(dt), (torch.randn(2 * 96, 64) * 0.2).to(dt), (torch.randn(64, 96) * 0.1).to(dt)
-    got = PA.sublayer_out(PA.swiglu_in(h.to(dev), w1.to(dev)), w2.to(dev))
+    got = PA.sublayer_out(PA.glu_in(h.to(dev), w1.to(dev)), w2.to(dev))
     want = O.dense(h.double(), {"gate": w1[:96].double(), "up": w1[96:].double(), "down": w2.double()})
     assert rel(got, want) < tol(where)
 
