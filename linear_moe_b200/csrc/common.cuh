@@ -82,6 +82,22 @@ template <> struct Vec<float> {
     __device__ __forceinline__ void set(int i, float v) { reinterpret_cast<float*>(&raw)[i] = v; }
 };
 
+// Four consecutive numbers as fp32 (16-byte aligned fp32, 8-byte aligned bf16).
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const bf16* p) {
+    const uint2 r = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void store4(float* y, float4 v) { *reinterpret_cast<float4*>(y) = v; }
+__device__ __forceinline__ void store4(bf16* y, float4 v) {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    uint2 r;
+    r.x = *reinterpret_cast<uint32_t*>(&lo);
+    r.y = *reinterpret_cast<uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(y) = r;
+}
+
 // Lets a kernel that was launched with programmatic stream serialization (the decode GEMM, csrc/gemm_skinny.cu) start while
 // this one is still running; that kernel waits for this one's completion before it reads anything this one writes.
 // Without such a dependent in the stream the instruction does nothing.

@@ -4,6 +4,9 @@
 //   packed_attn_step_kernel   one token per request from the cache (bf16 fast path: packed_attn_step.cu)
 //   qk_norm_rope_kernel       RMS norm of all query rows of a projection and of all key rows, before the heads are split, then
 //                             interleaved rotary positions, in place; the new keys and values enter the cache
+//   head_norm_rope_kernel     RMS norm of every query, key and value head, rotary positions in either pairing, values mixed with another
+//                             layer's, in place; the new keys and values enter the cache
+//   head_mix_kernel           talking heads: the outputs of every head's weights over every value head -> the heads' outputs
 //   latent_norm_kernel        RMS norm of a latent projection into a matrix of its own and into the cache
 //   gather_rows_kernel        rows of a matrix and of a cache -> rows of a buffer (a prompt that goes on from a cache)
 //   gate_rows_kernel          o *= sigmoid(g)
@@ -32,6 +35,7 @@ __global__ void __launch_bounds__(TQ * 4) packed_attn_rows_kernel(Prompt a) {
     const int* it = a.items + (long long)blockIdx.x * pa::I_N;
     const int row0 = it[pa::I_ROW], nq = it[pa::I_NQ], c0 = it[pa::I_C0], krow = it[pa::I_KROW];
     const int h = blockIdx.y, hk = h / (a.H / a.G);
+    const int hv = a.cross ? blockIdx.z : hk, ho = a.cross ? h * a.G + hv : h;      // value head, head of the output
     for (int i = threadIdx.x; i < TQ * dk; i += NT) {
         const int r = i / dk, d = i % dk;
         Q[r * ldk + d] = r < nq ? to_f(((const T*)a.q)[(row0 + r) * a.ldq + h * dk + d]) : 0.f;
@@ -49,7 +53,7 @@ __global__ void __launch_bounds__(TQ * 4) packed_attn_rows_kernel(Prompt a) {
         }
         for (int i = threadIdx.x; i < TK * dv; i += NT) {
             const int j = i / dv, d = i % dv;
-            V[i] = k0 + j < k_end ? to_f(((const T*)a.v)[(long long)(krow + k0 + j) * a.ldv + hk * dv + d]) : 0.f;
+            V[i] = k0 + j < k_end ? to_f(((const T*)a.v)[(long long)(krow + k0 + j) * a.ldv + hv * dv + d]) : 0.f;
         }
         __syncthreads();
         float s[KP];
@@ -90,7 +94,7 @@ __global__ void __launch_bounds__(TQ * 4) packed_attn_rows_kernel(Prompt a) {
         __syncwarp();
     }
     if (r < nq) {
-        T* out = (T*)a.out + (row0 + r) * a.ldo + h * dv;
+        T* out = (T*)a.out + (row0 + r) * a.ldo + ho * dv;
         const T* g = a.gate == nullptr ? nullptr : (const T*)a.gate + (row0 + r) * a.ldg + h * dv;
         for (int d = part; d < dv; d += 4) {
             const float o = O[r * dv + d] / l;
@@ -105,14 +109,14 @@ static int launch_rows(const Prompt& a, cudaStream_t st) {
     if (smem > 227 * 1024) return -2;
     cudaError_t e = cudaFuncSetAttribute(packed_attn_rows_kernel<T, TQ>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
-    packed_attn_rows_kernel<T, TQ><<<dim3(a.n, a.H), TQ * 4, smem, st>>>(a);
+    packed_attn_rows_kernel<T, TQ><<<dim3(a.n, a.H, a.cross ? a.G : 1), TQ * 4, smem, st>>>(a);
     return (int)cudaGetLastError();
 }
 
 // ---------------------------------------------------------------------------------------------------------------- one token
 constexpr int ST = 256, SK = 64;         // threads, keys per tile
 
-// grid (H, n)
+// grid (H, n, cross ? G : 1)
 template <typename T>
 __global__ void __launch_bounds__(ST) packed_attn_step_kernel(Step a) {
     extern __shared__ float sm[];
@@ -122,6 +126,7 @@ __global__ void __launch_bounds__(ST) packed_attn_step_kernel(Step a) {
     __shared__ long long rows[SK];
     __shared__ float red[32];
     const int h = blockIdx.x, b = blockIdx.y, hk = h / (a.H / a.G);
+    const int hv = a.cross ? blockIdx.z : hk, ho = a.cross ? h * a.G + hv : h;
     const int w = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int slot = a.slots[b], pos = a.pos[b];
     const int first = a.c.table == nullptr ? max(0, pos + 1 - a.c.cap) : a.window > 0 ? max(0, pos + 1 - a.window) : 0;
@@ -132,10 +137,10 @@ __global__ void __launch_bounds__(ST) packed_attn_step_kernel(Step a) {
     for (int k0 = first; k0 <= pos; k0 += SK) {
         const int nt = min(SK, pos + 1 - k0);
         __syncthreads();
-        if (threadIdx.x < nt) rows[threadIdx.x] = a.c.row(slot, k0 + threadIdx.x) * a.G + hk;
+        if (threadIdx.x < nt) rows[threadIdx.x] = a.c.row(slot, k0 + threadIdx.x) * a.G;
         __syncthreads();
         for (int j = w; j < nt; j += ST / 32) {
-            const T* k = (const T*)a.c.k + rows[j] * a.dk;
+            const T* k = (const T*)a.c.k + (rows[j] + hk) * a.dk;
             float s = 0.f;
             for (int d = lane; d < a.dk; d += 32) s += Q[d] * to_f(k[d]);
             s = warp_sum(s);
@@ -152,11 +157,11 @@ __global__ void __launch_bounds__(ST) packed_attn_step_kernel(Step a) {
         m = mx;
         for (int d = threadIdx.x; d < a.dv; d += ST) {
             float o = O[d] * corr;
-            for (int j = 0; j < nt; ++j) o += P[j] * to_f(((const T*)a.c.v)[rows[j] * a.dv + d]);
+            for (int j = 0; j < nt; ++j) o += P[j] * to_f(((const T*)a.c.v)[(rows[j] + hv) * a.dv + d]);
             O[d] = o;
         }
     }
-    T* out = (T*)a.out + (long long)b * a.ldo + (long long)h * a.dv;
+    T* out = (T*)a.out + (long long)b * a.ldo + (long long)ho * a.dv;
     for (int d = threadIdx.x; d < a.dv; d += ST) out[d] = from_f<T>(O[d] / l);
 }
 
@@ -166,7 +171,7 @@ static int launch_step(const Step& a, cudaStream_t st) {
     if (smem > 200 * 1024) return -2;
     cudaError_t e = cudaFuncSetAttribute(packed_attn_step_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
-    packed_attn_step_kernel<T><<<dim3(a.H, a.n), ST, smem, st>>>(a);
+    packed_attn_step_kernel<T><<<dim3(a.H, a.n, a.cross ? a.G : 1), ST, smem, st>>>(a);
     return (int)cudaGetLastError();
 }
 
@@ -292,6 +297,166 @@ __global__ void __launch_bounds__(THREADS) qk_norm_rope_kernel(QkNorm a) {
         }
 }
 
+struct HeadNorm {
+    void* z;                             // [rows, ldz]: queries (H x dk), keys (G x dk), values (V x dv) from columns zq, zk, zv
+    const float *wq, *wk;                // norm weights [dk], shared by the heads (null: no norm)
+    const double* freq;                  // [rot / 2] rotation per position
+    const void* first;                   // [rows, ldf]: v <- (1 - *mix) v + *mix first (null: values as they are)
+    const float* mix;
+    Cache c;                             // k null: nothing is stored
+    const int *pos, *slots, *ends;       // as in QkNorm
+    long long ldz, ldf;
+    int zq, zk, zv, H, G, V, dk, dv;     // V: G, or 0: no values
+    int nk, nv;                          // numbers in a norm (the unpadded head sizes)
+    int rot, halves;                     // rotated dimensions; pairs (i, i + rot / 2) or neighbours
+    int norm_v;
+    float size, eps;                     // factor of cos and sin
+    int rows;
+};
+
+// grid (rows, parts): a warp takes every (8 parts)-th head; the head lies in shared memory in fp32 between the norm and the rotation
+template <typename T>
+__global__ void __launch_bounds__(THREADS) head_norm_rope_kernel(HeadNorm a) {
+    pdl_trigger();
+    extern __shared__ float4 sm4[];      // one head per warp, then [rot / 2] (cos, sin)
+    const int row = blockIdx.x, pos = a.pos[row], w = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int half = a.rot / 2, heads = a.H + a.G + a.V, size = max(a.dk, a.dv), stride = gridDim.y * (THREADS / 32);
+    float* X = reinterpret_cast<float*>(sm4) + w * size;
+    float2* turn = reinterpret_cast<float2*>(reinterpret_cast<float*>(sm4) + THREADS / 32 * size);
+    T* z = (T*)a.z + (long long)row * a.ldz;
+    auto start = [&](int i) { return z + (i < a.H ? a.zq + i * a.dk : i < a.H + a.G ? a.zk + (i - a.H) * a.dk : a.zv + (i - a.H - a.G) * a.dv); };
+    int i = blockIdx.y * (THREADS / 32) + w;
+    float4 ahead = make_float4(0.f, 0.f, 0.f, 0.f);          // the first head's first piece is on its way while the angles are made
+    if (i < heads && lane * 4 < (i < a.H + a.G ? a.dk : a.dv)) ahead = load4(start(i) + lane * 4);
+    for (int p = threadIdx.x; p < half; p += THREADS) {
+        // range reduction in double: the angle is exact to fp32 at any position
+        constexpr double TWO_PI = 6.283185307179586476925286766559, INV = 0.15915494309189533576888376337251;
+        const double angle = (double)pos * a.freq[p];
+        const float r = (float)(angle - TWO_PI * rint(angle * INV));
+        turn[p] = make_float2(cosf(r) * a.size, sinf(r) * a.size);
+    }
+    __syncthreads();
+    // a ring keeps the request's last `cap` positions: of the rows that share a place only the last one is stored
+    const bool store = a.c.k != nullptr && (a.ends == nullptr || a.c.table != nullptr || pos >= a.ends[row] - a.c.cap);
+    const long long place = store ? a.c.row(a.slots[row], pos) * a.G : 0;
+    const float mix = a.first != nullptr ? *a.mix : 0.f;
+    const bool aligned = a.halves && half % 4 == 0;          // four neighbours lie in one half, and so do their partners
+    for (bool first = true; i < heads; i += stride, first = false) {
+        const bool is_v = i >= a.H + a.G, is_k = !is_v && i >= a.H;
+        const int n = is_v ? a.dv : a.dk;
+        T* p = start(i);
+        float s = 0.f;
+        for (int c = lane * 4; c < n; c += 128) {
+            const float4 x = first && c == lane * 4 ? ahead : load4(p + c);
+            s += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+            *reinterpret_cast<float4*>(X + c) = x;
+        }
+        s = warp_sum(s);
+        __syncwarp();
+        const float* weight = is_v ? nullptr : is_k ? a.wk : a.wq;
+        const float r = (is_v ? a.norm_v != 0 : weight != nullptr) ? 1.f / sqrtf(s / (is_v ? a.nv : a.nk) + a.eps) : 1.f;
+        auto number = [&](int d) { return X[d] * r * (weight == nullptr ? 1.f : weight[d]); };
+        auto four = [&](int d) {
+            const float4 x = *reinterpret_cast<const float4*>(X + d), g = weight == nullptr ? make_float4(1.f, 1.f, 1.f, 1.f) : load4(weight + d);
+            return make_float4(x.x * r * g.x, x.y * r * g.y, x.z * r * g.z, x.w * r * g.w);
+        };
+        T* cached = !store || i < a.H ? nullptr : is_v ? (T*)a.c.v + (place + i - a.H - a.G) * a.dv : (T*)a.c.k + (place + i - a.H) * a.dk;
+        const T* other = is_v && a.first != nullptr ? (const T*)a.first + (long long)row * a.ldf + (i - a.H - a.G) * a.dv : nullptr;
+        for (int c = lane * 4; c < n; c += 128) {
+            float4 y = four(c);
+            if (!is_v && c < a.rot) {
+                if (aligned) {
+                    const bool low = c < half;
+                    const float4 o = four(low ? c + half : c - half);
+                    const float2* t = turn + (low ? c : c - half);
+                    const float sign = low ? -1.f : 1.f;
+                    y = make_float4(y.x * t[0].x + sign * o.x * t[0].y, y.y * t[1].x + sign * o.y * t[1].y, y.z * t[2].x + sign * o.z * t[2].y,
+                                    y.w * t[3].x + sign * o.w * t[3].y);
+                } else {
+                    float f[4] = {y.x, y.y, y.z, y.w};
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const int d = c + e;
+                        if (d < a.rot) {
+                            const bool low = a.halves ? d < half : (d & 1) == 0;
+                            const float2 t = turn[a.halves ? (low ? d : d - half) : d >> 1];
+                            const float o = number(a.halves ? (low ? d + half : d - half) : d ^ 1);
+                            f[e] = low ? f[e] * t.x - o * t.y : f[e] * t.x + o * t.y;
+                        }
+                    }
+                    y = make_float4(f[0], f[1], f[2], f[3]);
+                }
+            }
+            if (other != nullptr) {
+                const float4 o = load4(other + c);
+                y = make_float4((1.f - mix) * y.x + mix * o.x, (1.f - mix) * y.y + mix * o.y, (1.f - mix) * y.z + mix * o.z, (1.f - mix) * y.w + mix * o.w);
+            }
+            store4(p + c, y);
+            if (cached != nullptr) store4(cached + c, y);
+        }
+        __syncwarp();
+    }
+}
+
+// x [n, ldx]: [H, G, dv] per row -> out [n, ldo]: out[h] = sum over g of table[h, g] x[g, value head of h].  A thread takes 16 bytes of a
+// value head and up to 8 of the heads that share it.
+template <typename T>
+__global__ void __launch_bounds__(THREADS) head_mix_kernel(const T* __restrict__ x, long long ldx, const float* __restrict__ table, T* __restrict__ out,
+                                                           long long ldo, int n, int H, int G, int dv, int in_smem) {
+    pdl_trigger();
+    constexpr int W = Vec<T>::N, HT = 8;
+    extern __shared__ float sm[];
+    if (in_smem) {
+        for (int i = threadIdx.x; i < H * H; i += THREADS) sm[i] = table[i];
+        __syncthreads();
+    }
+    const float* tab = in_smem ? sm : table;
+    const int qpg = H / G, pieces = dv / W, tiles = (qpg + HT - 1) / HT;
+    const long long total = (long long)n * G * tiles * pieces;
+    for (long long i = blockIdx.x * (long long)THREADS + threadIdx.x; i < total; i += (long long)gridDim.x * THREADS) {
+        const int c = (int)(i % pieces) * W, tile = (int)(i / pieces % tiles), k = (int)(i / pieces / tiles % G);
+        const long long row = i / pieces / tiles / G;
+        const int h0 = k * qpg + tile * HT, nh = min(HT, k * qpg + qpg - h0);
+        float acc[HT][W];
+#pragma unroll
+        for (int h = 0; h < HT; ++h)
+#pragma unroll
+            for (int e = 0; e < W; ++e) acc[h][e] = 0.f;
+        const T* p = x + row * ldx + k * dv + c;
+#pragma unroll 4
+        for (int g = 0; g < H; ++g) {
+            Vec<T> v;
+            v.load(p + (long long)g * G * dv);
+#pragma unroll
+            for (int h = 0; h < HT; ++h) {
+                if (h < nh) {
+                    const float t = tab[(h0 + h) * H + g];
+#pragma unroll
+                    for (int e = 0; e < W; ++e) acc[h][e] += t * v.get(e);
+                }
+            }
+        }
+#pragma unroll
+        for (int h = 0; h < HT; ++h) {
+            if (h < nh) {
+                Vec<T> y;
+#pragma unroll
+                for (int e = 0; e < W; ++e) y.set(e, acc[h][e]);
+                y.store(out + row * ldo + (long long)(h0 + h) * dv + c);
+            }
+        }
+    }
+}
+
+template <typename T>
+static int launch_mix(const void* x, long long ldx, const float* table, void* out, long long ldo, int n, int H, int G, int dv, cudaStream_t st) {
+    const int qpg = H / G, in_smem = H * H * 4 <= 48 * 1024;
+    const long long total = (long long)n * G * ((qpg + 7) / 8) * (dv / Vec<T>::N), blocks = (total + THREADS - 1) / THREADS;
+    head_mix_kernel<T><<<(unsigned)(blocks < 148 * 8 ? blocks : 148 * 8), THREADS, in_smem ? H * H * 4 : 0, st>>>((const T*)x, ldx, table, (T*)out, ldo, n, H, G,
+                                                                                                                  dv, in_smem);
+    return (int)cudaGetLastError();
+}
+
 struct LatentNorm {
     const void* z;                       // [rows, ldz], latent projection from column 0 (pitch ldz)
     void* c;                             // [rows, ldc] normed rows
@@ -409,6 +574,31 @@ LMOE_API int lmoe_qk_norm_rope(const pag::QkNorm* ap, int dt, cudaStream_t st) {
     if (dt) pag::qk_norm_rope_kernel<bf16><<<a.rows, pag::THREADS, smem, st>>>(a);
     else pag::qk_norm_rope_kernel<float><<<a.rows, pag::THREADS, smem, st>>>(a);
     return (int)cudaGetLastError();
+}
+
+// dk, dv, ldz, ldf and the first columns multiples of 8 (bf16) or 4 (fp32), rot even
+LMOE_API int lmoe_head_norm_rope(const pag::HeadNorm* ap, int dt, cudaStream_t st) {
+    const pag::HeadNorm& a = *ap;
+    const int w = dt ? 8 : 4;
+    if (a.rows <= 0 || a.H <= 0 || a.G <= 0 || (a.V != 0 && a.V != a.G) || a.dk <= 0 || a.dk % w || a.dv < 0 || a.dv % w || a.ldz % w || a.ldf % w || a.zq % w ||
+        a.zk % w || a.zv % w || a.rot % 2 || a.rot < 0 || a.rot > a.dk || a.nk <= 0 || (a.V && a.nv <= 0) || !pag::aligned(a.z) || !pag::aligned(a.first) ||
+        !pag::aligned(a.wq) || !pag::aligned(a.wk) || !pag::aligned(a.c.k) || !pag::aligned(a.c.v) ||
+        (a.c.k != nullptr && ((a.c.table == nullptr && a.c.cap <= 0) || !a.V)) || (a.rot > 0 && a.freq == nullptr) || (a.first != nullptr && a.mix == nullptr))
+        return -1;
+    const size_t smem = sizeof(float2) * (a.rot / 2) + sizeof(float) * (pag::THREADS / 32) * (a.dk > a.dv ? a.dk : a.dv);
+    if (smem > 46 * 1024) return -2;
+    const int heads = a.H + a.G + a.V, parts = a.rows >= 1024 ? 1 : (heads + 7) / 8;
+    if (dt) pag::head_norm_rope_kernel<bf16><<<dim3(a.rows, parts), pag::THREADS, smem, st>>>(a);
+    else pag::head_norm_rope_kernel<float><<<dim3(a.rows, parts), pag::THREADS, smem, st>>>(a);
+    return (int)cudaGetLastError();
+}
+
+// x [n, ldx] with H * G * dv columns -> out [n, ldo] with H * dv columns; table [H, H]; dv and pitches multiples of 8 (bf16) or 4 (fp32)
+LMOE_API int lmoe_head_mix(const void* x, long long ldx, const float* table, void* out, long long ldo, int n, int H, int G, int dv, int dt,
+                           cudaStream_t st) {
+    const int w = dt ? 8 : 4;
+    if (n <= 0 || H <= 0 || G <= 0 || H % G || dv <= 0 || dv % w || ldx % w || ldo % w || !pag::aligned(x) || !pag::aligned(out)) return -1;
+    return dt ? pag::launch_mix<bf16>(x, ldx, table, out, ldo, n, H, G, dv, st) : pag::launch_mix<float>(x, ldx, table, out, ldo, n, H, G, dv, st);
 }
 
 LMOE_API int lmoe_latent_norm(const pag::LatentNorm* ap, int dt, cudaStream_t st) {

@@ -30,6 +30,7 @@ struct Prompt {
     int window;                       // <= 0: none
     int n, q_rows, k_rows;
     float scale;
+    int cross;                        // every query head's weights are applied to the values of every kv head: out [rows, H, G, dv]
 };
 
 struct Cache {
@@ -51,6 +52,7 @@ struct Step {
     int window;                       // <= 0: none
     int n;
     float scale;
+    int cross;                        // as in Prompt
 };
 
 }  // namespace pa

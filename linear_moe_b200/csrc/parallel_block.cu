@@ -14,16 +14,6 @@ namespace pb {
 
 constexpr int THREADS = 256;
 
-// stores 4 values at y[c .. c + 3] (c a multiple of 4)
-__device__ __forceinline__ void store4(float* y, float4 v) { *reinterpret_cast<float4*>(y) = v; }
-__device__ __forceinline__ void store4(bf16* y, float4 v) {
-    __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
-    uint2 r;
-    r.x = *reinterpret_cast<uint32_t*>(&lo);
-    r.y = *reinterpret_cast<uint32_t*>(&hi);
-    *reinterpret_cast<uint2*>(y) = r;
-}
-
 // x [rows, ldx] fp32, y [rows, ldy]; columns width .. pad of x hold zeros, and y gets zeros there
 template <typename T>
 __global__ void __launch_bounds__(THREADS) stream_norm_kernel(const float* __restrict__ x, long long ldx, T* __restrict__ y,

@@ -10,20 +10,6 @@ namespace sb {
 
 constexpr int THREADS = 256, NV = 4;         // float4s a thread keeps in registers (rows up to 4096 wide)
 
-__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 load4(const bf16* p) {
-    const uint2 r = *reinterpret_cast<const uint2*>(p);
-    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
-    return make_float4(a.x, a.y, b.x, b.y);
-}
-__device__ __forceinline__ void store4(float* y, float4 v) { *reinterpret_cast<float4*>(y) = v; }
-__device__ __forceinline__ void store4(bf16* y, float4 v) {
-    __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
-    uint2 r;
-    r.x = *reinterpret_cast<uint32_t*>(&lo);
-    r.y = *reinterpret_cast<uint32_t*>(&hi);
-    *reinterpret_cast<uint2*>(y) = r;
-}
 __device__ __forceinline__ float dot4(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
 __device__ __forceinline__ float4 mul4(float4 v, float r, float4 w) { return make_float4(v.x * r * w.x, v.y * r * w.y, v.z * r * w.z, v.w * r * w.w); }
 __device__ __forceinline__ float4 add4(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
