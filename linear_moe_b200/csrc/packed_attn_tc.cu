@@ -10,6 +10,8 @@
 //               (shared memory and a named barrier), P = exp2(S - m), bf16 pack into the 128-byte-swizzled P tile
 // O accumulates in tensor memory over all key tiles.  The maximum a row is scaled by may lag behind the true one by LAG (in
 // units of log2), so that P stays below 2^LAG; only when a row runs ahead of that is O multiplied in tensor memory.
+// With `cross`, a query head's weights are applied to the values of every kv head (talking heads, which mix these results afterwards): a
+// CTA takes as many kv heads as fit 256 columns of tensor memory, and the values come in stages of 64 keys.
 // Every mbarrier wait is bounded; on expiry the error word is set and the CTA drains and frees its tensor memory.
 #include "attn_math.cuh"
 #include "flash_tc_utils.cuh"
@@ -22,11 +24,13 @@ using pa::Prompt;
 
 constexpr float LAG = 8.f;
 
-template <int DQ, int DV>
+// DQ: key dims, DT: value columns of a CTA
+template <int DQ, int DT>
 struct __align__(1024) Smem {
+    static constexpr int VK = DT > 128 ? 64 : BN;           // keys per stage of values
     uint8_t q[BM * DQ * 2];
     uint8_t k[2][BN * DQ * 2];
-    uint8_t v[2][BN * DV * 2];
+    uint8_t v[2][VK * DT * 2];
     uint8_t p[BM * BN * 2];
     float mx[2][SPLIT][BM], ls[SPLIT][BM];
     uint64_t q_full, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[2], pv_done, p_ready;
@@ -41,18 +45,20 @@ __device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t (&r)[16
 }
 __device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 
-template <int DQ, int DV>
+// DV: value dims of a head, NB: value heads of a CTA
+template <int DQ, int DV, int NB>
 __global__ void __launch_bounds__(THREADS, 1)
 packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                       const __grid_constant__ CUtensorMap tmV, Prompt a) {
     extern __shared__ uint8_t smem_raw[];
-    Smem<DQ, DV>& sm = *reinterpret_cast<Smem<DQ, DV>*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-    constexpr int KQ = DQ / 64, KV = DV / 64;               // 64-element blocks along the head dimensions
+    constexpr int DT = NB * DV, VK = Smem<DQ, DT>::VK, VS = BN / VK;         // VS: stages of values per tile of keys
+    Smem<DQ, DT>& sm = *reinterpret_cast<Smem<DQ, DT>*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+    constexpr int KQ = DQ / 64, KV = DT / 64;               // 64-element blocks along the head dimensions
     constexpr uint32_t TMEM_COLS = 512, O_COL = 2 * BN;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int* it = a.items + (long long)blockIdx.x * pa::I_N;
     const int row0 = it[pa::I_ROW], nq = it[pa::I_NQ], c0 = it[pa::I_C0], krow = it[pa::I_KROW];
-    const int h = blockIdx.y, hk = h / (a.H / a.G);
+    const int h = blockIdx.y, hk = h / (a.H / a.G), hv = a.cross ? blockIdx.z * NB : hk;       // hv: first value head
     const int nb_lo = a.window > 0 ? max(0, c0 - a.window + 1) / BN : 0;
     const int n_it = (c0 + nq + BN - 1) / BN - nb_lo;       // at least 1: a query sees its own key
     volatile int* abort_flag = &sm.abort_flag;
@@ -92,19 +98,27 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
                 mbar_expect_tx(&sm.k_full[s], BN * DQ * 2);
 #pragma unroll
                 for (int kb = 0; kb < KQ; ++kb) tma_load_4d(sm.k[s] + kb * BN * 128, &tmK, &sm.k_full[s], kb * 64, hk, key0, 0);
-                if (!mbar_wait_suspend(&sm.v_empty[s], ph ^ 1, abort_flag, err, 0x7200 | s)) break;
-                mbar_expect_tx(&sm.v_full[s], BN * DV * 2);
+                bool ok = true;
 #pragma unroll
-                for (int kk = 0; kk < BN / 64; ++kk)        // MN-major operand: per 64 keys, DV/64 boxes of {64 d, 64 keys}
+                for (int u = 0; u < VS; ++u) {
+                    const int vi = j * VS + u, t = vi & 1;
+                    ok = mbar_wait_suspend(&sm.v_empty[t], ((vi >> 1) & 1) ^ 1, abort_flag, err, 0x7200 | t);
+                    if (!ok) break;
+                    mbar_expect_tx(&sm.v_full[t], VK * DT * 2);
 #pragma unroll
-                    for (int nb = 0; nb < KV; ++nb)
-                        tma_load_4d(sm.v[s] + (kk * KV + nb) * 8192, &tmV, &sm.v_full[s], nb * 64, hk, key0 + kk * 64, 0);
+                    for (int kk = 0; kk < VK / 64; ++kk)    // MN-major operand: per 64 keys, DT/64 boxes of {64 d, 64 keys}
+#pragma unroll
+                        for (int nb = 0; nb < KV; ++nb)     // (heads behind the last one read zeros)
+                            tma_load_4d(sm.v[t] + (kk * KV + nb) * 8192, &tmV, &sm.v_full[t], nb % (DV / 64) * 64, hv + nb / (DV / 64),
+                                        key0 + u * VK + kk * 64, 0);
+                }
+                if (!ok) break;
             }
         }
     } else if (warp == 1) {
         const uint32_t issue = lane == 0 ? 1u : 0u;
         constexpr uint32_t idesc_s = idesc_bf16<false, BN>();
-        constexpr uint32_t idesc_o = idesc_bf16<true, DV>();
+        constexpr uint32_t idesc_o = idesc_bf16<true, DT>();
         bool ok = mbar_wait_suspend(&sm.q_full, 0, abort_flag, err, 0x8000);
         auto issue_s = [&](int j) -> bool {
             const int s = j & 1;
@@ -124,25 +138,31 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
         for (int j = 0; ok && j < n_it; ++j) {
             // score buffer (j + 1) & 1 was last read for P_{j-1}, whose p_ready was waited for in the previous iteration
             if (j + 1 < n_it) { ok = issue_s(j + 1); if (!ok) break; }
-            const int s = j & 1;
-            if (!mbar_wait_suspend(&sm.v_full[s], (j >> 1) & 1, abort_flag, err, 0x8200 | s)) break;
-            if (!mbar_wait_suspend(&sm.p_ready, j & 1, abort_flag, err, 0x8300)) break;
-            tc_fence_after();
-            const uint32_t pl = desc_lo<false>(s32(sm.p)), vl = desc_lo<true>(s32(sm.v[s]));
 #pragma unroll
-            for (int kk = 0; kk < BN / UMMA_K; ++kk) {
-                const uint32_t aoff = ((kk / 4) * (BM * 128) + (kk % 4) * 32) >> 4;
-                const uint32_t boff = ((kk / 4) * (KV * 8192) + (kk % 4) * 2048) >> 4;
-                umma_lo(tmem_base + O_COL, pl + aoff, vl + boff, idesc_o, (j > 0 || kk > 0) ? 1u : 0u, issue);
+            for (int u = 0; u < VS; ++u) {
+                const int vi = j * VS + u, t = vi & 1;
+                ok = mbar_wait_suspend(&sm.v_full[t], (vi >> 1) & 1, abort_flag, err, 0x8200 | t);
+                if (ok && u == 0) ok = mbar_wait_suspend(&sm.p_ready, j & 1, abort_flag, err, 0x8300);
+                if (!ok) break;
+                tc_fence_after();
+                const uint32_t pl = desc_lo<false>(s32(sm.p)), vl = desc_lo<true>(s32(sm.v[t]));
+#pragma unroll
+                for (int kk = 0; kk < VK / UMMA_K; ++kk) {
+                    const int kp = u * (VK / UMMA_K) + kk;  // 16-key step of the tile
+                    const uint32_t aoff = ((kp / 4) * (BM * 128) + (kp % 4) * 32) >> 4;
+                    const uint32_t boff = ((kk / 4) * (KV * 8192) + (kk % 4) * 2048) >> 4;
+                    umma_lo(tmem_base + O_COL, pl + aoff, vl + boff, idesc_o, (j > 0 || kp > 0) ? 1u : 0u, issue);
+                }
+                umma_commit_if(&sm.v_empty[t], issue);
             }
-            umma_commit_if(&sm.v_empty[s], issue);
+            if (!ok) break;
             umma_commit_if(&sm.pv_done, issue);
         }
     } else if (warp >= 4) {
         const int qd = warp & 3, part = (warp - 4) >> 2;
         const int r = qd * 32 + lane;                         // query row inside the tile
         const uint32_t lane_addr = tmem_base + ((uint32_t)(qd * 32) << 16);
-        constexpr int CW = BN / SPLIT, OW = DV / SPLIT;       // score / output columns of this thread
+        constexpr int CW = BN / SPLIT, OW = DT / SPLIT;       // score / output columns of this thread
         static_assert(CW == 32 && OW % 16 == 0, "tensor-memory load widths");
         const float sc = a.scale * LOG2E, lag = LAG / sc;
         uint8_t* prow = sm.p + ((part * CW) >> 6) * (BM * 128) + (r >> 3) * 1024 + (r & 7) * 128;
@@ -233,11 +253,11 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
             const float w = 1.f / l;
             const long long row = row0 + r;
             const bf16* gp = a.gate == nullptr ? nullptr : (const bf16*)a.gate + row * a.ldg + h * a.dv;
-            bf16* op = (bf16*)a.out + row * a.ldo + h * a.dv;
 #pragma unroll
             for (int c = 0; c < OW; c += 8) {
-                const int col = part * OW + c;
-                if (col < a.dv) {
+                const int col = (part * OW + c) % DV, nb = (part * OW + c) / DV;
+                bf16* op = (bf16*)a.out + row * a.ldo + (long long)(a.cross ? h * a.G + hv + nb : h) * a.dv;
+                if (col < a.dv && hv + nb < a.G) {
                     Vec<bf16> g, y;
                     if (gp != nullptr) g.load(gp + col);
 #pragma unroll
@@ -258,14 +278,21 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
     }
 }
 
-template <int DQ, int DV>
+template <int DQ, int DV, int NB>
 static int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const Prompt& a, cudaStream_t st) {
-    const size_t smem = sizeof(Smem<DQ, DV>) + 1024;
-    static_assert(sizeof(Smem<DQ, DV>) + 1024 <= 227 * 1024, "shared memory of one CTA");
-    cudaError_t e = cudaFuncSetAttribute(packed_attn_tc_kernel<DQ, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    const size_t smem = sizeof(Smem<DQ, NB * DV>) + 1024;
+    static_assert(sizeof(Smem<DQ, NB * DV>) + 1024 <= 227 * 1024 && NB * DV <= 256, "shared and tensor memory of one CTA");
+    cudaError_t e = cudaFuncSetAttribute(packed_attn_tc_kernel<DQ, DV, NB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
-    packed_attn_tc_kernel<DQ, DV><<<dim3(a.n, a.H), THREADS, smem, st>>>(mq, mk, mv, a);
+    packed_attn_tc_kernel<DQ, DV, NB><<<dim3(a.n, a.H, a.cross ? (a.G + NB - 1) / NB : 1), THREADS, smem, st>>>(mq, mk, mv, a);
     return (int)cudaGetLastError();
+}
+
+template <int DQ>
+static int by_values(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const Prompt& a, cudaStream_t st) {
+    const int heads = a.cross ? a.G : 1;
+    if (a.dv <= 64) return heads > 2 ? launch<DQ, 64, 4>(mq, mk, mv, a, st) : heads > 1 ? launch<DQ, 64, 2>(mq, mk, mv, a, st) : launch<DQ, 64, 1>(mq, mk, mv, a, st);
+    return heads > 1 ? launch<DQ, 128, 2>(mq, mk, mv, a, st) : launch<DQ, 128, 1>(mq, mk, mv, a, st);
 }
 
 }  // namespace patc
@@ -280,7 +307,7 @@ LMOE_API int lmoe_packed_attn_tc(const pa::Prompt* ap, cudaStream_t st) {
     const Prompt& a = *ap;
     if (a.n <= 0 || a.q_rows <= 0 || a.k_rows <= 0 || a.H <= 0 || a.G <= 0 || a.H % a.G || a.dk <= 0 || a.dk > 128 || a.dv <= 0 || a.dv > 128 ||
         a.dk % 8 || a.dv % 8 || a.ldq % 8 || a.ldk % 8 || a.ldv % 8 || a.ldo % 8 || (a.gate != nullptr && a.ldg % 8) || !(a.scale > 0.f) ||
-        ((reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.k) | reinterpret_cast<uintptr_t>(a.v) |
+        (a.cross && a.gate != nullptr) || ((reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.k) | reinterpret_cast<uintptr_t>(a.v) |
           reinterpret_cast<uintptr_t>(a.gate) | reinterpret_cast<uintptr_t>(a.out)) & 15))
         return -1;
     CUtensorMap mq, mk, mv;
@@ -288,6 +315,5 @@ LMOE_API int lmoe_packed_attn_tc(const pa::Prompt* ap, cudaStream_t st) {
     if (rc == 0) rc = make_map_4d(&mk, a.k, 1, a.k_rows, a.G, a.dk, (long long)a.k_rows * a.ldk, a.ldk, a.dk, BN);
     if (rc == 0) rc = make_map_4d(&mv, a.v, 1, a.k_rows, a.G, a.dv, (long long)a.k_rows * a.ldv, a.ldv, a.dv, 64);
     if (rc) return rc;
-    if (a.dk <= 64) return a.dv <= 64 ? launch<64, 64>(mq, mk, mv, a, st) : launch<64, 128>(mq, mk, mv, a, st);
-    return a.dv <= 64 ? launch<128, 64>(mq, mk, mv, a, st) : launch<128, 128>(mq, mk, mv, a, st);
+    return a.dk <= 64 ? by_values<64>(mq, mk, mv, a, st) : by_values<128>(mq, mk, mv, a, st);
 }
