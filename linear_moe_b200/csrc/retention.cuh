@@ -21,7 +21,7 @@ enum { R_SLOT, R_FLAGS, R_STATE, R_GROUPS, R_TOKENS };
 struct Args {
     void *z, *out;                       // [rows, ldz]: queries, keys (H x dk), values, gate (H x dv); [rows, ldo]: H x dv
     float* state;                        // [slots, H, dk, dv] or null
-    float* scratch;                      // [groups that are not last, H, dk, dv]
+    float* scratch;                      // [places, H, dk, dv]
     float* raw;                          // general kernel: [rows, H * dv]
     const float* powers;                 // [H, CH + 1] decay^0 ..
     const double* decay;                 // [H]

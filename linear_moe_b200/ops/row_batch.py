@@ -123,7 +123,7 @@ class RowBatch:
         """Every request's new tokens in groups of at most ``tokens``: ``(groups, states, requests)`` as int32 tables (``csrc/retention.cuh``).
         A group is (first row, tokens, slot, flags, state in front, state behind): flag 1: the request's first group, flag 2: its last one,
         flag 4: the request has a past; the states are places in a buffer of ``states`` (-1: none).  Requests of more than one group are
-        listed as (slot, flags, first state, groups, tokens of a group); ``None`` when there are none."""
+        listed as (slot, flags, first state, groups, tokens of a group), with one state per group; ``None`` when there are none."""
         key = ("recurrent", tokens)
         if key not in self._items:
             groups, many, states = [], [], 0
@@ -134,8 +134,8 @@ class RowBatch:
                 for i in range(count):
                     last = i == count - 1
                     groups.append((self.row0[r] + i * tokens, n - i * tokens if last else tokens, slot, past + (i == 0) + 2 * last,
-                                   states + i - 1 if i else -1, -1 if last else states + i, 0, 0))
-                states += count - 1
+                                   states + i if count > 1 else -1, -1 if last else states + i + 1, 0, 0))
+                states += count if count > 1 else 0
             self._items[key] = (self._table(key + (0,), groups), states, self._table(key + (1,), many) if many else None)
         return self._items[key]
 
