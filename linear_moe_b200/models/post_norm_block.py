@@ -48,7 +48,7 @@ class Retention(Part):
     def forward(self, h, step: RowStep, layer: int) -> torch.Tensor:
         z = ops.linear(h, self.linear_in)
         out = activation_rows(h, self.linear_out, self.s.heads * self.s.dv)
-        ops.retention(z, out, self.lay, self.s, self.powers, self.decay, self.freq, self.eps, step.batch, step.cache(layer))
+        ops.retention_rows(z, out, self.lay, self.s, self.powers, self.decay, self.freq, self.eps, step.batch, step.cache(layer))
         return ops.sublayer_out(out, self.linear_out)
 
 

@@ -327,7 +327,7 @@ from .group_norm import embed_rows, group_norm, residual_group_norm, softcap_   
 from .moe_rows import experts_relu2   # noqa: E402,F401
 from .packed_attn import (causal_attention, gather_rows, glu_in, head_norm_rope_, latent_absorb, latent_norm, latent_up,   # noqa: E402,F401
                           qk_norm_rope_, residual_norm, rotate_heads_, step_attention, sublayer_out)
-from .retention import retention   # noqa: E402,F401
+from .retention import retention_rows   # noqa: E402,F401
 
 
 # ---- linear sequence models -----------------------------------------------

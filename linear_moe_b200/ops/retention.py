@@ -91,11 +91,11 @@ def group_tokens(counts, heads: int, sms: int) -> int:
     return min(per, longest) * CHUNK
 
 
-def retention(z, out, lay: RetentionLayout, s: RetentionSpec, powers, decay, freq, eps: float, batch: RowBatch, cache: Optional[dict]):
+def retention_rows(z, out, lay: RetentionLayout, s: RetentionSpec, powers, decay, freq, eps: float, batch: RowBatch, cache: Optional[dict]):
     """``out[:, :heads * dv]`` from the projection rows ``z`` (whose queries and keys a prompt rotates in place); ``cache["s"]``
     ``[slots, heads, dk, dv]`` (fp32) holds the requests' states.  ``powers``, ``decay``, ``freq``: the spec's tables."""
     if not z.is_cuda:
-        return RR.retention(z, out, lay, s, freq, eps, batch, cache)
+        return RR.retention_rows(z, out, lay, s, freq, eps, batch, cache)
     from . import cuda as K
     _no_grad(z)
     dev, dt, dk, dv, H = z.device, K._dt(z), s.dk, s.dv, s.heads

@@ -1,4 +1,4 @@
-"""Eager definition of :func:`linear_moe_b200.ops.retention.retention` (what CPU tensors run): token by token in fp32."""
+"""Eager definition of :func:`linear_moe_b200.ops.retention.retention_rows` (what CPU tensors run): token by token in fp32."""
 from __future__ import annotations
 
 import torch
@@ -6,7 +6,7 @@ import torch
 from .packed_attn import rotate_heads_
 
 
-def retention(z, out, lay, s, freq, eps, batch, cache):
+def retention_rows(z, out, lay, s, freq, eps, batch, cache):
     H, dk, dv = s.heads, s.dk, s.dv
     if s.rot_dims:
         rotate_heads_(z, lay.q, lay.k, H, H, dk, True, freq, 1.0, batch)

@@ -166,3 +166,35 @@ def greedy(w, cfg, prompt, steps):
     for _ in range(steps):
         tokens.append(int(logits(w, cfg, tokens)[-1].argmax()))
     return tokens[len(prompt):]
+
+
+def random_model(cfg, seed=0, gain=1.5):
+    """bf16 weights of a configuration; ``gain`` sharpens the attention."""
+    g = torch.Generator().manual_seed(seed)
+
+    def rnd(*shape, std=1.0):
+        return (torch.randn(*shape, generator=g) * std).bfloat16()
+
+    def weight(n, around=1.0):
+        return (around * (0.7 + 0.6 * torch.rand(n, generator=g))).bfloat16()
+    d, V = cfg["width"], cfg["vocab"]
+    w = {"embed": rnd(V, d), "final.norm": weight(d), "head": rnd(V, d, std=0.8 * cfg["logit_softcap"] * d ** -0.5)}
+    for n, layer in enumerate(cfg["layers"]):
+        m, l, x = layer["mixer"], f"l{n}.", f"l{n}.mix."
+        H, dk, dv = m["heads"], m["dim"], m["vdim"]
+        w[l + "norm1"], w[l + "ls1"] = weight(d), weight(d, 0.6)
+        if layer["type"] == "retention":
+            w[x + "q"], w[x + "k"], w[x + "v"], w[x + "g"] = (rnd(H * e, d, std=d ** -0.5) for e in (dk, dk, dv, dv))
+        else:
+            G = m["kv_heads"]
+            w[x + "q"], w[x + "k"], w[x + "v"] = rnd(H * dk, d, std=d ** -0.5), rnd(G * dk, d, std=d ** -0.5), rnd(G * dv, d, std=d ** -0.5)
+            w[x + "q.norm"], w[x + "k.norm"] = weight(dk, gain), weight(dk)
+            w[x + "talk"] = (0.8 * torch.eye(H) + 0.5 * H ** -0.5 * torch.randn(H, H, generator=g)).bfloat16()
+            if m.get("v_mix", False):
+                w[x + "vmix"] = torch.tensor(0.2 + 0.6 * float(torch.rand((), generator=g))).bfloat16()
+        w[x + "o"] = rnd(d, H * dv, std=(H * dv) ** -0.5)
+        if layer.get("mlp") is not None:
+            f, x = layer["mlp"]["ff"], l + "mlp."
+            w[l + "norm2"], w[l + "ls2"] = weight(d), weight(d, 0.5)
+            w[x + "gate"], w[x + "up"], w[x + "down"] = rnd(f, d, std=d ** -0.5), rnd(f, d, std=d ** -0.5), rnd(d, f, std=f ** -0.5)
+    return w

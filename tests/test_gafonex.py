@@ -1,0 +1,782 @@
+"""The Gafonex design against its plain definition (tests/gafonex_oracle.py): every mechanism alone, whole models, the slot cache and
+step function under many schedules, generation, the command line and trace replay.  The same cases run on the CPU (eager definitions,
+fp32) and, with ``-m gpu``, on the kernels in fp32 and bf16."""
+import io
+import json
+import os
+import subprocess
+import sys
+
+import pytest
+import torch
+
+import gafonex_oracle as O
+from linear_moe_b200 import ops
+from linear_moe_b200.infer.generation import generate_tokens
+from linear_moe_b200.infer.kv_cache import LayerPages, LayerRows, LayerState, SlotCache
+from linear_moe_b200.infer.session import InferenceSession
+from linear_moe_b200.models.registry import load_model
+from linear_moe_b200.ops import packed_attn as PA
+from linear_moe_b200.ops import retention as RT
+from linear_moe_b200.ops.row_batch import RowBatch, round_up
+from linear_moe_b200.ref.packed_attn import cache_rows, store
+from serving_utils import GPU, ROOT, folder, padded, prompt, rel, tol, where
+
+YARN = {"factor": 4.0, "original": 24, "fast": 3.0, "slow": 0.5}
+
+
+def retention(heads, dim, vdim, decay, rot, base=1000.0):
+    return "retention", {"heads": heads, "dim": dim, "vdim": vdim, "decay": list(decay), "rot": {"dims": rot, "base": base}}
+
+
+def attention(heads, kv_heads, dim, vdim, rot, base=500.0, scaling=None, scale=None, v_mix=False):
+    r = {"dims": rot, "base": base}
+    return "attention", {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5 if scale is None else scale,
+                         "v_mix": v_mix, "rot": r if scaling is None else {**r, "scaling": scaling}}
+
+
+def config(*layers, width=80, vocab=90, eps=1e-5, groups=2, cap=6.0):
+    return {"architecture": "Gafonex", "width": width, "vocab": vocab, "norm": {"eps": eps, "groups": groups}, "logit_softcap": cap,
+            "layers": [{"type": kind, "mixer": m, "mlp": None if ff is None else {"kind": "dense", "ff": ff}} for (kind, m), ff in layers]}
+
+
+CONFIGS = {
+    # every branch, sizes that differ by layer; the first attention layer keeps its values to itself, the second one lends them
+    "mixed": config((retention(3, 24, 40, (0.9, 0.98, 0.999), 16), 112), (attention(6, 3, 24, 40, 16, scaling=YARN), 72),
+                    (attention(4, 2, 32, 24, 32, base=90.0, scaling={**YARN, "factor": 8.0}, v_mix=True), None), (retention(2, 16, 16, (0.5, 0.995), 16), None),
+                    (attention(6, 2, 48, 24, 20, scale=0.3, v_mix=True), 40), (attention(2, 2, 16, 24, 16, scaling=YARN, v_mix=True), 96), width=96, groups=4),
+    # nothing divides by 8, groups of ten columns, pairs three apart; two layers share values
+    "odd": config((attention(5, 5, 10, 7, 6, scaling={**YARN, "original": 100}, v_mix=True), 45), (retention(3, 9, 7, (0.8, 0.97, 0.9999), 6), 13),
+                  (attention(10, 5, 9, 7, 2, v_mix=True), None), (retention(1, 22, 13, (0.99,), 22), 10), width=50, vocab=77, groups=5, cap=30.0),
+    # full tensor-core tiles, one and many heads on a key and value, more value heads than a tile holds
+    "wide": config((retention(2, 128, 128, (0.97, 0.9995), 128), 256), (attention(24, 1, 128, 64, 32, scaling=YARN), 96),
+                   (attention(4, 4, 64, 128, 64), 64), (attention(10, 5, 128, 32, 128, scaling=YARN, v_mix=True), None), (retention(3, 64, 128, (0.9, 0.99, 0.999), 48), 128),
+                   (attention(15, 5, 32, 32, 32, v_mix=True), 64), width=128, groups=1),
+    # heads too large for the fast kernels
+    "large": config((retention(2, 144, 272, (0.96, 0.998), 144), 64), (attention(4, 2, 144, 160, 100, scaling=YARN), 32), (retention(1, 32, 144, (0.99,), 16), None),
+                    width=64, groups=2),
+    # numbers at the ends of their ranges: one head, decays of one and zero, nothing rotated, no scaling to speak of, more groups than warps
+    "extremes": config((retention(2, 16, 16, (1.0, 0.0), 0), 24), (attention(1, 1, 16, 16, 16, scaling={**YARN, "factor": 1.0}, v_mix=True), None),
+                       (retention(1, 16, 32, (1.0,), 16), 16), (attention(2, 1, 16, 16, 0, v_mix=True), 16), width=64, groups=16),
+}
+
+
+@pytest.fixture(scope="module")
+def build(tmp_path_factory):
+    """``build(name, where) -> (model, weights, config)``; a model is made once per module."""
+    made = {}
+
+    def get(name, where):
+        gain = 3.0 if where[1] == "float32" else 1.5      # sharper attention in fp32 (in bf16 near ties between keys would hide the rest)
+        key = (name, where)
+        if key not in made:
+            cfg = CONFIGS[name]
+            w = O.random_model(cfg, seed=len(name), gain=gain)
+            d = folder(tmp_path_factory.mktemp("model") / "m", cfg, w)
+            made[key] = (load_model(d, getattr(torch, where[1]), where[0]), w, cfg)
+        return made[key]
+    return get
+
+
+def laid_out(x, size):
+    """``[n, heads, d]`` -> ``[n, heads * size]`` with zeros behind every head."""
+    return torch.nn.functional.pad(x, (0, size - x.shape[2])).reshape(x.shape[0], -1)
+
+
+def heads_of(x, heads, size, d):
+    return x.reshape(x.shape[0], heads, size)[:, :, :d].double().cpu()
+
+
+# ------------------------------------------------------------------------------------------------------- single mechanisms
+@pytest.mark.parametrize("dims,base", [(64, 50000.0), (16, 500.0), (6, 10.0), (2, 7.0), (128, 1e6)])
+def test_rotary_scaling(dims, base):
+    for s in (None, YARN, {"factor": 8.0, "original": 1024, "fast": 32.0, "slow": 1.0}, {"factor": 2.5, "original": 4096, "fast": 1.0, "slow": 1.0},
+              {"factor": 0.5, "original": 7, "fast": 100.0, "slow": 0.01}, {"factor": 1.0, "original": 1, "fast": 2.0, "slow": 1.0}):
+        want, size = O.frequencies(dims, base, s)
+        scaling = None if s is None else PA.RotaryScaling(**s)
+        assert torch.allclose(PA.rotary_frequencies(dims, base, scaling), want, rtol=1e-12, atol=0)
+        assert s is None or abs(scaling.size - size) < 1e-12
+    assert not torch.equal(O.frequencies(16, 500.0, YARN)[0], O.frequencies(16, 500.0)[0])
+
+
+@where
+@pytest.mark.parametrize("ring", [False, True])
+@pytest.mark.parametrize("heads,kv_heads,dim,vdim,rot,halves", [(4, 2, 16, 16, 16, True), (3, 1, 10, 7, 6, True), (6, 3, 72, 24, 20, True), (32, 8, 128, 128, 128, True),
+                                                                (2, 2, 16, 160, 0, True), (4, 4, 24, 32, 10, False)])
+def test_head_norms_rotation_and_values(where, heads, kv_heads, dim, vdim, rot, halves, ring):
+    """Each head by itself; pairs half the rotated width apart (or neighbours); values normed, then mixed; positions far out keep their angles."""
+    dev, dt = where[0], getattr(torch, where[1])
+    yarn = {**YARN, "original": 64}
+    s = PA.AttentionSpec(heads, kv_heads, dim, vdim, 1.0, 30 if ring else None, rot, 777.0, head_norm=True, rot_halves=halves, value_norm=True,
+                         rot_scaling=PA.RotaryScaling(**yarn) if halves and rot else None)
+    lay, pos = PA.QkvLayout.of(s), [0, 1, 29, 30, 63, 64, 5000]
+    n = len(pos)
+    x = [torch.randn(n, h, d) * torch.tensor([1.0, 0.01, 30.0, 1.0, 2.0, 1.0, 1.0])[:, None, None] for h, d in ((heads, dim), (kv_heads, dim), (kv_heads, vdim))]
+    q, k, v = (t.to(dt) for t in x)
+    other, mix = torch.randn(n, kv_heads, vdim).to(dt), torch.tensor(0.37)
+    wq, wk = torch.rand(dim) + 0.5, torch.rand(dim) + 0.5
+    far = pos + [262143] if ring else pos                                      # (pages up to there would be many)
+    for mixed in (False, True):
+        z = torch.cat([laid_out(q, s.dk), laid_out(k, s.dk), laid_out(v, s.dv)], 1).to(dev)
+        cache = SlotCache([LayerRows(30, kv_heads, s.dk, s.dv) if ring else LayerPages(kv_heads, s.dk, s.dv)], n, dev, dt)
+        slots = cache.acquire(n)
+        at = far[-n:]
+        cache.reserve(slots, [p + 1 for p in at])
+        batch = RowBatch(at, [1] * n, slots, dev)
+        norms = [torch.nn.functional.pad(w, (0, s.dk - dim)).to(dev) for w in (wq, wk)]
+        PA.head_norm_rope_(z, lay, s, *norms, s.frequencies(dev), 1e-3, batch, cache[0], *((laid_out(other, s.dv).to(dev), mix.to(dev)) if mixed else ()))
+        positions = torch.tensor(at)
+
+        def turned(t):
+            if halves:
+                return O.rotate(t, positions, rot, 777.0, yarn if rot else None)
+            y = t.clone()                                                      # neighbours: the same turn on shuffled dimensions
+            order = list(range(0, rot, 2)) + list(range(1, rot, 2))
+            y[:, :, order] = O.rotate(t[:, :, order], positions, rot, 777.0)
+            return y
+        for t, w, h, c in ((q, wq, heads, lay.q), (k, wk, kv_heads, lay.k)):
+            want = turned(O.head_norm(t.double(), 1e-3, w.double()))
+            got = z[:, c:c + h * s.dk]
+            assert rel(heads_of(got, h, s.dk, dim), want) < tol(where)
+            assert float(got.reshape(n, h, s.dk)[:, :, dim:].float().abs().sum()) == 0
+        want = O.head_norm(v.double(), 1e-3)
+        if mixed:
+            want = (1 - 0.37) * want + 0.37 * other.double()
+        assert rel(heads_of(z[:, lay.v:], kv_heads, s.dv, vdim), want) < tol(where)
+        cpu = {name: t.cpu() for name, t in cache[0].items()}
+        for i, p in enumerate(at):
+            for name, c, e in (("k", lay.k, lay.v), ("v", lay.v, lay.width)):
+                assert torch.equal(cache_rows(cpu, name, slots[i], torch.tensor([p])).flatten(), z[i, c:e].cpu())
+
+
+@where
+@pytest.mark.parametrize("rows,width,groups", [(1, 32, 1), (5, 50, 5), (5, 50, 1), (3, 96, 3), (2, 64, 16), (4, 36, 12), (3, 4104, 2), (2, 5000, 8), (2, 2560, 10), (2, 49, 7),
+                                               (1, 9000, 1)])
+def test_group_norms(where, rows, width, groups):
+    dev, dt, pad, eps = where[0], getattr(torch, where[1]), round_up(width, 32), 1e-3
+    x, gain = torch.zeros(rows, pad), torch.zeros(pad)
+    loud = torch.repeat_interleave(torch.logspace(-2, 1, groups), width // groups)           # groups of unequal size
+    x[:, :width], gain[:width] = torch.randn(rows, width) * loud, torch.rand(width) + 0.5
+    got = ops.group_norm(x.to(dev), width, groups, gain.to(dev), eps, dt)
+    assert rel(got[:, :width], O.group_norm(x[:, :width].double(), gain[:width].double(), groups, eps)) < tol(where)
+    assert float(got[:, width:].float().abs().sum()) == 0 and got.dtype == dt
+    for ydt in {torch.float32, dt}:
+        y = torch.zeros(rows, pad, dtype=ydt)
+        y[:, :width] = (torch.randn(rows, width) * loud * 0.1).to(ydt)
+        want = x[:, :width].double() + O.group_norm(y[:, :width].double(), gain[:width].double(), groups, eps)
+        for asked in (True, False):
+            xs = x.clone().to(dev)
+            h = ops.residual_group_norm(xs, y.to(dev), width, groups, gain.to(dev), eps, dt, asked)
+            assert rel(xs[:, :width], want) < 2e-6 and float(xs[:, width:].abs().sum()) == 0
+            assert h is None if not asked else torch.equal(h, xs.to(dt)) and h.data_ptr() != xs.data_ptr()
+    emb, ids = torch.randn(9, width).to(dt), torch.tensor([8, 0, 3])
+    xs, h = ops.embed_rows(ids.to(dev), emb.to(dev), pad)
+    assert torch.equal(xs[:, :width].cpu(), emb[ids].float()) and torch.equal(h.float(), xs) and float(xs[:, width:].abs().sum()) == 0 and h.data_ptr() != xs.data_ptr()
+
+
+@where
+def test_softcap(where):
+    z = torch.randn(7, 33) * 20
+    assert rel(ops.softcap_(z.clone().to(where[0]), 5.0), O.softcap(z.double(), 5.0)) < 1e-6
+
+
+@where
+@pytest.mark.parametrize("rows", [1, 16, 17, 300])
+def test_gated_relu_feed_forward(where, rows):
+    dev, dt = where[0], getattr(torch, where[1])
+    h, w1, w2 = torch.randn(rows, 64).to(dt), (torch.randn(2 * 96, 64) * 0.2).to(dt), (torch.randn(64, 96) * 0.1).to(dt)
+    got = PA.sublayer_out(PA.glu_in(h.to(dev), w1.to(dev), "relu"), w2.to(dev))
+    assert rel(got, O.relu_mlp(h.double(), {"gate": w1[:96].double(), "up": w1[96:].double(), "down": w2.double()})) < tol(where)
+
+
+def talk_case(where, H, G, dk, dv, window, starts, counts, sharp=(), seed=0, scale=None, table=None):
+    """Random queries, keys, values and mixing table through the prompt or step kernels, cached keys included; the result and the
+    definition's, row by row.  ``sharp``: (request, query position, key position, head) whose score is made to stand out."""
+    dev, dt = where[0], getattr(torch, where[1])
+    g = torch.Generator().manual_seed(seed)
+    scale = dk ** -0.5 if scale is None else scale
+    ends = [s + c for s, c in zip(starts, counts)]
+    qs, ks, vs = ([torch.randn(e, n, d, generator=g) for e in ends] for n, d in ((H, dk), (G, dk), (G, dv)))
+    for r, i, j, h in sharp:
+        qs[r][i, h] = 3.0 * ks[r][j, h // (H // G)]
+    qs, ks, vs = ([t.to(dt) for t in x] for x in (qs, ks, vs))
+    if table is None:
+        table = torch.eye(H) + 0.7 * H ** -0.5 * torch.randn(H, H, generator=g)
+    cache = SlotCache([LayerPages(G, dk, dv) if window is None else LayerRows(window, G, dk, dv)], 2, dev, dt)
+    for t in cache[0].values():
+        if t.dtype == dt:
+            t.fill_(1e3)                                                      # what nobody has written must not matter
+    cache.acquire(3)
+    slots = cache.acquire(len(starts))
+    cache.reserve(slots[::-1], ends[::-1])
+    batch = RowBatch(starts, counts, slots, dev)
+    cpu = {name: t.cpu() for name, t in cache[0].items()}
+    for r, slot in enumerate(slots):
+        upto = ends[r] if batch.decode else starts[r]
+        if upto:
+            keep = torch.arange(0 if window is None else max(0, upto - window), upto)
+            store(cpu, "k", slot, keep, ks[r][keep])
+            store(cpu, "v", slot, keep, vs[r][keep])
+    for name, t in cache[0].items():
+        t.copy_(cpu[name])
+    new = [slice(s, e) for s, e in zip(starts, ends)]
+    q = torch.cat([t[s] for t, s in zip(qs, new)]).reshape(-1, H * dk).to(dev)
+    out = torch.full((q.shape[0], H * dv), 7.0, dtype=dt, device=dev)
+    if batch.decode:
+        PA.step_attention(q, out, H, G, dk, dv, scale, window, cache[0], batch, table.to(dev))
+    else:
+        mats = []
+        for name, src, d in (("k", ks, dk), ("v", vs, dv)):
+            m = torch.full((batch.key_rows(window), G * d), float("nan"), dtype=dt, device=dev)
+            ops.gather_rows(m, None, cache[0], name, batch.key_sources(window, True))
+            ops.gather_rows(m, torch.cat([t[s] for t, s in zip(src, new)]).reshape(-1, G * d).to(dev), cache[0], name, batch.key_sources(window, False))
+            mats.append(m)
+        PA.causal_attention(q, *mats, out, H, G, dk, dv, scale, window, batch, None, table.to(dev))
+    want = []
+    for a, b, c, s in zip(qs, ks, vs, new):
+        i = torch.arange(len(a))
+        seen = (i[None, :] <= i[:, None]) & (i[:, None] - i[None, :] < (window or len(a)))
+        want.append(O.apply_weights(O.talk(O.softmax_weights(a.double(), b.double(), scale, seen), table.double()), c.double())[s])
+    return out, torch.cat(want)
+
+
+SHAPES = [(4, 2, 32, 32, None), (2, 1, 16, 64, None), (3, 3, 48, 16, None), (10, 1, 80, 112, None), (2, 2, 128, 128, None), (10, 5, 128, 64, None), (20, 5, 64, 32, None),
+          (9, 3, 128, 128, None), (1, 1, 16, 16, None), (4, 2, 160, 32, None), (2, 2, 400, 416, None), (4, 2, 32, 48, 20), (6, 2, 64, 64, 64), (40, 2, 16, 16, None)]
+shapes = pytest.mark.parametrize("shape", SHAPES, ids=lambda s: f"h{s[0]}g{s[1]}d{s[2]}v{s[3]}w{s[4]}")
+
+
+@where
+@shapes
+def test_talking_heads_in_prompts(where, shape):
+    """Requests that end inside, on and past tiles, from their first token and from the middle."""
+    got, want = talk_case(where, *shape, [0] * 5, [131, 64, 1, 63, 129])
+    assert rel(got, want) < tol(where)
+    got, want = talk_case(where, *shape, [64, 5, 0, 63, 200, 64], [2, 128, 7, 1, 131, 64], seed=1)
+    assert rel(got, want) < tol(where)
+
+
+@where
+@shapes
+def test_talking_heads_in_steps(where, shape):
+    starts = [1, 15, 16, 17, 62, 63, 64, 65, 700]
+    got, want = talk_case(where, *shape, starts, [1] * len(starts))
+    assert rel(got, want) < tol(where)
+    assert all(rel(g, w) < 2 * tol(where) for g, w in zip(got, want))
+    got, want = talk_case(where, *shape, [400], [1], seed=1)                  # alone: the keys are split over a cluster
+    assert rel(got, want) < tol(where)
+
+
+@where
+def test_a_window_of_pages(where):
+    """Steps of a layer whose window is shorter than what its pages hold."""
+    dev, dt, (H, G, d, n, window) = where[0], getattr(torch, where[1]), (4, 2, 32, 150, 40)
+    q, k, v, table = torch.randn(n, H, d).to(dt), torch.randn(n, G, d).to(dt), torch.randn(n, G, d).to(dt), torch.eye(H) + 0.3 * torch.randn(H, H)
+    cache = SlotCache([LayerPages(G, d, d)], 1, "cpu", dt)
+    slots = cache.acquire(1)
+    cache.reserve(slots, [n])
+    store(cache[0], "k", 0, torch.arange(n), k)
+    store(cache[0], "v", 0, torch.arange(n), v)
+    c, i = {name: t.to(dev) for name, t in cache[0].items()}, torch.arange(n)
+    seen = (i[None, :] <= i[:, None]) & (i[:, None] - i[None, :] < window)
+    want = O.apply_weights(O.talk(O.softmax_weights(q.double(), k.double(), 0.2, seen), table.double()), v.double())
+    for p in (1, 38, 39, 40, 41, 63, 64, 103, 104, 149):
+        out = torch.zeros(1, H * d, dtype=dt, device=dev)
+        PA.step_attention(q[p:p + 1].reshape(1, -1).to(dev), out, H, G, d, d, 0.2, window, c, RowBatch([p], [1], slots, dev), table.to(dev))
+        assert rel(out[0], want[p]) < tol(where), p
+
+
+@where
+@pytest.mark.parametrize("decode", [False, True])
+def test_one_key_of_one_head_stands_out(where, decode):
+    """One head looks at one key, at page and tile borders, near and far: what the other heads see of it is what the table says."""
+    H, G, d = 6, 3, 32
+    table = torch.zeros(H, H)
+    for h in range(H):
+        table[h, (h + 1) % H], table[h, 2] = 1.0, -0.5 * (h % 3)             # nobody uses its own weights
+    for i, j in ((300, 0), (300, 1), (300, 63), (300, 64), (300, 127), (300, 128), (300, 299), (300, 300), (129, 128), (128, 0), (640, 5), (64, 63)):
+        for h in (0, 2, 5):
+            got, want = talk_case(where, H, G, d, 48, None, [i] if decode else [0], [1 if decode else i + 1], [(0, i, j, h)], i + j, 0.3, table)
+            assert rel(got[-1], want[-1]) < tol(where), (i, j, h)
+
+
+@where
+@pytest.mark.parametrize("decode", [False, True])
+def test_scores_that_rise(where, decode):
+    """Scores far beyond the range of exp, growing along the keys: the running maximum has to follow."""
+    H, d, n = 2, 64, 400
+    dev, dt = where[0], getattr(torch, where[1])
+    k = torch.randn(n, H, d)
+    k[:, :, 0] = torch.linspace(-300, 300, n)[:, None]
+    q, v, table = torch.randn(n, H, d) * 0.1, torch.randn(n, H, d), torch.tensor([[1.0, 0.4], [-0.3, 0.9]])
+    q[:, :, 0] = 1.0
+    q, k, v = q.to(dt), k.to(dt), v.to(dt)
+    seen = torch.ones(n, n, dtype=torch.bool).tril()
+    want = O.apply_weights(O.talk(O.softmax_weights(q.double(), k.double(), 1.0, seen), table.double()), v.double())
+    out = torch.zeros(n if not decode else 1, H * d, dtype=dt, device=dev)
+    if decode:
+        cache = SlotCache([LayerPages(H, d, d)], 1, "cpu", dt)
+        slots = cache.acquire(1)
+        cache.reserve(slots, [n])
+        store(cache[0], "k", 0, torch.arange(n), k)
+        store(cache[0], "v", 0, torch.arange(n), v)
+        c = {name: t.to(dev) for name, t in cache[0].items()}
+        PA.step_attention(q[-1:].reshape(1, -1).to(dev), out, H, H, d, d, 1.0, None, c, RowBatch([n - 1], [1], slots, dev), table.to(dev))
+        want = want[-1:]
+    else:
+        PA.causal_attention(*(t.reshape(n, -1).to(dev) for t in (q, k, v)), out, H, H, d, d, 1.0, None, RowBatch([0], [n], None, dev), None, table.to(dev))
+    assert rel(out, want) < tol(where)
+
+
+@where
+def test_long_prompts_go_in_parts(where, monkeypatch):
+    monkeypatch.setattr(PA, "TALK_BYTES", 1)                                  # one tile of queries at a time
+    got, want = talk_case(where, 4, 2, 32, 32, None, [0, 70, 0], [300, 130, 5])
+    assert rel(got, want) < tol(where)
+    monkeypatch.setattr(PA, "TALK_BYTES", 200 * 4 * 2 * 32 * 4)
+    got, want = talk_case(where, 4, 2, 32, 32, None, [0, 70, 0], [300, 130, 5])
+    assert rel(got, want) < tol(where)
+
+
+def test_parts_of_work_lists():
+    b = RowBatch([0, 5, 0], [300, 130, 7], [0, 1, 2], "cpu")
+    parts = b.causal_parts(None, 128, 180)
+    assert [(r, e) for r, e, _ in parts] == [(0, 128), (128, 300), (300, 437)]
+    every = sorted(t for _, _, items in parts for t in items.tolist())
+    assert every == sorted(b.causal_items(None, 128).tolist())
+    for r, e, items in parts:
+        assert all(r <= t[0] and t[0] + t[1] <= e for t in items.tolist())
+
+
+def test_groups_of_a_recurrence():
+    """Groups cover every row once; the states of a request of several groups are places of its own."""
+    b = RowBatch([0, 9, 0, 3], [130, 64, 1, 200], [5, 0, 2, 1], "cpu")
+    groups, states, many = b.recurrent_groups(64)
+    assert states == 3 + 4 and many.tolist() == [[5, 0, 0, 3, 64, 0, 0, 0], [1, 4, 3, 4, 64, 0, 0, 0]]
+    assert groups.tolist() == [[0, 64, 5, 1, 0, 1, 0, 0], [64, 64, 5, 0, 1, 2, 0, 0], [128, 2, 5, 2, 2, -1, 0, 0], [130, 64, 0, 7, -1, -1, 0, 0],
+                               [194, 1, 2, 3, -1, -1, 0, 0], [195, 64, 1, 5, 3, 4, 0, 0], [259, 64, 1, 4, 4, 5, 0, 0], [323, 64, 1, 4, 5, 6, 0, 0],
+                               [387, 8, 1, 6, 6, -1, 0, 0]]
+    for counts, heads in (([4096] * 4, 16), ([4096], 16), ([1], 4), ([100, 5000, 3], 2), ([64] * 300, 8), ([131072], 32)):
+        per = RT.group_tokens(counts, heads, 148)
+        assert per % RT.CHUNK == 0 and sum(-(-c // per) for c in counts) <= max(148 // heads, len(counts))
+        assert per >= min(8 * RT.CHUNK, round_up(max(counts), RT.CHUNK))
+
+
+def retention_case(where, heads, dim, vdim, starts, counts, rot=None, decay=None, sharp=(), seed=0, keep_cache=True):
+    """Random projections of several requests; those that start in the middle come with the state the definition left."""
+    dev, dt = where[0], getattr(torch, where[1])
+    g = torch.Generator().manual_seed(seed)
+    rot = dim // 2 * 2 if rot is None else rot
+    decay = tuple(1 - 2.0 ** -(3 + 2 * h) for h in range(heads)) if decay is None else decay
+    s = RT.RetentionSpec(heads, dim, vdim, decay, rot, 300.0)
+    lay, eps = RT.RetentionLayout.of(s), 1e-3
+    ends = [a + c for a, c in zip(starts, counts)]
+    q, k, v, gate = ([torch.randn(e, heads, d, generator=g) for e in ends] for d in (dim, dim, vdim, vdim))
+    for r, i, j in sharp:
+        t = torch.tensor([i, j])
+        for h in range(heads):                                                # the same vector seen from both positions
+            u = torch.randn(1, 1, dim, generator=g)
+            q[r][i, h] = 2 * O.rotate(u.double(), -t[:1], rot, 300.0)[0, 0]
+            k[r][j, h] = 8 * O.rotate(u.double(), -t[1:], rot, 300.0)[0, 0]
+    q, k, v, gate = ([t.to(dt) for t in x] for x in (q, k, v, gate))
+    want, states = [], []
+    cache = SlotCache([LayerState(heads, s.dk, s.dv)], 2, dev, dt) if keep_cache else None
+    if keep_cache:
+        cache[0]["s"].fill_(1e3)                                              # what others have left must not matter
+        cache.acquire(1)
+        slots = cache.acquire(len(starts))
+        cache[0]["s"][slots] = 1e3
+    for r, (a, e) in enumerate(zip(starts, ends)):
+        pos = torch.arange(e)
+        qr, kr = (O.rotate(t[r].double(), pos, rot, 300.0) for t in (q, k))
+        kr = kr * dim ** -0.5
+        o, S = O.decayed_recurrence(qr, kr, v[r].double(), decay)
+        x = gate[r].double()
+        want.append((O.head_norm(o, eps) * x * torch.sigmoid(x))[a:])
+        states.append(S * dim ** 0.5)                                         # the kernels scale the queries instead of the keys
+        if a:
+            before = O.decayed_recurrence(qr[:a], kr[:a], v[r][:a].double(), decay)[1] * dim ** 0.5
+            cache[0]["s"][slots[r]] = torch.nn.functional.pad(before, (0, s.dv - vdim, 0, s.dk - dim)).float().to(dev)
+    z = torch.cat([torch.cat([laid_out(t[r][a:], d) for t, d in ((q, s.dk), (k, s.dk), (v, s.dv), (gate, s.dv))], 1) for r, a in enumerate(starts)]).to(dev)
+    batch = RowBatch(starts, counts, slots if keep_cache else None, dev)
+    out = torch.full((z.shape[0], round_up(heads * s.dv, 32)), 7.0, dtype=dt, device=dev)
+    RT.retention_rows(z, out, lay, s, s.powers(dev), s.decays(dev), s.frequencies(dev), eps, batch, None if cache is None else cache[0])
+    got = heads_of(out[:, :heads * s.dv], heads, s.dv, vdim)
+    assert float(out[:, :heads * s.dv].reshape(-1, heads, s.dv)[:, :, vdim:].float().abs().sum()) == 0
+    if keep_cache:
+        for r, slot in enumerate(slots):
+            assert rel(cache[0]["s"][slot][:, :dim, :vdim], states[r]) < tol(where)
+        assert float((cache[0]["s"][0] - 1e3).abs().max()) == 0
+    return got, torch.cat(want)
+
+
+RETENTION = [(3, 24, 40), (2, 64, 64), (2, 128, 128), (1, 16, 16), (5, 9, 7), (2, 144, 32), (2, 32, 272), (1, 48, 256), (2, 112, 64), (4, 32, 96)]
+retentions = pytest.mark.parametrize("shape", RETENTION, ids=lambda s: f"h{s[0]}d{s[1]}v{s[2]}")
+
+
+@where
+@retentions
+def test_retention_in_prompts(where, shape):
+    """Requests that end inside, on and past chunks, from their first token and from a state."""
+    got, want = retention_case(where, *shape, [0] * 6, [1, 2, 63, 64, 65, 130])
+    assert rel(got, want) < tol(where)
+    got, want = retention_case(where, *shape, [5, 0, 64, 63], [2, 70, 129, 64], seed=1)
+    assert rel(got, want) < tol(where)
+    got, want = retention_case(where, *shape, [0, 0], [3, 80], seed=2, keep_cache=False)
+    assert rel(got, want) < tol(where)
+
+
+@where
+@retentions
+def test_retention_in_steps(where, shape):
+    starts = [1, 2, 63, 64, 65, 0, 130]                                       # one of them has its first token here
+    got, want = retention_case(where, *shape, starts, [1] * len(starts))
+    assert rel(got, want) < tol(where)
+
+
+@where
+@pytest.mark.parametrize("starts,counts", [([0], [1541]), ([70], [1100]), ([0, 40, 0], [600, 1030, 3])])
+def test_long_prompts_are_cut_into_groups(where, starts, counts):
+    """States between the groups of a request, with a past and without; the last group is not whole."""
+    got, want = retention_case(where, 2, 32, 48, starts, counts, decay=(0.97, 0.9999))
+    assert rel(got, want) < tol(where)
+    assert rel(got[-3:], want[-3:]) < tol(where)
+
+
+@where
+@pytest.mark.parametrize("decode", [False, True])
+def test_a_far_key_stays_in_the_state(where, decode):
+    """A loud key far back, at chunk borders, with decays of (almost) one; a decay of zero remembers nothing."""
+    for i, j in ((300, 0), (300, 63), (300, 64), (200, 127), (200, 128), (129, 128), (64, 63), (600, 1)):
+        got, want = retention_case(where, 3, 32, 32, [i] if decode else [0], [1 if decode else i + 1], decay=(1.0, 0.9999, 0.0), sharp=[(0, i, j)], seed=i + j)
+        assert rel(got[-1], want[-1]) < tol(where), (i, j)
+
+
+@where
+def test_rotation_dimensions_of_retention(where):
+    for dim, rot in ((32, 0), (32, 2), (32, 10), (64, 48), (24, 24)):
+        for starts, counts in (([0, 20], [40, 9]), ([7, 100], [1, 1])):
+            got, want = retention_case(where, 2, dim, 16, starts, counts, rot=rot)
+            assert rel(got, want) < tol(where), (dim, rot)
+
+
+def test_states_and_slots():
+    c = SlotCache([LayerState(2, 16, 32), LayerPages(1, 16, 16)], 1, "cpu", torch.bfloat16)
+    assert c[0]["s"].shape == (1, 2, 16, 32) and c[0]["s"].dtype == torch.float32
+    a = c.acquire(1)
+    c[0]["s"][a] = 3.0
+    was = c.generation
+    c.acquire(3)                                                              # more slots than there were
+    assert c.generation > was and c[0]["s"].shape[0] == 4 and bool((c[0]["s"][a] == 3.0).all())
+    assert c.nbytes() == 4 * 2 * 16 * 32 * 4 + 2 * c[1]["k"].numel() * 2
+
+
+# ------------------------------------------------------------------------------------------------------------- whole models
+@where
+@pytest.mark.parametrize("name", list(CONFIGS))
+def test_model_matches_definition(build, where, name):
+    model, w, cfg = build(name, where)
+    ids = prompt(cfg, 330 if name == "wide" else 150)
+    model.residual_taps = taps = []
+    with torch.no_grad():
+        got = model(ids[None].to(where[0]))[0]
+    model.residual_taps = None
+    stream = O.hidden_states(w, cfg, ids)
+    for n, t in enumerate(taps):
+        assert rel(t, stream[n]) < tol(where), f"layer {n}"
+    assert rel(got, O.logits(w, cfg, ids)) < 1.5 * tol(where)
+
+
+@where
+@pytest.mark.parametrize("name", list(CONFIGS))
+def test_prompt_then_one_by_one(build, where, name):
+    """Unequal requests in one batch, decoded together over pages and chunks; each against the definition alone."""
+    model, w, cfg = build(name, where)
+    lens, extra = ([149, 1, 300, 17] if name == "wide" else [36, 1, 62, 17]), (4 if name in ("wide", "large") else 12)
+    seqs = [prompt(cfg, n + extra, seed=n) for n in lens]
+    want = [O.logits(w, cfg, s) for s in seqs]
+    ses = InferenceSession(model, slots=2)                               # fewer than needed: the cache grows
+    slots, lg = ses.start([s[:n] for s, n in zip(seqs, lens)], [list(range(n)) for n in lens])
+    at = 0
+    for k, n in enumerate(lens):
+        assert rel(lg[at:at + n], want[k][:n]) < 1.5 * tol(where), k
+        at += n
+    for t in range(extra):
+        lg = ses.step(slots, torch.stack([s[n + t] for s, n in zip(seqs, lens)]))
+        for k, n in enumerate(lens):
+            assert rel(lg[k], want[k][n + t]) < 1.5 * tol(where), (t, k)
+    ses.finish(slots)
+    assert ses.cache.lengths == {} and sorted(ses.cache.free_pages) == list(range(ses.cache.pages))
+
+
+@where
+@pytest.mark.parametrize("portion", [1, 2, 3, 7, 21, 64, 70])
+def test_portions_of_a_prompt(build, where, portion):
+    model, w, cfg = build("mixed", where)
+    ids = prompt(cfg, 140 if portion > 1 else 70, seed=5)
+    want = O.logits(w, cfg, ids)
+    ses = InferenceSession(model)
+    slot, got, at = ses.cache.acquire(1), [], 0
+    while at < len(ids):
+        part = ids[at:at + portion]
+        got.append(ses.extend(slot, [part], [list(range(len(part)))]))
+        at += len(part)
+    assert rel(torch.cat(got), want) < 1.5 * tol(where)
+
+
+@where
+def test_mixed_batches(build, where):
+    """New prompts, portions of prompts and single tokens in the same call."""
+    model, w, cfg = build("mixed", where)
+    seqs = [prompt(cfg, n, seed=n) for n in (90, 80, 70, 5)]
+    want = [O.logits(w, cfg, s) for s in seqs]
+    cuts = [[40, 41, 42, 90], [0, 30, 79, 80], [0, 0, 1, 70], [2, 2, 3, 5]]   # lengths of the requests after every call
+    ses = InferenceSession(model)
+    slots, at = ses.cache.acquire(4), [0] * 4
+    for call in range(4):
+        go = [r for r in range(4) if cuts[r][call] > at[r]]
+        parts = [seqs[r][at[r]:cuts[r][call]] for r in go]
+        lg = ses.extend([slots[r] for r in go], parts, [list(range(len(p))) for p in parts])
+        row = 0
+        for r, p in zip(go, parts):
+            assert rel(lg[row:row + len(p)], want[r][at[r]:at[r] + len(p)]) < 1.5 * tol(where), (call, r)
+            at[r], row = at[r] + len(p), row + len(p)
+
+
+@where
+def test_slots_and_pages_are_used_again(build, where):
+    """Requests that start in slots and pages others have left (full of their keys, states and garbage), while a third one lives on; some
+    of them start with a single token, together with a step of the one that lives on."""
+    model, w, cfg = build("mixed", where)
+    ses = InferenceSession(model, slots=3, tokens=400)
+    pages = ses.cache.pages
+    keep = prompt(cfg, 90, seed=9)
+    kept, _ = ses.start([keep[:60]])
+    at, used = 60, set()
+    for turn, n in enumerate((130, 5, 64, 1)):
+        a, b = prompt(cfg, n + 3, seed=turn), prompt(cfg, 63 + turn, seed=20 + turn)
+        if n == 1:
+            sa, = ses.cache.acquire(1)
+            lg = ses.extend([kept[0], sa], [keep[at:at + 1], a[:1]])
+            assert rel(lg[0], O.logits(w, cfg, keep[:at + 1])[-1]) < 1.5 * tol(where) and rel(lg[1], O.logits(w, cfg, a[:1])[-1]) < 1.5 * tol(where)
+            at += 1
+        else:
+            (sa,), _ = ses.start([a[:n]])
+        (sb,), lb = ses.start([b])
+        used |= {sa, sb}
+        assert rel(lb[0], O.logits(w, cfg, b)[-1]) < 1.5 * tol(where)
+        for t in range(3):
+            lg = ses.step([kept[0], sa], torch.stack([keep[at], a[n + t]]))
+            assert rel(lg[0], O.logits(w, cfg, keep[:at + 1])[-1]) < 1.5 * tol(where)
+            assert rel(lg[1], O.logits(w, cfg, a[:n + t + 1])[-1]) < 1.5 * tol(where)
+            at += 1
+        ses.finish([sb, sa])
+        for spec, layer in zip(ses.cache.spec, ses.cache.layers):
+            for name, t in layer.items():
+                if name != "table":
+                    t[ses.cache.free_pages if isinstance(spec, LayerPages) else ses.cache.free] = 50.0
+    assert used == {1, 2} and ses.cache.slots == 3 and ses.cache.pages == pages
+
+
+@where
+@pytest.mark.parametrize("graph", [False, True])
+def test_long_decoding(build, where, graph):
+    """From one token over many pages, without a prompt; the pool and its table grow on the way."""
+    model, w, cfg = build("mixed", where)
+    ids = prompt(cfg, 200, seed=2)
+    want = O.logits(w, cfg, ids)
+    ses = InferenceSession(model, cuda_graph=graph)
+    slot, lg = ses.start([ids[:1]])
+    worst = rel(lg[0], want[0])
+    for t in range(1, len(ids)):
+        worst = max(worst, rel(ses.step(slot, ids[t:t + 1])[0], want[t]))
+    assert worst < 2 * tol(where)
+
+
+@where
+def test_logits_do_not_depend_on_the_batch(build, where):
+    model, w, cfg = build("wide", where)
+    seqs = [prompt(cfg, n, seed=n) for n in (3, 160, 129, 40)]
+    alone = [InferenceSession(model).start([s])[1][0].clone() for s in seqs]
+    together = InferenceSession(model).start(seqs)[1]
+    for a, b in zip(alone, together):
+        assert rel(b, a.double().cpu()) < (2e-2 if where[1] == "bfloat16" else 1e-5)
+
+
+@GPU
+def test_many_requests_together(build):
+    """More tokens per step than the weight-streaming kernels take."""
+    where = ("cuda", "bfloat16")
+    model, w, cfg = build("mixed", where)
+    for n in (20, 70):
+        seqs = [prompt(cfg, 4 + k % 40, seed=k) for k in range(n)]
+        ses = InferenceSession(model, cuda_graph=True)
+        slots, _ = ses.start([s[:-3] for s in seqs])
+        for t in range(3):
+            lg = ses.step(slots, torch.stack([s[t - 3] for s in seqs])).clone()
+        for k in range(0, n, 7):
+            assert rel(lg[k], O.logits(w, cfg, seqs[k])[-1]) < 2 * tol(where), k
+
+
+# --------------------------------------------------------------------------------------- generation, folders, command line
+@where
+@pytest.mark.parametrize("graph", [False, True])
+def test_greedy_generation(build, where, graph):
+    model, w, cfg = build("mixed", where)
+    prompts = [prompt(cfg, n, seed=n) for n in (60, 66, 9)]
+    t, n = padded(prompts, 12)
+    got, lens, lp = generate_tokens(model, t.to(where[0]), n.to(where[0]), top_k=1, return_log_probs=True, cuda_graph=graph)
+    got, lp = got.cpu(), lp.cpu()
+    assert lens.tolist() == [78] * 3
+    for b, p in enumerate(prompts):
+        seq = got[b].tolist()
+        assert seq[:len(p)] == p.tolist()
+        lg = O.logits(w, cfg, seq)
+        ref = torch.log_softmax(lg, -1)[torch.arange(len(seq) - 1), torch.tensor(seq[1:])]
+        assert float((lp[b].double() - ref).abs().max()) < (0.5 if where[1] == "bfloat16" else 1e-3)
+        for i in range(len(p), len(seq)):                              # every token is the largest logit, up to rounding
+            assert float(lg[i - 1].max() - lg[i - 1][seq[i]]) < (0.3 if where[1] == "bfloat16" else 1e-4)
+        if where[1] == "float32" and b < 2:
+            assert seq[len(p):] == O.greedy(w, cfg, p.tolist(), len(seq) - len(p))
+
+
+def test_existing_loops_run_the_model(build):
+    """Scoring, beam search and plain calls with ``caches`` and ``position_offset``, as the other models take them."""
+    from linear_moe_b200.infer.generation import beam_search, score_tokens
+    model, w, cfg = build("odd", ("cpu", "float32"))
+    ids = torch.stack([prompt(cfg, 70, seed=s) for s in (1, 2)])
+    want = torch.stack([O.logits(w, cfg, s) for s in ids])
+    lp = torch.log_softmax(want, -1)[:, :-1].gather(2, ids[:, 1:, None]).squeeze(2)
+    assert float((score_tokens(model, ids).double() - lp).abs().max()) < 2e-4
+    caches, got = model.new_cache(), []
+    for lo, hi in ((0, 9), (9, 10), (10, 31), (31, 70)):
+        got.append(model(ids[:, lo:hi], caches=caches, position_offset=lo))
+    assert rel(torch.cat(got, 1), want) < 3e-5
+    loss = model(ids[:, :-1], labels=ids[:, 1:])
+    assert float((loss.double() + lp).abs().max()) < 2e-4
+    toks, _ = beam_search(model, ids[:1, :5], 1, 6, eod=-1)
+    assert toks[0, :11].tolist() == ids[0, :5].tolist() + O.greedy(w, cfg, ids[0, :5].tolist(), 6)
+
+
+def test_training_is_refused(build):
+    from linear_moe_b200.config.model_config import ParallelConfig, TrainConfig
+    from linear_moe_b200.train.loop import Trainer
+    model, _, _ = build("odd", ("cpu", "float32"))
+    with pytest.raises(ValueError, match="serve"):
+        Trainer(model.cfg, ParallelConfig(), TrainConfig())
+
+
+def test_folder_errors(tmp_path):
+    cfg = CONFIGS["mixed"]
+    w = O.random_model(cfg)
+
+    def refused(cfg_, w_, match, exc=ValueError):
+        with pytest.raises(exc, match=match):
+            load_model(folder(tmp_path / "m", cfg_, w_), torch.float32, "cpu")
+
+    def changed(layer, **kw):
+        c = json.loads(json.dumps(cfg))
+        for k, v in kw.items():
+            (c["layers"][layer] if k in ("type", "mlp") else c["layers"][layer]["mixer"])[k] = v
+        return c
+    load_model(folder(tmp_path / "m", cfg, w), torch.float32, "cpu")
+    refused(cfg, {k: v for k, v in w.items() if k != "l1.mix.talk"}, "l1.mix.talk", KeyError)
+    refused(cfg, {k: v for k, v in w.items() if k != "l4.mix.vmix"}, "l4.mix.vmix", KeyError)
+    refused(cfg, {k: v for k, v in w.items() if k != "l0.ls2"}, "l0.ls2", KeyError)
+    refused(cfg, {**w, "l0.mix.g": w["l0.mix.g"][:-1]}, "mix.g")
+    refused(cfg, {**w, "l1.mix.q.norm": w["l1.mix.q.norm"][:-1]}, "q.norm")
+    refused(cfg, {**w, "final.norm": w["final.norm"][:-1]}, "final.norm")
+    refused(changed(1, type="pooling"), w, "pooling")
+    refused(changed(1, mlp={"kind": "other"}), w, "other")
+    refused(changed(0, decay=[0.5, 0.5]), w, "decays")
+    refused(changed(0, decay=[0.5, 0.5, 1.5]), w, "decays")
+    refused(changed(4, vdim=16), w, "layer 2")
+    refused(changed(1, kv_heads=4), w, "evenly")
+    refused(changed(1, rot={"dims": 26, "base": 10.0}), w, "rotated")
+    refused(changed(1, rot={"dims": 16, "base": 10.0, "scaling": {**YARN, "factor": 0.0}}), w, "scaling")
+    refused(changed(1, scale=0.0), w, "scale")
+    refused({**cfg, "norm": {"eps": 1e-5, "groups": 7}}, w, "equal parts")
+    refused({**cfg, "logit_softcap": -1.0}, w, "cap")
+
+
+def test_trace_replay(build, tmp_path):
+    """The replayer's protocol on the CPU: file contents, order of the rows, steps without a file, slots given back."""
+    import numpy as np
+    from linear_moe_b200.infer.trace import replay
+    model, w, cfg = build("mixed", ("cpu", "float32"))
+    a, b = prompt(cfg, 66, seed=1), prompt(cfg, 12, seed=2)
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": a[:64].tolist(), "want": [63, 0]}, {"id": "b", "tokens": b[:11].tolist(), "want": []}], "end": []},
+             {"step": 1, "entries": [{"id": "b", "tokens": b[11:].tolist(), "want": [0]}, {"id": "a", "tokens": a[64:65].tolist(), "want": [0]}], "end": ["b"]},
+             {"step": 2, "entries": [{"id": "a", "tokens": a[65:].tolist(), "want": []}], "end": ["a"]}]
+    said, ses = [], InferenceSession(model)
+    replay(ses, io.StringIO("\n".join(json.dumps(s) for s in steps) + "\n"), str(tmp_path), said.append)
+    assert said == ["done 0", "done 1", "done 2"] and sorted(os.listdir(tmp_path)) == ["0.f32", "1.f32"] and ses.cache.lengths == {}
+    la, lb = O.logits(w, cfg, a), O.logits(w, cfg, b)
+    for name, want in (("0.f32", torch.stack([la[63], la[0]])), ("1.f32", torch.stack([lb[11], la[64]]))):
+        got = torch.from_numpy(np.fromfile(tmp_path / name, dtype="<f4").reshape(2, cfg["vocab"]).copy())
+        assert rel(got, want) < 3e-5
+
+
+@GPU
+@pytest.mark.parametrize("dtype,graph", [("float32", []), ("bfloat16", []), ("bfloat16", ["--cuda-graph"])])
+def test_trace_program(tmp_path, dtype, graph):
+    import numpy as np
+    cfg = CONFIGS["mixed"]
+    w = O.random_model(cfg, seed=3, gain=3.0 if dtype == "float32" else 1.5)
+    d, a = folder(tmp_path / "m", cfg, w), prompt(cfg, 69, seed=1)
+    steps = [{"step": 0, "entries": [{"id": "q", "tokens": a[:60].tolist(), "want": [59]}], "end": []}]
+    steps += [{"step": t, "entries": [{"id": "q", "tokens": [int(a[59 + t])], "want": [0]}], "end": ["q"] if t == 9 else []} for t in range(1, 10)]
+    out = tmp_path / "out"
+    out.mkdir()
+    r = subprocess.run([os.path.join(ROOT, "bin", "trace_run"), "--model", d, "--dtype", dtype, "--out", str(out), "--max-tokens", "69", *graph],
+                       input="\n".join(json.dumps(s) for s in steps) + "\n", capture_output=True, text=True, timeout=600)
+    assert r.returncode == 0, r.stderr[-2000:]
+    assert [l for l in r.stdout.splitlines() if l.startswith("done")] == [f"done {t}" for t in range(10)]
+    want = O.logits(w, cfg, a)
+    for t in range(10):
+        got = torch.from_numpy(np.fromfile(out / f"{t}.f32", dtype="<f4").copy())
+        assert rel(got, want[59 + t]) < (0.04 if dtype == "bfloat16" else 3e-5)
+
+
+@pytest.mark.parametrize("device", ["cpu", pytest.param("cuda", marks=GPU)])
+def test_command_line(tmp_path, device):
+    cfg = CONFIGS["odd"]
+    w = O.random_model(cfg, seed=4, gain=2.0)
+    d = folder(tmp_path / "m", cfg, w)
+    prompts = ["5 6 7 8 9 10 11", "3"]
+    (tmp_path / "in.txt").write_text("\n".join(prompts) + "\n")
+    env = dict(os.environ, **({"CUDA_VISIBLE_DEVICES": ""} if device == "cpu" else {}))
+    r = subprocess.run([sys.executable, os.path.join(ROOT, "examples", "generate.py"), "--model-dir", d, "--model-dtype", "float32",
+                        "--text-generate-input-file", str(tmp_path / "in.txt"), "--text-generate-output-file", str(tmp_path / "out.jsonl"),
+                        "--out-seq-length", "6", "--top-k", "1", "--cuda-graph-decode"], capture_output=True, text=True, timeout=600, env=env)
+    assert r.returncode == 0, r.stderr[-2000:]
+    for p, line in zip(prompts, open(tmp_path / "out.jsonl")):
+        ids = [int(t) for t in p.split()]
+        new = O.greedy(w, cfg, ids, 6)
+        if cfg["vocab"] - 1 in new:                                     # the tokenizer's end token
+            new = new[:new.index(cfg["vocab"] - 1) + 1]
+        assert [int(t) for t in json.loads(line)["output"].split()] == ids + new
+
+
+def test_server_request(build):
+    from linear_moe_b200.data.tokenizer import NullTokenizer
+    from linear_moe_b200.infer.server import run_request
+    model, w, cfg = build("odd", ("cpu", "float32"))
+    out = run_request(model, NullTokenizer(cfg["vocab"]), {"prompts": ["1 2 3", "4 5 6 7 8"], "tokens_to_generate": 4, "top_k": 1,
+                                                           "use_eod_token_for_early_termination": False})
+    for p, toks in zip(([1, 2, 3], [4, 5, 6, 7, 8]), out["tokens"]):
+        assert toks == p + O.greedy(w, cfg, p, 9 - len(p))
+
+
+@GPU
+def test_kernels_are_the_ones_that_run(build):
+    """The bf16 and fp32 paths launch this library's kernels, and the tcgen05 waits report no error."""
+    from linear_moe_b200.ops import cuda as K
+    from linear_moe_b200.ops import gemm
+    for where in (("cuda", "bfloat16"), ("cuda", "float32")):
+        model, w, cfg = build("wide", where)
+        K.reset_launch_count()
+        ses = InferenceSession(model)
+        slots, _ = ses.start([prompt(cfg, 200)])
+        ses.step(slots, torch.tensor([1]))
+        assert K.reset_launch_count() >= 2 * 3 * len(cfg["layers"])
+        gemm.check_error()
