@@ -185,6 +185,9 @@ def random_model(cfg, seed=0, gain=1.5):
         w[l + "norm1"], w[l + "ls1"] = weight(d), weight(d, 0.6)
         if layer["type"] == "retention":
             w[x + "q"], w[x + "k"], w[x + "v"], w[x + "g"] = (rnd(H * e, d, std=d ** -0.5) for e in (dk, dk, dv, dv))
+            # a token's key resembles its query: a first token's output is its value times their product, and the norm behind it would
+            # turn a product of about zero into a coin toss
+            w[x + "k"] = (0.8 * w[x + "q"].float() + 0.6 * w[x + "k"].float()).bfloat16()
         else:
             G = m["kv_heads"]
             w[x + "q"], w[x + "k"], w[x + "v"] = rnd(H * dk, d, std=d ** -0.5), rnd(G * dk, d, std=d ** -0.5), rnd(G * dv, d, std=d ** -0.5)

@@ -471,6 +471,12 @@ def test_states_and_slots():
 
 
 # ------------------------------------------------------------------------------------------------------------- whole models
+def one(where):
+    """Allowed error of the logits at one position.  In bf16 the worst of many positions of these random models is some four times the
+    average one by rounding alone (the CPU's bf16 shows the same); a lost key or state is several times that."""
+    return 0.1 if where[1] == "bfloat16" else 4e-5
+
+
 @where
 @pytest.mark.parametrize("name", list(CONFIGS))
 def test_model_matches_definition(build, where, name):
@@ -498,12 +504,15 @@ def test_prompt_then_one_by_one(build, where, name):
     slots, lg = ses.start([s[:n] for s, n in zip(seqs, lens)], [list(range(n)) for n in lens])
     at = 0
     for k, n in enumerate(lens):
-        assert rel(lg[at:at + n], want[k][:n]) < 1.5 * tol(where), k
+        assert rel(lg[at:at + n], want[k][:n]) < (1.5 * tol(where) if n > 8 else one(where)), k
         at += n
+    steps = []
     for t in range(extra):
         lg = ses.step(slots, torch.stack([s[n + t] for s, n in zip(seqs, lens)]))
+        steps.append(lg.clone())
         for k, n in enumerate(lens):
-            assert rel(lg[k], want[k][n + t]) < 1.5 * tol(where), (t, k)
+            assert rel(lg[k], want[k][n + t]) < one(where), (t, k)
+    assert rel(torch.stack(steps), torch.stack([torch.stack([s[n + t] for s, n in zip(want, lens)]) for t in range(extra)])) < 1.5 * tol(where)
     ses.finish(slots)
     assert ses.cache.lengths == {} and sorted(ses.cache.free_pages) == list(range(ses.cache.pages))
 
@@ -538,7 +547,7 @@ def test_mixed_batches(build, where):
         lg = ses.extend([slots[r] for r in go], parts, [list(range(len(p))) for p in parts])
         row = 0
         for r, p in zip(go, parts):
-            assert rel(lg[row:row + len(p)], want[r][at[r]:at[r] + len(p)]) < 1.5 * tol(where), (call, r)
+            assert rel(lg[row:row + len(p)], want[r][at[r]:at[r] + len(p)]) < (1.5 * tol(where) if len(p) > 8 else one(where)), (call, r)
             at[r], row = at[r] + len(p), row + len(p)
 
 
@@ -557,17 +566,17 @@ def test_slots_and_pages_are_used_again(build, where):
         if n == 1:
             sa, = ses.cache.acquire(1)
             lg = ses.extend([kept[0], sa], [keep[at:at + 1], a[:1]])
-            assert rel(lg[0], O.logits(w, cfg, keep[:at + 1])[-1]) < 1.5 * tol(where) and rel(lg[1], O.logits(w, cfg, a[:1])[-1]) < 1.5 * tol(where)
+            assert rel(lg[0], O.logits(w, cfg, keep[:at + 1])[-1]) < one(where) and rel(lg[1], O.logits(w, cfg, a[:1])[-1]) < one(where)
             at += 1
         else:
             (sa,), _ = ses.start([a[:n]])
         (sb,), lb = ses.start([b])
         used |= {sa, sb}
-        assert rel(lb[0], O.logits(w, cfg, b)[-1]) < 1.5 * tol(where)
+        assert rel(lb[0], O.logits(w, cfg, b)[-1]) < one(where)
         for t in range(3):
             lg = ses.step([kept[0], sa], torch.stack([keep[at], a[n + t]]))
-            assert rel(lg[0], O.logits(w, cfg, keep[:at + 1])[-1]) < 1.5 * tol(where)
-            assert rel(lg[1], O.logits(w, cfg, a[:n + t + 1])[-1]) < 1.5 * tol(where)
+            assert rel(lg[0], O.logits(w, cfg, keep[:at + 1])[-1]) < one(where)
+            assert rel(lg[1], O.logits(w, cfg, a[:n + t + 1])[-1]) < one(where)
             at += 1
         ses.finish([sb, sa])
         for spec, layer in zip(ses.cache.spec, ses.cache.layers):
@@ -586,10 +595,11 @@ def test_long_decoding(build, where, graph):
     want = O.logits(w, cfg, ids)
     ses = InferenceSession(model, cuda_graph=graph)
     slot, lg = ses.start([ids[:1]])
-    worst = rel(lg[0], want[0])
+    got = [lg[0].clone()]
     for t in range(1, len(ids)):
-        worst = max(worst, rel(ses.step(slot, ids[t:t + 1])[0], want[t]))
-    assert worst < 2 * tol(where)
+        got.append(ses.step(slot, ids[t:t + 1])[0].clone())
+    assert max(rel(g, r) for g, r in zip(got, want)) < one(where)
+    assert rel(torch.stack(got), want) < 1.5 * tol(where)
 
 
 @where
@@ -599,7 +609,7 @@ def test_logits_do_not_depend_on_the_batch(build, where):
     alone = [InferenceSession(model).start([s])[1][0].clone() for s in seqs]
     together = InferenceSession(model).start(seqs)[1]
     for a, b in zip(alone, together):
-        assert rel(b, a.double().cpu()) < (2e-2 if where[1] == "bfloat16" else 1e-5)
+        assert rel(b, a.double().cpu()) < (3e-2 if where[1] == "bfloat16" else 1e-5)
 
 
 @GPU
@@ -613,8 +623,8 @@ def test_many_requests_together(build):
         slots, _ = ses.start([s[:-3] for s in seqs])
         for t in range(3):
             lg = ses.step(slots, torch.stack([s[t - 3] for s in seqs])).clone()
-        for k in range(0, n, 7):
-            assert rel(lg[k], O.logits(w, cfg, seqs[k])[-1]) < 2 * tol(where), k
+        some = range(0, n, 7)
+        assert rel(lg[list(some)], torch.stack([O.logits(w, cfg, seqs[k])[-1] for k in some])) < 1.5 * tol(where)
 
 
 # --------------------------------------------------------------------------------------- generation, folders, command line
