@@ -127,14 +127,15 @@ def kernels(size: str) -> list:
     batch = RowBatch([0] * B, [T] * B, None, dev)
     lay = RT.RetentionLayout.of(ret)
     z, o = rnd(rows, lay.width), torch.empty(rows, H * D, dtype=bf, device=dev)
-    tables = (ret.powers(dev), ret.decays(dev), ret.frequencies(dev))
+    tables, turn = (ret.powers(dev), ret.decays(dev)), ops.rotary_rows(batch.pos, ret.frequencies(dev))
+    row("rotary_rows, once per call", "rotary table", timeit(lambda: ops.rotary_rows(batch.pos, ret.frequencies(dev))), bytes_=rows * D * 4)
     still = RT.RetentionSpec(H, D, D, ret.decay)
-    row("retention_tc (norm and gate inside)", "retention", timeit(lambda: RT.retention_rows(z, o, lay, still, *tables[:2], None, 1e-5, batch, None)),
+    row("retention_tc (norm and gate inside)", "retention", timeit(lambda: RT.retention_rows(z, o, lay, still, *tables, None, 1e-5, batch, None)),
         bytes_=rows * H * D * 10)
-    row("rotation of its queries and keys", "rotary", timeit(lambda: ops.rotate_heads_(z, lay.q, lay.k, H, H, D, D, True, tables[2], 1.0, batch)),
+    row("rotation of its queries and keys", "rotary", timeit(lambda: ops.rotate_heads_(z, lay.q, lay.k, H, H, D, D, True, turn, batch)),
         bytes_=rows * H * D * 8)
     long = RowBatch([0], [rows], None, dev)
-    row(f"retention_tc, one prompt of {rows}", "retention long", timeit(lambda: RT.retention_rows(z, o, lay, still, *tables[:2], None, 1e-5, long, None)),
+    row(f"retention_tc, one prompt of {rows}", "retention long", timeit(lambda: RT.retention_rows(z, o, lay, still, *tables, None, 1e-5, long, None)),
         bytes_=rows * H * D * 10)
     qkv = rnd(B, T, H, 3 * D)
     q, k, v = qkv.split([D, D, D], -1)
@@ -147,9 +148,10 @@ def kernels(size: str) -> list:
     row("head_norm_gate (hybrid)", "norm and gate", timeit(lambda: ops.head_norm_gate(ol, ones, gate)), bytes_=rows * H * D * 6)
     del z, qkv, q, k, v, ol, gate
     lay = PA.QkvLayout.of(att)
-    z, wq, wk, freq, mix = rnd(rows, lay.width), torch.ones(D, device=dev), torch.ones(D, device=dev), att.frequencies(dev), torch.tensor(0.5, device=dev)
+    z, wq, wk, turn, mix = rnd(rows, lay.width), torch.ones(D, device=dev), torch.ones(D, device=dev), \
+        ops.rotary_rows(batch.pos, att.frequencies(dev), att.rot_size), torch.tensor(0.5, device=dev)
     first = rnd(rows, G * D)
-    row("head_norm_rope, values mixed", "norm + rotary", timeit(lambda: ops.head_norm_rope_(z, lay, att, wq, wk, freq, 1e-5, batch, None, first, mix)),
+    row("head_norm_rope, values mixed", "norm + rotary", timeit(lambda: ops.head_norm_rope_(z, lay, att, wq, wk, turn, 1e-5, batch, None, first, mix)),
         bytes_=rows * (lay.width * 4 + G * D * 2))
     qf, kf, vf = rnd(B, T, H, D), rnd(B, T, G, D), rnd(B, T, G, D)
     cos, sin = torch.randn(T, D // 2, device=dev), torch.randn(T, D // 2, device=dev)
@@ -198,11 +200,12 @@ def kernels(size: str) -> list:
                 c_.reserve(slots, [CTX] * n)
                 made.append((c_[0],))
             return made
+        t1 = ops.rotary_rows(one_tok.pos, att.frequencies(dev))
         zr, orr = rnd(n, lr.width), torch.empty(n, H * D, dtype=bf, device=dev)
         by = n * H * D * D * 8
         sets = caches(LayerState(H, D, D), by)
         row(f"retention_step (rotation, norm, gate inside), batch {n}", "retention decode", _graph_ms(
-            lambda c_: RT.retention_rows(zr, orr, lr, ret, *tables, 1e-5, one_tok, c_), sets), bytes_=by)
+            lambda c_: RT.retention_rows(zr, orr, lr, ret, *tables, t1, 1e-5, one_tok, c_), sets), bytes_=by)
         q, k, v = rnd(n, 1, H, 3 * D).split([D, D, D], -1)
         row(f"lsm_scalar_step (hybrid), batch {n}", "retention decode", _graph_ms(lambda c_: ops.lsm_scalar(q, k, v, g, None, c_["s"]), sets), bytes_=by)
         del sets
@@ -222,7 +225,7 @@ def kernels(size: str) -> list:
         page = SlotCache([LayerPages(G, D, D)], n, dev, bf, tokens=n * CTX)
         page.reserve(page.acquire(n), [CTX] * n)
         row(f"head_norm_rope + store, batch {n}", "row kernel decode", _graph_ms(
-            lambda: ops.head_norm_rope_(za, lay, att, wq, wk, freq, 1e-5, one_tok, page[0], fa, mix), [()] * 100))
+            lambda: ops.head_norm_rope_(za, lay, att, wq, wk, t1, 1e-5, one_tok, page[0], fa, mix), [()] * 100))
         qr, cs = rnd(n, 1, H, D), torch.randn(1, D // 2, device=dev)
         row(f"apply_rope (hybrid), batch {n}", "row kernel decode", _graph_ms(lambda: ops.apply_rope(qr, cs, cs), [()] * 100))
         xf, yf, hn = torch.randn(n, w, device=dev), torch.randn(n, w, device=dev), rnd(n, w)

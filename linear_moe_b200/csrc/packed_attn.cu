@@ -4,6 +4,7 @@
 //   packed_attn_step_kernel   one token per request from the cache (bf16 fast path: packed_attn_step.cu)
 //   qk_norm_rope_kernel       RMS norm of all query rows of a projection and of all key rows, before the heads are split, then
 //                             interleaved rotary positions, in place; the new keys and values enter the cache
+//   rotary_rows_kernel        cos and sin of every row's angles, for all layers that rotate alike
 //   head_norm_rope_kernel     RMS norm of every query, key and value head, rotary positions in either pairing, values mixed with another
 //                             layer's, in place; the new keys and values enter the cache
 //   head_mix_kernel           talking heads: the outputs of every head's weights over every value head -> the heads' outputs
@@ -300,7 +301,7 @@ __global__ void __launch_bounds__(THREADS) qk_norm_rope_kernel(QkNorm a) {
 struct HeadNorm {
     void* z;                             // [rows, ldz]: queries (H x dk), keys (G x dk), values (V x dv) from columns zq, zk, zv
     const float *wq, *wk;                // norm weights [dk], shared by the heads (null: no norm)
-    const double* freq;                  // [rot / 2] rotation per position
+    const float2* turn;                  // [rows, rot / 2] (cos, sin)
     const void* first;                   // [rows, ldf]: v <- (1 - *mix) v + *mix first (null: values as they are)
     const float* mix;
     Cache c;                             // k null: nothing is stored
@@ -310,47 +311,53 @@ struct HeadNorm {
     int nk, nv;                          // numbers in a norm (the unpadded head sizes)
     int rot, halves;                     // rotated dimensions; pairs (i, i + rot / 2) or neighbours
     int norm_v;
-    float size, eps;                     // factor of cos and sin
+    float eps;
     int rows;
 };
+
+// turn [rows, half] = size (cos, sin) of pos * freq
+__global__ void __launch_bounds__(THREADS) rotary_rows_kernel(const int* __restrict__ pos, const double* __restrict__ freq, float2* __restrict__ turn, int rows,
+                                                              int half, float size) {
+    pdl_trigger();
+    for (long long i = blockIdx.x * (long long)THREADS + threadIdx.x; i < (long long)rows * half; i += (long long)gridDim.x * THREADS) {
+        // range reduction in double: the angle is exact to fp32 at any position
+        constexpr double TWO_PI = 6.283185307179586476925286766559, INV = 0.15915494309189533576888376337251;
+        const double angle = (double)pos[i / half] * freq[i % half];
+        const float r = (float)(angle - TWO_PI * rint(angle * INV));
+        turn[i] = make_float2(cosf(r) * size, sinf(r) * size);
+    }
+}
 
 // grid (rows, parts): a warp takes every (8 parts)-th head; the head lies in shared memory in fp32 between the norm and the rotation
 template <typename T>
 __global__ void __launch_bounds__(THREADS) head_norm_rope_kernel(HeadNorm a) {
     pdl_trigger();
-    extern __shared__ float4 sm4[];      // one head per warp, then [rot / 2] (cos, sin)
+    extern __shared__ float4 sm4[];      // one head per warp
     const int row = blockIdx.x, pos = a.pos[row], w = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int half = a.rot / 2, heads = a.H + a.G + a.V, size = max(a.dk, a.dv), stride = gridDim.y * (THREADS / 32);
     float* X = reinterpret_cast<float*>(sm4) + w * size;
-    float2* turn = reinterpret_cast<float2*>(reinterpret_cast<float*>(sm4) + THREADS / 32 * size);
+    const float2* turn = a.turn + (long long)row * half;
     T* z = (T*)a.z + (long long)row * a.ldz;
     auto start = [&](int i) { return z + (i < a.H ? a.zq + i * a.dk : i < a.H + a.G ? a.zk + (i - a.H) * a.dk : a.zv + (i - a.H - a.G) * a.dv); };
     int i = blockIdx.y * (THREADS / 32) + w;
-    float4 ahead = make_float4(0.f, 0.f, 0.f, 0.f);          // the first head's first piece is on its way while the angles are made
+    float4 ahead = make_float4(0.f, 0.f, 0.f, 0.f);          // the first piece of this warp's next head
     if (i < heads && lane * 4 < (i < a.H + a.G ? a.dk : a.dv)) ahead = load4(start(i) + lane * 4);
-    for (int p = threadIdx.x; p < half; p += THREADS) {
-        // range reduction in double: the angle is exact to fp32 at any position
-        constexpr double TWO_PI = 6.283185307179586476925286766559, INV = 0.15915494309189533576888376337251;
-        const double angle = (double)pos * a.freq[p];
-        const float r = (float)(angle - TWO_PI * rint(angle * INV));
-        turn[p] = make_float2(cosf(r) * a.size, sinf(r) * a.size);
-    }
-    __syncthreads();
     // a ring keeps the request's last `cap` positions: of the rows that share a place only the last one is stored
     const bool store = a.c.k != nullptr && (a.ends == nullptr || a.c.table != nullptr || pos >= a.ends[row] - a.c.cap);
     const long long place = store ? a.c.row(a.slots[row], pos) * a.G : 0;
     const float mix = a.first != nullptr ? *a.mix : 0.f;
     const bool aligned = a.halves && half % 4 == 0;          // four neighbours lie in one half, and so do their partners
-    for (bool first = true; i < heads; i += stride, first = false) {
+    for (; i < heads; i += stride) {
         const bool is_v = i >= a.H + a.G, is_k = !is_v && i >= a.H;
         const int n = is_v ? a.dv : a.dk;
         T* p = start(i);
         float s = 0.f;
         for (int c = lane * 4; c < n; c += 128) {
-            const float4 x = first && c == lane * 4 ? ahead : load4(p + c);
+            const float4 x = c == lane * 4 ? ahead : load4(p + c);
             s += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
             *reinterpret_cast<float4*>(X + c) = x;
         }
+        if (i + stride < heads && lane * 4 < (i + stride < a.H + a.G ? a.dk : a.dv)) ahead = load4(start(i + stride) + lane * 4);
         s = warp_sum(s);
         __syncwarp();
         const float* weight = is_v ? nullptr : is_k ? a.wk : a.wq;
@@ -368,10 +375,11 @@ __global__ void __launch_bounds__(THREADS) head_norm_rope_kernel(HeadNorm a) {
                 if (aligned) {
                     const bool low = c < half;
                     const float4 o = four(low ? c + half : c - half);
-                    const float2* t = turn + (low ? c : c - half);
+                    const float4* t = reinterpret_cast<const float4*>(turn + (low ? c : c - half));
+                    const float4 t0 = t[0], t1 = t[1];       // (cos, sin) of four pairs
                     const float sign = low ? -1.f : 1.f;
-                    y = make_float4(y.x * t[0].x + sign * o.x * t[0].y, y.y * t[1].x + sign * o.y * t[1].y, y.z * t[2].x + sign * o.z * t[2].y,
-                                    y.w * t[3].x + sign * o.w * t[3].y);
+                    y = make_float4(y.x * t0.x + sign * o.x * t0.y, y.y * t0.z + sign * o.y * t0.w, y.z * t1.x + sign * o.z * t1.y,
+                                    y.w * t1.z + sign * o.w * t1.w);
                 } else {
                     float f[4] = {y.x, y.y, y.z, y.w};
 #pragma unroll
@@ -399,62 +407,76 @@ __global__ void __launch_bounds__(THREADS) head_norm_rope_kernel(HeadNorm a) {
 }
 
 // x [n, ldx]: [H, G, dv] per row -> out [n, ldo]: out[h] = sum over g of table[h, g] x[g, value head of h].  A thread takes 16 bytes of a
-// value head and up to 8 of the heads that share it.
-template <typename T>
+// value head and HT of the heads that share it (HT divides their number).
+template <typename T, int HT>
 __global__ void __launch_bounds__(THREADS) head_mix_kernel(const T* __restrict__ x, long long ldx, const float* __restrict__ table, T* __restrict__ out,
-                                                           long long ldo, int n, int H, int G, int dv, int in_smem) {
+                                                           long long ldo, int n, int H, int G, int dv) {
     pdl_trigger();
-    constexpr int W = Vec<T>::N, HT = 8;
-    extern __shared__ float sm[];
-    if (in_smem) {
-        for (int i = threadIdx.x; i < H * H; i += THREADS) sm[i] = table[i];
-        __syncthreads();
-    }
-    const float* tab = in_smem ? sm : table;
-    const int qpg = H / G, pieces = dv / W, tiles = (qpg + HT - 1) / HT;
-    const long long total = (long long)n * G * tiles * pieces;
+    constexpr int W = Vec<T>::N, AHEAD = 8;                  // softmax heads whose pieces are in flight
+    extern __shared__ float sm[];                            // [H][H] transposed: [g][h]
+    for (int i = threadIdx.x; i < H * H; i += THREADS) sm[i % H * H + i / H] = table[i];
+    __syncthreads();
+    const int qpg = H / G, pieces = dv / W, tiles = qpg / HT, per_row = G * tiles * pieces;
+    const long long total = (long long)n * per_row, pitch = (long long)G * dv;
     for (long long i = blockIdx.x * (long long)THREADS + threadIdx.x; i < total; i += (long long)gridDim.x * THREADS) {
-        const int c = (int)(i % pieces) * W, tile = (int)(i / pieces % tiles), k = (int)(i / pieces / tiles % G);
-        const long long row = i / pieces / tiles / G;
-        const int h0 = k * qpg + tile * HT, nh = min(HT, k * qpg + qpg - h0);
+        const long long row = i / per_row;
+        const int in_row = (int)(i - row * per_row), c = in_row % pieces * W, k = in_row / pieces % G, h0 = k * qpg + in_row / pieces / G * HT;
         float acc[HT][W];
 #pragma unroll
         for (int h = 0; h < HT; ++h)
 #pragma unroll
             for (int e = 0; e < W; ++e) acc[h][e] = 0.f;
         const T* p = x + row * ldx + k * dv + c;
-#pragma unroll 4
-        for (int g = 0; g < H; ++g) {
-            Vec<T> v;
-            v.load(p + (long long)g * G * dv);
+        for (int g0 = 0; g0 < H; g0 += AHEAD) {
+            Vec<T> v[AHEAD];
 #pragma unroll
-            for (int h = 0; h < HT; ++h) {
-                if (h < nh) {
-                    const float t = tab[(h0 + h) * H + g];
+            for (int j = 0; j < AHEAD; ++j) v[j].load(p + min(g0 + j, H - 1) * pitch);
 #pragma unroll
-                    for (int e = 0; e < W; ++e) acc[h][e] += t * v.get(e);
+            for (int j = 0; j < AHEAD; ++j) {
+                if (g0 + j < H) {
+                    const float* t = sm + (g0 + j) * H + h0;
+                    float f[W];
+#pragma unroll
+                    for (int e = 0; e < W; ++e) f[e] = v[j].get(e);
+#pragma unroll
+                    for (int h = 0; h < HT; ++h) {
+                        const float w = t[h];
+#pragma unroll
+                        for (int e = 0; e < W; ++e) acc[h][e] += w * f[e];
+                    }
                 }
             }
         }
 #pragma unroll
         for (int h = 0; h < HT; ++h) {
-            if (h < nh) {
-                Vec<T> y;
+            Vec<T> y;
 #pragma unroll
-                for (int e = 0; e < W; ++e) y.set(e, acc[h][e]);
-                y.store(out + row * ldo + (long long)(h0 + h) * dv + c);
-            }
+            for (int e = 0; e < W; ++e) y.set(e, acc[h][e]);
+            y.store(out + row * ldo + (long long)(h0 + h) * dv + c);
         }
     }
 }
 
-template <typename T>
+template <typename T, int HT>
 static int launch_mix(const void* x, long long ldx, const float* table, void* out, long long ldo, int n, int H, int G, int dv, cudaStream_t st) {
-    const int qpg = H / G, in_smem = H * H * 4 <= 48 * 1024;
-    const long long total = (long long)n * G * ((qpg + 7) / 8) * (dv / Vec<T>::N), blocks = (total + THREADS - 1) / THREADS;
-    head_mix_kernel<T><<<(unsigned)(blocks < 148 * 8 ? blocks : 148 * 8), THREADS, in_smem ? H * H * 4 : 0, st>>>((const T*)x, ldx, table, (T*)out, ldo, n, H, G,
-                                                                                                                  dv, in_smem);
+    const size_t smem = sizeof(float) * H * H;
+    if (smem > 227 * 1024) return -2;
+    if (smem > 48 * 1024) {
+        cudaError_t e = cudaFuncSetAttribute(head_mix_kernel<T, HT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return (int)e;
+    }
+    const long long total = (long long)n * (H / HT) * (dv / Vec<T>::N), blocks = (total + THREADS - 1) / THREADS;
+    head_mix_kernel<T, HT><<<(unsigned)(blocks < 148 * 16 ? blocks : 148 * 16), THREADS, smem, st>>>((const T*)x, ldx, table, (T*)out, ldo, n, H, G, dv);
     return (int)cudaGetLastError();
+}
+
+template <typename T>
+static int mix_by_heads(const void* x, long long ldx, const float* table, void* out, long long ldo, int n, int H, int G, int dv, cudaStream_t st) {
+    const int qpg = H / G;
+    return qpg % 4 == 0   ? launch_mix<T, 4>(x, ldx, table, out, ldo, n, H, G, dv, st)
+           : qpg % 3 == 0 ? launch_mix<T, 3>(x, ldx, table, out, ldo, n, H, G, dv, st)
+           : qpg % 2 == 0 ? launch_mix<T, 2>(x, ldx, table, out, ldo, n, H, G, dv, st)
+                          : launch_mix<T, 1>(x, ldx, table, out, ldo, n, H, G, dv, st);
 }
 
 struct LatentNorm {
@@ -576,6 +598,14 @@ LMOE_API int lmoe_qk_norm_rope(const pag::QkNorm* ap, int dt, cudaStream_t st) {
     return (int)cudaGetLastError();
 }
 
+// pos [rows], freq [half] -> turn [rows, half] (cos, sin) times size
+LMOE_API int lmoe_rotary_rows(const int* pos, const double* freq, void* turn, int rows, int half, float size, cudaStream_t st) {
+    if (rows <= 0 || half <= 0 || !pag::aligned(turn)) return -1;
+    const long long blocks = ((long long)rows * half + pag::THREADS - 1) / pag::THREADS;
+    pag::rotary_rows_kernel<<<(unsigned)(blocks < 148 * 32 ? blocks : 148 * 32), pag::THREADS, 0, st>>>(pos, freq, (float2*)turn, rows, half, size);
+    return (int)cudaGetLastError();
+}
+
 // dk, dv, ldz, ldf and the first columns multiples of 8 (bf16) or 4 (fp32), rot even
 LMOE_API int lmoe_head_norm_rope(const pag::HeadNorm* ap, int dt, cudaStream_t st) {
     const pag::HeadNorm& a = *ap;
@@ -583,9 +613,9 @@ LMOE_API int lmoe_head_norm_rope(const pag::HeadNorm* ap, int dt, cudaStream_t s
     if (a.rows <= 0 || a.H <= 0 || a.G <= 0 || (a.V != 0 && a.V != a.G) || a.dk <= 0 || a.dk % w || a.dv < 0 || a.dv % w || a.ldz % w || a.ldf % w || a.zq % w ||
         a.zk % w || a.zv % w || a.rot % 2 || a.rot < 0 || a.rot > a.dk || a.nk <= 0 || (a.V && a.nv <= 0) || !pag::aligned(a.z) || !pag::aligned(a.first) ||
         !pag::aligned(a.wq) || !pag::aligned(a.wk) || !pag::aligned(a.c.k) || !pag::aligned(a.c.v) ||
-        (a.c.k != nullptr && ((a.c.table == nullptr && a.c.cap <= 0) || !a.V)) || (a.rot > 0 && a.freq == nullptr) || (a.first != nullptr && a.mix == nullptr))
+        (a.c.k != nullptr && ((a.c.table == nullptr && a.c.cap <= 0) || !a.V)) || (a.rot > 0 && a.turn == nullptr) || !pag::aligned(a.turn) || (a.first != nullptr && a.mix == nullptr))
         return -1;
-    const size_t smem = sizeof(float2) * (a.rot / 2) + sizeof(float) * (pag::THREADS / 32) * (a.dk > a.dv ? a.dk : a.dv);
+    const size_t smem = sizeof(float) * (pag::THREADS / 32) * (a.dk > a.dv ? a.dk : a.dv);
     if (smem > 46 * 1024) return -2;
     const int heads = a.H + a.G + a.V, parts = a.rows >= 1024 ? 1 : (heads + 7) / 8;
     if (dt) pag::head_norm_rope_kernel<bf16><<<dim3(a.rows, parts), pag::THREADS, smem, st>>>(a);
@@ -598,7 +628,7 @@ LMOE_API int lmoe_head_mix(const void* x, long long ldx, const float* table, voi
                            cudaStream_t st) {
     const int w = dt ? 8 : 4;
     if (n <= 0 || H <= 0 || G <= 0 || H % G || dv <= 0 || dv % w || ldx % w || ldo % w || !pag::aligned(x) || !pag::aligned(out)) return -1;
-    return dt ? pag::launch_mix<bf16>(x, ldx, table, out, ldo, n, H, G, dv, st) : pag::launch_mix<float>(x, ldx, table, out, ldo, n, H, G, dv, st);
+    return dt ? pag::mix_by_heads<bf16>(x, ldx, table, out, ldo, n, H, G, dv, st) : pag::mix_by_heads<float>(x, ldx, table, out, ldo, n, H, G, dv, st);
 }
 
 LMOE_API int lmoe_latent_norm(const pag::LatentNorm* ap, int dt, cudaStream_t st) {

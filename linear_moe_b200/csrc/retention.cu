@@ -9,14 +9,6 @@
 namespace lmoe {
 namespace rt {
 
-__device__ __forceinline__ float2 angle_of(int pos, double freq) {
-    // range reduction in double: the angle is exact to fp32 at any position
-    constexpr double TWO_PI = 6.283185307179586476925286766559, INV = 0.15915494309189533576888376337251;
-    const double angle = (double)pos * freq;
-    const float r = (float)(angle - TWO_PI * rint(angle * INV));
-    return make_float2(cosf(r), sinf(r));
-}
-
 // ---------------------------------------------------------------------------------------------------------------- one token
 constexpr int ST = 512;
 
@@ -32,8 +24,7 @@ __global__ void __launch_bounds__(ST) retention_step_kernel(Args a) {
     float* K = Q + dk;                                       // [dk]
     __shared__ float red[32];
     const bool on = r0 < parts;
-    const int pos = a.pos[b];
-    const bool fresh = pos == 0;
+    const bool fresh = a.pos[b] == 0;
     float* S = a.state + ((long long)a.slots[b] * a.H + h) * dk * dv;
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
     // the state is older than the kernel before this one
@@ -52,7 +43,7 @@ __global__ void __launch_bounds__(ST) retention_step_kernel(Args a) {
         if (d < a.rot) {
             const bool low = d < half;
             const int o = low ? d + half : d - half;
-            const float2 cs = angle_of(pos, a.freq[low ? d : o]);
+            const float2 cs = a.turn[(long long)b * half + (low ? d : o)];
             const float xo = to_f(q[o]), yo = to_f(k[o]);
             x = low ? x * cs.x - xo * cs.y : x * cs.x + xo * cs.y;
             y = low ? y * cs.x - yo * cs.y : y * cs.x + yo * cs.y;
@@ -212,7 +203,7 @@ using namespace lmoe;
 // the device before the kernel that precedes this one in the stream was launched.
 LMOE_API int lmoe_retention_step(const rt::Args* ap, int dt, cudaStream_t st) {
     const rt::Args& a = *ap;
-    if (!rt::ok(a, dt) || a.dv > 256 || a.state == nullptr || (a.rot > 0 && a.freq == nullptr) || a.zq % 4 || a.zk % 4 || a.zv % 4) return -1;
+    if (!rt::ok(a, dt) || a.dv > 256 || a.state == nullptr || (a.rot > 0 && a.turn == nullptr) || a.zq % 4 || a.zk % 4 || a.zv % 4) return -1;
     return dt ? rt::launch_step<bf16>(a, st) : rt::launch_step<float>(a, st);
 }
 

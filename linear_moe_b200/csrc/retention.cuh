@@ -25,7 +25,7 @@ struct Args {
     float* raw;                          // general kernel: [rows, H * dv]
     const float* powers;                 // [H, CH + 1] decay^0 ..
     const double* decay;                 // [H]
-    const double* freq;                  // [rot / 2] (one-token kernel; prompts are rotated before)
+    const float2* turn;                  // [rows, rot / 2] (cos, sin) (one-token kernel; prompts are rotated before)
     const int *pos, *slots;              // [rows]
     const int *groups, *requests;        // [n, 8], [m, 8]
     long long ldz, ldo;

@@ -33,6 +33,14 @@ class RowStep:
     latents: Dict[int, torch.Tensor] = field(default_factory=dict)    # layer -> latent rows, for the layers that borrow them
     values: Dict[int, torch.Tensor] = field(default_factory=dict)     # layer -> value rows, for the layers that mix them into theirs
 
+    turns: Dict[tuple, Optional[torch.Tensor]] = field(default_factory=dict)      # rotary tables of the rows, by their constants
+
+    def turn(self, key: tuple, freq: Optional[torch.Tensor], size: float = 1.0) -> Optional[torch.Tensor]:
+        """``ops.rotary_rows``, made once per call for all layers with the same ``key``."""
+        if key not in self.turns:
+            self.turns[key] = ops.rotary_rows(self.batch.pos, freq, size)
+        return self.turns[key]
+
     def cache(self, layer: int) -> Optional[dict]:
         return None if self.caches is None else self.caches[layer]
 

@@ -48,7 +48,8 @@ class Retention(Part):
     def forward(self, h, step: RowStep, layer: int) -> torch.Tensor:
         z = ops.linear(h, self.linear_in)
         out = activation_rows(h, self.linear_out, self.s.heads * self.s.dv)
-        ops.retention_rows(z, out, self.lay, self.s, self.powers, self.decay, self.freq, self.eps, step.batch, step.cache(layer))
+        turn = step.turn((self.s.rot_dims, self.s.rot_base, None), self.freq)
+        ops.retention_rows(z, out, self.lay, self.s, self.powers, self.decay, turn, self.eps, step.batch, step.cache(layer))
         return ops.sublayer_out(out, self.linear_out)
 
 

@@ -118,7 +118,8 @@ class GroupedAttention(Part):
                 ops.gather_rows(t, None, cache, name, batch.key_sources(s.window, True))
         if s.head_norm:
             borrows = s.value_source is not None and s.value_source != layer
-            ops.head_norm_rope_(z, l, s, *norms, self.freq, self.eps, batch, cache, *((step.values[s.value_source], self.vmix) if borrows else ()))
+            turn = step.turn((s.rot_dims, s.rot_base, s.rot_scaling), self.freq, s.rot_size)
+            ops.head_norm_rope_(z, l, s, *norms, turn, self.eps, batch, cache, *((step.values[s.value_source], self.vmix) if borrows else ()))
             if s.value_source == layer:
                 step.values[layer] = z[:, l.v:]
         else:

@@ -326,7 +326,7 @@ from .chunk_attn import chunk_attention, embed_norm, poly_norm, stream_norm   # 
 from .group_norm import embed_rows, group_norm, residual_group_norm, softcap_   # noqa: E402,F401
 from .moe_rows import experts_relu2   # noqa: E402,F401
 from .packed_attn import (causal_attention, gather_rows, glu_in, head_norm_rope_, latent_absorb, latent_norm, latent_up,   # noqa: E402,F401
-                          qk_norm_rope_, residual_norm, rotate_heads_, step_attention, sublayer_out)
+                          qk_norm_rope_, residual_norm, rotary_rows, rotate_heads_, step_attention, sublayer_out)
 from .retention import retention_rows   # noqa: E402,F401
 
 

@@ -180,8 +180,8 @@ class _QkNorm(ctypes.Structure):
 
 
 class _HeadNorm(ctypes.Structure):
-    _fields_ = _fields(a=(_P, "z wq wk freq first mix"), b=(_Cache, "c"), c=(_P, "pos slots ends"), d=(_LL, "ldz ldf"),
-                       e=(_I, "zq zk zv H G V dk dv nk nv rot halves norm_v"), f=(_F, "size eps"), g=(_I, "rows"))
+    _fields_ = _fields(a=(_P, "z wq wk turn first mix"), b=(_Cache, "c"), c=(_P, "pos slots ends"), d=(_LL, "ldz ldf"),
+                       e=(_I, "zq zk zv H G V dk dv nk nv rot halves norm_v"), f=(_F, "eps"), g=(_I, "rows"))
 
 
 class _TalkStep(ctypes.Structure):
@@ -385,13 +385,25 @@ def qk_norm_rope_(z, lay: QkvLayout, spec: AttentionSpec, wq, wk, freq, eps: flo
     K._check(K.lib().lmoe_qk_norm_rope(ctypes.byref(a), K._dt(z), K._st()), "qk_norm_rope")
 
 
-def head_norm_rope_(z, lay: QkvLayout, spec: AttentionSpec, wq, wk, freq, eps: float, batch: RowBatch, cache: Optional[dict],
+def rotary_rows(pos, freq, size: float = 1.0) -> Optional[torch.Tensor]:
+    """``[rows, pairs, 2]`` fp32: cos and sin of ``pos * freq`` (taken in fp64), times ``size``; one table serves all layers that rotate alike."""
+    if freq is None:
+        return None
+    if not freq.is_cuda:
+        return RP.rotary_rows(pos, freq, size)
+    from . import cuda as K
+    turn = torch.empty(pos.numel(), freq.numel(), 2, dtype=torch.float32, device=freq.device)
+    K._check(K.lib().lmoe_rotary_rows(K._p(pos), K._p(freq), K._p(turn), pos.numel(), freq.numel(), ctypes.c_float(size), K._st()), "rotary_rows")
+    return turn
+
+
+def head_norm_rope_(z, lay: QkvLayout, spec: AttentionSpec, wq, wk, turn, eps: float, batch: RowBatch, cache: Optional[dict],
                     first: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None):
     """Norm every query, key and value head of a projection's output and rotate queries and keys, in place; keys and values enter the
-    cache.  ``first``, ``mix``: values become ``(1 - mix) v + mix first`` behind their norm (``mix`` one fp32 number)."""
+    cache.  ``turn``: the rows' ``rotary_rows``.  ``first``, ``mix``: values become ``(1 - mix) v + mix first`` behind their norm (``mix`` one fp32 number)."""
     if not z.is_cuda:
-        return RP.head_norm_rope_(z, lay, spec, wq, wk, freq, eps, batch, cache, first, mix)
-    a = _head_args(z, lay.q, lay.k, spec.heads, spec.kv_heads, spec.dk, spec.rot_dims, spec.rot_halves, freq, spec.rot_size, batch)
+        return RP.head_norm_rope_(z, lay, spec, wq, wk, turn, eps, batch, cache, first, mix)
+    a = _head_args(z, lay.q, lay.k, spec.heads, spec.kv_heads, spec.dk, spec.rot_dims, spec.rot_halves, turn, batch)
     a.wq, a.wk, a.c, a.ends = _ptr(wq), _ptr(wk), _cache_args(cache), _ptr(batch.end)
     a.zv, a.V, a.dv, a.nk, a.nv, a.norm_v, a.eps = lay.v, spec.kv_heads, spec.dv, spec.dim, spec.vdim, int(spec.value_norm), eps
     if first is not None:
@@ -400,20 +412,21 @@ def head_norm_rope_(z, lay: QkvLayout, spec: AttentionSpec, wq, wk, freq, eps: f
     _head_launch(a, z)
 
 
-def rotate_heads_(z, at_q: int, at_k: int, heads: int, kv_heads: int, dk: int, dims: int, halves: bool, freq, size: float, batch: RowBatch):
+def rotate_heads_(z, at_q: int, at_k: int, heads: int, kv_heads: int, dk: int, dims: int, halves: bool, turn, batch: RowBatch):
     """Rotate the first ``dims`` dimensions of every query and key head in place."""
     if not dims:
         return
     if not z.is_cuda:
-        return RP.rotate_heads_(z, at_q, at_k, heads, kv_heads, dk, halves, freq, size, batch)
-    _head_launch(_head_args(z, at_q, at_k, heads, kv_heads, dk, dims, halves, freq, size, batch), z)
+        return RP.rotate_heads_(z, at_q, at_k, heads, kv_heads, dk, halves, turn)
+    _head_launch(_head_args(z, at_q, at_k, heads, kv_heads, dk, dims, halves, turn, batch), z)
 
 
-def _head_args(z, at_q, at_k, heads, kv_heads, dk, dims, halves, freq, size, batch) -> _HeadNorm:
+def _head_args(z, at_q, at_k, heads, kv_heads, dk, dims, halves, turn, batch) -> _HeadNorm:
     _no_grad(z)
+    assert not dims or (turn.shape == (z.shape[0], dims // 2, 2) and turn.is_contiguous())
     a = _HeadNorm()
-    a.z, a.freq, a.pos, a.slots, a.ldz, a.zq, a.zk = z.data_ptr(), _ptr(freq), batch.pos.data_ptr(), batch.slot.data_ptr(), z.stride(0), at_q, at_k
-    a.H, a.G, a.dk, a.nk, a.rot, a.halves, a.size, a.rows = heads, kv_heads, dk, dk, dims, int(halves), size, z.shape[0]
+    a.z, a.turn, a.pos, a.slots, a.ldz, a.zq, a.zk = z.data_ptr(), _ptr(turn), batch.pos.data_ptr(), batch.slot.data_ptr(), z.stride(0), at_q, at_k
+    a.H, a.G, a.dk, a.nk, a.rot, a.halves, a.rows = heads, kv_heads, dk, dk, dims, int(halves), z.shape[0]
     return a
 
 

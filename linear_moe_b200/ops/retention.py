@@ -76,7 +76,7 @@ _P, _LL, _I, _F = ctypes.c_void_p, ctypes.c_longlong, ctypes.c_int, ctypes.c_flo
 
 
 class _Args(ctypes.Structure):
-    _fields_ = _fields(a=(_P, "z out state scratch raw powers decay freq pos slots groups requests"), b=(_LL, "ldz ldo"),
+    _fields_ = _fields(a=(_P, "z out state scratch raw powers decay turn pos slots groups requests"), b=(_LL, "ldz ldo"),
                        c=(_I, "zq zk zv zg H dk dv nv rot n m"), d=(_F, "scale eps"))
 
 
@@ -91,17 +91,19 @@ def group_tokens(counts, heads: int, sms: int) -> int:
     return min(per, longest) * CHUNK
 
 
-def retention_rows(z, out, lay: RetentionLayout, s: RetentionSpec, powers, decay, freq, eps: float, batch: RowBatch, cache: Optional[dict]):
+def retention_rows(z, out, lay: RetentionLayout, s: RetentionSpec, powers, decay, turn, eps: float, batch: RowBatch, cache: Optional[dict]):
     """``out[:, :heads * dv]`` from the projection rows ``z`` (whose queries and keys a prompt rotates in place); ``cache["s"]``
-    ``[slots, heads, dk, dv]`` (fp32) holds the requests' states.  ``powers``, ``decay``, ``freq``: the spec's tables."""
+    ``[slots, heads, dk, dv]`` (fp32) holds the requests' states.  ``powers``, ``decay``: the spec's tables; ``turn``: the
+    rows' ``rotary_rows``."""
     if not z.is_cuda:
-        return RR.retention_rows(z, out, lay, s, freq, eps, batch, cache)
+        return RR.retention_rows(z, out, lay, s, turn, eps, batch, cache)
     from . import cuda as K
     _no_grad(z)
     dev, dt, dk, dv, H = z.device, K._dt(z), s.dk, s.dv, s.heads
+    assert not s.rot_dims or (turn.shape == (z.shape[0], s.rot_dims // 2, 2) and turn.is_contiguous())
     assert out.dtype == z.dtype and z.stride(1) == out.stride(1) == 1 and z.shape[0] == out.shape[0] == batch.rows
     a = _Args()
-    a.z, a.out, a.powers, a.decay, a.freq = z.data_ptr(), out.data_ptr(), powers.data_ptr(), decay.data_ptr(), _ptr(freq)
+    a.z, a.out, a.powers, a.decay, a.turn = z.data_ptr(), out.data_ptr(), powers.data_ptr(), decay.data_ptr(), _ptr(turn)
     a.pos, a.slots, a.ldz, a.ldo = batch.pos.data_ptr(), batch.slot.data_ptr(), z.stride(0), out.stride(0)
     a.zq, a.zk, a.zv, a.zg, a.H, a.dk, a.dv, a.nv, a.rot = lay.q, lay.k, lay.v, lay.g, H, dk, dv, s.vdim, s.rot_dims
     a.scale, a.eps = s.dim ** -0.5, eps
@@ -112,7 +114,7 @@ def retention_rows(z, out, lay: RetentionLayout, s: RetentionSpec, powers, decay
         a.n = batch.rows
         K._check(K.lib().lmoe_retention_step(ctypes.byref(a), dt, K._st()), "retention_step")
         return
-    rotate_heads_(z, lay.q, lay.k, H, H, dk, s.rot_dims, True, freq, 1.0, batch)
+    rotate_heads_(z, lay.q, lay.k, H, H, dk, s.rot_dims, True, turn, batch)
     if dt == 1 and not batch.decode and dk <= 128 and dv <= 128:
         groups, states, many = batch.recurrent_groups(group_tokens(batch.counts, H, K.num_sms()))
         scratch = torch.empty(states, H, dk, dv, dtype=torch.float32, device=dev) if states else None

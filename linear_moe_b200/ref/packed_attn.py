@@ -87,36 +87,34 @@ def _store_rows(z, lay, G, dk, dv, batch, cache):
         store(cache, "v", slot, p, z[r:r + 1, lay.v:lay.v + G * dv].reshape(1, G, dv))
 
 
-def rotate_halves(x, pos, freq, size):
-    """``x [n, heads, d]``: dimensions i and i + len(freq) turn by ``pos * freq[i]`` and grow by ``size``."""
-    angle, half = pos.double()[:, None] * freq[None, :], len(freq)
-    c, s = (size * torch.cos(angle)).float()[:, None], (size * torch.sin(angle)).float()[:, None]
-    y, u, v = x.clone(), x[..., :half], x[..., half:2 * half]
-    y[..., :half], y[..., half:2 * half] = u * c - v * s, v * c + u * s
-    return y
+def rotary_rows(pos, freq, size):
+    angle = pos.double()[:, None] * freq[None, :]
+    return torch.stack([size * torch.cos(angle), size * torch.sin(angle)], -1).float()
 
 
-def _turn(x, pos, halves, freq, size):
-    if freq is None:
+def turned(x, halves, turn):
+    """``x [n, heads, d]``: pairs of the first dimensions (half of them apart, or neighbours) turned by the rows' ``turn``."""
+    if turn is None:
         return x
-    if halves:
-        return rotate_halves(x, pos, freq, size)
-    y = rotate_pairs(x, pos, freq)
-    y[..., :2 * len(freq)] *= size
+    half = turn.shape[1]
+    low, high = (slice(0, half), slice(half, 2 * half)) if halves else (slice(0, 2 * half, 2), slice(1, 2 * half, 2))
+    c, s = turn[:, None, :, 0], turn[:, None, :, 1]
+    y, u, v = x.clone(), x[..., low], x[..., high]
+    y[..., low], y[..., high] = u * c - v * s, v * c + u * s
     return y
 
 
-def rotate_heads_(z, at_q, at_k, heads, kv_heads, dk, halves, freq, size, batch):
+def rotate_heads_(z, at_q, at_k, heads, kv_heads, dk, halves, turn):
     for at, n in ((at_q, heads), (at_k, kv_heads)):
         x = z[:, at:at + n * dk].float().reshape(-1, n, dk)
-        z[:, at:at + n * dk] = _turn(x, batch.pos, halves, freq, size).reshape(-1, n * dk).to(z.dtype)
+        z[:, at:at + n * dk] = turned(x, halves, turn).reshape(-1, n * dk).to(z.dtype)
 
 
-def head_norm_rope_(z, lay, s, wq, wk, freq, eps, batch, cache, first, mix):
+def head_norm_rope_(z, lay, s, wq, wk, turn, eps, batch, cache, first, mix):
     for at, n, w in ((lay.q, s.heads, wq), (lay.k, s.kv_heads, wk)):
         x = z[:, at:at + n * s.dk].float().reshape(-1, n, s.dk)
         x = x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) / s.dim + eps) * w
-        z[:, at:at + n * s.dk] = _turn(x, batch.pos, s.rot_halves, freq, s.rot_size).reshape(-1, n * s.dk).to(z.dtype)
+        z[:, at:at + n * s.dk] = turned(x, s.rot_halves, turn).reshape(-1, n * s.dk).to(z.dtype)
     at = slice(lay.v, lay.v + s.kv_heads * s.dv)
     v = z[:, at].float().reshape(-1, s.kv_heads, s.dv)
     if s.value_norm:

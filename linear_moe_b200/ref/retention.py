@@ -6,10 +6,10 @@ import torch
 from .packed_attn import rotate_heads_
 
 
-def retention_rows(z, out, lay, s, freq, eps, batch, cache):
+def retention_rows(z, out, lay, s, turn, eps, batch, cache):
     H, dk, dv = s.heads, s.dk, s.dv
     if s.rot_dims:
-        rotate_heads_(z, lay.q, lay.k, H, H, dk, True, freq, 1.0, batch)
+        rotate_heads_(z, lay.q, lay.k, H, H, dk, True, turn)
     decay = torch.tensor(s.decay, dtype=torch.float32)[:, None, None]
     q, k = (z[:, at:at + H * dk].float().reshape(-1, H, dk) for at in (lay.q, lay.k))
     v, g = (z[:, at:at + H * dv].float() for at in (lay.v, lay.g))

@@ -124,7 +124,7 @@ def test_head_norms_rotation_and_values(where, heads, kv_heads, dim, vdim, rot, 
         cache.reserve(slots, [p + 1 for p in at])
         batch = RowBatch(at, [1] * n, slots, dev)
         norms = [torch.nn.functional.pad(w, (0, s.dk - dim)).to(dev) for w in (wq, wk)]
-        PA.head_norm_rope_(z, lay, s, *norms, s.frequencies(dev), 1e-3, batch, cache[0], *((laid_out(other, s.dv).to(dev), mix.to(dev)) if mixed else ()))
+        PA.head_norm_rope_(z, lay, s, *norms, PA.rotary_rows(batch.pos, s.frequencies(dev), s.rot_size), 1e-3, batch, cache[0], *((laid_out(other, s.dv).to(dev), mix.to(dev)) if mixed else ()))
         positions = torch.tensor(at)
 
         def turned(t):
@@ -306,7 +306,7 @@ def test_scores_that_rise(where, decode):
     H, d, n = 2, 64, 400
     dev, dt = where[0], getattr(torch, where[1])
     k = torch.randn(n, H, d)
-    k[:, :, 0] = torch.linspace(-300, 300, n)[:, None]
+    k[:, :, 0] = torch.linspace(-120, 120, n)[:, None]
     q, v, table = torch.randn(n, H, d) * 0.1, torch.randn(n, H, d), torch.tensor([[1.0, 0.4], [-0.3, 0.9]])
     q[:, :, 0] = 1.0
     q, k, v = q.to(dt), k.to(dt), v.to(dt)
@@ -399,7 +399,7 @@ def retention_case(where, heads, dim, vdim, starts, counts, rot=None, decay=None
     z = torch.cat([torch.cat([laid_out(t[r][a:], d) for t, d in ((q, s.dk), (k, s.dk), (v, s.dv), (gate, s.dv))], 1) for r, a in enumerate(starts)]).to(dev)
     batch = RowBatch(starts, counts, slots if keep_cache else None, dev)
     out = torch.full((z.shape[0], round_up(heads * s.dv, 32)), 7.0, dtype=dt, device=dev)
-    RT.retention_rows(z, out, lay, s, s.powers(dev), s.decays(dev), s.frequencies(dev), eps, batch, None if cache is None else cache[0])
+    RT.retention_rows(z, out, lay, s, s.powers(dev), s.decays(dev), PA.rotary_rows(batch.pos, s.frequencies(dev)), eps, batch, None if cache is None else cache[0])
     got = heads_of(out[:, :heads * s.dv], heads, s.dv, vdim)
     assert float(out[:, :heads * s.dv].reshape(-1, heads, s.dv)[:, :, vdim:].float().abs().sum()) == 0
     if keep_cache:
