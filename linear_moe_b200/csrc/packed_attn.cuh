@@ -31,6 +31,7 @@ struct Prompt {
     int n, q_rows, k_rows;
     float scale;
     int cross;                        // every query head's weights are applied to the values of every kv head: out [rows, H, G, dv]
+    int bounded;                      // cross, tensor-core kernel: |q . k * scale| <= 60 everywhere, so that exp needs no running maximum
 };
 
 struct Cache {

@@ -11,7 +11,9 @@
 // O accumulates in tensor memory over all key tiles.  The maximum a row is scaled by may lag behind the true one by LAG (in
 // units of log2), so that P stays below 2^LAG; only when a row runs ahead of that is O multiplied in tensor memory.
 // With `cross`, a query head's weights are applied to the values of every kv head (talking heads, which mix these results afterwards): a
-// CTA takes as many kv heads as fit 256 columns of tensor memory, and the values come in stages of 64 keys.
+// CTA takes as many kv heads as fit 256 columns of tensor memory, and the values come in stages of 64 keys.  Where the scores are known to
+// be `bounded` (normed queries and keys), P = exp2(S) as it is: no maximum, no exchange between threads, and two P tiles, so that the
+// exponentials of a tile run beside the value product of the one before.
 // Every mbarrier wait is bounded; on expiry the error word is set and the CTA drains and frees its tensor memory.
 #include "attn_math.cuh"
 #include "flash_tc_utils.cuh"
@@ -24,16 +26,16 @@ using pa::Prompt;
 
 constexpr float LAG = 8.f;
 
-// DQ: key dims, DT: value columns of a CTA
-template <int DQ, int DT>
+// DQ: key dims, DT: value columns of a CTA, PB: P tiles (2: bounded scores)
+template <int DQ, int DT, int PB>
 struct __align__(1024) Smem {
     static constexpr int VK = DT > 128 ? 64 : BN;           // keys per stage of values
     uint8_t q[BM * DQ * 2];
     uint8_t k[2][BN * DQ * 2];
     uint8_t v[2][VK * DT * 2];
-    uint8_t p[BM * BN * 2];
-    float mx[2][SPLIT][BM], ls[SPLIT][BM];
-    uint64_t q_full, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[2], pv_done, p_ready;
+    uint8_t p[PB][BM * BN * 2];
+    float mx[PB == 1 ? 2 : 1][PB == 1 ? SPLIT : 1][PB == 1 ? BM : 1];
+    uint64_t q_full, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[2], pv_done[PB], p_ready[PB];
     uint32_t tmem_base;
     int abort_flag;
 };
@@ -45,14 +47,15 @@ __device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t (&r)[16
 }
 __device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 
-// DV: value dims of a head, NB: value heads of a CTA
-template <int DQ, int DV, int NB>
+// DV: value dims of a head, NB: value heads of a CTA, BOUNDED: see above
+template <int DQ, int DV, int NB, bool BOUNDED>
 __global__ void __launch_bounds__(THREADS, 1)
 packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                       const __grid_constant__ CUtensorMap tmV, Prompt a) {
     extern __shared__ uint8_t smem_raw[];
-    constexpr int DT = NB * DV, VK = Smem<DQ, DT>::VK, VS = BN / VK;         // VS: stages of values per tile of keys
-    Smem<DQ, DT>& sm = *reinterpret_cast<Smem<DQ, DT>*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+    constexpr int DT = NB * DV, PB = BOUNDED ? 2 : 1;
+    constexpr int VK = Smem<DQ, DT, PB>::VK, VS = BN / VK;  // VS: stages of values per tile of keys
+    Smem<DQ, DT, PB>& sm = *reinterpret_cast<Smem<DQ, DT, PB>*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
     constexpr int KQ = DQ / 64, KV = DT / 64;               // 64-element blocks along the head dimensions
     constexpr uint32_t TMEM_COLS = 512, O_COL = 2 * BN;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -61,6 +64,8 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
     const int h = blockIdx.y, hk = h / (a.H / a.G), hv = a.cross ? blockIdx.z * NB : hk;       // hv: first value head
     const int nb_lo = a.window > 0 ? max(0, c0 - a.window + 1) / BN : 0;
     const int n_it = (c0 + nq + BN - 1) / BN - nb_lo;       // at least 1: a query sees its own key
+    auto buf = [](int j) { return j & (PB - 1); };          // P tile and barriers of key tile j, and their phase
+    auto phase = [](int j) { return (uint32_t)(PB == 2 ? (j >> 1) & 1 : j & 1); };
     volatile int* abort_flag = &sm.abort_flag;
     int* err = a.err;
 
@@ -71,8 +76,10 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
             mbar_init(&sm.v_full[s], 1); mbar_init(&sm.v_empty[s], 1);
             mbar_init(&sm.s_full[s], 1);
         }
-        mbar_init(&sm.pv_done, 1);
-        mbar_init(&sm.p_ready, 4 * SPLIT);
+        for (int b = 0; b < PB; ++b) {
+            mbar_init(&sm.pv_done[b], 1);
+            mbar_init(&sm.p_ready[b], 4 * SPLIT);
+        }
         sm.abort_flag = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
@@ -142,10 +149,10 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
             for (int u = 0; u < VS; ++u) {
                 const int vi = j * VS + u, t = vi & 1;
                 ok = mbar_wait_suspend(&sm.v_full[t], (vi >> 1) & 1, abort_flag, err, 0x8200 | t);
-                if (ok && u == 0) ok = mbar_wait_suspend(&sm.p_ready, j & 1, abort_flag, err, 0x8300);
+                if (ok && u == 0) ok = mbar_wait_suspend(&sm.p_ready[buf(j)], phase(j), abort_flag, err, 0x8300);
                 if (!ok) break;
                 tc_fence_after();
-                const uint32_t pl = desc_lo<false>(s32(sm.p)), vl = desc_lo<true>(s32(sm.v[t]));
+                const uint32_t pl = desc_lo<false>(s32(sm.p[buf(j)])), vl = desc_lo<true>(s32(sm.v[t]));
 #pragma unroll
                 for (int kk = 0; kk < VK / UMMA_K; ++kk) {
                     const int kp = u * (VK / UMMA_K) + kk;  // 16-key step of the tile
@@ -156,7 +163,7 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
                 umma_commit_if(&sm.v_empty[t], issue);
             }
             if (!ok) break;
-            umma_commit_if(&sm.pv_done, issue);
+            umma_commit_if(&sm.pv_done[buf(j)], issue);
         }
     } else if (warp >= 4) {
         const int qd = warp & 3, part = (warp - 4) >> 2;
@@ -165,7 +172,7 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
         constexpr int CW = BN / SPLIT, OW = DT / SPLIT;       // score / output columns of this thread
         static_assert(CW == 32 && OW % 16 == 0, "tensor-memory load widths");
         const float sc = a.scale * LOG2E, lag = LAG / sc;
-        uint8_t* prow = sm.p + ((part * CW) >> 6) * (BM * 128) + (r >> 3) * 1024 + (r & 7) * 128;
+        uint8_t* prow = sm.p[0] + ((part * CW) >> 6) * (BM * 128) + (r >> 3) * 1024 + (r & 7) * 128;
         const int ch0 = ((part * CW) & 63) >> 3;
         float m = -INFINITY, l = 0.f;
         bool alive = true;
@@ -183,39 +190,41 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
                 for (int c = 0; c < CW; ++c)
                     if (c > hi || c <= lo) v[c] = 0xff800000u;                  // -inf
             }
-            float mx4[4];
+            if constexpr (!BOUNDED) {
+                float mx4[4];
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                mx4[e] = fmaxf(__uint_as_float(v[e]), __uint_as_float(v[e + 4]));
+                for (int e = 0; e < 4; ++e) {
+                    mx4[e] = fmaxf(__uint_as_float(v[e]), __uint_as_float(v[e + 4]));
 #pragma unroll
-                for (int c = 8; c < CW; c += 8) mx4[e] = max3(mx4[e], __uint_as_float(v[c + e]), __uint_as_float(v[c + e + 4]));
-            }
-            sm.mx[s][part][r] = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-            asm volatile("bar.sync %0, %1;" :: "r"(1 + qd), "n"(32 * SPLIT) : "memory");
-            float mx = sm.mx[s][0][r];
-#pragma unroll
-            for (int p = 1; p < SPLIT; ++p) mx = fmaxf(mx, sm.mx[s][p][r]);
-            // the four parts of a row see the same numbers and decide alike
-            const bool grow = mx > m + lag;                   // also the first visible key of the row (m = -inf)
-            const bool scaled = grow && m != -INFINITY;
-            const float corr = scaled ? ex2((m - mx) * sc) : 1.f;
-            if (grow) m = mx;
-            l *= corr;
-            if (__any_sync(0xffffffffu, scaled)) {            // not before tile 1: O holds something
-                if (!mbar_wait_suspend(&sm.pv_done, (j - 1) & 1, abort_flag, err, 0x9200)) { alive = false; break; }
-                tc_fence_after();
-#pragma unroll
-                for (int c = 0; c < OW; c += 16) {
-                    uint32_t o[16];
-                    tmem_ld16(lane_addr + O_COL + part * OW + c, o);
-                    tmem_ld_wait();
-#pragma unroll
-                    for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * corr);
-                    tmem_st16(lane_addr + O_COL + part * OW + c, o);
+                    for (int c = 8; c < CW; c += 8) mx4[e] = max3(mx4[e], __uint_as_float(v[c + e]), __uint_as_float(v[c + e + 4]));
                 }
-                tmem_st_wait();
+                sm.mx[s][part][r] = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
+                asm volatile("bar.sync %0, %1;" :: "r"(1 + qd), "n"(32 * SPLIT) : "memory");
+                float mx = sm.mx[s][0][r];
+#pragma unroll
+                for (int p = 1; p < SPLIT; ++p) mx = fmaxf(mx, sm.mx[s][p][r]);
+                // the four parts of a row see the same numbers and decide alike
+                const bool grow = mx > m + lag;                   // also the first visible key of the row (m = -inf)
+                const bool scaled = grow && m != -INFINITY;
+                const float corr = scaled ? ex2((m - mx) * sc) : 1.f;
+                if (grow) m = mx;
+                l *= corr;
+                if (__any_sync(0xffffffffu, scaled)) {            // not before tile 1: O holds something
+                    if (!mbar_wait_suspend(&sm.pv_done[0], (j - 1) & 1, abort_flag, err, 0x9200)) { alive = false; break; }
+                    tc_fence_after();
+#pragma unroll
+                    for (int c = 0; c < OW; c += 16) {
+                        uint32_t o[16];
+                        tmem_ld16(lane_addr + O_COL + part * OW + c, o);
+                        tmem_ld_wait();
+#pragma unroll
+                        for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * corr);
+                        tmem_st16(lane_addr + O_COL + part * OW + c, o);
+                    }
+                    tmem_st_wait();
+                }
             }
-            const float nm = m == -INFINITY ? 0.f : -m * sc;
+            const float nm = BOUNDED || m == -INFINITY ? 0.f : -m * sc;
             const float2 sc2 = make_float2(sc, sc), nm2 = make_float2(nm, nm);
             float2 sum0 = make_float2(0.f, 0.f), sum1 = make_float2(0.f, 0.f);
 #pragma unroll
@@ -229,23 +238,24 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
                 v[(c >> 1) + 1] = pack_bf16(p2, p3);
             }
             l += (sum0.x + sum0.y) + (sum1.x + sum1.y);
-            // the P tile is free once O += P_{j-1} V_{j-1} has completed
-            if (j > 0 && !mbar_wait_suspend(&sm.pv_done, (j - 1) & 1, abort_flag, err, 0x9300)) { alive = false; break; }
+            // a P tile is free once the product with the values that it was last used for has completed
+            if (j >= PB && !mbar_wait_suspend(&sm.pv_done[buf(j)], phase(j - PB), abort_flag, err, 0x9300)) { alive = false; break; }
 #pragma unroll
             for (int c = 0; c < 4; ++c)
-                *reinterpret_cast<uint4*>(prow + (((ch0 + c) ^ (r & 7)) << 4)) = make_uint4(v[4 * c], v[4 * c + 1], v[4 * c + 2], v[4 * c + 3]);
+                *reinterpret_cast<uint4*>(prow + buf(j) * (BM * BN * 2) + (((ch0 + c) ^ (r & 7)) << 4)) = make_uint4(v[4 * c], v[4 * c + 1], v[4 * c + 2], v[4 * c + 3]);
             tc_fence_before();
             asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
             __syncwarp();
-            if (lane == 0) mbar_arrive(&sm.p_ready);
+            if (lane == 0) mbar_arrive(&sm.p_ready[buf(j)]);
         }
-        if (alive) alive = mbar_wait_suspend(&sm.pv_done, (n_it - 1) & 1, abort_flag, err, 0x9400);
+        if (alive) alive = mbar_wait_suspend(&sm.pv_done[buf(n_it - 1)], phase(n_it - 1), abort_flag, err, 0x9400);
         tc_fence_after();
-        sm.ls[part][r] = l;
+        float* ls = reinterpret_cast<float*>(sm.q);           // [SPLIT][BM]; every product has completed, the queries are not read any more
+        ls[part * BM + r] = l;
         asm volatile("bar.sync %0, %1;" :: "r"(1 + qd), "n"(32 * SPLIT) : "memory");
         l = 0.f;
 #pragma unroll
-        for (int p = 0; p < SPLIT; ++p) l += sm.ls[p][r];
+        for (int p = 0; p < SPLIT; ++p) l += ls[p * BM + r];
         uint32_t o[OW];
         tmem_ld<OW>(lane_addr + O_COL + part * OW, o);
         tmem_ld_wait();
@@ -278,21 +288,24 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
     }
 }
 
-template <int DQ, int DV, int NB>
+template <int DQ, int DV, int NB, bool BOUNDED>
 static int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const Prompt& a, cudaStream_t st) {
-    const size_t smem = sizeof(Smem<DQ, NB * DV>) + 1024;
-    static_assert(sizeof(Smem<DQ, NB * DV>) + 1024 <= 227 * 1024 && NB * DV <= 256, "shared and tensor memory of one CTA");
-    cudaError_t e = cudaFuncSetAttribute(packed_attn_tc_kernel<DQ, DV, NB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    const size_t smem = sizeof(Smem<DQ, NB * DV, BOUNDED ? 2 : 1>) + 1024;
+    static_assert(sizeof(Smem<DQ, NB * DV, BOUNDED ? 2 : 1>) + 1024 <= 227 * 1024 && NB * DV <= 256, "shared and tensor memory of one CTA");
+    cudaError_t e = cudaFuncSetAttribute(packed_attn_tc_kernel<DQ, DV, NB, BOUNDED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
-    packed_attn_tc_kernel<DQ, DV, NB><<<dim3(a.n, a.H, a.cross ? (a.G + NB - 1) / NB : 1), THREADS, smem, st>>>(mq, mk, mv, a);
+    packed_attn_tc_kernel<DQ, DV, NB, BOUNDED><<<dim3(a.n, a.H, a.cross ? (a.G + NB - 1) / NB : 1), THREADS, smem, st>>>(mq, mk, mv, a);
     return (int)cudaGetLastError();
 }
 
-template <int DQ>
+template <int DQ, bool BOUNDED>
 static int by_values(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const Prompt& a, cudaStream_t st) {
     const int heads = a.cross ? a.G : 1;
-    if (a.dv <= 64) return heads > 2 ? launch<DQ, 64, 4>(mq, mk, mv, a, st) : heads > 1 ? launch<DQ, 64, 2>(mq, mk, mv, a, st) : launch<DQ, 64, 1>(mq, mk, mv, a, st);
-    return heads > 1 ? launch<DQ, 128, 2>(mq, mk, mv, a, st) : launch<DQ, 128, 1>(mq, mk, mv, a, st);
+    if (a.dv <= 64)
+        return heads > 2   ? launch<DQ, 64, 4, BOUNDED>(mq, mk, mv, a, st)
+               : heads > 1 ? launch<DQ, 64, 2, BOUNDED>(mq, mk, mv, a, st)
+                           : launch<DQ, 64, 1, BOUNDED>(mq, mk, mv, a, st);
+    return heads > 1 ? launch<DQ, 128, 2, BOUNDED>(mq, mk, mv, a, st) : launch<DQ, 128, 1, BOUNDED>(mq, mk, mv, a, st);
 }
 
 }  // namespace patc
@@ -315,5 +328,6 @@ LMOE_API int lmoe_packed_attn_tc(const pa::Prompt* ap, cudaStream_t st) {
     if (rc == 0) rc = make_map_4d(&mk, a.k, 1, a.k_rows, a.G, a.dk, (long long)a.k_rows * a.ldk, a.ldk, a.dk, BN);
     if (rc == 0) rc = make_map_4d(&mv, a.v, 1, a.k_rows, a.G, a.dv, (long long)a.k_rows * a.ldv, a.ldv, a.dv, 64);
     if (rc) return rc;
-    return a.dk <= 64 ? by_values<64>(mq, mk, mv, a, st) : by_values<128>(mq, mk, mv, a, st);
+    if (a.cross && a.bounded) return a.dk <= 64 ? by_values<64, true>(mq, mk, mv, a, st) : by_values<128, true>(mq, mk, mv, a, st);
+    return a.dk <= 64 ? by_values<64, false>(mq, mk, mv, a, st) : by_values<128, false>(mq, mk, mv, a, st);
 }

@@ -60,7 +60,7 @@ class Part(nn.Module):
 class GroupedAttention(Part):
     def __init__(self, cfg, s: AttentionSpec, device):
         super().__init__()
-        self.s, self.lay, self.width, self.eps = s, QkvLayout.of(s), cfg.hidden_size, cfg.norm_eps
+        self.s, self.lay, self.width, self.eps, self._bound = s, QkvLayout.of(s), cfg.hidden_size, cfg.norm_eps, None
         pad = round_up(cfg.hidden_size, ROW_PAD)
         self.linear_in = blank((self.lay.width, pad), cfg, device)
         self.linear_out = blank((pad, round_up(s.heads * s.dv, ROW_PAD)), cfg, device)
@@ -98,6 +98,14 @@ class GroupedAttention(Part):
             with torch.no_grad():
                 self.talk.add_(torch.eye(self.s.heads, device=self.talk.device))
 
+    def score_bound(self) -> float:
+        """No |score| is larger: queries and keys are unit vectors times sqrt(dim), their norms' weights and the rotation's size, rounded to
+        16 bits.  Made anew when a weight has changed or moved."""
+        s, now = self.s, tuple((w.data_ptr(), w._version) for w in (self.q_norm, self.k_norm))
+        if self._bound is None or self._bound[0] != now:
+            self._bound = now, float(self.q_norm.abs().max() * self.k_norm.abs().max()) * s.dim * s.rot_size ** 2 * s.scale * 1.02
+        return self._bound[1]
+
     def cache_spec(self, limit: int):
         s = self.s
         if s.window is None or min(s.window, limit) > RING_MAX:
@@ -133,7 +141,7 @@ class GroupedAttention(Part):
                     ops.gather_rows(t, src, cache, name, batch.key_sources(s.window, False))
             else:
                 k, v = zk, zv
-            ops.causal_attention(z[:, :l.k], k, v, o, *sizes, batch, None, talk)
+            ops.causal_attention(z[:, :l.k], k, v, o, *sizes, batch, None, talk, self.score_bound() if s.head_norm else None)
         return ops.sublayer_out(out, self.linear_out)
 
 

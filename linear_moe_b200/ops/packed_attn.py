@@ -18,6 +18,7 @@ from typing import Optional
 import torch
 
 from ..ref import packed_attn as RP
+from .chunk_attn import SCORE_BOUND
 from .row_batch import RowBatch, round_up
 
 ROWS_SMEM = 227 * 1024 // 4   # floats of shared memory a prompt kernel for any head size may use
@@ -162,7 +163,7 @@ def _fields(**groups):
 
 class _Prompt(ctypes.Structure):
     _fields_ = _fields(a=(_P, "q k v gate out items err"), b=(_LL, "ldq ldk ldv ldg ldo"), c=(_I, "H G dk dv window n q_rows k_rows"), d=(_F, "scale"),
-                       e=(_I, "cross"))
+                       e=(_I, "cross bounded"))
 
 
 class _Cache(ctypes.Structure):
@@ -218,10 +219,10 @@ def _ptr(t: Optional[torch.Tensor]) -> int:
 
 # --------------------------------------------------------------------------------------------------------------- attention
 def causal_attention(q, k, v, out, heads: int, kv_heads: int, dk: int, dv: int, scale: float, window: Optional[int], batch: RowBatch,
-                     gate: Optional[torch.Tensor] = None, talk: Optional[torch.Tensor] = None):
+                     gate: Optional[torch.Tensor] = None, talk: Optional[torch.Tensor] = None, score_bound: Optional[float] = None):
     """Prompts: ``out [rows, heads * dv] = softmax(q . k * scale) v`` (times ``sigmoid(gate)``), ``q [rows, heads * dk]``; ``k``, ``v``
     ``[key rows, kv_heads * d]`` in the order of ``batch.key_sources`` (the rows themselves when no request goes on from a cache).
-    ``talk [heads, heads]`` (fp32): head h mixes its values with ``sum_g talk[h, g] softmax_g``."""
+    ``talk [heads, heads]`` (fp32): head h mixes its values with ``sum_g talk[h, g] softmax_g``; ``score_bound``: no |score| is larger."""
     if not q.is_cuda:
         return RP.causal_attention(q, k, v, out, heads, kv_heads, dk, dv, scale, window, batch, gate, talk)
     from . import cuda as K
@@ -237,6 +238,7 @@ def causal_attention(q, k, v, out, heads: int, kv_heads: int, dk: int, dv: int, 
     dt = K._dt(q)
     fast = dt == 1 and dk <= 128 and dv <= 128
     if talk is not None:
+        a.bounded = int(score_bound is not None and score_bound <= SCORE_BOUND)
         return _talk_prompt(a, q, out, talk, window, batch, fast)
     tile = 128 if fast else 32 if 64 * (dk + 1) + 64 * dv + 32 * 33 <= ROWS_SMEM else 16
     items = batch.causal_items(window, tile)

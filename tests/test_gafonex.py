@@ -189,7 +189,7 @@ def test_gated_relu_feed_forward(where, rows):
     assert rel(got, O.relu_mlp(h.double(), {"gate": w1[:96].double(), "up": w1[96:].double(), "down": w2.double()})) < tol(where)
 
 
-def talk_case(where, H, G, dk, dv, window, starts, counts, sharp=(), seed=0, scale=None, table=None):
+def talk_case(where, H, G, dk, dv, window, starts, counts, sharp=(), seed=0, scale=None, table=None, bound=None):
     """Random queries, keys, values and mixing table through the prompt or step kernels, cached keys included; the result and the
     definition's, row by row.  ``sharp``: (request, query position, key position, head) whose score is made to stand out."""
     dev, dt = where[0], getattr(torch, where[1])
@@ -231,7 +231,7 @@ def talk_case(where, H, G, dk, dv, window, starts, counts, sharp=(), seed=0, sca
             ops.gather_rows(m, None, cache[0], name, batch.key_sources(window, True))
             ops.gather_rows(m, torch.cat([t[s] for t, s in zip(src, new)]).reshape(-1, G * d).to(dev), cache[0], name, batch.key_sources(window, False))
             mats.append(m)
-        PA.causal_attention(q, *mats, out, H, G, dk, dv, scale, window, batch, None, table.to(dev))
+        PA.causal_attention(q, *mats, out, H, G, dk, dv, scale, window, batch, None, table.to(dev), bound)
     want = []
     for a, b, c, s in zip(qs, ks, vs, new):
         i = torch.arange(len(a))
@@ -247,11 +247,14 @@ shapes = pytest.mark.parametrize("shape", SHAPES, ids=lambda s: f"h{s[0]}g{s[1]}
 
 @where
 @shapes
-def test_talking_heads_in_prompts(where, shape):
-    """Requests that end inside, on and past tiles, from their first token and from the middle."""
-    got, want = talk_case(where, *shape, [0] * 5, [131, 64, 1, 63, 129])
+@pytest.mark.parametrize("bound", [None, 60.0])
+def test_talking_heads_in_prompts(where, shape, bound):
+    """Requests that end inside, on and past tiles, from their first token and from the middle; scores known to be bounded, or not."""
+    got, want = talk_case(where, *shape, [0] * 5, [131, 64, 1, 63, 129], bound=bound)
     assert rel(got, want) < tol(where)
-    got, want = talk_case(where, *shape, [64, 5, 0, 63, 200, 64], [2, 128, 7, 1, 131, 64], seed=1)
+    got, want = talk_case(where, *shape, [64, 5, 0, 63, 200, 64], [2, 128, 7, 1, 131, 64], seed=1, bound=bound)
+    assert rel(got, want) < tol(where)
+    got, want = talk_case(where, *shape, [0, 300], [700, 400], seed=2, bound=bound)             # many tiles of keys
     assert rel(got, want) < tol(where)
 
 
@@ -295,8 +298,9 @@ def test_one_key_of_one_head_stands_out(where, decode):
         table[h, (h + 1) % H], table[h, 2] = 1.0, -0.5 * (h % 3)             # nobody uses its own weights
     for i, j in ((300, 0), (300, 1), (300, 63), (300, 64), (300, 127), (300, 128), (300, 299), (300, 300), (129, 128), (128, 0), (640, 5), (64, 63)):
         for h in (0, 2, 5):
-            got, want = talk_case(where, H, G, d, 48, None, [i] if decode else [0], [1 if decode else i + 1], [(0, i, j, h)], i + j, 0.3, table)
-            assert rel(got[-1], want[-1]) < tol(where), (i, j, h)
+            for bound in (None,) if decode else (None, 50.0):
+                got, want = talk_case(where, H, G, d, 48, None, [i] if decode else [0], [1 if decode else i + 1], [(0, i, j, h)], i + j, 0.3, table, bound)
+                assert rel(got[-1], want[-1]) < tol(where), (i, j, h)
 
 
 @where
@@ -335,6 +339,40 @@ def test_long_prompts_go_in_parts(where, monkeypatch):
     monkeypatch.setattr(PA, "TALK_BYTES", 200 * 4 * 2 * 32 * 4)
     got, want = talk_case(where, 4, 2, 32, 32, None, [0, 70, 0], [300, 130, 5])
     assert rel(got, want) < tol(where)
+
+
+@where
+@pytest.mark.parametrize("size", [58.0, 64.0])
+def test_scores_at_the_bound(where, size):
+    """Scores as large as the bound lets them be, of both signs, in the form that the bound selects; and just beyond it."""
+    H, d, n = 2, 32, 300
+    dev, dt = where[0], getattr(torch, where[1])
+    q, k, v = (torch.randn(n, H, d, generator=torch.Generator().manual_seed(s)) for s in (1, 2, 3))
+    q, k = ((t / t.norm(dim=-1, keepdim=True)) for t in (q, k))
+    k[::3], k[1::3] = q[0], -q[0]
+    q[5:] = q[0]
+    q, k, v, table = q.to(dt), k.to(dt), v.to(dt), torch.tensor([[1.0, 0.4], [-0.3, 0.9]])
+    seen = torch.ones(n, n, dtype=torch.bool).tril()
+    want = O.apply_weights(O.talk(O.softmax_weights(q.double(), k.double(), size, seen), table.double()), v.double())
+    out = torch.zeros(n, H * d, dtype=dt, device=dev)
+    PA.causal_attention(*(t.reshape(n, -1).to(dev) for t in (q, k, v)), out, H, H, d, d, size, None, RowBatch([0], [n], None, dev), None, table.to(dev), size * 1.02)
+    assert rel(out, want) < tol(where)
+
+
+def test_bound_of_the_scores(build):
+    """Normed and rotated queries and keys of a layer stay inside the bound that its weights give."""
+    model, w, cfg = build("mixed", ("cpu", "float32"))
+    mix, m, p = model.decoder.layers[1].mix, cfg["layers"][1]["mixer"], {k[7:]: t.double() for k, t in w.items() if k.startswith("l1.mix.")}
+    h = torch.randn(60, cfg["width"], dtype=torch.float64) * 3
+    q, k = (O.rotate(O.head_norm((h @ p[n].T).reshape(60, -1, m["dim"]), 1e-5, p[n + ".norm"]), torch.arange(60), m["rot"]["dims"], m["rot"]["base"], m["rot"]["scaling"])
+            for n in ("q", "k"))
+    largest = float(torch.einsum("ihd,jgd->ijhg", q, k).abs().max()) * m["scale"]
+    assert 0.2 * mix.score_bound() < largest <= mix.score_bound()
+    with torch.no_grad():
+        was = mix.score_bound()
+        mix.q_norm.mul_(2)
+        assert abs(mix.score_bound() / was - 2) < 1e-5
+        mix.q_norm.mul_(0.5)
 
 
 def test_parts_of_work_lists():
