@@ -12,8 +12,9 @@
 // units of log2), so that P stays below 2^LAG; only when a row runs ahead of that is O multiplied in tensor memory.
 // With `cross`, a query head's weights are applied to the values of every kv head (talking heads, which mix these results afterwards): a
 // CTA takes as many kv heads as fit 256 columns of tensor memory, and the values come in stages of 64 keys.  Where the scores are known to
-// be `bounded` (normed queries and keys), P = exp2(S) as it is: no maximum, no exchange between threads, and two P tiles, so that the
-// exponentials of a tile run beside the value product of the one before.
+// be `bounded` (normed queries and keys), P = exp2(S) as it is: no maximum, no exchange between threads, and P goes back to tensor memory
+// into the columns its scores came from, from where the value product reads it; the shared memory of the P tile holds more stages of
+// values.
 // Every mbarrier wait is bounded; on expiry the error word is set and the CTA drains and frees its tensor memory.
 #include "attn_math.cuh"
 #include "flash_tc_utils.cuh"
@@ -26,16 +27,17 @@ using pa::Prompt;
 
 constexpr float LAG = 8.f;
 
-// DQ: key dims, DT: value columns of a CTA, PB: P tiles (2: bounded scores)
-template <int DQ, int DT, int PB>
+// DQ: key dims, DT: value columns of a CTA
+template <int DQ, int DT, bool BOUNDED>
 struct __align__(1024) Smem {
     static constexpr int VK = DT > 128 ? 64 : BN;           // keys per stage of values
+    static constexpr int ST = DT > 128 && BOUNDED ? 4 : 2;               // stages of values
     uint8_t q[BM * DQ * 2];
     uint8_t k[2][BN * DQ * 2];
-    uint8_t v[2][VK * DT * 2];
-    uint8_t p[PB][BM * BN * 2];
-    float mx[PB == 1 ? 2 : 1][PB == 1 ? SPLIT : 1][PB == 1 ? BM : 1];
-    uint64_t q_full, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[2], pv_done[PB], p_ready[PB];
+    uint8_t v[ST][VK * DT * 2];
+    uint8_t p[BOUNDED ? 16 : BM * BN * 2];
+    float mx[BOUNDED ? 1 : 2][BOUNDED ? 1 : SPLIT][BOUNDED ? 1 : BM];
+    uint64_t q_full, k_full[2], k_empty[2], v_full[ST], v_empty[ST], s_full[2], pv_done, p_ready[2];
     uint32_t tmem_base;
     int abort_flag;
 };
@@ -45,6 +47,13 @@ __device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t (&r)[16
                  :: "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]),
                     "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(taddr) : "memory");
 }
+// D += A B with A in tensor memory: row r in lane r, two consecutive k per column
+__device__ __forceinline__ void umma_ta(uint32_t tmem_d, uint32_t tmem_a, uint32_t b_lo, uint32_t idesc, uint32_t accumulate, uint32_t issue) {
+    asm volatile("{\n.reg .pred p, q;\n.reg .b64 db;\nsetp.ne.b32 p, %4, 0;\nsetp.ne.b32 q, %5, 0;\n"
+                 "mov.b64 db, {%2, %6};\n"
+                 "@q tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], db, %3, p;\n}"
+                 :: "r"(tmem_d), "r"(tmem_a), "r"(b_lo), "r"(idesc), "r"(accumulate), "r"(issue), "r"(DESC_HI) : "memory");
+}
 __device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 
 // DV: value dims of a head, NB: value heads of a CTA, BOUNDED: see above
@@ -53,9 +62,10 @@ __global__ void __launch_bounds__(THREADS, 1)
 packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                       const __grid_constant__ CUtensorMap tmV, Prompt a) {
     extern __shared__ uint8_t smem_raw[];
-    constexpr int DT = NB * DV, PB = BOUNDED ? 2 : 1;
-    constexpr int VK = Smem<DQ, DT, PB>::VK, VS = BN / VK;  // VS: stages of values per tile of keys
-    Smem<DQ, DT, PB>& sm = *reinterpret_cast<Smem<DQ, DT, PB>*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+    constexpr int DT = NB * DV;
+    using Sm = Smem<DQ, DT, BOUNDED>;
+    constexpr int VK = Sm::VK, VS = BN / VK, ST = Sm::ST;   // VS: stages of values per tile of keys
+    Sm& sm = *reinterpret_cast<Sm*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
     constexpr int KQ = DQ / 64, KV = DT / 64;               // 64-element blocks along the head dimensions
     constexpr uint32_t TMEM_COLS = 512, O_COL = 2 * BN;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -64,8 +74,9 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
     const int h = blockIdx.y, hk = h / (a.H / a.G), hv = a.cross ? blockIdx.z * NB : hk;       // hv: first value head
     const int nb_lo = a.window > 0 ? max(0, c0 - a.window + 1) / BN : 0;
     const int n_it = (c0 + nq + BN - 1) / BN - nb_lo;       // at least 1: a query sees its own key
-    auto buf = [](int j) { return j & (PB - 1); };          // P tile and barriers of key tile j, and their phase
-    auto phase = [](int j) { return (uint32_t)(PB == 2 ? (j >> 1) & 1 : j & 1); };
+    // bounded: a warp may be done with tile j + 1 while another one works on tile j, so neighbouring tiles have barriers of their own
+    auto p_bar = [&](int j) { return &sm.p_ready[BOUNDED ? j & 1 : 0]; };
+    auto p_phase = [](int j) { return (uint32_t)(BOUNDED ? (j >> 1) & 1 : j & 1); };
     volatile int* abort_flag = &sm.abort_flag;
     int* err = a.err;
 
@@ -73,13 +84,11 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
         mbar_init(&sm.q_full, 1);
         for (int s = 0; s < 2; ++s) {
             mbar_init(&sm.k_full[s], 1); mbar_init(&sm.k_empty[s], 1);
-            mbar_init(&sm.v_full[s], 1); mbar_init(&sm.v_empty[s], 1);
             mbar_init(&sm.s_full[s], 1);
         }
-        for (int b = 0; b < PB; ++b) {
-            mbar_init(&sm.pv_done[b], 1);
-            mbar_init(&sm.p_ready[b], 4 * SPLIT);
-        }
+        for (int s = 0; s < ST; ++s) { mbar_init(&sm.v_full[s], 1); mbar_init(&sm.v_empty[s], 1); }
+        mbar_init(&sm.pv_done, 1);
+        for (int s = 0; s < 2; ++s) mbar_init(&sm.p_ready[s], 4 * SPLIT);
         sm.abort_flag = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
@@ -108,8 +117,8 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
                 bool ok = true;
 #pragma unroll
                 for (int u = 0; u < VS; ++u) {
-                    const int vi = j * VS + u, t = vi & 1;
-                    ok = mbar_wait_suspend(&sm.v_empty[t], ((vi >> 1) & 1) ^ 1, abort_flag, err, 0x7200 | t);
+                    const int vi = j * VS + u, t = vi % ST;
+                    ok = mbar_wait_suspend(&sm.v_empty[t], (vi / ST & 1) ^ 1, abort_flag, err, 0x7200 | t);
                     if (!ok) break;
                     mbar_expect_tx(&sm.v_full[t], VK * DT * 2);
 #pragma unroll
@@ -143,27 +152,31 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
         };
         if (ok) ok = issue_s(0);
         for (int j = 0; ok && j < n_it; ++j) {
-            // score buffer (j + 1) & 1 was last read for P_{j-1}, whose p_ready was waited for in the previous iteration
+            // score buffer (j + 1) & 1 was last read for P_{j-1}, whose p_ready was waited for in the previous iteration; with P_{j-1} in its
+            // place, the product that reads it has to complete
+            if (BOUNDED && j > 0 && j + 1 < n_it && !mbar_wait_suspend(&sm.pv_done, (j - 1) & 1, abort_flag, err, 0x8400)) break;
             if (j + 1 < n_it) { ok = issue_s(j + 1); if (!ok) break; }
 #pragma unroll
             for (int u = 0; u < VS; ++u) {
-                const int vi = j * VS + u, t = vi & 1;
-                ok = mbar_wait_suspend(&sm.v_full[t], (vi >> 1) & 1, abort_flag, err, 0x8200 | t);
-                if (ok && u == 0) ok = mbar_wait_suspend(&sm.p_ready[buf(j)], phase(j), abort_flag, err, 0x8300);
+                const int vi = j * VS + u, t = vi % ST;
+                ok = mbar_wait_suspend(&sm.v_full[t], vi / ST & 1, abort_flag, err, 0x8200 | t);
+                if (ok && u == 0) ok = mbar_wait_suspend(p_bar(j), p_phase(j), abort_flag, err, 0x8300);
                 if (!ok) break;
                 tc_fence_after();
-                const uint32_t pl = desc_lo<false>(s32(sm.p[buf(j)])), vl = desc_lo<true>(s32(sm.v[t]));
+                const uint32_t pl = BOUNDED ? tmem_base + (j & 1) * BN : desc_lo<false>(s32(sm.p)), vl = desc_lo<true>(s32(sm.v[t]));
 #pragma unroll
                 for (int kk = 0; kk < VK / UMMA_K; ++kk) {
                     const int kp = u * (VK / UMMA_K) + kk;  // 16-key step of the tile
                     const uint32_t aoff = ((kp / 4) * (BM * 128) + (kp % 4) * 32) >> 4;
                     const uint32_t boff = ((kk / 4) * (KV * 8192) + (kk % 4) * 2048) >> 4;
-                    umma_lo(tmem_base + O_COL, pl + aoff, vl + boff, idesc_o, (j > 0 || kp > 0) ? 1u : 0u, issue);
+                    if (BOUNDED)                            // every 32 scores left 16 columns of P at their beginning
+                        umma_ta(tmem_base + O_COL, pl + kp / 2 * 32 + kp % 2 * 8, vl + boff, idesc_o, (j > 0 || kp > 0) ? 1u : 0u, issue);
+                    else umma_lo(tmem_base + O_COL, pl + aoff, vl + boff, idesc_o, (j > 0 || kp > 0) ? 1u : 0u, issue);
                 }
                 umma_commit_if(&sm.v_empty[t], issue);
             }
             if (!ok) break;
-            umma_commit_if(&sm.pv_done[buf(j)], issue);
+            umma_commit_if(&sm.pv_done, issue);
         }
     } else if (warp >= 4) {
         const int qd = warp & 3, part = (warp - 4) >> 2;
@@ -172,7 +185,7 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
         constexpr int CW = BN / SPLIT, OW = DT / SPLIT;       // score / output columns of this thread
         static_assert(CW == 32 && OW % 16 == 0, "tensor-memory load widths");
         const float sc = a.scale * LOG2E, lag = LAG / sc;
-        uint8_t* prow = sm.p[0] + ((part * CW) >> 6) * (BM * 128) + (r >> 3) * 1024 + (r & 7) * 128;
+        uint8_t* prow = sm.p + ((part * CW) >> 6) * (BM * 128) + (r >> 3) * 1024 + (r & 7) * 128;
         const int ch0 = ((part * CW) & 63) >> 3;
         float m = -INFINITY, l = 0.f;
         bool alive = true;
@@ -210,7 +223,7 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
                 if (grow) m = mx;
                 l *= corr;
                 if (__any_sync(0xffffffffu, scaled)) {            // not before tile 1: O holds something
-                    if (!mbar_wait_suspend(&sm.pv_done[0], (j - 1) & 1, abort_flag, err, 0x9200)) { alive = false; break; }
+                    if (!mbar_wait_suspend(&sm.pv_done, (j - 1) & 1, abort_flag, err, 0x9200)) { alive = false; break; }
                     tc_fence_after();
 #pragma unroll
                     for (int c = 0; c < OW; c += 16) {
@@ -238,17 +251,28 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
                 v[(c >> 1) + 1] = pack_bf16(p2, p3);
             }
             l += (sum0.x + sum0.y) + (sum1.x + sum1.y);
-            // a P tile is free once the product with the values that it was last used for has completed
-            if (j >= PB && !mbar_wait_suspend(&sm.pv_done[buf(j)], phase(j - PB), abort_flag, err, 0x9300)) { alive = false; break; }
+            if constexpr (BOUNDED) {
+                uint32_t p[16];
 #pragma unroll
-            for (int c = 0; c < 4; ++c)
-                *reinterpret_cast<uint4*>(prow + buf(j) * (BM * BN * 2) + (((ch0 + c) ^ (r & 7)) << 4)) = make_uint4(v[4 * c], v[4 * c + 1], v[4 * c + 2], v[4 * c + 3]);
-            tc_fence_before();
-            asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+                for (int c = 0; c < 16; ++c) p[c] = v[c];
+                tmem_st16(lane_addr + s * BN + part * CW, p);
+                tmem_st_wait();
+                tc_fence_before();
+            } else {
+                // the P tile is free once O += P_{j-1} V_{j-1} has completed
+                if (j > 0 && !mbar_wait_suspend(&sm.pv_done, (j - 1) & 1, abort_flag, err, 0x9300)) { alive = false; break; }
+#pragma unroll
+                for (int c = 0; c < 4; ++c)
+                    *reinterpret_cast<uint4*>(prow + (((ch0 + c) ^ (r & 7)) << 4)) = make_uint4(v[4 * c], v[4 * c + 1], v[4 * c + 2], v[4 * c + 3]);
+                tc_fence_before();
+                asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+            }
             __syncwarp();
-            if (lane == 0) mbar_arrive(&sm.p_ready[buf(j)]);
+            if (lane == 0) mbar_arrive(p_bar(j));
         }
-        if (alive) alive = mbar_wait_suspend(&sm.pv_done[buf(n_it - 1)], phase(n_it - 1), abort_flag, err, 0x9400);
+        // (the product before the last one first: a barrier that is two phases behind looks like one that is done)
+        if (BOUNDED && alive && n_it > 1) alive = mbar_wait_suspend(&sm.pv_done, (n_it - 2) & 1, abort_flag, err, 0x9500);
+        if (alive) alive = mbar_wait_suspend(&sm.pv_done, (n_it - 1) & 1, abort_flag, err, 0x9400);
         tc_fence_after();
         float* ls = reinterpret_cast<float*>(sm.q);           // [SPLIT][BM]; every product has completed, the queries are not read any more
         ls[part * BM + r] = l;
@@ -290,8 +314,8 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
 
 template <int DQ, int DV, int NB, bool BOUNDED>
 static int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const Prompt& a, cudaStream_t st) {
-    const size_t smem = sizeof(Smem<DQ, NB * DV, BOUNDED ? 2 : 1>) + 1024;
-    static_assert(sizeof(Smem<DQ, NB * DV, BOUNDED ? 2 : 1>) + 1024 <= 227 * 1024 && NB * DV <= 256, "shared and tensor memory of one CTA");
+    const size_t smem = sizeof(Smem<DQ, NB * DV, BOUNDED>) + 1024;
+    static_assert(sizeof(Smem<DQ, NB * DV, BOUNDED>) + 1024 <= 227 * 1024 && NB * DV <= 256, "shared and tensor memory of one CTA");
     cudaError_t e = cudaFuncSetAttribute(packed_attn_tc_kernel<DQ, DV, NB, BOUNDED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     packed_attn_tc_kernel<DQ, DV, NB, BOUNDED><<<dim3(a.n, a.H, a.cross ? (a.G + NB - 1) / NB : 1), THREADS, smem, st>>>(mq, mk, mv, a);

@@ -14,7 +14,7 @@ constexpr int ST = 512;
 
 // grid (H, n).  A thread owns 4 columns of the state and every `parts`-th row (parts = ST / (dv / 4)), NB of them in flight.
 template <typename T>
-__global__ void __launch_bounds__(ST) retention_step_kernel(Args a) {
+__global__ void __launch_bounds__(ST, 2) retention_step_kernel(Args a) {
     constexpr int NB = 8;
     extern __shared__ float4 sm4[];
     const int h = blockIdx.x, b = blockIdx.y, dk = a.dk, dv = a.dv, half = a.rot / 2;
