@@ -186,7 +186,7 @@ def _gafonex_config(raw: dict, shapes: Dict[str, Tuple[int, ...]]) -> ModelConfi
         layers.append({"mixer": _gafonex_mixer(i, raw["layers"], lender), "ff": None if mlp is None else mlp["ff"]})
     first = layers[0]["mixer"]
     return ModelConfig(base_model="gafonex", layers=tuple(layers), hidden_size=raw["width"], vocab_size=raw["vocab"], norm_eps=raw["norm"]["eps"],
-                       norm_groups=raw["norm"]["groups"], logit_softcap=raw.get("logit_softcap"), max_position_embeddings=UNBOUNDED,
+                       norm_groups=raw["norm"].get("groups", 1), logit_softcap=raw.get("logit_softcap"), max_position_embeddings=UNBOUNDED,
                        num_attention_heads=first.heads, kv_channels=first.dim)
 
 
