@@ -119,7 +119,7 @@ def kernels(size: str) -> list:
     from ..ops import gemm
     from ..ops import packed_attn as PA
     from ..ops.moe_fused import fused_moe
-    from ..ops.moe_rows import ExpertsSpec, experts_relu2, route_rows
+    from ..ops.moe_rows import ExpertsSpec, experts_rows, route_rows
     from ..ops.row_batch import RowBatch
     from ..parallel import fused_comm
     dev, bf = torch.device("cuda", 0), torch.bfloat16
@@ -183,10 +183,10 @@ def kernels(size: str) -> list:
     up, down = rnd(E, ff, w) * 0.02, rnd(E, w, ff) * 0.02
     e, logits = ExpertsSpec(E, top, ff), torch.randn(rows, E, device=dev)
     fl = 2 * rows * top * 2 * ff * w
-    row("experts_relu2, whole", "experts", timeit(lambda: experts_relu2(h, logits, up, down, e)), flops=fl)
+    row("experts_rows, whole", "experts", timeit(lambda: experts_rows(h, logits, up, down, e)), flops=fl)
     wr = rnd(E, w)
     row("router product (gemm_dense, fp32)", "router gemm", timeit(lambda: ops.linear_f32(h, wr)), bytes_=rows * w * 2)
-    row("route_rows", "router", timeit(lambda: route_rows(logits, E, top)), bytes_=rows * (E + 2 * top) * 4)
+    row("route_rows", "router", timeit(lambda: route_rows(logits, ExpertsSpec(E, top, ff))), bytes_=rows * (E + 2 * top) * 4)
     lb = logits.bfloat16()
     row("router_topk (qwen2)", "router", timeit(lambda: ops.router_topk(lb, top)), bytes_=rows * (E + 2 * top) * 4)
     ws = fused_comm.MoeWorkspace(None, E, w, rows * top + 256 * E, dev)
@@ -256,10 +256,10 @@ def kernels(size: str) -> list:
         row(f"out projection (gemm, fp32 result), batch {n}", "skinny gemm", _graph_ms(lambda m: PA.sublayer_out(oa, m), ms), bytes_=by)
         del ms
         lg = torch.randn(n, E, device=dev)
-        used = int(torch.unique(route_rows(lg, E, top)[1]).numel())
+        used = int(torch.unique(route_rows(lg, ExpertsSpec(E, top, ff))[1]).numel())
         by = used * ff * w * 4
         sets = [(up, down)] + [(torch.randn_like(up), torch.randn_like(down)) for _ in range(2)]
-        row(f"route + moe_step up + down, batch {n}", "experts decode", _graph_ms(lambda u, d: experts_relu2(x8, lg, u, d, e), sets), bytes_=by)
+        row(f"route + moe_step up + down, batch {n}", "experts decode", _graph_ms(lambda u, d: experts_rows(x8, lg, u, d, e), sets), bytes_=by)
         pk, ix, _ = ops.router_topk(lg.bfloat16(), top)
         del sets
         row(f"fused_moe (qwen2), gated experts, batch {n} (eager calls)", "experts decode", timeit(lambda: fused_moe(x8, pk, ix, w1, w2, ws)), bytes_=by * 1.5)
@@ -276,7 +276,7 @@ def kernels(size: str) -> list:
         page.reserve(page.acquire(n), [CTX] * n)
         zl = rnd(n, R)
         row(f"latent_norm + store, batch {n}", "row kernel decode", _graph_ms(lambda: PA.latent_norm(zl, wc, R, 1e-5, one_tok, page[0]), [()] * 100))
-        row(f"route_rows, batch {n}", "row kernel decode", _graph_ms(lambda: route_rows(lg, E, top), [()] * 100))
+        row(f"route_rows, batch {n}", "row kernel decode", _graph_ms(lambda: route_rows(lg, ExpertsSpec(E, top, ff)), [()] * 100))
     gemm.check_error()
     return out
 

@@ -20,8 +20,21 @@ LA_MODULES = (
     "gated_deltanet", "gsa", "based", "rebased", "hgrn2", "rwkv6", "rwkv7",
     "mamba2", "lasp2", "mom_gla", "mom_gated_deltanet", "mom_linear_attention",
 )
-BASE_MODELS = ("qwen2", "llama3", "mixtral", "deepseek_v2", "lagisun", "sonodra", "gafonex")
-LAYER_LIST_MODELS = ("lagisun", "sonodra", "gafonex")        # described by ModelConfig.layers; run packed rows, serve only
+BASE_MODELS = ("qwen2", "llama3", "mixtral", "deepseek_v2", "lagisun", "sonodra", "gafonex", "zelinex")
+LAYER_LIST_MODELS = ("lagisun", "sonodra", "gafonex", "zelinex")        # described by ModelConfig.layers; run packed rows, serve only
+
+
+@dataclass(frozen=True)
+class LayerLoop:
+    """Layers ``start .. stop - 1`` run ``times`` times in a row with the same weights.  In front of every pass the stream gets the pass's
+    own vector, and in front of every pass but the first the embedding's rows again."""
+    start: int
+    stop: int
+    times: int
+
+    def __post_init__(self):
+        if not 0 <= self.start < self.stop or self.times < 1:
+            raise ValueError(f"layers {self.start} .. {self.stop} run {self.times} times")
 
 
 @dataclass
@@ -140,7 +153,10 @@ class ModelConfig:
     #   {"mixer": ops.packed_attn.AttentionSpec or LatentSpec, "ff": width (gated), ops.moe_rows.ExpertsSpec, or None}
     # gafonex: sequential blocks with a norm behind a sublayer only, one entry per layer
     #   {"mixer": ops.packed_attn.AttentionSpec or ops.retention.RetentionSpec, "ff": width (gated, ReLU) or None}
+    # zelinex: blocks as sonodra's, scaled by residual_multiplier, some of them run several times
+    #   {"mixer": models.sandwich_block.ParallelSpec or ops.delta_rule.GeneralDeltaSpec, "ff": ops.moe_rows.MlpSpec or ExpertsSpec, or None}
     layers: Optional[Tuple[dict, ...]] = None
+    loop: Optional["LayerLoop"] = None            # layer-list designs: layers that run several times in a row
     norm_groups: int = 1                          # layer-list designs: parts of a row that are normed by themselves
     logit_softcap: Optional[float] = None         # layer-list designs: logits become cap * tanh(logits / cap)
     residual_multiplier: float = 1.0              # factor of every block's output before it joins the residual stream
@@ -164,6 +180,8 @@ class ModelConfig:
             raise ValueError(f"{', '.join(LAYER_LIST_MODELS)} models are described by their layer list (and no other family has one)")
         if self.layers is not None:
             self.num_layers = len(self.layers)
+        if self.loop is not None and (self.layers is None or self.loop.stop > len(self.layers)):
+            raise ValueError(f"{self.loop} of a model without these layers")
         if self.norm_groups < 1 or self.hidden_size % self.norm_groups:
             raise ValueError(f"a width of {self.hidden_size} has no {self.norm_groups} equal parts")
         if self.logit_softcap is not None and not self.logit_softcap > 0:
@@ -190,6 +208,14 @@ class ModelConfig:
             self.shared_expert_gate = False
 
     # -- derived ----------------------------------------------------------
+    def layer_runs(self) -> List[Tuple[int, Optional[int]]]:
+        """Layer-list designs: the layers in the order they run; with the first layer of a loop's pass, the number of the pass."""
+        n, loop = len(self.layers), self.loop
+        if loop is None:
+            return [(i, None) for i in range(n)]
+        passes = [(i, t if i == loop.start else None) for t in range(loop.times) for i in range(loop.start, loop.stop)]
+        return [(i, None) for i in range(loop.start)] + passes + [(i, None) for i in range(loop.stop, n)]
+
     @property
     def is_moe(self) -> bool:
         return self.num_experts is not None and self.num_experts > 0

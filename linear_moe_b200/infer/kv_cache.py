@@ -9,16 +9,17 @@ token until it is released; each layer says what it needs (``None``: nothing of 
 * :class:`LayerPages`  one row per token, in pages of :data:`PAGE` rows taken from a pool as a request grows.  Page numbers hold for
   all paged layers alike, so one table ``[slots, pages]`` (int32, on the device) serves the model.  A row is a key and a value
   (``[pages, PAGE, heads, dim]``) or, with ``v_dim = 0``, one vector that is both (a latent).
+* :class:`LayerInputs` the last rows that went into a short convolution (row = position modulo rows), not cleared either.
 * :class:`LayerState`  one fp32 matrix per head, ``[slots, heads, k_dim, v_dim]``: the state of a recurrence, whatever the context.  It is not
   cleared when a slot is handed out; a request's first call starts from zero instead of reading it.
 
-Because the buffers never move while a request lives (unless they have to grow, which changes ``generation``), one-token steps
+A layer that keeps several of these says so with a tuple.  Because the buffers never move while a request lives (unless they have to grow, which changes ``generation``), one-token steps
 can be captured in a CUDA graph.
 """
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Dict, List, Optional, Sequence, Union
+from typing import Dict, List, Optional, Sequence, Tuple, Union
 
 import torch
 
@@ -50,16 +51,27 @@ class LayerState:
     v_dim: int
 
 
+@dataclass(frozen=True)
+class LayerInputs:
+    """The last ``rows`` inputs of a short convolution."""
+    rows: int
+    width: int
+
+
+Kept = Union[LayerRows, LayerPages, LayerState, LayerInputs]
+
+
 class SlotCache:
-    def __init__(self, layers: Sequence[Optional[Union[LayerRows, LayerPages, LayerState]]], slots: int, device, dtype, tokens: int = 0):
+    def __init__(self, layers: Sequence[Optional[Union[Kept, Tuple[Kept, ...]]]], slots: int, device, dtype, tokens: int = 0):
         """``tokens``: live tokens to make room for from the start (paged layers; the pool grows when there are more)."""
         self.spec, self.device, self.dtype = list(layers), torch.device(device), dtype
         self.layers: List[Dict[str, torch.Tensor]] = [{} for _ in self.spec]
+        self._kept = [(s, c) for kept, c in zip(self.spec, self.layers) if kept is not None for s in (kept if isinstance(kept, tuple) else (kept,))]
         self.free: List[int] = []
         self.slots = 0
         self.generation = 0                     # changes when the buffers move (captured graphs are then stale)
         self.lengths: Dict[int, int] = {}       # tokens of every live slot
-        self.paged = any(isinstance(s, LayerPages) for s in self.spec)
+        self.paged = any(isinstance(s, LayerPages) for s, _ in self._kept)
         self.pages = 0                          # pages of the pool
         self.free_pages: List[int] = []
         self.owned: Dict[int, List[int]] = {}   # slot -> its pages, in order of position
@@ -82,12 +94,14 @@ class SlotCache:
         c[name] = t
 
     def _resize(self, slots: int):
-        for s, c in zip(self.spec, self.layers):
+        for s, c in self._kept:
             if isinstance(s, LayerRows):
                 for name, dim in (("k", s.k_dim), ("v", s.v_dim)):
                     self._buffer(c, name, (slots, s.rows, s.heads, dim), self.slots)
             elif isinstance(s, LayerState):
                 self._buffer(c, "s", (slots, s.heads, s.k_dim, s.v_dim), self.slots, torch.float32)
+            elif isinstance(s, LayerInputs):
+                self._buffer(c, "c", (slots, s.rows, s.width), self.slots)
         if self.paged:
             self._resize_table(slots, max(self._table_host.shape[1], 16))
         self.free += range(self.slots, slots)
@@ -99,12 +113,12 @@ class SlotCache:
         self._table_host = torch.zeros(slots, pages, dtype=torch.int32)
         self._table_host[: old.shape[0], : old.shape[1]] = old
         self.table = self._table_host.to(self.device)
-        for s, c in zip(self.spec, self.layers):
+        for s, c in self._kept:
             if isinstance(s, LayerPages):
                 c["table"] = self.table
 
     def _grow_pool(self, pages: int):
-        for s, c in zip(self.spec, self.layers):
+        for s, c in self._kept:
             if isinstance(s, LayerPages):
                 self._buffer(c, "k", (pages, PAGE, s.heads, s.k_dim), self.pages)
                 if s.v_dim:

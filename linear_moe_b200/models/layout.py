@@ -24,7 +24,7 @@ from typing import List, Optional, Tuple
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: Optional[str]      # 'lsm' | 'attn' | 'mla' | 'mamba' | 'chunk_attn' | 'packed_attn' | 'packed_latent' | 'retention' | None
+    mixer: Optional[str]      # 'lsm' | 'attn' | 'mla' | 'mamba' | 'chunk_attn' | 'packed_attn' | 'packed_latent' | 'retention' | 'parallel' | 'general_delta' | None
     ffn: Optional[str]        # 'mlp' | 'moe' | 'poly_mlp' | None
     symbol: str               # source symbol, for logs and checkpoints
     index: int                # global index in the expanded list
@@ -89,6 +89,9 @@ def expand_layer_pattern(cfg) -> List[LayerSpec]:
         if cfg.base_model == "gafonex":
             return [LayerSpec("retention" if hasattr(l["mixer"], "decay") else "packed_attn", None if l["ff"] is None else "mlp", "P", i)
                     for i, l in enumerate(cfg.layers)]
+        if cfg.base_model == "zelinex":
+            return [LayerSpec("parallel" if hasattr(l["mixer"], "left") else "general_delta", None if l["ff"] is None else "moe" if hasattr(l["ff"], "experts") else "mlp",
+                              "S", i) for i, l in enumerate(cfg.layers)]
         if cfg.base_model == "sonodra":
             return [LayerSpec("packed_latent" if hasattr(l["mixer"], "rank") else "packed_attn",
                               None if l["ff"] is None else "mlp" if isinstance(l["ff"], int) else "moe", "S", i) for i, l in enumerate(cfg.layers)]

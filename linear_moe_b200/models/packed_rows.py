@@ -33,6 +33,7 @@ class RowStep:
     latents: Dict[int, torch.Tensor] = field(default_factory=dict)    # layer -> latent rows, for the layers that borrow them
     values: Dict[int, torch.Tensor] = field(default_factory=dict)     # layer -> value rows, for the layers that mix them into theirs
 
+    place: Dict[int, int] = field(default_factory=dict)               # layer -> its current run (a layer of a loop has one cache per run)
     turns: Dict[tuple, Optional[torch.Tensor]] = field(default_factory=dict)      # rotary tables of the rows, by their constants
 
     def turn(self, key: tuple, freq: Optional[torch.Tensor], size: float = 1.0) -> Optional[torch.Tensor]:
@@ -42,12 +43,24 @@ class RowStep:
         return self.turns[key]
 
     def cache(self, layer: int) -> Optional[dict]:
-        return None if self.caches is None else self.caches[layer]
+        return None if self.caches is None else self.caches[self.place[layer]]
+
+
+def fill(view, t: torch.Tensor):
+    """Put a checkpoint's tensor into its place (``RowBlock.places``)."""
+    if isinstance(view, list):
+        at = 0
+        for v in view:
+            n = v.shape[0] * (v.shape[1] if v.dim() > t.dim() else 1)
+            v.copy_(t[at:at + n].reshape(v.shape))
+            at += n
+    else:
+        view.copy_(t.reshape(view.shape))
 
 
 class RowBlock(nn.Module):
     """A block of such a model.  ``places()`` maps the checkpoint's tensor names (without the layer) to views inside the block's
-    parameters and the tensors' shapes; weights may be stored fused and padded."""
+    parameters (a list of views: consecutive rows of the tensor) and the tensors' shapes; weights may be stored fused and padded."""
     reads_stream = False
 
     def places(self) -> Dict[str, Tuple[torch.Tensor, Tuple[int, ...]]]:
@@ -59,13 +72,13 @@ class RowBlock(nn.Module):
             t = get(name)
             if tuple(t.shape) != tuple(shape):
                 raise ValueError(f"{name}: shape {tuple(t.shape)}, the configuration asks for {tuple(shape)}")
-            view.copy_(t.reshape(view.shape))
+            fill(view, t)
 
 
 def new_slot_cache(model, slots: int = 1, tokens: int = 0) -> SlotCache:
     limit = model.cfg.max_position_embeddings
     p = model.embedding.word_embeddings.weight
-    return SlotCache([b.cache_spec(limit) for b in model.decoder.layers], slots, p.device, p.dtype, tokens)
+    return SlotCache([model.decoder.layers[i].cache_spec(limit) for i, _ in model.cfg.layer_runs()], slots, p.device, p.dtype, tokens)
 
 
 def forward_rows(model, input_ids, labels, caches, position_offset: int, batch: Optional[RowBatch], logit_rows, return_hidden: bool):
@@ -86,15 +99,21 @@ def forward_rows(model, input_ids, labels, caches, position_offset: int, batch: 
         raise ValueError(f"position {batch.reach() - 1} is beyond the model's table of {cfg.max_position_embeddings} positions")
     emb, w, blocks = model.embedding, cfg.hidden_size, model.decoder.layers
     pos = getattr(emb, "position_embeddings", None)
+    ids, table = input_ids.reshape(-1), emb.word_embeddings.weight
+    steps = getattr(model.decoder, "loop_step", None)
     if blocks[0].reads_stream:
-        x, h = ops.embed_rows(input_ids.reshape(-1), emb.word_embeddings.weight, round_up(w, ROW_PAD))
+        x, h = ops.embed_rows(ids, table, round_up(w, ROW_PAD))
     else:
-        x, h = ops.embed_norm(input_ids.reshape(-1), batch.pos, emb.word_embeddings.weight, None if pos is None else pos.weight,
-                              round_up(w, ROW_PAD), cfg.norm_eps, blocks[0].input_gain())
+        x, h = ops.embed_norm(ids, batch.pos, table, None if pos is None else pos.weight, round_up(w, ROW_PAD), cfg.norm_eps, blocks[0].input_gain(),
+                              None if cfg.loop is None or cfg.loop.start else steps[0])
     taps = getattr(model, "residual_taps", None)                    # a list here receives the stream after every layer
-    step, dtype = RowStep(batch, caches), h.dtype
-    for blk, nxt in zip(blocks, [*blocks[1:], None]):
-        h = blk(x, h, step, nxt)
+    step, dtype, runs = RowStep(batch, caches), h.dtype, cfg.layer_runs()
+    for n, (i, start) in enumerate(runs):
+        if start is not None and n:                                 # a pass of the loop begins
+            h = ops.restart_norm(x, ids, table if start else None, steps[start], w, cfg.norm_eps, blocks[i].input_gain(), dtype)
+        step.place[i] = n
+        after, again = runs[n + 1] if n + 1 < len(runs) else (None, None)
+        h = blocks[i](x, h, step, None if after is None or again is not None else blocks[after])
         if taps is not None:
             taps.append(x[:, :w].clone())
     if logit_rows is not None:

@@ -13,11 +13,14 @@ from typing import Callable, Dict, Optional, Tuple
 import torch
 
 from ..ckpt.safetensors_io import read_header, read_tensors
-from ..config.model_config import ModelConfig
+from ..config.model_config import LayerLoop, ModelConfig
 from ..ops.chunk_attn import ChunkAttnSpec
-from ..ops.moe_rows import ExpertsSpec
+from ..ops.delta_rule import GeneralDeltaSpec
+from ..ops.moe_rows import ExpertsSpec, MlpSpec
 from ..ops.packed_attn import AttentionSpec, LatentSpec, RotaryScaling
 from ..ops.retention import RetentionSpec
+from ..ops.ssd import SsdSpec
+from .sandwich_block import ParallelSpec
 from .transformer import CausalLM
 
 UNBOUNDED = 1 << 30           # positions of a model without a position table
@@ -137,12 +140,14 @@ def _sonodra_load(model: CausalLM, tensors: Dict[str, torch.Tensor]):
 
 @torch.no_grad()
 def _load_rows(model: CausalLM, tensors: Dict[str, torch.Tensor], more: Dict[str, torch.Tensor]):
-    """Tensors of a packed-row model: ``embed``, ``final.norm``, ``head``, those in ``more``, and every layer's under ``l<i>.``."""
+    """Tensors of a packed-row model: ``embed``, ``final.norm``, ``head`` (unless the embedding is the head), those in ``more``, and every layer's under ``l<i>.``."""
     norm = model.decoder.final_layernorm.weight
     if norm.dim():                                                  # padded rows: nothing behind the width
         norm.zero_()
         norm = norm[:model.cfg.hidden_size]
-    whole = {"embed": model.embedding.word_embeddings.weight, "final.norm": norm, "head": model.output_layer.weight, **more}
+    whole = {"embed": model.embedding.word_embeddings.weight, "final.norm": norm, **more}
+    if not model.cfg.tie_embeddings:
+        whole["head"] = model.output_layer.weight
     for name, dst in whole.items():
         t = tensors[name]
         if t.shape != dst.shape:
@@ -195,3 +200,52 @@ def _gafonex_load(model: CausalLM, tensors: Dict[str, torch.Tensor]):
 
 
 register(Architecture("Gafonex", _gafonex_config, _gafonex_load, "post_norm_block"))
+
+
+# ---------------------------------------------------------------------------------------------------------------- Zelinex
+def _zelinex_attention(m: dict) -> AttentionSpec:
+    rot, mask = m.get("rot"), m.get("mask")
+    return AttentionSpec(heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"], scale=m["scale"], rot_halves=True, sigmoid=True,
+                         window=None if mask is None else mask["size"], rot_dims=0 if rot is None else rot["dims"],
+                         rot_base=1.0 if rot is None else rot["base"])
+
+
+def _zelinex_mixer(i: int, layer: dict, shapes: Dict[str, Tuple[int, ...]]):
+    kind, m = layer["type"], layer["mixer"]
+    if kind == "general_delta":
+        return GeneralDeltaSpec(heads=m["heads"], dim=m["dim"], rank=shapes[f"l{i}.mix.w1"][0])
+    if kind == "parallel":
+        r = m["right"]
+        right = SsdSpec(heads=r["heads"], groups=r["groups"], state=r["state"], vdim=r["vdim"], taps=r["conv"], norm_groups=r["norm_groups"])
+        return ParallelSpec(left=_zelinex_attention(m["left"]), right=right, left_scale=m["left_scale"], right_scale=m["right_scale"])
+    raise ValueError(f"layer {i}: unknown mixer {kind!r}")
+
+
+def _zelinex_ff(i: int, mlp: Optional[dict]):
+    if mlp is None:
+        return None
+    if mlp["kind"] == "dense":
+        return MlpSpec(mlp["ff"], "xielu")
+    if mlp["kind"] == "moe":
+        r, shared = mlp["router"], mlp.get("shared")
+        return ExpertsSpec(r["experts"], r["top"], mlp["expert"]["ff"], act="silu", scores="softmax", normalise=True, scale=r["scale"],
+                           shared=None if shared is None else shared["ff"])
+    raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+
+
+def _zelinex_config(raw: dict, shapes: Dict[str, Tuple[int, ...]]) -> ModelConfig:
+    layers = [{"mixer": _zelinex_mixer(i, l, shapes), "ff": _zelinex_ff(i, l.get("mlp"))} for i, l in enumerate(raw["layers"])]
+    loop, first = raw.get("loop"), layers[0]["mixer"]
+    first = getattr(first, "left", first)
+    return ModelConfig(base_model="zelinex", layers=tuple(layers), hidden_size=raw["width"], vocab_size=raw["vocab"], norm_eps=raw["norm"]["eps"],
+                       residual_multiplier=raw.get("residual_mult", 1.0), tie_embeddings=True, max_position_embeddings=UNBOUNDED,
+                       loop=None if loop is None else LayerLoop(loop["start"], loop["stop"], loop["times"]), num_attention_heads=first.heads,
+                       kv_channels=first.dim)
+
+
+def _zelinex_load(model: CausalLM, tensors: Dict[str, torch.Tensor]):
+    steps = getattr(model.decoder, "loop_step", None)
+    _load_rows(model, tensors, {} if steps is None else {"loop.step": steps[:, :model.cfg.hidden_size]})
+
+
+register(Architecture("Zelinex", _zelinex_config, _zelinex_load, "zelinex"))

@@ -185,6 +185,8 @@ class CausalLM(nn.Module):
                 self.decoder.final_layernorm = nn.Module()         # one number, or one per column of the padded rows
                 shape = () if cfg.normalization == "ScalarRMSNorm" else (-(-cfg.hidden_size // ROW_PAD) * ROW_PAD,)
                 self.decoder.final_layernorm.weight = nn.Parameter(torch.ones(shape, device=device))
+                if cfg.loop is not None:
+                    self.decoder.loop_step = nn.Parameter(torch.zeros(cfg.loop.times, -(-cfg.hidden_size // ROW_PAD) * ROW_PAD, device=device))
             else:
                 self.decoder.final_layernorm = Norm(cfg, device)
             tied = self.embedding.word_embeddings.weight if (cfg.tie_embeddings and pre_process) else None

@@ -322,12 +322,14 @@ def softmax_attention(q, k, v, scale=None, causal=True, q_offset: int = 0, windo
 
 
 # ---- packed-row operators (serving only) -----------------------------------------------------------
-from .chunk_attn import chunk_attention, embed_norm, poly_norm, stream_norm   # noqa: E402,F401
+from .chunk_attn import chunk_attention, embed_norm, poly_norm, restart_norm, stream_norm   # noqa: E402,F401
 from .group_norm import embed_rows, group_norm, residual_group_norm, softcap_   # noqa: E402,F401
-from .moe_rows import experts_relu2   # noqa: E402,F401
+from .delta_rule import general_delta_rows   # noqa: E402,F401
+from .moe_rows import experts_rows   # noqa: E402,F401
 from .packed_attn import (causal_attention, gather_rows, glu_in, head_norm_rope_, latent_absorb, latent_norm, latent_up,   # noqa: E402,F401
-                          qk_norm_rope_, residual_norm, rotary_rows, rotate_heads_, step_attention, sublayer_out)
+                          qk_norm_rope_, residual_norm, rotary_rows, rotate_heads_, step_attention, sublayer_out, xielu_in)
 from .retention import retention_rows   # noqa: E402,F401
+from .ssd import ssd_rows   # noqa: E402,F401
 
 
 # ---- linear sequence models -----------------------------------------------

@@ -178,13 +178,15 @@ def stream_norm(x: torch.Tensor, width: int, eps: float, dtype, gain: Optional[t
 
 
 def embed_norm(ids: torch.Tensor, pos: torch.Tensor, emb: torch.Tensor, ptab: Optional[torch.Tensor], pad: int, eps: float,
-               gain: Optional[torch.Tensor] = None):
-    """``x = emb[ids] (+ ptab[pos])`` as fp32 rows padded to ``pad`` columns, and ``x / rms(x)`` (times ``gain [pad]``) in the
+               gain: Optional[torch.Tensor] = None, shift: Optional[torch.Tensor] = None):
+    """``x = emb[ids] (+ ptab[pos]) (+ shift [pad])`` as fp32 rows padded to ``pad`` columns, and ``x / rms(x)`` (times ``gain [pad]``) in the
     table's dtype."""
     width = emb.shape[1]
     if not emb.is_cuda:
         x = torch.zeros(ids.numel(), pad)
         x[:, :width] = emb[ids].float() + (0 if ptab is None else ptab[pos.long()].float())
+        if shift is not None:
+            x += shift
         y = RC.unit_norm(x[:, :width], eps, pad)
         return x, (y if gain is None else y * gain).to(emb.dtype)
     from . import cuda as K
@@ -194,8 +196,29 @@ def embed_norm(ids: torch.Tensor, pos: torch.Tensor, emb: torch.Tensor, ptab: Op
     y = torch.empty(ids.numel(), pad, dtype=emb.dtype, device=emb.device)
     K._check(K.lib().lmoe_embed_norm(K._p(ids), K._p(pos), K._p(emb), K._p(ptab), K._p(x), ctypes.c_longlong(pad), K._p(y),
                                      ctypes.c_longlong(pad), ids.numel(), width, pad, emb.shape[0], 0 if ptab is None else ptab.shape[0],
-                                     ctypes.c_float(eps), K._p(gain), K._dt(emb), K._st()), "embed_norm")
+                                     ctypes.c_float(eps), K._p(gain), K._p(shift), 0, K._dt(emb), K._st()), "embed_norm")
     return x, y
+
+
+def restart_norm(x: torch.Tensor, ids: torch.Tensor, emb: Optional[torch.Tensor], shift: torch.Tensor, width: int, eps: float, gain: Optional[torch.Tensor],
+                 dtype) -> torch.Tensor:
+    """``x += emb[ids] + shift`` on the fp32 stream, in place (``emb`` ``None``: the shift only); returns ``x / rms(x)`` (times ``gain [pad]``) in
+    ``dtype``."""
+    if not x.is_cuda:
+        if emb is not None:
+            x[:, :width] += emb[ids].float()
+        x += shift
+        y = RC.unit_norm(x[:, :width], eps, x.shape[1])
+        return (y if gain is None else y * gain).to(dtype)
+    from . import cuda as K
+    _no_grad(x)
+    ids, pad = ids.contiguous(), x.shape[1]
+    y = torch.empty(x.shape, dtype=dtype, device=x.device)
+    assert (emb is None or emb.dtype == dtype) and shift.shape == (pad,)
+    K._check(K.lib().lmoe_embed_norm(K._p(ids), K._p(None), K._p(emb), K._p(None), K._p(x), ctypes.c_longlong(x.stride(0)), K._p(y), ctypes.c_longlong(pad),
+                                     x.shape[0], width, pad, 1 if emb is None else emb.shape[0], 0, ctypes.c_float(eps), K._p(gain), K._p(shift), 1, K._dt(y),
+                                     K._st()), "embed_norm")
+    return y
 
 
 def poly_norm(z: torch.Tensor, out: torch.Tensor, ff: int, gain: torch.Tensor, act: torch.Tensor, eps: float, mul: float = 1.0):

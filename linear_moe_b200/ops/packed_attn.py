@@ -1,8 +1,8 @@
-"""Softmax attention over packed rows with a cache, and the row operators of blocks that norm both ends of a sublayer.
+"""Attention over packed rows with a cache, and the row operators of blocks that norm both ends of a sublayer.
 
 Two kinds of attention share the kernels: grouped-query attention (optional norm over the whole query and key projections or over every
-head, optional rotary positions in either pairing, optional sliding window, optional talking heads, optional norm and mixing of the values)
-and latent attention (keys and values are products of one cached latent row per token).  Operators work on packed rows (:class:`~linear_moe_b200.ops.row_batch.RowBatch`).  CUDA tensors (bf16 or fp32) take the kernels of
+head, optional rotary positions in either pairing, optional sliding window, optional talking heads, optional norm and mixing of the values,
+softmax weights or sigmoid weights of every pair by itself) and latent attention (keys and values are products of one cached latent row per token).  Operators work on packed rows (:class:`~linear_moe_b200.ops.row_batch.RowBatch`).  CUDA tensors (bf16 or fp32) take the kernels of
 ``csrc/packed_attn*.cu``, ``csrc/talk_step.cu``, ``csrc/latent_step.cu`` and ``csrc/sandwich_block.cu``; CPU tensors take the eager definitions of
 :mod:`linear_moe_b200.ref.packed_attn`.  These operators serve (no backward pass).
 
@@ -75,6 +75,7 @@ class AttentionSpec:
     value_norm: bool = False          # every value head over its root mean square (with head_norm)
     talk: bool = False                # the softmax weights of the heads are mixed by a [heads, heads] table
     value_source: Optional[int] = None    # layer whose values are mixed into this one's (its own number: it only lends them)
+    sigmoid: bool = False             # a visible key's weight is sigmoid(score + a number of the head); nothing sums to one
 
     def __post_init__(self):
         if min(self.heads, self.kv_heads, self.dim, self.vdim) < 1 or (self.window is not None and self.window < 1):
@@ -85,9 +86,18 @@ class AttentionSpec:
             raise ValueError(f"{self.rot_dims} rotated dimensions in a head of {self.dim}")
         if self.qk_norm and self.head_norm:
             raise ValueError("queries and keys are normed as a whole or by head")
-        if not self.head_norm and (self.rot_halves or self.value_norm or self.rot_scaling or self.value_source is not None):
-            raise ValueError("rotation of halves, rotary scaling and operations on values come with the norm by head")
-        _check_scale(self.scale)
+        if not self.head_norm and (self.value_norm or self.rot_scaling or self.value_source is not None):
+            raise ValueError("rotary scaling and operations on values come with the norm by head")
+        if self.qk_norm and self.rot_halves:
+            raise ValueError("rotation of halves comes without the norm over whole projections")
+        if self.sigmoid and self.talk:
+            raise ValueError("talking heads mix softmax weights")
+        if not self.sigmoid:
+            _check_scale(self.scale)
+
+    @property
+    def by_head(self) -> bool:        # queries and keys are prepared head by head (``head_norm_rope_``)
+        return self.head_norm or self.rot_halves
 
     @property
     def dk(self) -> int:              # as laid out
@@ -163,7 +173,7 @@ def _fields(**groups):
 
 class _Prompt(ctypes.Structure):
     _fields_ = _fields(a=(_P, "q k v gate out items err"), b=(_LL, "ldq ldk ldv ldg ldo"), c=(_I, "H G dk dv window n q_rows k_rows"), d=(_F, "scale"),
-                       e=(_I, "cross bounded"))
+                       e=(_I, "cross bounded"), f=(_P, "bias"), g=(_F, "mul"))
 
 
 class _Cache(ctypes.Structure):
@@ -172,7 +182,7 @@ class _Cache(ctypes.Structure):
 
 class _Step(ctypes.Structure):
     _fields_ = _fields(a=(_P, "q out"), b=(_Cache, "c"), c=(_P, "pos slots"), d=(_LL, "ldq ldo"), e=(_I, "H G dk dv window n"), f=(_F, "scale"),
-                       g=(_I, "cross"))
+                       g=(_I, "cross"), h=(_P, "bias"), i=(_F, "mul"))
 
 
 class _QkNorm(ctypes.Structure):
@@ -219,12 +229,15 @@ def _ptr(t: Optional[torch.Tensor]) -> int:
 
 # --------------------------------------------------------------------------------------------------------------- attention
 def causal_attention(q, k, v, out, heads: int, kv_heads: int, dk: int, dv: int, scale: float, window: Optional[int], batch: RowBatch,
-                     gate: Optional[torch.Tensor] = None, talk: Optional[torch.Tensor] = None, score_bound: Optional[float] = None):
+                     gate: Optional[torch.Tensor] = None, talk: Optional[torch.Tensor] = None, score_bound: Optional[float] = None,
+                     sigmoid: Optional[torch.Tensor] = None, mul: float = 1.0):
     """Prompts: ``out [rows, heads * dv] = softmax(q . k * scale) v`` (times ``sigmoid(gate)``), ``q [rows, heads * dk]``; ``k``, ``v``
     ``[key rows, kv_heads * d]`` in the order of ``batch.key_sources`` (the rows themselves when no request goes on from a cache).
-    ``talk [heads, heads]`` (fp32): head h mixes its values with ``sum_g talk[h, g] softmax_g``; ``score_bound``: no |score| is larger."""
+    ``talk [heads, heads]`` (fp32): head h mixes its values with ``sum_g talk[h, g] softmax_g``; ``score_bound``: no |score| is larger.
+    ``sigmoid [heads]`` (fp32): weights ``sigmoid(q . k * scale + sigmoid[h])`` instead of the softmax, and the output times ``mul``."""
+    assert sigmoid is not None or mul == 1.0
     if not q.is_cuda:
-        return RP.causal_attention(q, k, v, out, heads, kv_heads, dk, dv, scale, window, batch, gate, talk)
+        return RP.causal_attention(q, k, v, out, heads, kv_heads, dk, dv, scale, window, batch, gate, talk, sigmoid, mul)
     from . import cuda as K
     from . import gemm
     _no_grad(q, k, v, gate)
@@ -236,7 +249,8 @@ def causal_attention(q, k, v, out, heads: int, kv_heads: int, dk: int, dv: int, 
     a.H, a.G, a.dk, a.dv, a.window, a.scale = heads, kv_heads, dk, dv, window or 0, scale
     a.q_rows, a.k_rows = q.shape[0], k.shape[0]
     dt = K._dt(q)
-    fast = dt == 1 and dk <= 128 and dv <= 128
+    fast = dt == 1 and dk <= 128 and dv <= (128 if sigmoid is None else 256)
+    a.bias, a.mul = _head_bias(sigmoid, heads, gate, talk), mul
     if talk is not None:
         a.bounded = int(score_bound is not None and score_bound <= SCORE_BOUND)
         return _talk_prompt(a, q, out, talk, window, batch, fast)
@@ -282,6 +296,13 @@ def head_mix(x, talk, out, heads: int, kv_heads: int, dv: int):
              "head_mix")
 
 
+def _head_bias(sigmoid: Optional[torch.Tensor], heads: int, gate=None, talk=None) -> int:
+    if sigmoid is None:
+        return 0
+    assert gate is None and talk is None and sigmoid.shape == (heads,) and sigmoid.dtype == torch.float32 and sigmoid.is_contiguous()
+    return sigmoid.data_ptr()
+
+
 def step_splits(requests: int, heads: int, kv_heads: int, dk: int, dv: int, shared: bool, rows: Optional[int], sms: int) -> int:
     """CTAs (1 - 8, one cluster) that share the keys of one (request, 16 heads of a kv head): as many as stay resident together, two
     per SM while their stages of keys fit.  ``rows``: the most keys there can be, where that is known."""
@@ -301,11 +322,12 @@ def _step_bytes(dk: int, dv: int, shared: bool) -> int:
 
 
 def step_attention(q, out, heads: int, kv_heads: int, dk: int, dv: int, scale: float, window: Optional[int], cache: dict, batch: RowBatch,
-                   talk: Optional[torch.Tensor] = None):
-    """One token per request, whose key and value are in the cache already: ``q [n, heads * dk]`` -> ``out [n, heads * dv]``; ``talk`` as
-    in ``causal_attention``."""
+                   talk: Optional[torch.Tensor] = None, sigmoid: Optional[torch.Tensor] = None, mul: float = 1.0):
+    """One token per request, whose key and value are in the cache already: ``q [n, heads * dk]`` -> ``out [n, heads * dv]``; ``talk``,
+    ``sigmoid``, ``mul`` as in ``causal_attention``."""
+    assert sigmoid is not None or mul == 1.0
     if not q.is_cuda:
-        return RP.step_attention(q, out, heads, kv_heads, dk, dv, scale, window, cache, batch, talk)
+        return RP.step_attention(q, out, heads, kv_heads, dk, dv, scale, window, cache, batch, talk, sigmoid, mul)
     from . import cuda as K
     from . import gemm
     _no_grad(q)
@@ -314,6 +336,7 @@ def step_attention(q, out, heads: int, kv_heads: int, dk: int, dv: int, scale: f
     a.q, a.out, a.c, a.pos, a.slots = q.data_ptr(), out.data_ptr(), _cache_args(cache), batch.pos.data_ptr(), batch.slot.data_ptr()
     a.ldq, a.ldo, a.H, a.G, a.dk, a.dv, a.window, a.n, a.scale = q.stride(0), out.stride(0), heads, kv_heads, dk, dv, window or 0, q.shape[0], scale
     dt, shared = K._dt(q), cache["v"].data_ptr() == cache["k"].data_ptr()
+    a.bias, a.mul = _head_bias(sigmoid, heads, None, talk), mul
     if talk is not None:
         return _talk_step(a, q, out, talk, cache)
     if dt == 1 and dk % 16 == 0 and dv % 16 == 0 and max(dk, dv) <= 512 and _step_bytes(dk, dv, shared) < 224 * 1024:
@@ -485,17 +508,21 @@ def latent_up(x, w_uv, gate, heads: int, dv: int) -> torch.Tensor:
     return out
 
 
-def residual_norm(x, y, width: int, post, pre: Optional[torch.Tensor], eps: float, dtype, dest: Optional[torch.Tensor] = None, top: int = 0):
-    """``x += y / rms(y) * post`` on the fp32 stream, in place; returns ``x / rms(x) * pre`` in ``dtype`` (``pre`` ``None``: nothing).
-    With ``top``, token t's y is the sum of rows ``dest[t * top + k]`` (``dest`` ``None``: of rows ``t * top + k``)."""
+def residual_norm(x, y, width: int, post, pre: Optional[torch.Tensor], eps: float, dtype, dest: Optional[torch.Tensor] = None, top: int = 0,
+                  plus: Optional[torch.Tensor] = None, mul: float = 1.0):
+    """``x += mul * y / rms(y) * post`` on the fp32 stream, in place; returns ``x / rms(x) * pre`` in ``dtype`` (``pre`` ``None``: nothing).
+    With ``top``, token t's y is the sum of rows ``dest[t * top + k]`` (``dest`` ``None``: of rows ``t * top + k``); ``plus`` (one row per
+    token, in y's dtype) is added to y."""
     if not x.is_cuda:
-        return RP.residual_norm(x, y, width, post, pre, eps, dtype, dest, top)
+        return RP.residual_norm(x, y, width, post, pre, eps, dtype, dest, top, plus, mul)
     from . import cuda as K
     _no_grad(x, y)
     ld = ctypes.c_longlong
     h = None if pre is None else torch.empty(x.shape, dtype=dtype, device=x.device)
     assert y.shape[1] >= x.shape[1] and y.stride(1) == 1 and (top or y.shape[0] == x.shape[0])
-    K._check(K.lib().lmoe_residual_norm(K._p(x), ld(x.stride(0)), K._p(y), ld(y.stride(0)), K._dt(y), K._p(dest), top, K._p(post), K._p(pre), K._p(h),
+    assert plus is None or (plus.dtype == y.dtype and plus.shape[0] == x.shape[0] and plus.shape[1] >= x.shape[1] and plus.stride(1) == 1)
+    K._check(K.lib().lmoe_residual_norm(K._p(x), ld(x.stride(0)), K._p(y), ld(y.stride(0)), K._dt(y), K._p(dest), top, K._p(plus),
+                                        ld(0 if plus is None else plus.stride(0)), ctypes.c_float(mul), K._p(post), K._p(pre), K._p(h),
                                         ld(0 if h is None else h.stride(0)), x.shape[0], width, x.shape[1], ctypes.c_float(eps),
                                         1 if dtype == torch.bfloat16 else 0, K._st()), "residual_norm")
     return h
@@ -504,10 +531,10 @@ def residual_norm(x, y, width: int, post, pre: Optional[torch.Tensor], eps: floa
 FEW_ROWS = 256                # products of this few rows keep their fp32 result (their cost is reading the weights)
 
 
-def sublayer_out(x, weight) -> torch.Tensor:
-    """The last product of a sublayer, in fp32 for few rows."""
+def sublayer_out(x, weight, dtype=None) -> torch.Tensor:
+    """The last product of a sublayer, in ``dtype``, or in fp32 for few rows."""
     from . import linear, linear_f32
-    return linear_f32(x, weight) if x.shape[0] <= FEW_ROWS else linear(x, weight)
+    return linear_f32(x, weight) if dtype == torch.float32 or (dtype is None and x.shape[0] <= FEW_ROWS) else linear(x, weight)
 
 
 ACTIVATIONS = ("silu", "relu")            # as numbered in csrc/gemm_dense.cu and csrc/sandwich_block.cu
@@ -529,3 +556,18 @@ def glu_in(h, w1, act: str = "silu") -> torch.Tensor:
     out = torch.empty(z.shape[0], ff, dtype=z.dtype, device=z.device)
     K._check(K.lib().lmoe_glu_rows(K._p(z), ld(z.stride(0)), K._p(out), ld(ff), z.shape[0], ff, ACTIVATIONS.index(act), K._dt(z), K._st()), "glu_rows")
     return out
+
+
+def xielu_in(h, w1, act) -> torch.Tensor:
+    """``xielu(h W1^T)``: ``a0 z^2 + z / 2`` for positive z, else ``a1 (e^z - 1 - z) + z / 2``, with ``act = (a0, a1)`` (fp32)."""
+    from . import linear
+    if not h.is_cuda:
+        return RP.xielu(linear(h, w1).float(), act).to(h.dtype)
+    from . import cuda as K
+    from . import gemm
+    _no_grad(h, w1)
+    if h.shape[0] > 16 and gemm.dense_ok(h, w1) and w1.shape[0] % 8 == 0:
+        return gemm.dense_xielu(h, w1, act)
+    z, ld = linear(h, w1), ctypes.c_longlong
+    K._check(K.lib().lmoe_xielu_rows(K._p(z), ld(z.stride(0)), z.shape[0], z.shape[1], K._p(act), K._dt(z), K._st()), "xielu_rows")
+    return z

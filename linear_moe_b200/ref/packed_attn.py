@@ -27,35 +27,38 @@ def store(cache: dict, name: str, slot: int, positions: torch.Tensor, rows: torc
     buf.view(-1, *buf.shape[2:])[_places(cache, slot, positions)] = rows.to(buf.dtype)
 
 
-def mix(q, k, v, scale: float, first_query: int, window: Optional[int], talk=None):
+def mix(q, k, v, scale: float, first_query: int, window: Optional[int], talk=None, sigmoid=None, mul: float = 1.0):
     """``q [n, H, d]`` at key indices ``first_query ..``, ``k [m, G, d]``, ``v [m, G, e]`` -> ``[n, H, e]`` (fp32).  ``talk [H, H]`` mixes
-    the heads' weights."""
+    the heads' weights; ``sigmoid [H]``: sigmoid weights with that bias."""
     n, H, G = q.shape[0], q.shape[1], k.shape[1]
     i, j = torch.arange(first_query, first_query + n)[:, None], torch.arange(k.shape[0])[None, :]
     hidden = j > i if window is None else (j > i) | (j <= i - window)
     s = torch.einsum("ihd,jhd->hij", q.float(), k.float().repeat_interleave(H // G, 1)) * scale
-    w = s.masked_fill(hidden, float("-inf")).softmax(-1)
+    if sigmoid is not None:
+        w = torch.sigmoid(s + sigmoid[:, None, None]).masked_fill(hidden, 0.0) * mul
+    else:
+        w = s.masked_fill(hidden, float("-inf")).softmax(-1)
     if talk is not None:
         w = torch.einsum("hg,gij->hij", talk.float(), w)
     return torch.einsum("hij,jhd->ihd", w, v.float().repeat_interleave(H // G, 1))
 
 
-def causal_attention(q, k, v, out, H, G, dk, dv, scale, window, batch, gate, talk=None):
+def causal_attention(q, k, v, out, H, G, dk, dv, scale, window, batch, gate, talk=None, sigmoid=None, mul=1.0):
     krow = 0
     for r, (past, n) in enumerate(zip(batch.past(window), batch.counts)):
         a, b = batch.row0[r], batch.row0[r + 1]
         ks = slice(krow, krow + past + n)
-        o = mix(q[a:b].reshape(n, H, dk), k[ks].reshape(-1, G, dk), v[ks].reshape(-1, G, dv), scale, past, window, talk).reshape(n, H * dv)
+        o = mix(q[a:b].reshape(n, H, dk), k[ks].reshape(-1, G, dk), v[ks].reshape(-1, G, dv), scale, past, window, talk, sigmoid, mul).reshape(n, H * dv)
         out[a:b] = (o if gate is None else o * torch.sigmoid(gate[a:b].float())).to(out.dtype)
         krow += past + n
 
 
-def step_attention(q, out, H, G, dk, dv, scale, window, cache, batch, talk=None):
+def step_attention(q, out, H, G, dk, dv, scale, window, cache, batch, talk=None, sigmoid=None, mul=1.0):
     for r, (p, slot) in enumerate(zip(batch.pos.tolist(), batch.slot.tolist())):
         span = window if "table" in cache else cache["k"].shape[1]
         at = torch.arange(0 if span is None else max(0, p + 1 - span), p + 1)
         k, v = cache_rows(cache, "k", slot, at), cache_rows(cache, "v", slot, at)
-        out[r] = mix(q[r:r + 1].reshape(1, H, dk), k, v, scale, len(at) - 1, None, talk).reshape(-1).to(out.dtype)
+        out[r] = mix(q[r:r + 1].reshape(1, H, dk), k, v, scale, len(at) - 1, None, talk, sigmoid, mul).reshape(-1).to(out.dtype)
 
 
 def rotate_pairs(x, pos, freq):
@@ -113,7 +116,8 @@ def rotate_heads_(z, at_q, at_k, heads, kv_heads, dk, halves, turn):
 def head_norm_rope_(z, lay, s, wq, wk, turn, eps, batch, cache, first, mix):
     for at, n, w in ((lay.q, s.heads, wq), (lay.k, s.kv_heads, wk)):
         x = z[:, at:at + n * s.dk].float().reshape(-1, n, s.dk)
-        x = x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) / s.dim + eps) * w
+        if w is not None:
+            x = x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) / s.dim + eps) * w
         z[:, at:at + n * s.dk] = turned(x, s.rot_halves, turn).reshape(-1, n * s.dk).to(z.dtype)
     at = slice(lay.v, lay.v + s.kv_heads * s.dv)
     v = z[:, at].float().reshape(-1, s.kv_heads, s.dv)
@@ -122,7 +126,8 @@ def head_norm_rope_(z, lay, s, wq, wk, turn, eps, batch, cache, first, mix):
     v = v.reshape(-1, s.kv_heads * s.dv)
     if first is not None:
         v = (1 - mix) * v + mix * first.float()
-    z[:, at] = v.to(z.dtype)
+    if s.value_norm or first is not None:
+        z[:, at] = v.to(z.dtype)
     _store_rows(z, lay, s.kv_heads, s.dk, s.dv, batch, cache)
 
 
@@ -140,24 +145,39 @@ def gather_rows(dst, src, name, cache, meta):
         dst[d] = src[s] if s >= 0 else cache_rows(cache, name, slot, torch.tensor([pos]))[0].reshape(-1)
 
 
-def residual_norm(x, y, width, post, pre, eps, dtype, dest, top):
+def residual_norm(x, y, width, post, pre, eps, dtype, dest, top, plus=None, mul=1.0):
     if top:
         y = y.float()[torch.arange(x.shape[0] * top) if dest is None else dest.long()].reshape(x.shape[0], top, -1).sum(1)
     y = y[:, :x.shape[1]].float()
-    x.add_(y * torch.rsqrt(y.pow(2).sum(-1, keepdim=True) / width + eps) * post)
+    if plus is not None:
+        y = y + plus[:, :x.shape[1]].float()
+    x.add_(y * (mul * torch.rsqrt(y.pow(2).sum(-1, keepdim=True) / width + eps)) * post)
     return None if pre is None else (x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) / width + eps) * pre).to(dtype)
 
 
-def route(logits, top):
-    z, idx = torch.topk(logits, top, -1)
-    return torch.sigmoid(z), idx
+def xielu(z, act):
+    """``softplus(p) z^2 + z / 2`` for positive z, else ``(1/2 + softplus(q)) (e^z - 1 - z) + z / 2``; ``act = (softplus(p), 1/2 + softplus(q))``."""
+    return torch.where(z > 0, act[0] * z * z, act[1] * (torch.expm1(z.clamp(max=0)) - z)) + z / 2
 
 
-def experts_relu2(h, logits, up, down, top):
-    """Rows ``[n * top, width]``: expert(weight * h) of every (token, expert)."""
-    w, idx = route(logits, top)
-    y = torch.zeros(h.shape[0] * top, down.shape[1])
+def route(logits, spec):
+    z, idx = torch.topk(logits, spec.top, -1)
+    w = torch.sigmoid(z) if spec.scores == "sigmoid" else torch.softmax(logits, -1).gather(-1, idx)
+    if spec.normalise:
+        w = w / (w.sum(-1, keepdim=True) + 1e-20)
+    return w * spec.scale, idx
+
+
+def experts_rows(h, logits, up, down, spec):
+    """Rows ``[n * top, width]``: every (token, expert)'s output times its weight."""
+    w, idx = route(logits, spec)
+    y = torch.zeros(h.shape[0] * spec.top, down.shape[1])
     for p, (wt, e) in enumerate(zip(w.flatten().tolist(), idx.flatten().tolist())):
-        a = (wt * torch.relu(up[e].float() @ h[p // top].float())).pow(2).to(h.dtype)
-        y[p] = down[e].float() @ a.float()
+        z = up[e].float() @ h[p // spec.top].float()
+        if spec.act == "relu2":
+            a = (wt * torch.relu(z)).pow(2)
+        else:
+            gate, value = z.chunk(2)
+            a = wt * torch.nn.functional.silu(gate) * value
+        y[p] = down[e].float() @ a.to(h.dtype).float()
     return y

@@ -17,7 +17,7 @@ from linear_moe_b200.infer.kv_cache import PAGE, LayerPages, LayerRows, SlotCach
 from linear_moe_b200.infer.session import InferenceSession
 from linear_moe_b200.models.registry import load_model
 from linear_moe_b200.ops import packed_attn as PA
-from linear_moe_b200.ops.moe_rows import ExpertsSpec, experts_relu2
+from linear_moe_b200.ops.moe_rows import ExpertsSpec, experts_rows
 from linear_moe_b200.ops.row_batch import RowBatch, round_up
 from serving_utils import GPU, ROOT, folder, padded, prompt, rel, tol, where
 
@@ -204,7 +204,7 @@ def test_experts(where, experts, top, ff, width, rows):
         logits[:, 1] = -9.0
     wide = torch.full((rows, round_up(experts, 8)), 99.0)
     wide[:, :experts] = logits
-    y, dest = experts_relu2(h.to(dev), wide.to(dev), up.to(dev), down.to(dev), ExpertsSpec(experts, top, ff))
+    y, dest = experts_rows(h.to(dev), wide.to(dev), up.to(dev), down.to(dev), ExpertsSpec(experts, top, ff))
     y = y.double().cpu()
     got = (y[:rows * top] if dest is None else y[dest.long().cpu()]).reshape(rows, top, width).sum(1)
     # an identity in front of the definition's router: its logits are the given ones
