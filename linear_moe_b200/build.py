@@ -23,13 +23,16 @@ OBJ = os.path.join(ROOT, "build")
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "--use_fast_math",
               "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden"]
 # sources whose fp32 instantiations serve models in true 32-bit: IEEE division and the accurate exp / tanh
-PRECISE = {"chunk_attn.cu", "parallel_block.cu", "packed_attn.cu", "sandwich_block.cu", "moe_rows.cu", "post_norm.cu", "retention.cu"}
+PRECISE = {"chunk_attn.cu", "parallel_block.cu", "packed_attn.cu", "sandwich_block.cu", "moe_rows.cu", "post_norm.cu", "retention.cu", "ssd.cu",
+           "delta_rule.cu"}
 # what serving a model of the listed kind needs (``build_serving``); everything else is training, communication and fp8
 SERVING = {"parallel_block": ("chunk_attn.cu", "chunk_attn_step.cu", "chunk_attn_tc.cu", "parallel_block.cu", "gemm_dense.cu", "gemm_skinny.cu"),
            "sandwich_block": ("packed_attn.cu", "packed_attn_step.cu", "packed_attn_tc.cu", "latent_step.cu", "moe_rows.cu", "sandwich_block.cu",
                               "parallel_block.cu", "gemm_dense.cu", "gemm_grouped.cu", "gemm_skinny.cu"),
            "post_norm_block": ("packed_attn.cu", "packed_attn_tc.cu", "talk_step.cu", "retention.cu", "retention_tc.cu", "post_norm.cu", "sandwich_block.cu",
-                               "parallel_block.cu", "gemm_dense.cu", "gemm_skinny.cu")}
+                               "parallel_block.cu", "gemm_dense.cu", "gemm_skinny.cu"),
+           "zelinex": ("packed_attn.cu", "packed_attn_step.cu", "packed_attn_tc.cu", "ssd.cu", "delta_rule.cu", "moe_rows.cu",
+                       "sandwich_block.cu", "parallel_block.cu", "gemm_dense.cu", "gemm_grouped.cu", "gemm_skinny.cu")}
 
 
 def _nvcc() -> str:

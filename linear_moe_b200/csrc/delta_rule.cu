@@ -1,0 +1,294 @@
+// Generalized delta rule over packed rows, head by head in fp32,
+//     S <- diag(w) S - (a u)(u^T S) + k v^T,    o = S^T r,    out = o / rms(o) * weight * sigmoid(gate)
+// with the unit key u, decays w = exp(-DECAY sigmoid(W2 tanh(.) + w0)) and rates a = sigmoid(. + bias) per channel:
+//   delta_low_kernel    prompts: tanh of the decay's inner activations (the second projection is a matrix product)
+//   delta_rows_kernel   prompts of any size, bf16 or fp32, token by token (bf16 fast path: delta_rule_tc.cu), and
+//   delta_norm_kernel   the norm and gate behind it
+//   delta_step_kernel   one token per request, everything in one pass over the state
+// With the old state S, p = S^T u and q = S^T (w r), the output is o = q - (r . a u) p + (r . k) v: one reduction over the rows of S.
+// Compiled without fast-math: the fp32 instantiations serve models in true 32-bit.
+#include "common.cuh"
+#include "delta_rule.cuh"
+
+namespace lmoe {
+namespace dlt {
+
+__device__ __forceinline__ float sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
+
+template <typename T>
+__global__ void __launch_bounds__(256) delta_low_kernel(Args a) {
+    pdl_trigger();
+    const long long total = (long long)a.rows * (a.rank / 4);
+    for (long long i = blockIdx.x * 256LL + threadIdx.x; i < total; i += gridDim.x * 256LL) {
+        const long long row = i / (a.rank / 4);
+        const int c = (int)(i - row * (a.rank / 4)) * 4;
+        const float4 x = load4((const T*)a.z + row * a.ldz + a.zw + c);
+        store4((T*)a.low + row * a.ldl + c, make_float4(tanhf(x.x), tanhf(x.y), tanhf(x.z), tanhf(x.w)));
+    }
+}
+
+// ------------------------------------------------------------------------------------------------------------------ prompts
+constexpr int RT = 256, COLS = 64, TOK = 16, LD = COLS + 8;
+
+// grid (requests, H, column slices of 64).  Thread 4 j + r owns rows r mod 4 of column j of the state, which lies in shared memory.
+template <typename T>
+__global__ void __launch_bounds__(RT) delta_rows_kernel(Args a) {
+    extern __shared__ float sm[];
+    const int d = a.d;
+    float* S = sm;                       // [d][COLS + 8]
+    float* R = S + d * LD;               // [TOK][d] each
+    float* K = R + TOK * d;
+    float* U = K + TOK * d;
+    float* A = U + TOK * d;              // a u
+    float* W = A + TOK * d;
+    float* V = W + TOK * d;              // [TOK][COLS]
+    const int h = blockIdx.y, c0 = blockIdx.z * COLS, nc = min(COLS, d - c0);
+    int row0 = blockIdx.x, n = 1, slot, flags;
+    if (a.groups != nullptr) {
+        const int* g = a.groups + blockIdx.x * rt::G_INTS;
+        row0 = g[rt::G_ROW], n = g[rt::G_N], slot = g[rt::G_SLOT], flags = g[rt::G_FLAGS];
+    } else {                             // one token per request, positions only known here
+        slot = a.slots[row0], flags = a.pos[row0] > 0 ? 7 : 3;
+    }
+    float* state = a.state == nullptr ? nullptr : a.state + ((long long)slot * a.H + h) * d * d;
+    for (int i = threadIdx.x; i < d * COLS; i += RT) {
+        const int r = i / COLS, c = i % COLS;
+        S[r * LD + c] = (flags & 4) && state != nullptr && c < nc ? state[(long long)r * d + c0 + c] : 0.f;
+    }
+    const int j = threadIdx.x >> 2, part = threadIdx.x & 3, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int t0 = 0; t0 < n; t0 += TOK) {
+        const int nt = min(TOK, n - t0);
+        __syncthreads();
+        for (int t = warp; t < nt; t += RT / 32) {           // a warp prepares a token
+            const long long row = row0 + t0 + t;
+            const T* z = (const T*)a.z + row * a.ldz + h * d;
+            float s = 0.f;
+            for (int c = lane; c < d; c += 32) {
+                const float k = to_f(z[a.zk + c]);
+                s += k * k;
+            }
+            const float inv = 1.f / sqrtf(warp_sum(s) + UNIT_EPS);
+            for (int c = lane; c < d; c += 32) {
+                const float k = to_f(z[a.zk + c]), u = k * inv;
+                R[t * d + c] = to_f(z[a.zr + c]);
+                K[t * d + c] = k;
+                U[t * d + c] = u;
+                A[t * d + c] = u * sigmoid(to_f(z[a.za + c]) + a.a_bias[h * d + c]);
+                W[t * d + c] = expf(-DECAY * sigmoid(a.w[row * a.ldw + h * d + c] + a.w0[h * d + c]));
+            }
+        }
+        for (int i = threadIdx.x; i < nt * COLS; i += RT)
+            V[i] = i % COLS < nc ? to_f(((const T*)a.z)[(long long)(row0 + t0 + i / COLS) * a.ldz + a.zv + h * d + c0 + i % COLS]) : 0.f;
+        __syncthreads();
+        for (int t = 0; t < nt; ++t) {
+            const float v = V[t * COLS + j];
+            float p = 0.f, o = 0.f;
+            for (int r = part; r < d; r += 4) p += U[t * d + r] * S[r * LD + j];
+            p += __shfl_xor_sync(0xffffffffu, p, 1);
+            p += __shfl_xor_sync(0xffffffffu, p, 2);
+            for (int r = part; r < d; r += 4) {
+                const float s = W[t * d + r] * S[r * LD + j] - A[t * d + r] * p + K[t * d + r] * v;
+                S[r * LD + j] = s;
+                o += R[t * d + r] * s;
+            }
+            o += __shfl_xor_sync(0xffffffffu, o, 1);
+            o += __shfl_xor_sync(0xffffffffu, o, 2);
+            if (part == 0 && j < nc) a.raw[((long long)(row0 + t0 + t) * a.H + h) * d + c0 + j] = o;
+        }
+    }
+    __syncthreads();
+    if (state != nullptr)
+        for (int i = threadIdx.x; i < d * nc; i += RT) state[(long long)(i / nc) * d + c0 + i % nc] = S[i / nc * LD + i % nc];
+}
+
+// one warp per (row, head)
+template <typename T>
+__global__ void __launch_bounds__(256) delta_norm_kernel(Args a) {
+    const long long i = blockIdx.x * 8LL + (threadIdx.x >> 5);
+    const int lane = threadIdx.x & 31, h = (int)(i % a.H);
+    const long long row = i / a.H;
+    if (row >= a.rows) return;
+    const float* o = a.raw + (row * a.H + h) * a.d;
+    float s = 0.f;
+    for (int c = lane; c < a.d; c += 32) s += o[c] * o[c];
+    const float r = 1.f / sqrtf(warp_sum(s) / a.nd + a.eps);
+    const T* g = (const T*)a.z + row * a.ldz + a.zg + h * a.d;
+    for (int c = lane; c < a.d; c += 32) ((T*)a.out)[row * a.ldo + h * a.d + c] = from_f<T>(o[c] * r * a.norm[h * a.d + c] * sigmoid(to_f(g[c])));
+}
+
+template <typename T>
+static int launch_rows(const Args& a, cudaStream_t st) {
+    const size_t smem = sizeof(float) * ((size_t)a.d * LD + 5 * TOK * a.d + TOK * COLS);
+    if (smem > 227 * 1024) return -2;
+    cudaError_t e = cudaFuncSetAttribute(delta_rows_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    delta_rows_kernel<T><<<dim3(a.n, a.H, (a.d + COLS - 1) / COLS), RT, smem, st>>>(a);
+    if ((e = cudaGetLastError()) != cudaSuccess) return (int)e;
+    delta_norm_kernel<T><<<(unsigned)(((long long)a.rows * a.H + 7) / 8), 256, 0, st>>>(a);
+    return (int)cudaGetLastError();
+}
+
+// ---------------------------------------------------------------------------------------------------------------- one token
+constexpr int ST = 512, NW = ST / 32;
+
+// grid (H, n).  A thread owns 4 columns of the state and every `parts`-th row (parts = ST / (d / 4)); the first NB of them stay in registers
+// between the reduction and the update.  staged: the head's rows of w2 lie in shared memory.
+template <typename T>
+__global__ void __launch_bounds__(ST) delta_step_kernel(Args a, int staged) {
+    constexpr int NB = 8;
+    extern __shared__ float4 sm4[];
+    const int h = blockIdx.x, b = blockIdx.y, d = a.d, rank = a.rank;
+    const int cols = d / 4, parts = ST / cols, c = threadIdx.x % cols * 4, r0 = threadIdx.x / cols;
+    float* P = reinterpret_cast<float*>(sm4);                // [parts][d] partial p, then
+    float* Q = P + parts * d;                                // [parts][d] partial q
+    float* R = Q + parts * d;                                // [d]
+    float* K = R + d;
+    float* U = K + d;
+    float* A = U + d;                                        // a u
+    float* W = A + d;
+    float* L = W + d;                                        // [rank]
+    T* W2 = reinterpret_cast<T*>(L + rank);                  // [d][rank]
+    __shared__ float red[32];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const bool on = r0 < parts;
+    // the state is older than the kernel before this one, and weights do not change
+    const bool fresh = a.pos[b] == 0;
+    float* S = a.state + ((long long)a.slots[b] * a.H + h) * d * d;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 s[NB];
+#pragma unroll
+    for (int i = 0; i < NB; ++i) {
+        const int r = r0 + i * parts;
+        s[i] = on && r < d && !fresh ? *reinterpret_cast<const float4*>(S + (long long)r * d + c) : zero;
+    }
+    const T* w2 = (const T*)a.w2 + (long long)h * d * rank;
+    if (staged)
+        for (int i = threadIdx.x * 4; i < d * rank; i += ST * 4) store4(W2 + i, load4(w2 + i));
+    pdl_trigger();
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    const T* z = (const T*)a.z + (long long)b * a.ldz + h * d;
+    float ks = 0.f;
+    for (int i = threadIdx.x; i < d; i += ST) {
+        const float k = to_f(z[a.zk + i]);
+        R[i] = to_f(z[a.zr + i]);
+        K[i] = k;
+        A[i] = sigmoid(to_f(z[a.za + i]) + a.a_bias[h * d + i]);
+        ks += k * k;
+    }
+    for (int i = threadIdx.x; i < rank; i += ST) L[i] = tanhf(to_f(((const T*)a.z + (long long)b * a.ldz + a.zw)[i]));
+    const float inv = 1.f / sqrtf(block_sum(ks, red) + UNIT_EPS);        // (its barriers also cover R, K, A and L)
+    const T* rows = staged ? W2 : w2;
+    for (int i = warp; i < d; i += NW) {
+        float x = 0.f;
+        for (int k = lane; k < rank; k += 32) x += L[k] * to_f(rows[(long long)i * rank + k]);
+        x = warp_sum(x);
+        if (lane == 0) {
+            W[i] = expf(-DECAY * sigmoid(x + a.w0[h * d + i]));
+            U[i] = K[i] * inv;
+            A[i] *= K[i] * inv;
+        }
+    }
+    __syncthreads();
+    float4 p = zero, q = zero;
+    auto gather = [&](float4 x, int r) {
+        const float u = U[r], f = W[r] * R[r];
+        p.x += u * x.x; p.y += u * x.y; p.z += u * x.z; p.w += u * x.w;
+        q.x += f * x.x; q.y += f * x.y; q.z += f * x.z; q.w += f * x.w;
+    };
+    if (on) {
+#pragma unroll
+        for (int i = 0; i < NB; ++i)
+            if (r0 + i * parts < d) gather(s[i], r0 + i * parts);
+        if (!fresh)
+            for (int r = r0 + NB * parts; r < d; r += parts) gather(*reinterpret_cast<const float4*>(S + (long long)r * d + c), r);
+        *reinterpret_cast<float4*>(P + r0 * d + c) = p;
+        *reinterpret_cast<float4*>(Q + r0 * d + c) = q;
+    }
+    float ra = 0.f, rk = 0.f;                                // r . a u, r . k
+    for (int i = threadIdx.x; i < d; i += ST) ra += R[i] * A[i], rk += R[i] * K[i];
+    ra = block_sum(ra, red);
+    rk = block_sum(rk, red);                                 // (the barriers also cover P and Q)
+    float y = 0.f;                                           // d <= ST: a thread finishes one column
+    if (threadIdx.x < d) {
+        float ps = 0.f, qs = 0.f;
+        for (int r = 0; r < parts; ++r) ps += P[r * d + threadIdx.x], qs += Q[r * d + threadIdx.x];
+        y = qs - ra * ps + rk * to_f(z[a.zv + threadIdx.x]);
+        Q[threadIdx.x] = ps;                                 // nobody else reads this column's partial q
+    }
+    const float rms = 1.f / sqrtf(block_sum(y * y, red) / a.nd + a.eps);
+    if (threadIdx.x < d) {
+        const int i = h * d + threadIdx.x;
+        ((T*)a.out)[(long long)b * a.ldo + i] = from_f<T>(y * rms * a.norm[i] * sigmoid(to_f(z[a.zg + threadIdx.x])));
+    }
+    if (!on) return;
+    p = *reinterpret_cast<const float4*>(Q + c);
+    const float4 v = load4(z + a.zv + c);
+    auto update = [&](float4 x, int r) {
+        const float w = W[r], m = A[r], k = K[r];
+        x = make_float4(w * x.x - m * p.x + k * v.x, w * x.y - m * p.y + k * v.y, w * x.z - m * p.z + k * v.z, w * x.w - m * p.w + k * v.w);
+        *reinterpret_cast<float4*>(S + (long long)r * d + c) = x;
+    };
+#pragma unroll
+    for (int i = 0; i < NB; ++i)
+        if (r0 + i * parts < d) update(s[i], r0 + i * parts);
+    for (int r = r0 + NB * parts; r < d; r += parts) update(fresh ? zero : *reinterpret_cast<const float4*>(S + (long long)r * d + c), r);
+}
+
+template <typename T>
+static int launch_step(const Args& a, cudaStream_t st) {
+    const size_t base = sizeof(float) * (2 * (ST / (a.d / 4)) * a.d + 5 * a.d + a.rank), table = sizeof(T) * (size_t)a.d * a.rank;
+    const int staged = base + table <= 100 * 1024;
+    const size_t smem = base + (staged ? table : 0);
+    if (smem > 200 * 1024) return -2;
+    cudaError_t e = cudaFuncSetAttribute(delta_step_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(a.H, a.n);
+    cfg.blockDim = dim3(ST);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = st;
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = 1;
+    return (int)cudaLaunchKernelEx(&cfg, delta_step_kernel<T>, a, staged);
+}
+
+static bool aligned(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
+static bool ok(const Args& a, int dt) {
+    const int w = dt ? 8 : 4;
+    return a.rows > 0 && a.H > 0 && a.d > 0 && a.d % 16 == 0 && a.nd > 0 && a.nd <= a.d && a.rank > 0 && a.rank % 32 == 0 && a.ldz % w == 0 && a.ldo % w == 0 &&
+           ((a.zr | a.zk | a.zv | a.za | a.zg | a.zw) & 7) == 0 && aligned(a.z) && aligned(a.out) && aligned(a.state) && aligned(a.w2);
+}
+
+}  // namespace dlt
+}  // namespace lmoe
+
+using namespace lmoe;
+
+// z -> low; dt: 1 bf16, 0 fp32
+LMOE_API int lmoe_delta_low(const dlt::Args* ap, int dt, cudaStream_t st) {
+    const dlt::Args& a = *ap;
+    if (!dlt::ok(a, dt) || a.low == nullptr || a.ldl % 4) return -1;
+    const long long blocks = ((long long)a.rows * (a.rank / 4) + 255) / 256;
+    const unsigned grid = (unsigned)(blocks < 148 * 16 ? blocks : 148 * 16);
+    if (dt) dlt::delta_low_kernel<bf16><<<grid, 256, 0, st>>>(a);
+    else dlt::delta_low_kernel<float><<<grid, 256, 0, st>>>(a);
+    return (int)cudaGetLastError();
+}
+
+// Groups that are whole requests (flags 3 or 7), or (a.groups null) one token per request; a.w, a.raw
+LMOE_API int lmoe_delta_rows(const dlt::Args* ap, int dt, cudaStream_t st) {
+    const dlt::Args& a = *ap;
+    if (!dlt::ok(a, dt) || a.n <= 0 || a.raw == nullptr || a.w == nullptr) return -1;
+    return dt ? dlt::launch_rows<bf16>(a, st) : dlt::launch_rows<float>(a, st);
+}
+
+// One token per request, state in place: a.state, d <= 256; rows with position 0 start from zero.  Slots and positions must have been on the
+// device before the kernel that precedes this one in the stream was launched.
+LMOE_API int lmoe_delta_step(const dlt::Args* ap, int dt, cudaStream_t st) {
+    const dlt::Args& a = *ap;
+    if (!dlt::ok(a, dt) || a.n != a.rows || a.d > 256 || a.state == nullptr || a.w2 == nullptr) return -1;
+    return dt ? dlt::launch_step<bf16>(a, st) : dlt::launch_step<float>(a, st);
+}

@@ -51,6 +51,7 @@ struct Params {
     int* err;
     const bf16* bias;  // out mode 0 without epilogue function: [N] added to every row, or null
     int relu = 0;      // epi 1: relu(gate) * up instead of silu(gate) * up
+    const float* act = nullptr;       // epi 3: {a0, a1} of xielu
 };
 
 __device__ __forceinline__ void tma_store_2d(const CUtensorMap* map, const void* src, int c0, int c1) {
@@ -88,6 +89,15 @@ __device__ __forceinline__ void add_bias32(uint32_t (&v)[32], const bf16* bias, 
                 v[g * 8 + 2 * i + 1] = __float_as_uint(__uint_as_float(v[g * 8 + 2 * i + 1]) + f.y);
             }
         }
+    }
+}
+
+// a0 z^2 + z / 2 for positive z, else a1 (e^z - 1 - z) + z / 2
+__device__ __forceinline__ void xielu32(uint32_t (&v)[32], float a0, float a1) {
+#pragma unroll
+    for (int i = 0; i < 32; ++i) {
+        const float z = __uint_as_float(v[i]);
+        v[i] = __float_as_uint((z > 0.f ? a0 * z * z : a1 * (__expf(fminf(z, 0.f)) - 1.f - z)) + 0.5f * z);
     }
 }
 
@@ -328,6 +338,7 @@ gemm_dense_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant
                 }
             } else if (OUT == 0) {
                 const int col_base = tn * 256;
+                const float act0 = EPI == 3 ? p.act[0] : 0.f, act1 = EPI == 3 ? p.act[1] : 0.f;
 #pragma unroll 1
                 for (int c = 0; c < 256; c += 64) {
                     uint32_t v0[32], v1[32];
@@ -340,6 +351,10 @@ gemm_dense_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant
                     if (p.bias != nullptr) {
                         add_bias32(v0, p.bias + col_base + c, p.N - (col_base + c));
                         add_bias32(v1, p.bias + col_base + c + 32, p.N - (col_base + c + 32));
+                    }
+                    if (EPI == 3) {
+                        xielu32(v0, act0, act1);
+                        xielu32(v1, act0, act1);
                     }
                     stage_bf16(s, lane, 0, v0); stage_bf16(s, lane, 1, v1);
                     fence_async_smem();
@@ -468,6 +483,22 @@ LMOE_API int lmoe_gemm_dense(const void* A, int lda, int a_mn, const void* B, in
 LMOE_API int lmoe_gemm_dense_bias(const void* A, int lda, int a_mn, const void* B, int ldb, int b_mn, void* C, int ldc,
                                   const void* bias, int M, int N, int K, int band, int* err, int num_sms, cudaStream_t st) {
     return gemm_dense_impl(A, lda, a_mn, B, ldb, b_mn, C, ldc, 0, M, N, K, band, err, num_sms, st, bias);
+}
+
+// C[M,N] (bf16) = xielu(X[M,K] W[N,K]^T), act = {a0, a1} in device memory.
+LMOE_API int lmoe_gemm_dense_xielu(const void* X, int ldx, const void* W, int ldw, void* C, int ldc, int M, int N, int K, int band, const float* act,
+                                   int* err, int num_sms, cudaStream_t st) {
+    if (M <= 0 || N <= 0 || K <= 0 || act == nullptr) return -1;
+    if (ldx % 8 || ldw % 8 || K % 8 || ldc % 8 || N % 8) return -1;
+    if (((uintptr_t)X | (uintptr_t)W | (uintptr_t)C) & 15) return -2;
+    CUtensorMap ma, mb, mc;
+    int rc = make_map(&ma, X, (uint64_t)M, (uint64_t)K, (uint64_t)ldx, 128);
+    if (rc == 0) rc = make_map(&mb, W, (uint64_t)N, (uint64_t)K, (uint64_t)ldw, 128);
+    if (rc == 0) rc = make_map_any(&mc, C, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, M, N, ldc, 64, 32);
+    if (rc) return rc;
+    Params p;
+    p.M = M; p.N = N; p.K = K; p.band = band > 0 ? band : 8; p.f_half = 0; p.err = err; p.bias = nullptr; p.act = act;
+    return launch<false, false, 0, 3>(ma, mb, mc, mc, 0, p, num_sms, st);
 }
 
 // act[M,F] = silu(x Wg^T) * (x Wu^T) (kind 1: relu in place of silu) with W = [Wg ; Wu] of shape [2F, K] (pitch ldw); if Y != null the pre-activations

@@ -1,12 +1,14 @@
-// Mixture of experts over packed rows, for serving: sigmoid scores, the `top` largest are a token's experts and its weights as they
-// are; the weight multiplies the expert's input, and the expert is W_down relu(W_up h)^2.  Because a weight is positive,
-//     relu(W_up (w h))^2 = (w relu(W_up h))^2
+// Mixture of experts over packed rows, for serving.  Scores are the sigmoid of the router logits or their softmax over all experts; the
+// `top` largest are a token's experts, and its weights as they are or divided by their sum, times a factor.  Two kinds of experts:
+//     squared ReLU   W_down relu(W_up (w h))^2 = W_down (w relu(W_up h))^2, because a weight is positive
+//     gated          w W_down (silu(W_gate h) * (W_up h)) = W_down (w silu(W_gate h) * (W_up h))
 // so the weight is applied in fp32 where the activation is formed and the rows themselves are never scaled.
 //   route_rows_kernel     router logits -> experts and weights of every token (and the number of pairs per expert)
 //   place_offsets_kernel  pairs per expert -> padded segments of the expert-sorted rows
 //   place_rows_kernel     every (token, expert) pair gets a row of its expert's segment; its input row and weight go there
 //   moe_rows_kernel       per-expert products over the sorted rows, any size, bf16 or fp32, fp32 arithmetic (the bf16 products of a
 //                         prompt run on gemm_grouped.cu with the same activation in its epilogue)
+//   moe_glu_kernel        the gated activation of the sorted rows
 //   moe_step_kernel       the same products for few tokens (bf16): no sorting, every CTA finds its expert's pairs itself and streams 16
 //                         rows of that expert's matrix through mma.sync fragments (as gemm_skinny.cu)
 // Compiled without fast-math.
@@ -20,14 +22,22 @@ namespace mr {
 constexpr int RT = 128;
 
 // one warp per token; counts (null: not wanted) must be zero
-__global__ void __launch_bounds__(RT) route_rows_kernel(const float* __restrict__ logits, long long ldl, int n, int E, int top,
+__global__ void __launch_bounds__(RT) route_rows_kernel(const float* __restrict__ logits, long long ldl, int n, int E, int top, int softmax, int normalise, float scale,
                                                         int* __restrict__ idx, float* __restrict__ weight, int* counts) {
     pdl_trigger();
     const int t = blockIdx.x * (RT / 32) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (t >= n) return;
     const float* z = logits + (long long)t * ldl;
-    float last = INFINITY;                                   // the previous choice; the sigmoid keeps the order of the logits
+    float last = INFINITY;                                   // the previous choice; sigmoid and softmax keep the order of the logits
     int last_e = -1;
+    float zmax = 0.f, inv = 0.f, chosen = 0.f;               // softmax: largest logit, 1 / sum; sum of the chosen scores
+    if (softmax) {
+        zmax = -INFINITY;
+        for (int e = lane; e < E; e += 32) zmax = fmaxf(zmax, z[e]);
+        zmax = warp_max(zmax);
+        for (int e = lane; e < E; e += 32) inv += expf(z[e] - zmax);
+        inv = 1.f / warp_sum(inv);
+    }
     for (int k = 0; k < top; ++k) {
         float best = -INFINITY;
         int be = E;
@@ -47,10 +57,14 @@ __global__ void __launch_bounds__(RT) route_rows_kernel(const float* __restrict_
         if (lane == 0) {
             const int e = min(be, E - 1);                    // (logits that are no numbers leave nothing to choose)
             idx[(long long)t * top + k] = e;
-            weight[(long long)t * top + k] = be == E ? 0.f : 1.f / (1.f + expf(-best));
+            const float s = be == E ? 0.f : softmax ? expf(best - zmax) * inv : 1.f / (1.f + expf(-best));
+            weight[(long long)t * top + k] = normalise ? s : s * scale;
+            chosen += s;
             if (counts != nullptr) atomicAdd(counts + e, 1);
         }
     }
+    if (normalise && lane == 0)
+        for (int k = 0; k < top; ++k) weight[(long long)t * top + k] = weight[(long long)t * top + k] / (chosen + 1e-20f) * scale;
 }
 
 __global__ void place_offsets_kernel(const int* __restrict__ counts, int* __restrict__ offs, int E, int align) {
@@ -151,20 +165,48 @@ __global__ void __launch_bounds__(256) moe_rows_kernel(const T* __restrict__ X, 
     }
 }
 
+// z [rows, ldz]: gate in columns 0 .. ff, up in ff .. 2 ff -> out[row] = row_scale[row] silu(gate) * up for the rows in use
+template <typename T>
+__global__ void __launch_bounds__(256) moe_glu_kernel(const T* __restrict__ z, long long ldz, T* __restrict__ out, long long ldo, const int* __restrict__ used,
+                                                      const float* __restrict__ row_scale, int rows, int ff) {
+    pdl_trigger();
+    constexpr int W = Vec<T>::N;
+    const int pieces = ff / W;
+    const long long total = (long long)min(rows, *used) * pieces;
+    for (long long i = blockIdx.x * 256LL + threadIdx.x; i < total; i += gridDim.x * 256LL) {
+        const long long row = i / pieces;
+        const int c = (int)(i - row * pieces) * W;
+        const float w = row_scale[row];
+        Vec<T> g, u;
+        g.load(z + row * ldz + c);
+        u.load(z + row * ldz + ff + c);
+#pragma unroll
+        for (int e = 0; e < W; ++e) {
+            const float t = g.get(e);
+            g.set(e, w * (t / (1.f + expf(-t))) * u.get(e));
+        }
+        g.store(out + row * ldo + c);
+    }
+}
+
 // --------------------------------------------------------------------------------------------------------------- few tokens
 constexpr int SW = 8, MAX_PAIRS = 1024;
 
-// One product for every pair p (token p / top, expert idx[p]); grid (N / 16 rounded up, E).
-//   UP:   x row p / top of h,  y[p] = (weight[p] * relu(.))^2 in bf16
-//   else  x row p,             y[p] in fp32
-template <bool UP>
+// One product for every pair p (token p / top, expert idx[p]); grid (N / 16 rounded up, E; GATED: N / 8).
+//   RELU2  x row p / top of h,  y[p] = (weight[p] * relu(.))^2 in bf16
+//   GATED  x row p / top of h,  y[p] = weight[p] * silu(.) * (.) in bf16 with the N gate rows in front of the N up rows of an expert's matrix
+//   DOWN   x row p,             y[p] in fp32
+enum Kind { DOWN, RELU2, GATED };
+template <Kind KIND>
 __global__ void __launch_bounds__(SW * 32) moe_step_kernel(const bf16* __restrict__ x, long long ldx, const bf16* __restrict__ Wt, void* y,
                                                            long long ldy, const int* __restrict__ idx, const float* __restrict__ weight,
                                                            int pairs, int top, int N, int K) {
     __shared__ float red[SW][2][32][4];
     __shared__ int list[MAX_PAIRS], count;
     const int w = threadIdx.x >> 5, l = threadIdx.x & 31, g = l >> 2, q = l & 3;
-    const int e = blockIdx.y, r0 = blockIdx.x * 16;
+    constexpr bool UP = KIND != DOWN;
+    constexpr int ROWS = KIND == GATED ? 8 : 16;             // outputs of a CTA: its fragments' lower rows are up rows of the same outputs
+    const int e = blockIdx.y, r0 = blockIdx.x * ROWS;
     pdl_trigger();
     asm volatile("griddepcontrol.wait;" ::: "memory");
     if (w == 0) {                                            // this expert's pairs, in order
@@ -180,9 +222,10 @@ __global__ void __launch_bounds__(SW * 32) moe_step_kernel(const bf16* __restric
     __syncthreads();
     const int n = count;
     if (n == 0) return;
-    const bool lo_ok = r0 + g < N, hi_ok = r0 + g + 8 < N;
-    const bf16* w_lo = Wt + ((long long)e * N + (lo_ok ? r0 + g : 0)) * K + q * 8;
-    const bf16* w_hi = Wt + ((long long)e * N + (hi_ok ? r0 + g + 8 : 0)) * K + q * 8;
+    const bool lo_ok = r0 + g < N, hi_ok = KIND == GATED ? lo_ok : r0 + g + 8 < N;
+    const long long M = KIND == GATED ? 2LL * N : N;         // rows of an expert's matrix
+    const bf16* w_lo = Wt + (e * M + (lo_ok ? r0 + g : 0)) * K + q * 8;
+    const bf16* w_hi = Wt + (e * M + (hi_ok ? r0 + g + (KIND == GATED ? N : 8) : 0)) * K + q * 8;
     const uint4 zero = make_uint4(0, 0, 0, 0);
     for (int n0 = 0; n0 < n; n0 += 16) {                     // 16 pairs at a time; another round reads the weights from L1 / L2
         const bf16* xr[2];
@@ -217,14 +260,19 @@ __global__ void __launch_bounds__(SW * 32) moe_step_kernel(const bf16* __restric
         __syncthreads();
         if (w < 2) {
 #pragma unroll
-            for (int i = 0; i < 4; ++i) {
+            for (int i = 0; i < (KIND == GATED ? 2 : 4); ++i) {
                 const int b = n0 + 8 * w + 2 * q + (i & 1), r = r0 + g + 8 * (i >> 1);
                 if (b < n && r < N) {
                     float s = 0.f;
 #pragma unroll
                     for (int k = 0; k < SW; ++k) s += red[k][w][l][i];
                     const int p = list[b];
-                    if (UP) {
+                    if (KIND == GATED) {
+                        float u = 0.f;
+#pragma unroll
+                        for (int k = 0; k < SW; ++k) u += red[k][w][l][i + 2];
+                        ((bf16*)y)[(long long)p * ldy + r] = __float2bfloat16(weight[p] * (s / (1.f + expf(-s))) * u);
+                    } else if (KIND == RELU2) {
                         s = weight[p] * fmaxf(s, 0.f);
                         ((bf16*)y)[(long long)p * ldy + r] = __float2bfloat16(s * s);
                     } else {
@@ -237,11 +285,11 @@ __global__ void __launch_bounds__(SW * 32) moe_step_kernel(const bf16* __restric
     }
 }
 
-template <bool UP>
+template <Kind KIND>
 static int launch_step(const bf16* x, long long ldx, const bf16* W, void* y, long long ldy, const int* idx, const float* weight, int pairs,
                        int top, int E, int N, int K, cudaStream_t st) {
     cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3((N + 15) / 16, E);
+    cfg.gridDim = dim3(KIND == GATED ? (N + 7) / 8 : (N + 15) / 16, E);
     cfg.blockDim = dim3(SW * 32);
     cfg.stream = st;
     cudaLaunchAttribute attr[1];
@@ -249,7 +297,7 @@ static int launch_step(const bf16* x, long long ldx, const bf16* W, void* y, lon
     attr[0].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
     cfg.numAttrs = 1;
-    return (int)cudaLaunchKernelEx(&cfg, moe_step_kernel<UP>, x, ldx, W, y, ldy, idx, weight, pairs, top, N, K);
+    return (int)cudaLaunchKernelEx(&cfg, moe_step_kernel<KIND>, x, ldx, W, y, ldy, idx, weight, pairs, top, N, K);
 }
 
 }  // namespace mr
@@ -257,10 +305,12 @@ static int launch_step(const bf16* x, long long ldx, const bf16* W, void* y, lon
 
 using namespace lmoe;
 
-// logits [n, ldl] fp32 -> idx, weight [n, top] (largest first); counts [E] zeros or null
-LMOE_API int lmoe_route_rows(const float* logits, long long ldl, int n, int E, int top, int* idx, float* weight, int* counts, cudaStream_t st) {
+// logits [n, ldl] fp32 -> idx, weight [n, top] (largest first); softmax: scores over all experts instead of each one's sigmoid; normalise: weights
+// over their sum; counts [E] zeros or null
+LMOE_API int lmoe_route_rows(const float* logits, long long ldl, int n, int E, int top, int softmax, int normalise, float scale, int* idx, float* weight, int* counts, cudaStream_t st) {
     if (n <= 0 || E <= 0 || top <= 0 || top > E) return -1;
-    mr::route_rows_kernel<<<(n + mr::RT / 32 - 1) / (mr::RT / 32), mr::RT, 0, st>>>(logits, ldl, n, E, top, idx, weight, counts);
+    mr::route_rows_kernel<<<(n + mr::RT / 32 - 1) / (mr::RT / 32), mr::RT, 0, st>>>(logits, ldl, n, E, top, softmax, normalise, scale,
+                                                                                                idx, weight, counts);
     return (int)cudaGetLastError();
 }
 
@@ -290,12 +340,28 @@ LMOE_API int lmoe_moe_rows(const void* X, long long ldx, const void* W, void* C,
     return (int)cudaGetLastError();
 }
 
-// up: x [n, ldx] -> y [n * top, ldy] bf16;  down: x [n * top, ldx] -> y [n * top, ldy] fp32.  K a multiple of 32, ldx of 8, at most 1024 pairs
+// z [rows, ldz] -> out [rows, ldo]; offs [E + 1]: the rows in use end at offs[E]
+LMOE_API int lmoe_moe_glu(const void* z, long long ldz, void* out, long long ldo, const int* offs, const float* row_scale, int rows, int E, int ff, int dt,
+                          cudaStream_t st) {
+    const int w = dt ? 8 : 4;
+    if (rows <= 0 || E <= 0 || ff <= 0 || ff % w || ldz % w || ldo % w || offs == nullptr || row_scale == nullptr ||
+        ((reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(out)) & 15))
+        return -1;
+    const long long blocks = ((long long)rows * (ff / w) + 255) / 256;
+    const unsigned grid = (unsigned)(blocks < 148 * 16 ? blocks : 148 * 16);
+    if (dt) mr::moe_glu_kernel<bf16><<<grid, 256, 0, st>>>((const bf16*)z, ldz, (bf16*)out, ldo, offs + E, row_scale, rows, ff);
+    else mr::moe_glu_kernel<float><<<grid, 256, 0, st>>>((const float*)z, ldz, (float*)out, ldo, offs + E, row_scale, rows, ff);
+    return (int)cudaGetLastError();
+}
+
+// kind 1 (squared ReLU), 2 (gated): x [n, ldx] -> y [n * top, ldy] bf16;  0 (down): x [n * top, ldx] -> y [n * top, ldy] fp32.  K a multiple of 32, ldx of 8, at most 1024 pairs
 LMOE_API int lmoe_moe_step(const bf16* x, long long ldx, const bf16* W, void* y, long long ldy, const int* idx, const float* weight, int n,
-                           int top, int E, int N, int K, int up, cudaStream_t st) {
+                           int top, int E, int N, int K, int kind, cudaStream_t st) {
     if (n <= 0 || top <= 0 || (long long)n * top > mr::MAX_PAIRS || E <= 0 || E > 65535 || N <= 0 || K <= 0 || K % 32 || ldx % 8 ||
+        kind < 0 || kind > 2 ||
         ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(W)) & 15))
         return -1;
-    return up ? mr::launch_step<true>(x, ldx, W, y, ldy, idx, weight, n * top, top, E, N, K, st)
-              : mr::launch_step<false>(x, ldx, W, y, ldy, idx, weight, n * top, top, E, N, K, st);
+    return kind == 2   ? mr::launch_step<mr::GATED>(x, ldx, W, y, ldy, idx, weight, n * top, top, E, N, K, st)
+           : kind == 1 ? mr::launch_step<mr::RELU2>(x, ldx, W, y, ldy, idx, weight, n * top, top, E, N, K, st)
+                       : mr::launch_step<mr::DOWN>(x, ldx, W, y, ldy, idx, weight, n * top, top, E, N, K, st);
 }

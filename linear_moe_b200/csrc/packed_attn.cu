@@ -1,4 +1,4 @@
-// Packed-row softmax attention for any head size, bf16 or fp32 (arithmetic in fp32), and the row kernels around it:
+// Packed-row attention (softmax or sigmoid weights) for any head size, bf16 or fp32 (arithmetic in fp32), and the row kernels around it:
 //   packed_attn_rows_kernel   prompts (mathematics and work items: packed_attn_tc.cu, the bf16 fast path): tiles of TQ queries x TQ
 //                             keys, online softmax
 //   packed_attn_step_kernel   one token per request from the cache (bf16 fast path: packed_attn_step.cu)
@@ -65,27 +65,37 @@ __global__ void __launch_bounds__(TQ * 4) packed_attn_rows_kernel(Prompt a) {
 #pragma unroll
             for (int e = 0; e < KP; ++e) s[e] += q * K[(part + 4 * e) * ldk + d];
         }
-        float mx = m;
+        float mx = m, corr = 1.f;
+        if (a.bias != nullptr) {
 #pragma unroll
-        for (int e = 0; e < KP; ++e) {
-            const int key = k0 + part + 4 * e;
-            s[e] = key <= qi && (a.window <= 0 || key > qi - a.window) ? s[e] * a.scale : -INFINITY;
-            mx = fmaxf(mx, s[e]);
-        }
-        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
-        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-        const float corr = m == -INFINITY ? 0.f : expf(m - mx);
-        float ps = 0.f;
+            for (int e = 0; e < KP; ++e) {
+                const int key = k0 + part + 4 * e;
+                const bool seen = key <= qi && (a.window <= 0 || key > qi - a.window);
+                S[r * (TK + 1) + part + 4 * e] = seen ? a.mul / (1.f + expf(-(s[e] * a.scale + a.bias[h]))) : 0.f;
+            }
+            l = 1.f;
+        } else {
 #pragma unroll
-        for (int e = 0; e < KP; ++e) {
-            const float p = mx == -INFINITY ? 0.f : expf(s[e] - mx);   // no visible key yet
-            S[r * (TK + 1) + part + 4 * e] = p;
-            ps += p;
+            for (int e = 0; e < KP; ++e) {
+                const int key = k0 + part + 4 * e;
+                s[e] = key <= qi && (a.window <= 0 || key > qi - a.window) ? s[e] * a.scale : -INFINITY;
+                mx = fmaxf(mx, s[e]);
+            }
+            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+            corr = m == -INFINITY ? 0.f : expf(m - mx);
+            float ps = 0.f;
+#pragma unroll
+            for (int e = 0; e < KP; ++e) {
+                const float p = mx == -INFINITY ? 0.f : expf(s[e] - mx);   // no visible key yet
+                S[r * (TK + 1) + part + 4 * e] = p;
+                ps += p;
+            }
+            ps += __shfl_xor_sync(0xffffffffu, ps, 1);
+            ps += __shfl_xor_sync(0xffffffffu, ps, 2);
+            l = l * corr + ps;
+            m = mx;
         }
-        ps += __shfl_xor_sync(0xffffffffu, ps, 1);
-        ps += __shfl_xor_sync(0xffffffffu, ps, 2);
-        l = l * corr + ps;
-        m = mx;
         __syncwarp();
         for (int d = part; d < dv; d += 4) {
             float o = O[r * dv + d] * corr;
@@ -148,14 +158,21 @@ __global__ void __launch_bounds__(ST) packed_attn_step_kernel(Step a) {
             if (lane == 0) P[j] = s * a.scale;
         }
         __syncthreads();
-        const float x = threadIdx.x < nt ? P[threadIdx.x] : -INFINITY;
-        const float mx = fmaxf(m, block_max(x, red));
-        const float p = threadIdx.x < nt ? expf(x - mx) : 0.f;
-        if (threadIdx.x < nt) P[threadIdx.x] = p;
-        const float ps = block_sum(p, red);                  // also orders the writes of P
-        const float corr = m == -INFINITY ? 0.f : expf(m - mx);
-        l = l * corr + ps;
-        m = mx;
+        float corr = 1.f;
+        if (a.bias != nullptr) {
+            if (threadIdx.x < nt) P[threadIdx.x] = a.mul / (1.f + expf(-(P[threadIdx.x] + a.bias[h])));
+            l = 1.f;
+            __syncthreads();
+        } else {
+            const float x = threadIdx.x < nt ? P[threadIdx.x] : -INFINITY;
+            const float mx = fmaxf(m, block_max(x, red));
+            const float p = threadIdx.x < nt ? expf(x - mx) : 0.f;
+            if (threadIdx.x < nt) P[threadIdx.x] = p;
+            const float ps = block_sum(p, red);              // also orders the writes of P
+            corr = m == -INFINITY ? 0.f : expf(m - mx);
+            l = l * corr + ps;
+            m = mx;
+        }
         for (int d = threadIdx.x; d < a.dv; d += ST) {
             float o = O[d] * corr;
             for (int j = 0; j < nt; ++j) o += P[j] * to_f(((const T*)a.c.v)[(rows[j] + hv) * a.dv + d]);

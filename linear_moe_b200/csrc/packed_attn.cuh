@@ -32,6 +32,8 @@ struct Prompt {
     float scale;
     int cross;                        // every query head's weights are applied to the values of every kv head: out [rows, H, G, dv]
     int bounded;                      // cross, tensor-core kernel: |q . k * scale| <= 60 everywhere, so that exp needs no running maximum
+    const float* bias;                // [H]: weights sigmoid(q . k * scale + bias[h]) that sum to nothing in particular (null: softmax)
+    float mul;                        // factor of the output with these
 };
 
 struct Cache {
@@ -54,6 +56,8 @@ struct Step {
     int n;
     float scale;
     int cross;                        // as in Prompt
+    const float* bias;                // as in Prompt
+    float mul;
 };
 
 }  // namespace pa

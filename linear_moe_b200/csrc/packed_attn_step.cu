@@ -1,4 +1,4 @@
-// One-token softmax attention over cached keys for bf16: grouped-query layers with a ring or pages, and latent layers, whose
+// One-token attention (softmax, or sigmoid weights of every key by itself) over cached keys for bf16: grouped-query layers with a ring or pages, and latent layers, whose
 // cached row is key and value at once (then it is read once).  Arguments and cache addressing: packed_attn.cuh.  The new token's key
 // and value are in the cache already; the order of the keys does not matter to a softmax, so a ring needs no unrolling.
 //
@@ -106,7 +106,9 @@ packed_attn_step_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_co
     const float sc = a.scale * LOG2E;
     const int bufs = min(WARPS, a.dk / 16);                  // warps with a step of the head dimension
     const int srow = threadIdx.x / TPR, sk0 = (threadIdx.x % TPR) * KPT;    // this thread's row and first key in the softmax
-    float m = -INFINITY, sum = 0.f;
+    const bool sigmoid = a.bias != nullptr;                  // then there is no maximum to follow: m stays 0
+    const float head_bias = sigmoid && srow < nh ? a.bias[h0 + srow] * LOG2E : 0.f;
+    float m = sigmoid ? 0.f : -INFINITY, sum = 0.f;
     float o[2 * N][4];
 #pragma unroll
     for (int j = 0; j < 2 * N; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
@@ -176,32 +178,43 @@ packed_attn_step_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_co
                         x[i + 1] += f.y;
                     }
                 }
-            float mx = m;
-            if (t * KT >= lo && (t + 1) * KT <= nk) {
+            if (sigmoid) {
 #pragma unroll
-                for (int i = 0; i < KPT; ++i) x[i] *= sc;
-            } else {
-#pragma unroll
-                for (int i = 0; i < KPT; ++i) {
+                for (int i = 0; i < KPT; i += 2) {
                     const int key = t * KT + sk0 + i;
-                    x[i] = key >= lo && key < nk ? x[i] * sc : -INFINITY;
+                    x[i] = key >= lo && key < nk ? rcp(1.f + ex2(-(x[i] * sc + head_bias))) : 0.f;
+                    x[i + 1] = key + 1 >= lo && key + 1 < nk ? rcp(1.f + ex2(-(x[i + 1] * sc + head_bias))) : 0.f;
+                    *reinterpret_cast<__nv_bfloat162*>(P + srow * (KT + 8) + sk0 + i) = __floats2bfloat162_rn(x[i], x[i + 1]);
                 }
+                if (sk0 == 0) ML[2 * ROWS + srow] = 1.f;
+            } else {
+                float mx = m;
+                if (t * KT >= lo && (t + 1) * KT <= nk) {
+#pragma unroll
+                    for (int i = 0; i < KPT; ++i) x[i] *= sc;
+                } else {
+#pragma unroll
+                    for (int i = 0; i < KPT; ++i) {
+                        const int key = t * KT + sk0 + i;
+                        x[i] = key >= lo && key < nk ? x[i] * sc : -INFINITY;
+                    }
+                }
+#pragma unroll
+                for (int i = 0; i < KPT; ++i) mx = fmaxf(mx, x[i]);
+#pragma unroll
+                for (int d = 1; d < TPR; d <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
+                const float corr = m == -INFINITY ? 0.f : ex2(m - mx);       // a tile of [lo, nk) has a visible key: mx is finite
+                sum *= corr;                                                 // this thread's keys only, added up at the end
+#pragma unroll
+                for (int i = 0; i < KPT; i += 2) {
+                    x[i] = ex2(x[i] - mx);
+                    x[i + 1] = ex2(x[i + 1] - mx);
+                    sum += x[i] + x[i + 1];
+                    *reinterpret_cast<__nv_bfloat162*>(P + srow * (KT + 8) + sk0 + i) = __floats2bfloat162_rn(x[i], x[i + 1]);
+                }
+                m = mx;
+                if (sk0 == 0) ML[2 * ROWS + srow] = corr;
             }
-#pragma unroll
-            for (int i = 0; i < KPT; ++i) mx = fmaxf(mx, x[i]);
-#pragma unroll
-            for (int d = 1; d < TPR; d <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
-            const float corr = m == -INFINITY ? 0.f : ex2(m - mx);       // a tile of [lo, nk) has a visible key: mx is finite
-            sum *= corr;                                                 // this thread's keys only, added up at the end
-#pragma unroll
-            for (int i = 0; i < KPT; i += 2) {
-                x[i] = ex2(x[i] - mx);
-                x[i + 1] = ex2(x[i + 1] - mx);
-                sum += x[i] + x[i + 1];
-                *reinterpret_cast<__nv_bfloat162*>(P + srow * (KT + 8) + sk0 + i) = __floats2bfloat162_rn(x[i], x[i + 1]);
-            }
-            m = mx;
-            if (sk0 == 0) ML[2 * ROWS + srow] = corr;
         }
         __syncthreads();
         {
@@ -280,7 +293,7 @@ packed_attn_step_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_co
                 ls += part[1][r][h] * f;
                 os.x += x.x * f; os.y += x.y * f; os.z += x.z * f; os.w += x.w * f;
             }
-            const float inv = 1.f / ls;
+            const float inv = sigmoid ? a.mul : 1.f / ls;
             __nv_bfloat162 y[2] = {__floats2bfloat162_rn(os.x * inv, os.y * inv), __floats2bfloat162_rn(os.z * inv, os.w * inv)};
             *reinterpret_cast<uint2*>((bf16*)a.out + (long long)b * a.ldo + (long long)(h0 + h) * a.dv + 4 * d) = *reinterpret_cast<uint2*>(y);
         }
@@ -352,7 +365,7 @@ using namespace lmoe;
 LMOE_API int lmoe_packed_attn_step(const pa::Step* ap, int rows, int splits, int* err, cudaStream_t st) {
     const pa::Step& a = *ap;
     if (a.n <= 0 || a.G <= 0 || a.H <= 0 || a.H % a.G || a.dk <= 0 || a.dv <= 0 || a.dk % 16 || a.dv % 16 || a.dk > 512 || a.dv > 512 || a.ldq % 8 || a.ldo % 8 ||
-        rows <= 0 || !(a.scale > 0.f) || (a.c.table == nullptr && a.c.cap <= 0) ||
+        rows <= 0 || (a.bias == nullptr && !(a.scale > 0.f)) || a.cross || (a.c.table == nullptr && a.c.cap <= 0) ||
         ((reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.c.k) | reinterpret_cast<uintptr_t>(a.c.v) |
           reinterpret_cast<uintptr_t>(a.out)) & 15) ||
         (splits != 1 && splits != 2 && splits != 4 && splits != 8 && splits != 16))

@@ -1,4 +1,4 @@
-// Causal softmax attention over packed prompts on the 5th-generation tensor cores (bf16, head sizes up to 128 in multiples of 8),
+// Causal attention over packed prompts on the 5th-generation tensor cores (bf16, head sizes up to 128 in multiples of 8),
 // with an optional sliding window and an optional output gate:
 //     o = sigmoid(gate) * softmax(q . k * scale) v          key j visible to query i when 0 <= i - j (< window)
 // Queries, keys and values are rows of separate matrices (packed_attn.cuh); a work item is up to 128 queries of one request.
@@ -15,6 +15,8 @@
 // be `bounded` (normed queries and keys), P = exp2(S) as it is: no maximum, no exchange between threads, and P goes back to tensor memory
 // into the columns its scores came from, from where the value product reads it; the shared memory of the P tile holds more stages of
 // values.
+// Sigmoid weights (every visible pair by itself, o = mul * sum of sigmoid(q . k * scale + bias[h]) v) are bounded too and take that form, with
+// value heads up to 256.
 // Every mbarrier wait is bounded; on expiry the error word is set and the CTA drains and frees its tensor memory.
 #include "attn_math.cuh"
 #include "flash_tc_utils.cuh"
@@ -26,6 +28,7 @@ using namespace lmoe::fatc;
 using pa::Prompt;
 
 constexpr float LAG = 8.f;
+enum Weights { LAGGING, BOUNDED_SOFTMAX, SIGMOID };
 
 // DQ: key dims, DT: value columns of a CTA
 template <int DQ, int DT, bool BOUNDED>
@@ -56,13 +59,14 @@ __device__ __forceinline__ void umma_ta(uint32_t tmem_d, uint32_t tmem_a, uint32
 }
 __device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 
-// DV: value dims of a head, NB: value heads of a CTA, BOUNDED: see above
-template <int DQ, int DV, int NB, bool BOUNDED>
+// DV: value dims of a head, NB: value heads of a CTA
+template <int DQ, int DV, int NB, Weights W>
 __global__ void __launch_bounds__(THREADS, 1)
 packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                       const __grid_constant__ CUtensorMap tmV, Prompt a) {
     extern __shared__ uint8_t smem_raw[];
     constexpr int DT = NB * DV;
+    constexpr bool BOUNDED = W != LAGGING;
     using Sm = Smem<DQ, DT, BOUNDED>;
     constexpr int VK = Sm::VK, VS = BN / VK, ST = Sm::ST;   // VS: stages of values per tile of keys
     Sm& sm = *reinterpret_cast<Sm*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -184,7 +188,7 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
         const uint32_t lane_addr = tmem_base + ((uint32_t)(qd * 32) << 16);
         constexpr int CW = BN / SPLIT, OW = DT / SPLIT;       // score / output columns of this thread
         static_assert(CW == 32 && OW % 16 == 0, "tensor-memory load widths");
-        const float sc = a.scale * LOG2E, lag = LAG / sc;
+        const float sc = a.scale * LOG2E, lag = LAG / sc, head_bias = W == SIGMOID ? a.bias[h] * LOG2E : 0.f;
         uint8_t* prow = sm.p + ((part * CW) >> 6) * (BM * 128) + (r >> 3) * 1024 + (r & 7) * 128;
         const int ch0 = ((part * CW) & 63) >> 3;
         float m = -INFINITY, l = 0.f;
@@ -201,7 +205,7 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
                 const int lo = a.window > 0 ? hi - a.window : -1;
 #pragma unroll
                 for (int c = 0; c < CW; ++c)
-                    if (c > hi || c <= lo) v[c] = 0xff800000u;                  // -inf
+                    if (c > hi || c <= lo) v[c] = W == SIGMOID && sc < 0.f ? 0x7f800000u : 0xff800000u;         // a weight of zero
             }
             if constexpr (!BOUNDED) {
                 float mx4[4];
@@ -237,16 +241,20 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
                     tmem_st_wait();
                 }
             }
-            const float nm = BOUNDED || m == -INFINITY ? 0.f : -m * sc;
-            const float2 sc2 = make_float2(sc, sc), nm2 = make_float2(nm, nm);
+            const float nm = W == SIGMOID ? -head_bias : BOUNDED || m == -INFINITY ? 0.f : -m * sc;
+            const float2 sc2 = W == SIGMOID ? make_float2(-sc, -sc) : make_float2(sc, sc), nm2 = make_float2(nm, nm);
             float2 sum0 = make_float2(0.f, 0.f), sum1 = make_float2(0.f, 0.f);
 #pragma unroll
             for (int c = 0; c < CW; c += 4) {
                 const float2 x01 = __ffma2_rn(make_float2(__uint_as_float(v[c]), __uint_as_float(v[c + 1])), sc2, nm2);
                 const float2 x23 = __ffma2_rn(make_float2(__uint_as_float(v[c + 2]), __uint_as_float(v[c + 3])), sc2, nm2);
-                const float p0 = ex2(x01.x), p1 = ex2(x01.y), p2 = ex2(x23.x), p3 = ex2(x23.y);
-                sum0 = __fadd2_rn(sum0, make_float2(p0, p1));
-                sum1 = __fadd2_rn(sum1, make_float2(p2, p3));
+                float p0 = ex2(x01.x), p1 = ex2(x01.y), p2 = ex2(x23.x), p3 = ex2(x23.y);
+                if constexpr (W == SIGMOID) {                 // (hidden: 1 / infinity)
+                    p0 = rcp(1.f + p0), p1 = rcp(1.f + p1), p2 = rcp(1.f + p2), p3 = rcp(1.f + p3);
+                } else {
+                    sum0 = __fadd2_rn(sum0, make_float2(p0, p1));
+                    sum1 = __fadd2_rn(sum1, make_float2(p2, p3));
+                }
                 v[c >> 1] = pack_bf16(p0, p1);
                 v[(c >> 1) + 1] = pack_bf16(p2, p3);
             }
@@ -281,10 +289,21 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
 #pragma unroll
         for (int p = 0; p < SPLIT; ++p) l += ls[p * BM + r];
         uint32_t o[OW];
-        tmem_ld<OW>(lane_addr + O_COL + part * OW, o);
-        tmem_ld_wait();
+        if constexpr (OW == 48) {
+#pragma unroll
+            for (int c = 0; c < OW; c += 16) {
+                uint32_t piece[16];
+                tmem_ld16(lane_addr + O_COL + part * OW + c, piece);
+                tmem_ld_wait();
+#pragma unroll
+                for (int i = 0; i < 16; ++i) o[c + i] = piece[i];
+            }
+        } else {
+            tmem_ld<OW>(lane_addr + O_COL + part * OW, o);
+            tmem_ld_wait();
+        }
         if (alive && r < nq) {
-            const float w = 1.f / l;
+            const float w = W == SIGMOID ? a.mul : 1.f / l;
             const long long row = row0 + r;
             const bf16* gp = a.gate == nullptr ? nullptr : (const bf16*)a.gate + row * a.ldg + h * a.dv;
 #pragma unroll
@@ -312,24 +331,32 @@ packed_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
     }
 }
 
-template <int DQ, int DV, int NB, bool BOUNDED>
+template <int DQ, int DV, int NB, Weights W>
 static int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const Prompt& a, cudaStream_t st) {
-    const size_t smem = sizeof(Smem<DQ, NB * DV, BOUNDED>) + 1024;
-    static_assert(sizeof(Smem<DQ, NB * DV, BOUNDED>) + 1024 <= 227 * 1024 && NB * DV <= 256, "shared and tensor memory of one CTA");
-    cudaError_t e = cudaFuncSetAttribute(packed_attn_tc_kernel<DQ, DV, NB, BOUNDED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    const size_t smem = sizeof(Smem<DQ, NB * DV, W != LAGGING>) + 1024;
+    static_assert(sizeof(Smem<DQ, NB * DV, W != LAGGING>) + 1024 <= 227 * 1024 && NB * DV <= 256, "shared and tensor memory of one CTA");
+    cudaError_t e = cudaFuncSetAttribute(packed_attn_tc_kernel<DQ, DV, NB, W>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
-    packed_attn_tc_kernel<DQ, DV, NB, BOUNDED><<<dim3(a.n, a.H, a.cross ? (a.G + NB - 1) / NB : 1), THREADS, smem, st>>>(mq, mk, mv, a);
+    packed_attn_tc_kernel<DQ, DV, NB, W><<<dim3(a.n, a.H, a.cross ? (a.G + NB - 1) / NB : 1), THREADS, smem, st>>>(mq, mk, mv, a);
     return (int)cudaGetLastError();
 }
 
-template <int DQ, bool BOUNDED>
+template <int DQ, Weights W>
 static int by_values(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const Prompt& a, cudaStream_t st) {
     const int heads = a.cross ? a.G : 1;
     if (a.dv <= 64)
-        return heads > 2   ? launch<DQ, 64, 4, BOUNDED>(mq, mk, mv, a, st)
-               : heads > 1 ? launch<DQ, 64, 2, BOUNDED>(mq, mk, mv, a, st)
-                           : launch<DQ, 64, 1, BOUNDED>(mq, mk, mv, a, st);
-    return heads > 1 ? launch<DQ, 128, 2, BOUNDED>(mq, mk, mv, a, st) : launch<DQ, 128, 1, BOUNDED>(mq, mk, mv, a, st);
+        return heads > 2   ? launch<DQ, 64, 4, W>(mq, mk, mv, a, st)
+               : heads > 1 ? launch<DQ, 64, 2, W>(mq, mk, mv, a, st)
+                           : launch<DQ, 64, 1, W>(mq, mk, mv, a, st);
+    return heads > 1 ? launch<DQ, 128, 2, W>(mq, mk, mv, a, st) : launch<DQ, 128, 1, W>(mq, mk, mv, a, st);
+}
+
+template <int DQ>
+static int sigmoid_by_values(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const Prompt& a, cudaStream_t st) {
+    return a.dv <= 64    ? launch<DQ, 64, 1, SIGMOID>(mq, mk, mv, a, st)
+           : a.dv <= 128 ? launch<DQ, 128, 1, SIGMOID>(mq, mk, mv, a, st)
+           : a.dv <= 192 ? launch<DQ, 192, 1, SIGMOID>(mq, mk, mv, a, st)
+                         : launch<DQ, 256, 1, SIGMOID>(mq, mk, mv, a, st);
 }
 
 }  // namespace patc
@@ -338,12 +365,13 @@ static int by_values(const CUtensorMap& mq, const CUtensorMap& mk, const CUtenso
 using namespace lmoe;
 
 // bf16; q [q_rows, ldq], k / v [k_rows, ldk / ldv], gate [q_rows, ldg] or null: bases 16-byte aligned, pitches and head sizes
-// multiples of 8, head sizes up to 128, scale > 0.  items: up to 128 queries each; every row they name lies inside the matrices.
+// multiples of 8, head sizes up to 128 (with sigmoid weights: values up to 256), scale > 0 (sigmoid: of any sign).  items: up to 128 queries each; every row they name lies inside the matrices.
 LMOE_API int lmoe_packed_attn_tc(const pa::Prompt* ap, cudaStream_t st) {
     using namespace lmoe::patc;
     const Prompt& a = *ap;
-    if (a.n <= 0 || a.q_rows <= 0 || a.k_rows <= 0 || a.H <= 0 || a.G <= 0 || a.H % a.G || a.dk <= 0 || a.dk > 128 || a.dv <= 0 || a.dv > 128 ||
-        a.dk % 8 || a.dv % 8 || a.ldq % 8 || a.ldk % 8 || a.ldv % 8 || a.ldo % 8 || (a.gate != nullptr && a.ldg % 8) || !(a.scale > 0.f) ||
+    if (a.n <= 0 || a.q_rows <= 0 || a.k_rows <= 0 || a.H <= 0 || a.G <= 0 || a.H % a.G || a.dk <= 0 || a.dk > 128 || a.dv <= 0 || a.dv > (a.bias != nullptr ? 256 : 128) ||
+        a.dk % 8 || a.dv % 8 || a.ldq % 8 || a.ldk % 8 || a.ldv % 8 || a.ldo % 8 || (a.gate != nullptr && a.ldg % 8) ||
+        (a.bias == nullptr ? !(a.scale > 0.f) : a.cross || a.gate != nullptr) ||
         (a.cross && a.gate != nullptr) || ((reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.k) | reinterpret_cast<uintptr_t>(a.v) |
           reinterpret_cast<uintptr_t>(a.gate) | reinterpret_cast<uintptr_t>(a.out)) & 15))
         return -1;
@@ -352,6 +380,7 @@ LMOE_API int lmoe_packed_attn_tc(const pa::Prompt* ap, cudaStream_t st) {
     if (rc == 0) rc = make_map_4d(&mk, a.k, 1, a.k_rows, a.G, a.dk, (long long)a.k_rows * a.ldk, a.ldk, a.dk, BN);
     if (rc == 0) rc = make_map_4d(&mv, a.v, 1, a.k_rows, a.G, a.dv, (long long)a.k_rows * a.ldv, a.ldv, a.dv, 64);
     if (rc) return rc;
-    if (a.cross && a.bounded) return a.dk <= 64 ? by_values<64, true>(mq, mk, mv, a, st) : by_values<128, true>(mq, mk, mv, a, st);
-    return a.dk <= 64 ? by_values<64, false>(mq, mk, mv, a, st) : by_values<128, false>(mq, mk, mv, a, st);
+    if (a.bias != nullptr) return a.dk <= 64 ? sigmoid_by_values<64>(mq, mk, mv, a, st) : sigmoid_by_values<128>(mq, mk, mv, a, st);
+    if (a.cross && a.bounded) return a.dk <= 64 ? by_values<64, BOUNDED_SOFTMAX>(mq, mk, mv, a, st) : by_values<128, BOUNDED_SOFTMAX>(mq, mk, mv, a, st);
+    return a.dk <= 64 ? by_values<64, LAGGING>(mq, mk, mv, a, st) : by_values<128, LAGGING>(mq, mk, mv, a, st);
 }

@@ -3,7 +3,8 @@
 //                      one-number norm gain is a scalar on the projection's outputs, so two norms of the same stream
 //                      need one pass and one matrix product; the consumers of the projection apply their gain.  A gain with
 //                      one number per column (gain_n > 1, padded like x) is applied here.
-//   embed_norm         x = embedding[token] [+ position table[position]], in fp32, together with the first block's norm
+//   embed_norm         x = embedding[token] [+ position table[position]] [+ a vector], in fp32, together with the first block's norm; or the
+//                      same added to x (layers that run again)
 //   poly_norm          sum over p = 1, 2, 3 of w_p u^p / rms(u^p), plus w_4 (element-wise powers, rms over the row)
 // Rows are padded (stream and activations to a multiple of 32 elements, pad = 0), so that every product is aligned for TMA.
 // Compiled without fast-math: the same code serves the fp32 model.
@@ -52,19 +53,20 @@ template <typename T>
 __global__ void __launch_bounds__(THREADS) embed_norm_kernel(const long long* __restrict__ ids, const int* __restrict__ pos,
                                                              const T* __restrict__ emb, const T* __restrict__ ptab, float* __restrict__ x,
                                                              long long ldx, T* __restrict__ y, long long ldy, int width, int pad,
-                                                             int vocab, int npos, float eps, const float* gain) {
+                                                             int vocab, int npos, float eps, const float* gain, const float* shift, int keep) {
     pdl_trigger();
     __shared__ float red[32];
     // ids and positions are checked on the host; the clamp keeps a bad one from becoming a bad address
     const long long id = min(max(ids[blockIdx.x], 0LL), (long long)vocab - 1);
-    const T* er = emb + id * width;
+    const T* er = emb == nullptr ? nullptr : emb + id * width;
     const T* pr = ptab == nullptr ? nullptr : ptab + (long long)min(max(pos[blockIdx.x], 0), npos - 1) * width;
     float* xr = x + (long long)blockIdx.x * ldx;
     T* yr = y + (long long)blockIdx.x * ldy;
     float s = 0.f;
     for (int c = threadIdx.x; c < pad; c += THREADS) {
-        float v = 0.f;
-        if (c < width) v = to_f(er[c]) + (pr == nullptr ? 0.f : to_f(pr[c]));
+        float v = keep ? xr[c] : 0.f;
+        if (c < width) v += (er == nullptr ? 0.f : to_f(er[c])) + (pr == nullptr ? 0.f : to_f(pr[c]));
+        if (shift != nullptr) v += shift[c];
         xr[c] = v;
         s += v * v;
     }
@@ -142,15 +144,16 @@ LMOE_API int lmoe_stream_norm(const float* x, long long ldx, void* y, long long 
     return (int)cudaGetLastError();
 }
 
-// emb [vocab, width], ptab [npos, width] or null, in the model's dtype; ids int64, pos int32; gain [pad] or null
+// emb [vocab, width] or null, ptab [npos, width] or null, in the model's dtype; ids int64, pos int32; gain, shift [pad] (zeros behind the width) or
+// null; keep: added to x
 LMOE_API int lmoe_embed_norm(const long long* ids, const int* pos, const void* emb, const void* ptab, float* x, long long ldx, void* y,
-                             long long ldy, int rows, int width, int pad, int vocab, int npos, float eps, const float* gain, int dt,
-                             cudaStream_t st) {
+                             long long ldy, int rows, int width, int pad, int vocab, int npos, float eps, const float* gain,
+                             const float* shift, int keep, int dt, cudaStream_t st) {
     if (rows <= 0 || width <= 0 || pad < width || vocab <= 0 || (ptab != nullptr && npos <= 0)) return -1;
     if (dt) pb::embed_norm_kernel<bf16><<<rows, pb::THREADS, 0, st>>>(ids, pos, (const bf16*)emb, (const bf16*)ptab, x, ldx, (bf16*)y,
-                                                                      ldy, width, pad, vocab, npos, eps, gain);
+                                                                      ldy, width, pad, vocab, npos, eps, gain, shift, keep);
     else pb::embed_norm_kernel<float><<<rows, pb::THREADS, 0, st>>>(ids, pos, (const float*)emb, (const float*)ptab, x, ldx, (float*)y,
-                                                                    ldy, width, pad, vocab, npos, eps, gain);
+                                                                    ldy, width, pad, vocab, npos, eps, gain, shift, keep);
     return (int)cudaGetLastError();
 }
 

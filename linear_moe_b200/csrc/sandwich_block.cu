@@ -1,7 +1,8 @@
-// Row kernels of blocks that norm both ends of a sublayer, x += post(f(pre(x))), around an fp32 residual stream:
-//   residual_norm   y = the sublayer's output rows (or the sum of a token's expert rows);  x += y / rms(y) * post;
+// Row kernels of blocks that norm both ends of a sublayer, x += mul post(f(pre(x))), around an fp32 residual stream:
+//   residual_norm   y = the sublayer's output rows (or the sum of a token's expert rows, and of another row);  x += mul y / rms(y) * post;
 //                   h = x / rms(x) * pre, the input of the next sublayer: one pass over the stream per sublayer
 //   glu_rows        silu(gate) * up, or relu(gate) * up
+//   xielu_rows      a0 z^2 + z / 2 for positive z, else a1 (e^z - 1 - z) + z / 2, in place
 // Rows are padded to a multiple of 4 elements (pad = 0).  Compiled without fast-math: the same code serves the fp32 model.
 #include "common.cuh"
 
@@ -14,18 +15,19 @@ __device__ __forceinline__ float dot4(float4 v) { return v.x * v.x + v.y * v.y +
 __device__ __forceinline__ float4 mul4(float4 v, float r, float4 w) { return make_float4(v.x * r * w.x, v.y * r * w.y, v.z * r * w.z, v.w * r * w.w); }
 __device__ __forceinline__ float4 add4(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
 
-// top > 0: y holds one row per (token, expert); those of token t are rows dest[t * top + k] (dest null: t * top + k)
+// top > 0: y holds one row per (token, expert); those of token t are rows dest[t * top + k] (dest null: t * top + k).  plus: one more row per
+// token (null: none)
 template <typename Y, typename T>
 __global__ void __launch_bounds__(THREADS) residual_norm_kernel(float* __restrict__ x, long long ldx, const Y* __restrict__ y, long long ldy,
-                                                                const int* __restrict__ dest, int top, const float* __restrict__ post,
-                                                                const float* __restrict__ pre, T* __restrict__ h, long long ldh, int width,
+                                                                const int* __restrict__ dest, int top, const Y* __restrict__ plus, long long ldp,
+                                                                float mul, const float* __restrict__ post, const float* __restrict__ pre, T* __restrict__ h, long long ldh, int width,
                                                                 int pad, float eps) {
     pdl_trigger();
     __shared__ float red[32];
     float* xr = x + (long long)blockIdx.x * ldx;
     auto load_y = [&](int c) {
-        if (top <= 0) return load4(y + (long long)blockIdx.x * ldy + c);
-        float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+        float4 s = plus == nullptr ? make_float4(0.f, 0.f, 0.f, 0.f) : load4(plus + (long long)blockIdx.x * ldp + c);
+        if (top <= 0) return add4(s, load4(y + (long long)blockIdx.x * ldy + c));
         for (int k = 0; k < top; ++k) {
             const long long i = (long long)blockIdx.x * top + k;
             s = add4(s, load4(y + (dest == nullptr ? i : (long long)dest[i]) * ldy + c));
@@ -43,7 +45,7 @@ __global__ void __launch_bounds__(THREADS) residual_norm_kernel(float* __restric
         s += dot4(v[i]);
     }
     for (int c = (threadIdx.x + NV * THREADS) * 4; c < pad; c += THREADS * 4) s += dot4(load_y(c));
-    const float ry = 1.f / sqrtf(block_sum(s, red) / width + eps);
+    const float ry = mul / sqrtf(block_sum(s, red) / width + eps);
     s = 0.f;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
@@ -90,10 +92,28 @@ __global__ void __launch_bounds__(THREADS) glu_rows_kernel(const T* __restrict__
     }
 }
 
+template <typename T>
+__global__ void __launch_bounds__(THREADS) xielu_rows_kernel(T* __restrict__ z, long long ldz, int cols, const float* __restrict__ act) {
+    pdl_trigger();
+    constexpr int W = Vec<T>::N;
+    T* zr = z + (long long)blockIdx.x * ldz;
+    const float a0 = act[0], a1 = act[1];
+    for (int c = (threadIdx.x + blockIdx.y * THREADS) * W; c < cols; c += gridDim.y * THREADS * W) {
+        Vec<T> v;
+        v.load(zr + c);
+#pragma unroll
+        for (int i = 0; i < W; ++i) {
+            const float t = v.get(i);
+            v.set(i, (t > 0.f ? a0 * t * t : a1 * (expm1f(t) - t)) + 0.5f * t);
+        }
+        v.store(zr + c);
+    }
+}
+
 template <typename Y, typename T>
-static int launch(float* x, long long ldx, const void* y, long long ldy, const int* dest, int top, const float* post, const float* pre, void* h,
-                  long long ldh, int rows, int width, int pad, float eps, cudaStream_t st) {
-    residual_norm_kernel<Y, T><<<rows, THREADS, 0, st>>>(x, ldx, (const Y*)y, ldy, dest, top, post, pre, (T*)h, ldh, width, pad, eps);
+static int launch(float* x, long long ldx, const void* y, long long ldy, const int* dest, int top, const void* plus, long long ldp, float mul,
+                  const float* post, const float* pre, void* h, long long ldh, int rows, int width, int pad, float eps, cudaStream_t st) {
+    residual_norm_kernel<Y, T><<<rows, THREADS, 0, st>>>(x, ldx, (const Y*)y, ldy, dest, top, (const Y*)plus, ldp, mul, post, pre, (T*)h, ldh, width, pad, eps);
     return (int)cudaGetLastError();
 }
 
@@ -103,14 +123,14 @@ static int launch(float* x, long long ldx, const void* y, long long ldy, const i
 using namespace lmoe;
 
 // y_dt, dt: 1 bf16, 0 fp32 (of y and h).  pad: columns of x, h, post and pre (a multiple of 4, zeros from width on); y has at least pad
-// columns with zeros from width on.
-LMOE_API int lmoe_residual_norm(float* x, long long ldx, const void* y, long long ldy, int y_dt, const int* dest, int top, const float* post,
-                                const float* pre, void* h, long long ldh, int rows, int width, int pad, float eps, int dt, cudaStream_t st) {
-    if (rows <= 0 || width <= 0 || pad < width || pad % 4 || ldx % 4 || ldy % 4 || (pre != nullptr && ldh % 4)) return -1;
-    if (y_dt) return dt ? sb::launch<bf16, bf16>(x, ldx, y, ldy, dest, top, post, pre, h, ldh, rows, width, pad, eps, st)
-                        : sb::launch<bf16, float>(x, ldx, y, ldy, dest, top, post, pre, h, ldh, rows, width, pad, eps, st);
-    return dt ? sb::launch<float, bf16>(x, ldx, y, ldy, dest, top, post, pre, h, ldh, rows, width, pad, eps, st)
-              : sb::launch<float, float>(x, ldx, y, ldy, dest, top, post, pre, h, ldh, rows, width, pad, eps, st);
+// columns with zeros from width on, and so has plus (y's type).
+LMOE_API int lmoe_residual_norm(float* x, long long ldx, const void* y, long long ldy, int y_dt, const int* dest, int top, const void* plus,
+                                long long ldp, float mul, const float* post, const float* pre, void* h, long long ldh, int rows, int width, int pad, float eps, int dt, cudaStream_t st) {
+    if (rows <= 0 || width <= 0 || pad < width || pad % 4 || ldx % 4 || ldy % 4 || ldp % 4 || (pre != nullptr && ldh % 4)) return -1;
+    if (y_dt) return dt ? sb::launch<bf16, bf16>(x, ldx, y, ldy, dest, top, plus, ldp, mul, post, pre, h, ldh, rows, width, pad, eps, st)
+                        : sb::launch<bf16, float>(x, ldx, y, ldy, dest, top, plus, ldp, mul, post, pre, h, ldh, rows, width, pad, eps, st);
+    return dt ? sb::launch<float, bf16>(x, ldx, y, ldy, dest, top, plus, ldp, mul, post, pre, h, ldh, rows, width, pad, eps, st)
+              : sb::launch<float, float>(x, ldx, y, ldy, dest, top, plus, ldp, mul, post, pre, h, ldh, rows, width, pad, eps, st);
 }
 
 // kind: 0 silu, 1 relu
@@ -121,5 +141,15 @@ LMOE_API int lmoe_glu_rows(const void* z, long long ldz, void* out, long long ld
     if (rows > 1024) cols = 1;
     if (dt) sb::glu_rows_kernel<bf16><<<dim3(rows, cols), sb::THREADS, 0, st>>>((const bf16*)z, ldz, (bf16*)out, ldo, ff, kind);
     else sb::glu_rows_kernel<float><<<dim3(rows, cols), sb::THREADS, 0, st>>>((const float*)z, ldz, (float*)out, ldo, ff, kind);
+    return (int)cudaGetLastError();
+}
+
+// act: {a0, a1}
+LMOE_API int lmoe_xielu_rows(void* z, long long ldz, int rows, int cols, const float* act, int dt, cudaStream_t st) {
+    const int w = dt ? 8 : 4;
+    if (rows <= 0 || cols <= 0 || cols % w || ldz % w || act == nullptr || (reinterpret_cast<uintptr_t>(z) & 15)) return -1;
+    const int parts = rows > 1024 ? 1 : (cols + sb::THREADS * w - 1) / (sb::THREADS * w);
+    if (dt) sb::xielu_rows_kernel<bf16><<<dim3(rows, parts), sb::THREADS, 0, st>>>((bf16*)z, ldz, cols, act);
+    else sb::xielu_rows_kernel<float><<<dim3(rows, parts), sb::THREADS, 0, st>>>((float*)z, ldz, cols, act);
     return (int)cudaGetLastError();
 }

@@ -156,6 +156,18 @@ def dense_swiglu(x: torch.Tensor, w: torch.Tensor, want_pre: bool = True, band: 
     return act, pre
 
 
+def dense_xielu(x: torch.Tensor, w: torch.Tensor, act: torch.Tensor) -> torch.Tensor:
+    """``xielu(x w^T)`` with the activation (``ops.xielu_in``) in the GEMM epilogue."""
+    from . import cuda as K
+    M, Kd = x.shape
+    out = torch.empty(M, w.shape[0], dtype=torch.bfloat16, device=x.device)
+    rc = K.lib().lmoe_gemm_dense_xielu(K._p(x), ctypes.c_int(x.stride(0)), K._p(w), ctypes.c_int(w.stride(0)), K._p(out), ctypes.c_int(out.stride(0)),
+                                       ctypes.c_int(M), ctypes.c_int(w.shape[0]), ctypes.c_int(Kd), ctypes.c_int(BAND), K._p(act), K._p(_err(x.device)),
+                                       ctypes.c_int(K.NUM_SMS), K._st())
+    K._check(rc, "gemm_dense_xielu")
+    return out
+
+
 def dense_dswiglu(dy: torch.Tensor, w2: torch.Tensor, pre: torch.Tensor, band: Optional[int] = None) -> torch.Tensor:
     """``dPre = SwiGLU'(pre) applied to (dy @ w2)`` for ``w2 [H, F]`` (the fc2 weight as stored) and ``pre [M, 2F]``: the
     data-gradient GEMM of fc2 with the activation backward in its epilogue.  ``F`` must be a multiple of 64."""
