@@ -31,7 +31,7 @@ SERVING = {"parallel_block": ("chunk_attn.cu", "chunk_attn_step.cu", "chunk_attn
                               "parallel_block.cu", "gemm_dense.cu", "gemm_grouped.cu", "gemm_skinny.cu"),
            "post_norm_block": ("packed_attn.cu", "packed_attn_tc.cu", "talk_step.cu", "retention.cu", "retention_tc.cu", "post_norm.cu", "sandwich_block.cu",
                                "parallel_block.cu", "gemm_dense.cu", "gemm_skinny.cu"),
-           "zelinex": ("packed_attn.cu", "packed_attn_step.cu", "packed_attn_tc.cu", "ssd.cu", "delta_rule.cu", "moe_rows.cu",
+           "zelinex": ("packed_attn.cu", "packed_attn_step.cu", "packed_attn_tc.cu", "ssd.cu", "ssd_tc.cu", "delta_rule.cu", "delta_rule_tc.cu", "moe_rows.cu",
                        "sandwich_block.cu", "parallel_block.cu", "gemm_dense.cu", "gemm_grouped.cu", "gemm_skinny.cu")}
 
 

@@ -3,8 +3,6 @@
 namespace lmoe {
 namespace rt {
 
-constexpr int CH = 64;                   // tokens per chunk of the tensor-core kernel
-
 // a run of a request's new tokens: eight int32
 enum {
     G_ROW,       // first row
@@ -23,7 +21,7 @@ struct Args {
     float* state;                        // [slots, H, dk, dv] or null
     float* scratch;                      // [places, H, dk, dv]
     float* raw;                          // general kernel: [rows, H * dv]
-    const float* powers;                 // [H, CH + 1] decay^0 ..
+    const float* powers;                 // [H, 65] decay^0 ..
     const double* decay;                 // [H]
     const float2* turn;                  // [rows, rot / 2] (cos, sin) (one-token kernel; prompts are rotated before)
     const int *pos, *slots;              // [rows]

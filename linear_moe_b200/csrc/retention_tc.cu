@@ -6,94 +6,25 @@
 //   retention_combine_kernel   those sums -> the state in front of every group
 //   retention_out_kernel       outputs, each group from the state in front of it; a request's last group leaves the new state
 // A request of one group needs the last kernel only.  The powers are fp32; keys and scores are rounded once, behind their decay.
-#include "mma_utils.cuh"
+#include "chunk_state.cuh"
 #include "retention.cuh"
 
 namespace lmoe {
 namespace rtc {
+using namespace chk;
 using namespace rt;
 
-constexpr int NT = 256, PLD = CH + 8;
-constexpr float LOG2E = 1.4426950408889634f;
-
-template <int DK, int DV> struct Cfg {
-    static constexpr int LDK = DK + 8, LDV = DV + 8;         // row strides of the tiles
-    static constexpr int RB = DK / 16, S_NT = DV / 8 / (8 / RB);         // row blocks of the state, its n-tiles per warp
-    static constexpr int O_NT = DV / 16;                     // n-tiles of a warp's 16 x DV / 2 outputs
-    static constexpr int KV = CH * LDK * 2 + CH * LDV * 2;   // bytes of a stage of keys and values
-    static constexpr int STATE_SMEM = 2 * KV;
-    static constexpr int OUT_SMEM = 2 * (KV + CH * LDK * 2) + CH * LDV * 2 + DK * LDV * 2 + CH * PLD * 2;
+template <int DK, int DV> struct Cfg : Shape<DK, DV> {
+    using S = Shape<DK, DV>;
+    static constexpr int STATE_SMEM = 2 * S::KV;
+    static constexpr int OUT_SMEM = 2 * (S::KV + CH * S::LDK * 2) + CH * S::LDV * 2 + DK * S::LDV * 2 + CH * PLD * 2;
 };
 
-// [CH rows x cols] -> shared memory [CH][ld], columns up to D; rows from `valid` on and columns from `cols` on are zero
-template <int D, int LD>
-__device__ __forceinline__ void load_rows(bf16* smem, const bf16* g, long long pitch, int valid, int cols) {
-    for (int i = threadIdx.x; i < CH * (D / 8); i += NT) {
-        const int r = i / (D / 8), c = i % (D / 8) * 8;
-        const bool ok = r < valid && c < cols;
-        cp_async16(smem + r * LD + c, ok ? g + r * pitch + c : g, ok);
-    }
-}
-
+// adds a chunk of n tokens; pw: decay^0 ..
 template <int DK, int DV>
-struct State {
-    using C = Cfg<DK, DV>;
-    float s[C::S_NT][4];
-    int m0, n0;                          // first row and column of this warp's part
-
-    __device__ __forceinline__ State() {
-        const int w = threadIdx.x >> 5;
-        m0 = 16 * (w % C::RB), n0 = w / C::RB * (C::S_NT * 8);
-    }
-    __device__ __forceinline__ void load(const float* p, int dk, int dv) {           // null: zero
-        const int l = threadIdx.x & 31, r = m0 + (l >> 2), c = n0 + (l & 3) * 2;
-#pragma unroll
-        for (int t = 0; t < C::S_NT; ++t)
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                const bool ok = p != nullptr && r + 8 * e < dk && c + 8 * t < dv;
-                const float2 x = ok ? *reinterpret_cast<const float2*>(p + (long long)(r + 8 * e) * dv + c + 8 * t) : make_float2(0.f, 0.f);
-                s[t][2 * e] = x.x, s[t][2 * e + 1] = x.y;
-            }
-    }
-    __device__ __forceinline__ void store(float* p, int dk, int dv) const {
-        const int l = threadIdx.x & 31, r = m0 + (l >> 2), c = n0 + (l & 3) * 2;
-#pragma unroll
-        for (int t = 0; t < C::S_NT; ++t)
-#pragma unroll
-            for (int e = 0; e < 2; ++e)
-                if (r + 8 * e < dk && c + 8 * t < dv)
-                    *reinterpret_cast<float2*>(p + (long long)(r + 8 * e) * dv + c + 8 * t) = make_float2(s[t][2 * e], s[t][2 * e + 1]);
-    }
-    // n tokens of a chunk; pw: decay^0 ..
-    __device__ __forceinline__ void advance(const bf16* K, const bf16* V, const float* pw, int n) {
-        const int l = threadIdx.x & 31;
-        const float whole = pw[n];
-#pragma unroll
-        for (int t = 0; t < C::S_NT; ++t)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) s[t][e] *= whole;
-#pragma unroll
-        for (int k0 = 0; k0 < CH; k0 += 16) {
-            uint32_t a[4];
-            load_a_t(a, K, C::LDK, m0, k0);
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {                    // registers 0, 1: tokens 2q, 2q + 1; registers 2, 3: eight later
-                const int j = k0 + 8 * (e >> 1) + 2 * (l & 3);
-                const float2 f = __bfloat1622float2(*reinterpret_cast<__nv_bfloat162*>(&a[e]));
-                __nv_bfloat162 r = __floats2bfloat162_rn(f.x * pw[max(n - 1 - j, 0)], f.y * pw[max(n - 2 - j, 0)]);      // rows from n on are zero
-                a[e] = *reinterpret_cast<uint32_t*>(&r);
-            }
-#pragma unroll
-            for (int t = 0; t < C::S_NT; t += 2) {
-                uint32_t b[4];
-                load_b2_t(b, V, C::LDV, n0 + t * 8, k0);
-                mma16816(s[t], a, b[0], b[1]);
-                mma16816(s[t + 1], a, b[2], b[3]);
-            }
-        }
-    }
-};
+__device__ __forceinline__ void advance(State<DK, DV>& S, const bf16* K, const bf16* V, const float* pw, int n) {
+    S.advance(K, V, pw[n], [&](int j) { return pw[max(n - 1 - j, 0)]; });
+}
 
 // grid (groups, H); groups without a place behind them have nothing to do
 template <int DK, int DV>
@@ -123,7 +54,7 @@ __global__ void __launch_bounds__(NT) retention_state_kernel(Args a) {
         cp_async_commit();
         cp_async_wait<1>();
         __syncthreads();
-        S.advance(K(t0 / CH & 1), V(t0 / CH & 1), pw, min(CH, n - t0));
+        advance(S, K(t0 / CH & 1), V(t0 / CH & 1), pw, min(CH, n - t0));
         __syncthreads();
     }
     S.store(a.scratch + ((long long)to * a.H + h) * a.dk * a.dv, a.dk, a.dv);
@@ -209,7 +140,7 @@ __global__ void __launch_bounds__(NT) retention_out_kernel(Args a) {
                 *reinterpret_cast<__nv_bfloat162*>(P + i * PLD + j) = __floats2bfloat162_rn(y0, y1);
             }
         }
-        S.advance(K(s), V(s), pw, nt);
+        advance(S, K(s), V(s), pw, nt);
         __syncthreads();                                     // P is complete, nobody reads Sb any more
         for (int k0 = 0; k0 <= m0; k0 += 16) {               // keys behind row m0 + 15 are hidden
             uint32_t p[4];

@@ -17,6 +17,7 @@ import torch
 
 from ..ref import delta_rule as RD
 from .packed_attn import _fields, _no_grad, _ptr
+from .retention import CHUNK
 from .row_batch import RowBatch, round_up
 
 DECAY = math.exp(-0.5)                # a channel's log decay lies between -DECAY and 0
@@ -94,6 +95,14 @@ def general_delta_rows(z, out, lay: DeltaLayout, s: GeneralDeltaSpec, w2, p: dic
     K._check(K.lib().lmoe_delta_low(ctypes.byref(a), dt, K._st()), "delta_low")
     decay = linear_f32(low, w2)
     a.w, a.ldw = decay.data_ptr(), decay.stride(0)
+    if dt == 1 and not batch.decode and d <= 128:
+        table, chunks = batch.recurrent_chunks(CHUNK)
+        size = K.lib().lmoe_delta_tc_work
+        size.restype = ctypes.c_longlong
+        work = torch.empty(chunks * H * size(d), dtype=torch.uint8, device=dev)
+        a.groups, a.work = table.data_ptr(), work.data_ptr()
+        K._check(K.lib().lmoe_delta_tc(ctypes.byref(a), chunks, batch.requests, K._st()), "delta_tc", 3)
+        return
     raw = torch.empty(rows, H * d, dtype=torch.float32, device=dev)
     a.raw = raw.data_ptr()
     if batch.decode:

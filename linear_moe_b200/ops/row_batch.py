@@ -139,6 +139,19 @@ class RowBatch:
             self._items[key] = (self._table(key + (0,), groups), states, self._table(key + (1,), many) if many else None)
         return self._items[key]
 
+    def recurrent_chunks(self, tokens: int):
+        """Every request's new tokens in chunks of at most ``tokens``: ``(table, chunks)``, an int32 table of the chunks (as ``recurrent_groups``) and
+        behind them the requests: (slot, flag 4: it has a past, first chunk, chunks)."""
+        key = ("chunks", tokens)
+        if key not in self._items:
+            chunks, requests = [], []
+            for r, n in enumerate(self.counts):
+                slot, past, count = 0 if self.slots is None else self.slots[r], 4 if self.starts[r] else 0, -(-n // tokens)
+                requests.append((slot, past, len(chunks), count, 0, 0, 0, 0))
+                chunks += [(self.row0[r] + i, min(tokens, n - i), slot, past + (i == 0) + 2 * (i + tokens >= n), -1, -1, 0, 0) for i in range(0, n, tokens)]
+            self._items[key] = (self._table(key + (0,), chunks + requests), len(chunks))
+        return self._items[key]
+
     def key_sources(self, window: Optional[int], cached: bool) -> torch.Tensor:
         """Where rows of the key matrix come from, ``[n, 4]`` int32 (destination, new row or -1, slot, position): the cached
         ones, or the new ones."""

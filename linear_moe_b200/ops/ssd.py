@@ -102,7 +102,7 @@ def ssd_rows(z, out, lay: SsdLayout, s: SsdSpec, w: dict, mul: float, eps: float
         assert cache["s"].is_contiguous() and cache["s"].shape[1:] == (H, dn, dv) and cache["c"].is_contiguous() and cache["c"].dtype == z.dtype
         a.state, a.tail, a.ring = cache["s"].data_ptr(), cache["c"].data_ptr(), cache["c"].shape[1]
     step = batch.decode and dv <= 256
-    fast = False
+    fast = dt == 1 and not batch.decode and dn <= 128 and dv <= 128
     y = torch.empty(rows, H * dv, dtype=torch.bfloat16 if fast else torch.float32, device=dev)
     a.y, a.ldy, a.y_f32 = y.data_ptr(), H * dv, int(not fast)
     if step:
