@@ -19,7 +19,7 @@ from ..ops.delta_rule import GeneralDeltaSpec
 from ..ops.moe_rows import ExpertsSpec, MlpSpec
 from ..ops.packed_attn import AttentionSpec, LatentSpec, RotaryScaling
 from ..ops.retention import RetentionSpec
-from ..ops.ssd import SsdSpec
+from ..ops.state_space import SsdSpec
 from .sandwich_block import ParallelSpec
 from .transformer import CausalLM
 

@@ -25,7 +25,7 @@ from ..ops.delta_rule import DeltaLayout, GeneralDeltaSpec
 from ..ops.moe_rows import ExpertsSpec, MlpSpec
 from ..ops.packed_attn import AttentionSpec, LatentSpec, QkvLayout
 from ..ops.row_batch import round_up
-from ..ops.ssd import SsdLayout, SsdSpec
+from ..ops.state_space import SsdLayout, SsdSpec
 from ..parallel.tensor_parallel import init_normal
 from .layout import LayerSpec
 from .packed_rows import ROW_PAD, RowBlock, RowStep, fill

@@ -329,7 +329,7 @@ from .moe_rows import experts_rows   # noqa: E402,F401
 from .packed_attn import (causal_attention, gather_rows, glu_in, head_norm_rope_, latent_absorb, latent_norm, latent_up,   # noqa: E402,F401
                           qk_norm_rope_, residual_norm, rotary_rows, rotate_heads_, step_attention, sublayer_out, xielu_in)
 from .retention import retention_rows   # noqa: E402,F401
-from .ssd import ssd_rows   # noqa: E402,F401
+from .state_space import ssd_rows   # noqa: E402,F401
 
 
 # ---- linear sequence models -----------------------------------------------

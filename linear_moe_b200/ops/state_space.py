@@ -4,7 +4,7 @@
     out = mul * norm(y silu(z)) * weight                                             the norm by groups of the heads' numbers
 
 ``B`` and ``C`` belong to groups of heads.  CUDA tensors (bf16 or fp32) take ``csrc/ssd_tc.cu`` (bf16 prompts, state and head sizes up to 128)
-and ``csrc/ssd.cu`` (convolution, one-token steps, gate and norm, everything else); CPU tensors take :mod:`linear_moe_b200.ref.ssd`.  Serves
+and ``csrc/ssd.cu`` (convolution, one-token steps, gate and norm, everything else); CPU tensors take :mod:`linear_moe_b200.ref.state_space`.  Serves
 only (no backward pass).
 """
 from __future__ import annotations
@@ -15,7 +15,7 @@ from typing import Optional
 
 import torch
 
-from ..ref import ssd as RS
+from ..ref import state_space as RS
 from .packed_attn import _fields, _no_grad, _ptr
 from .retention import CHUNK
 from .row_batch import RowBatch, round_up

@@ -1,4 +1,4 @@
-"""Eager definition of :func:`linear_moe_b200.ops.ssd.ssd_rows` (what CPU tensors run): token by token in fp32."""
+"""Eager definition of :func:`linear_moe_b200.ops.state_space.ssd_rows` (what CPU tensors run): token by token in fp32."""
 from __future__ import annotations
 
 import torch

@@ -217,3 +217,69 @@ def greedy(w, cfg, prompt, steps):
     for _ in range(steps):
         tokens.append(int(logits(w, cfg, tokens)[-1].argmax()))
     return tokens[len(prompt):]
+
+
+def random_model(cfg, seed=0, gain=1.5):
+    """bf16 weights of a configuration; ``gain`` sharpens the attention.
+
+    The routers decide clearly: the first columns of the stream hold a random order of the experts for each token (no sublayer and no pass
+    of the loop adds to them) and the routers read mostly these, so that rounding does not send a token to another expert."""
+    g = torch.Generator().manual_seed(seed)
+
+    def rnd(*shape, std=1.0):
+        return (torch.randn(*shape, generator=g) * std).bfloat16()
+
+    def weight(n, around=1.0):
+        return (around * (0.7 + 0.6 * torch.rand(n, generator=g))).bfloat16()
+
+    def gates(x, f, std):
+        return {x + "gate": rnd(f, d, std=std), x + "up": rnd(f, d, std=std), x + "down": rnd(d, f, std=f ** -0.5)}
+    d, V = cfg["width"], cfg["vocab"]
+    w = {"embed": rnd(V, d), "final.norm": weight(d, 0.9 * d ** -0.5 * 1.5)}
+    E = max([l["mlp"]["router"]["experts"] for l in cfg["layers"] if l.get("mlp") and l["mlp"]["kind"] == "moe"], default=0)
+    w["embed"][:, :E] = torch.stack([torch.randperm(E, generator=g) for _ in range(V)]).bfloat16() * (3.0 / max(E, 1)) - 1.5
+    if cfg.get("loop") is not None:
+        w["loop.step"] = rnd(cfg["loop"]["times"], d, std=0.7)
+        w["loop.step"][:, :E] = 0
+    for n, layer in enumerate(cfg["layers"]):
+        m, l, x = layer["mixer"], f"l{n}.", f"l{n}.mix."
+        w[l + "norm1"], w[l + "norm1b"] = weight(d), weight(d, 0.8)
+        w[l + "norm1b"][:E] = 0
+        if layer["type"] == "parallel":
+            s, r = m["left"], m["right"]
+            H, G, dk, dv = s["heads"], s["kv_heads"], s["dim"], s["vdim"]
+            y = x + "left."
+            w[y + "q"], w[y + "k"], w[y + "v"] = rnd(H * dk, d, std=gain * d ** -0.5), rnd(G * dk, d, std=d ** -0.5), rnd(G * dv, d, std=d ** -0.5)
+            w[y + "pb"], w[y + "o"] = rnd(H) - 1.0, rnd(d, H * dv, std=(H * dv) ** -0.5)
+            H, G, e, N = r["heads"], r["groups"], r["vdim"], r["state"]
+            y, ch = x + "right.", H * e + 2 * G * N
+            w[y + "in"] = rnd(H * e + ch + H, d, std=d ** -0.5)
+            w[y + "conv"], w[y + "conv.b"] = rnd(ch, r["conv"], std=0.6), rnd(ch, std=0.3)
+            w[y + "dt_bias"], w[y + "A_log"], w[y + "D"] = rnd(H) - 2.0, rnd(H) - 1.0, rnd(H)
+            w[y + "norm"], w[y + "o"] = weight(H * e), rnd(d, H * e, std=(H * e) ** -0.5)
+        else:
+            H, e, rank = m["heads"], m["dim"], 5 + 3 * n
+            w[x + "r"], w[x + "k"], w[x + "v"], w[x + "g"], w[x + "a"] = (rnd(H * e, d, std=d ** -0.5) for _ in range(5))
+            # a token's key resembles what it reads with: a first token's output is its value times their product, and the norm behind it
+            # would turn a product of about zero into a coin toss
+            w[x + "k"] = (0.8 * w[x + "r"].float() + 0.6 * w[x + "k"].float()).bfloat16()
+            w[x + "a.b"], w[x + "w0"], w[x + "norm"] = rnd(H * e), rnd(H * e, std=2.0) - 3.0, weight(H * e)
+            w[x + "w1"], w[x + "w2"] = rnd(rank, d, std=d ** -0.5), rnd(H * e, rank, std=rank ** -0.5)
+            w[x + "o"] = rnd(d, H * e, std=(H * e) ** -0.5)
+        ff, x = layer.get("mlp"), l + "mlp."
+        if ff is None:
+            continue
+        w[l + "norm2"], w[l + "norm2b"] = weight(d), weight(d, 0.8)
+        w[l + "norm2b"][:E] = 0
+        if ff["kind"] == "dense":
+            w[x + "up"], w[x + "down"], w[x + "act"] = rnd(ff["ff"], d, std=d ** -0.5), rnd(d, ff["ff"], std=ff["ff"] ** -0.5), rnd(2)
+        else:
+            many = ff["router"]["experts"]
+            w[x + "router"] = rnd(many, d, std=0.1 * d ** -0.5)
+            w[x + "router"][torch.arange(many), torch.randperm(E, generator=g)[:many]] = 1.5
+            w[l + "norm2"][:E] = 1.0
+            for e in range(many):
+                w.update(gates(f"{x}e{e}.", ff["expert"]["ff"], 1.5 * d ** -0.5))
+            if ff.get("shared") is not None:
+                w.update(gates(x + "shared.", ff["shared"]["ff"], d ** -0.5))
+    return w
