@@ -73,7 +73,7 @@ def parse():
     p.add_argument("--no-e2e", action="store_true")
     p.add_argument("--serve", action="store_true", help="instead of the training benchmark: prefill / decode throughput and kernel "
                    "times of a served design beside the framework's closest other model at equal size (one GPU)")
-    p.add_argument("--serve-model", choices=["lagisun", "sonodra", "gafonex"], default="lagisun", help="design of --serve")
+    p.add_argument("--serve-model", choices=["lagisun", "sonodra", "gafonex", "zelinex"], default="lagisun", help="design of --serve")
     p.add_argument("--serve-sizes", type=str, default="1b,8b", help="sizes of --serve")
     p.add_argument("--overlap-grad-reduce", action=argparse.BooleanOptionalAction, default=False,
                    help="reduce-scatter the gradients of a block while the backward pass of the blocks before it runs "
@@ -100,7 +100,9 @@ def main():
     if args.impl == "reference":
         return reference_arm()
     if args.serve:
-        if args.serve_model == "gafonex":
+        if args.serve_model == "zelinex":
+            from linear_moe_b200.bench.serve_zelinex import main as serve
+        elif args.serve_model == "gafonex":
             from linear_moe_b200.bench.serve_gafonex import main as serve
         elif args.serve_model == "sonodra":
             from linear_moe_b200.bench.serve_sonodra import main as serve

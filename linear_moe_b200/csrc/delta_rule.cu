@@ -1,10 +1,10 @@
 // Generalized delta rule over packed rows, head by head in fp32,
 //     S <- diag(w) S - (a u)(u^T S) + k v^T,    o = S^T r,    out = o / rms(o) * weight * sigmoid(gate)
 // with the unit key u, decays w = exp(-DECAY sigmoid(W2 tanh(.) + w0)) and rates a = sigmoid(. + bias) per channel:
-//   delta_low_kernel    prompts: tanh of the decay's inner activations (the second projection is a matrix product)
+//   delta_low_kernel    tanh of the decay's inner activations (the second projection is a matrix product)
 //   delta_rows_kernel   prompts of any size, bf16 or fp32, token by token (bf16 fast path: delta_rule_tc.cu), and
 //   delta_norm_kernel   the norm and gate behind it
-//   delta_step_kernel   one token per request, everything in one pass over the state
+//   delta_step_kernel   one token per request, everything else in one pass over the state
 // With the old state S, p = S^T u and q = S^T (w r), the output is o = q - (r . a u) p + (r . k) v: one reduction over the rows of S.
 // Compiled without fast-math: the fp32 instantiations serve models in true 32-bit.
 #include "common.cuh"
@@ -16,14 +16,14 @@ namespace dlt {
 __device__ __forceinline__ float sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
 
 template <typename T>
-__global__ void __launch_bounds__(256) delta_low_kernel(Args a) {
+__global__ void __launch_bounds__(256) delta_low_kernel(const T* __restrict__ z, long long ldz, T* __restrict__ low, long long ldl, int rows, int cols) {
     pdl_trigger();
-    const long long total = (long long)a.rows * (a.rank / 4);
+    const long long total = (long long)rows * (cols / 4);
     for (long long i = blockIdx.x * 256LL + threadIdx.x; i < total; i += gridDim.x * 256LL) {
-        const long long row = i / (a.rank / 4);
-        const int c = (int)(i - row * (a.rank / 4)) * 4;
-        const float4 x = load4((const T*)a.z + row * a.ldz + a.zw + c);
-        store4((T*)a.low + row * a.ldl + c, make_float4(tanhf(x.x), tanhf(x.y), tanhf(x.z), tanhf(x.w)));
+        const long long row = i / (cols / 4);
+        const int c = (int)(i - row * (cols / 4)) * 4;
+        const float4 x = load4(z + row * ldz + c);
+        store4(low + row * ldl + c, make_float4(tanhf(x.x), tanhf(x.y), tanhf(x.z), tanhf(x.w)));
     }
 }
 
@@ -129,119 +129,122 @@ static int launch_rows(const Args& a, cudaStream_t st) {
 }
 
 // ---------------------------------------------------------------------------------------------------------------- one token
-constexpr int ST = 512, NW = ST / 32;
-
 // grid (H, n).  A thread owns 4 columns of the state and every `parts`-th row (parts = ST / (d / 4)); the first NB of them stay in registers
-// between the reduction and the update.  staged: the head's rows of w2 lie in shared memory.
-template <typename T>
-__global__ void __launch_bounds__(ST) delta_step_kernel(Args a, int staged) {
-    constexpr int NB = 8;
+// between the reduction and the update.
+template <typename T, int ST>
+__global__ void __launch_bounds__(ST, ST == 256 ? 5 : 2) delta_step_kernel(Args a) {
+    constexpr int NB = ST == 256 ? 4 : 8, NW = ST / 32;
     extern __shared__ float4 sm4[];
-    const int h = blockIdx.x, b = blockIdx.y, d = a.d, rank = a.rank;
-    const int cols = d / 4, parts = ST / cols, c = threadIdx.x % cols * 4, r0 = threadIdx.x / cols;
-    float* P = reinterpret_cast<float*>(sm4);                // [parts][d] partial p, then
-    float* Q = P + parts * d;                                // [parts][d] partial q
-    float* R = Q + parts * d;                                // [d]
-    float* K = R + d;
-    float* U = K + d;
-    float* A = U + d;                                        // a u
-    float* W = A + d;
-    float* L = W + d;                                        // [rank]
-    T* W2 = reinterpret_cast<T*>(L + rank);                  // [d][rank]
-    __shared__ float red[32];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int h = blockIdx.x, b = blockIdx.y, d = a.d, i = threadIdx.x;
+    const int cols = d / 4, parts = ST / cols, c = i % cols * 4, r0 = i / cols, warp = i >> 5, lane = i & 31;
+    const bool pairs = 32 % cols == 0;                       // threads of a warp that share columns add up among themselves
+    const int partial = pairs ? NW : parts;
+    float* P = reinterpret_cast<float*>(sm4);                // [partial][d] partial p
+    float* Q = P + partial * d;                              // [partial][d] partial q
+    float* U = Q + partial * d;                              // [d] u
+    float* F = U + d;                                        // [d] w r
+    float* W = F + d;                                        // [d]
+    float* A = W + d;                                        // [d] a k (a u without the key's length)
+    float* K = A + d;                                        // [d]
+    float* Ps = K + d;                                       // [d] p
+    __shared__ float red[4][NW];
     const bool on = r0 < parts;
-    // the state is older than the kernel before this one, and weights do not change
+    // the state is older than the kernel before this one
     const bool fresh = a.pos[b] == 0;
     float* S = a.state + ((long long)a.slots[b] * a.H + h) * d * d;
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
     float4 s[NB];
 #pragma unroll
-    for (int i = 0; i < NB; ++i) {
-        const int r = r0 + i * parts;
-        s[i] = on && r < d && !fresh ? *reinterpret_cast<const float4*>(S + (long long)r * d + c) : zero;
+    for (int k = 0; k < NB; ++k) {
+        const int r = r0 + k * parts;
+        s[k] = on && r < d && !fresh ? *reinterpret_cast<const float4*>(S + (long long)r * d + c) : zero;
     }
-    const T* w2 = (const T*)a.w2 + (long long)h * d * rank;
-    if (staged)
-        for (int i = threadIdx.x * 4; i < d * rank; i += ST * 4) store4(W2 + i, load4(w2 + i));
     pdl_trigger();
     asm volatile("griddepcontrol.wait;" ::: "memory");
     const T* z = (const T*)a.z + (long long)b * a.ldz + h * d;
-    float ks = 0.f;
-    for (int i = threadIdx.x; i < d; i += ST) {
-        const float k = to_f(z[a.zk + i]);
-        R[i] = to_f(z[a.zr + i]);
-        K[i] = k;
-        A[i] = sigmoid(to_f(z[a.za + i]) + a.a_bias[h * d + i]);
-        ks += k * k;
+    float kk = 0.f, ra = 0.f, rk = 0.f, v = 0.f, gate = 0.f; // d <= ST: a thread has one channel
+    if (i < d) {
+        const float k = to_f(z[a.zk + i]), r = to_f(z[a.zr + i]), m = sigmoid(to_f(z[a.za + i]) + a.a_bias[h * d + i]) * k;
+        const float w = expf(-DECAY * sigmoid(a.w[(long long)b * a.ldw + h * d + i] + a.w0[h * d + i]));
+        v = to_f(z[a.zv + i]);
+        gate = a.norm[h * d + i] * sigmoid(to_f(z[a.zg + i]));
+        U[i] = K[i] = k;
+        F[i] = w * r;
+        W[i] = w;
+        A[i] = m;
+        kk = k * k, ra = r * m, rk = r * k;
     }
-    for (int i = threadIdx.x; i < rank; i += ST) L[i] = tanhf(to_f(((const T*)a.z + (long long)b * a.ldz + a.zw)[i]));
-    const float inv = 1.f / sqrtf(block_sum(ks, red) + UNIT_EPS);        // (its barriers also cover R, K, A and L)
-    const T* rows = staged ? W2 : w2;
-    for (int i = warp; i < d; i += NW) {
-        float x = 0.f;
-        for (int k = lane; k < rank; k += 32) x += L[k] * to_f(rows[(long long)i * rank + k]);
-        x = warp_sum(x);
-        if (lane == 0) {
-            W[i] = expf(-DECAY * sigmoid(x + a.w0[h * d + i]));
-            U[i] = K[i] * inv;
-            A[i] *= K[i] * inv;
-        }
+    if (warp * 32 < d) {
+        kk = warp_sum(kk), ra = warp_sum(ra), rk = warp_sum(rk);
+        if (lane == 0) red[0][warp] = kk, red[1][warp] = ra, red[2][warp] = rk;
     }
     __syncthreads();
+    kk = ra = rk = 0.f;
+    for (int k = 0; k * 32 < d; ++k) kk += red[0][k], ra += red[1][k], rk += red[2][k];
+    const float inv = 1.f / sqrtf(kk + UNIT_EPS);
+    // with p of the key as it is: u = inv k, so p_u = inv p and a u p_u = inv^2 (a k) p
     float4 p = zero, q = zero;
     auto gather = [&](float4 x, int r) {
-        const float u = U[r], f = W[r] * R[r];
+        const float u = U[r], f = F[r];
         p.x += u * x.x; p.y += u * x.y; p.z += u * x.z; p.w += u * x.w;
         q.x += f * x.x; q.y += f * x.y; q.z += f * x.z; q.w += f * x.w;
     };
     if (on) {
 #pragma unroll
-        for (int i = 0; i < NB; ++i)
-            if (r0 + i * parts < d) gather(s[i], r0 + i * parts);
+        for (int k = 0; k < NB; ++k)
+            if (r0 + k * parts < d) gather(s[k], r0 + k * parts);
         if (!fresh)
             for (int r = r0 + NB * parts; r < d; r += parts) gather(*reinterpret_cast<const float4*>(S + (long long)r * d + c), r);
-        *reinterpret_cast<float4*>(P + r0 * d + c) = p;
-        *reinterpret_cast<float4*>(Q + r0 * d + c) = q;
     }
-    float ra = 0.f, rk = 0.f;                                // r . a u, r . k
-    for (int i = threadIdx.x; i < d; i += ST) ra += R[i] * A[i], rk += R[i] * K[i];
-    ra = block_sum(ra, red);
-    rk = block_sum(rk, red);                                 // (the barriers also cover P and Q)
-    float y = 0.f;                                           // d <= ST: a thread finishes one column
-    if (threadIdx.x < d) {
-        float ps = 0.f, qs = 0.f;
-        for (int r = 0; r < parts; ++r) ps += P[r * d + threadIdx.x], qs += Q[r * d + threadIdx.x];
-        y = qs - ra * ps + rk * to_f(z[a.zv + threadIdx.x]);
-        Q[threadIdx.x] = ps;                                 // nobody else reads this column's partial q
+    if (pairs)
+        for (int k = cols; k < 32; k <<= 1) {
+            p.x += __shfl_xor_sync(0xffffffffu, p.x, k); p.y += __shfl_xor_sync(0xffffffffu, p.y, k);
+            p.z += __shfl_xor_sync(0xffffffffu, p.z, k); p.w += __shfl_xor_sync(0xffffffffu, p.w, k);
+            q.x += __shfl_xor_sync(0xffffffffu, q.x, k); q.y += __shfl_xor_sync(0xffffffffu, q.y, k);
+            q.z += __shfl_xor_sync(0xffffffffu, q.z, k); q.w += __shfl_xor_sync(0xffffffffu, q.w, k);
+        }
+    if (pairs ? lane < cols : on) {
+        *reinterpret_cast<float4*>(P + (pairs ? warp : r0) * d + c) = p;
+        *reinterpret_cast<float4*>(Q + (pairs ? warp : r0) * d + c) = q;
     }
-    const float rms = 1.f / sqrtf(block_sum(y * y, red) / a.nd + a.eps);
-    if (threadIdx.x < d) {
-        const int i = h * d + threadIdx.x;
-        ((T*)a.out)[(long long)b * a.ldo + i] = from_f<T>(y * rms * a.norm[i] * sigmoid(to_f(z[a.zg + threadIdx.x])));
+    __syncthreads();
+    float y = 0.f;
+    if (warp * 32 < d) {
+        if (i < d) {                                         // this thread's column
+            float ps = 0.f, qs = 0.f;
+            for (int r = 0; r < partial; ++r) ps += P[r * d + i], qs += Q[r * d + i];
+            ps *= inv * inv;
+            y = qs - ra * ps + rk * v;
+            Ps[i] = ps;
+        }
+        const float s2 = warp_sum(y * y);
+        if (lane == 0) red[3][warp] = s2;
+    }
+    __syncthreads();
+    if (i < d) {
+        float s2 = 0.f;
+        for (int k = 0; k * 32 < d; ++k) s2 += red[3][k];
+        ((T*)a.out)[(long long)b * a.ldo + h * d + i] = from_f<T>(y / sqrtf(s2 / a.nd + a.eps) * gate);
     }
     if (!on) return;
-    p = *reinterpret_cast<const float4*>(Q + c);
-    const float4 v = load4(z + a.zv + c);
+    p = *reinterpret_cast<const float4*>(Ps + c);
+    const float4 vs = load4(z + a.zv + c);
     auto update = [&](float4 x, int r) {
         const float w = W[r], m = A[r], k = K[r];
-        x = make_float4(w * x.x - m * p.x + k * v.x, w * x.y - m * p.y + k * v.y, w * x.z - m * p.z + k * v.z, w * x.w - m * p.w + k * v.w);
+        x = make_float4(w * x.x - m * p.x + k * vs.x, w * x.y - m * p.y + k * vs.y, w * x.z - m * p.z + k * vs.z, w * x.w - m * p.w + k * vs.w);
         *reinterpret_cast<float4*>(S + (long long)r * d + c) = x;
     };
 #pragma unroll
-    for (int i = 0; i < NB; ++i)
-        if (r0 + i * parts < d) update(s[i], r0 + i * parts);
+    for (int k = 0; k < NB; ++k)
+        if (r0 + k * parts < d) update(s[k], r0 + k * parts);
     for (int r = r0 + NB * parts; r < d; r += parts) update(fresh ? zero : *reinterpret_cast<const float4*>(S + (long long)r * d + c), r);
 }
 
-template <typename T>
+template <typename T, int ST>
 static int launch_step(const Args& a, cudaStream_t st) {
-    const size_t base = sizeof(float) * (2 * (ST / (a.d / 4)) * a.d + 5 * a.d + a.rank), table = sizeof(T) * (size_t)a.d * a.rank;
-    const int staged = base + table <= 100 * 1024;
-    const size_t smem = base + (staged ? table : 0);
-    if (smem > 200 * 1024) return -2;
-    cudaError_t e = cudaFuncSetAttribute(delta_step_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e != cudaSuccess) return (int)e;
+    const int cols = a.d / 4, partial = 32 % cols == 0 ? ST / 32 : ST / cols;
+    const size_t smem = sizeof(float) * (2 * partial + 6) * a.d;
+    if (smem > 46 * 1024) return -2;
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(a.H, a.n);
     cfg.blockDim = dim3(ST);
@@ -252,14 +255,14 @@ static int launch_step(const Args& a, cudaStream_t st) {
     attr[0].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
     cfg.numAttrs = 1;
-    return (int)cudaLaunchKernelEx(&cfg, delta_step_kernel<T>, a, staged);
+    return (int)cudaLaunchKernelEx(&cfg, delta_step_kernel<T, ST>, a);
 }
 
 static bool aligned(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
 static bool ok(const Args& a, int dt) {
     const int w = dt ? 8 : 4;
-    return a.rows > 0 && a.H > 0 && a.d > 0 && a.d % 16 == 0 && a.nd > 0 && a.nd <= a.d && a.rank > 0 && a.rank % 32 == 0 && a.ldz % w == 0 && a.ldo % w == 0 &&
-           ((a.zr | a.zk | a.zv | a.za | a.zg | a.zw) & 7) == 0 && aligned(a.z) && aligned(a.out) && aligned(a.state) && aligned(a.w2);
+    return a.rows > 0 && a.H > 0 && a.d > 0 && a.d % 16 == 0 && a.nd > 0 && a.nd <= a.d && a.ldz % w == 0 && a.ldo % w == 0 &&
+           ((a.zr | a.zk | a.zv | a.za | a.zg) & 7) == 0 && aligned(a.z) && aligned(a.out) && aligned(a.state);
 }
 
 }  // namespace dlt
@@ -267,14 +270,13 @@ static bool ok(const Args& a, int dt) {
 
 using namespace lmoe;
 
-// z -> low; dt: 1 bf16, 0 fp32
-LMOE_API int lmoe_delta_low(const dlt::Args* ap, int dt, cudaStream_t st) {
-    const dlt::Args& a = *ap;
-    if (!dlt::ok(a, dt) || a.low == nullptr || a.ldl % 4) return -1;
-    const long long blocks = ((long long)a.rows * (a.rank / 4) + 255) / 256;
+// z [rows, ldz] -> low [rows, ldl], cols a multiple of 4; dt: 1 bf16, 0 fp32
+LMOE_API int lmoe_delta_low(const void* z, long long ldz, void* low, long long ldl, int rows, int cols, int dt, cudaStream_t st) {
+    if (rows <= 0 || cols <= 0 || cols % 4 || ldz % 4 || ldl % 4 || !dlt::aligned(z) || !dlt::aligned(low)) return -1;
+    const long long blocks = ((long long)rows * (cols / 4) + 255) / 256;
     const unsigned grid = (unsigned)(blocks < 148 * 16 ? blocks : 148 * 16);
-    if (dt) dlt::delta_low_kernel<bf16><<<grid, 256, 0, st>>>(a);
-    else dlt::delta_low_kernel<float><<<grid, 256, 0, st>>>(a);
+    if (dt) dlt::delta_low_kernel<bf16><<<grid, 256, 0, st>>>((const bf16*)z, ldz, (bf16*)low, ldl, rows, cols);
+    else dlt::delta_low_kernel<float><<<grid, 256, 0, st>>>((const float*)z, ldz, (float*)low, ldl, rows, cols);
     return (int)cudaGetLastError();
 }
 
@@ -289,6 +291,7 @@ LMOE_API int lmoe_delta_rows(const dlt::Args* ap, int dt, cudaStream_t st) {
 // device before the kernel that precedes this one in the stream was launched.
 LMOE_API int lmoe_delta_step(const dlt::Args* ap, int dt, cudaStream_t st) {
     const dlt::Args& a = *ap;
-    if (!dlt::ok(a, dt) || a.n != a.rows || a.d > 256 || a.state == nullptr || a.w2 == nullptr) return -1;
-    return dt ? dlt::launch_step<bf16>(a, st) : dlt::launch_step<float>(a, st);
+    if (!dlt::ok(a, dt) || a.n != a.rows || a.d > 256 || a.state == nullptr || a.w == nullptr) return -1;
+    if (a.d <= 64) return dt ? dlt::launch_step<bf16, 256>(a, st) : dlt::launch_step<float, 256>(a, st);
+    return dt ? dlt::launch_step<bf16, 512>(a, st) : dlt::launch_step<float, 512>(a, st);
 }

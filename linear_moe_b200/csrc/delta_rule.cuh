@@ -9,21 +9,19 @@ constexpr float DECAY = 0.60653065971263342f;               // exp(-1/2): a chan
 constexpr float UNIT_EPS = 1e-6f;                            // in the length of a key
 
 struct Args {
-    const void* z;                       // [rows, ldz]: r, k, v, removal rate, gate (H x d each) and the decay's inner activations (rank)
+    const void* z;                       // [rows, ldz]: r, k, v, removal rate, gate (H x d each)
     void* out;                           // [rows, ldo]: H x d
-    const float* w;                      // [rows, ldw]: second projection of the decay (prompts)
-    void* low;                           // [rows, ldl]: tanh of the inner activations (prompts)
-    const void* w2;                      // [H * d, rank] (one token)
+    const float* w;                      // [rows, ldw]: second projection of the decay
     const float *w0, *a_bias, *norm;     // [H * d]
     float* state;                        // [slots, H, d, d] or null
     float* raw;                          // general kernel: [rows, H * d]
     void* work;                          // tensor-core kernels: what the chunks leave for the pass over them
     const int *pos, *slots;              // [rows]
     const int* groups;                   // [n, 8]
-    long long ldz, ldo, ldw, ldl;
-    int zr, zk, zv, za, zg, zw, H, d;
+    long long ldz, ldo, ldw;
+    int zr, zk, zv, za, zg, H, d;
     int nd;                              // a head's numbers without padding
-    int rank, rows, n;
+    int rows, n;
     float eps;
 };
 

@@ -6,7 +6,7 @@
 //   ssd_step_kernel   one token per request: convolution, step size and state update in one pass over the state
 //   ssd_norm_kernel   y silu(z) over the root mean square of its part of the row, times weight and factor
 // Compiled without fast-math: the fp32 instantiations serve models in true 32-bit.
-#include "common.cuh"
+#include "mma_utils.cuh"
 #include "ssd.cuh"
 
 namespace lmoe {
@@ -180,92 +180,128 @@ static int launch_scan(const Args& a, cudaStream_t st) {
 }
 
 // ---------------------------------------------------------------------------------------------------------------- one token
-constexpr int ST = 256;
+constexpr int ST = 256, SW = ST / 32;
 
-// grid (H, n).  A thread owns 4 columns of the state and every `parts`-th row (parts = ST / (dv / 4)), NB of them in flight.
+// How a CTA goes over a state: a thread owns 4 columns and every `parts`-th row, `slots` of them.
+struct StepShape {
+    int cols, parts, slots, partial;     // partial: rows of partial sums over the state's rows that meet in shared memory
+    __host__ __device__ StepShape(int dn, int dv) {
+        cols = dv / 4, parts = ST / cols, slots = (dn + parts - 1) / parts;
+        partial = 32 % cols == 0 ? SW : parts;               // (threads of a warp that share columns add up among themselves)
+    }
+    __host__ __device__ int stage() const { return slots * ST * 16; }
+    __host__ __device__ int rest(int dn, int dv, int heads) const { return 4 * (heads * dv + 2 * dn + 2 * partial * dv); }
+};
+
+// grid (H / heads, n): `heads` heads of one group, one after the other; while one is worked on, the next one's state is on its way into
+// shared memory (every thread waits for its own pieces only).
 template <typename T>
-__global__ void __launch_bounds__(ST) ssd_step_kernel(Args a) {
-    constexpr int NB = 8;
+__global__ void __launch_bounds__(ST, 3) ssd_step_kernel(Args a, int heads) {
     extern __shared__ float4 sm4[];
-    const int h = blockIdx.x, b = blockIdx.y, dn = a.dn, dv = a.dv, g = h / (a.H / a.G), ch = a.channels();
-    const int cols = dv / 4, parts = ST / cols, c = threadIdx.x % cols * 4, r0 = threadIdx.x / cols;
-    float* O = reinterpret_cast<float*>(sm4);                // [parts][dv]
-    float* X = O + parts * dv;                               // [dv]
-    float* B = X + dv;                                       // [dn]
+    const int h0 = blockIdx.x * heads, b = blockIdx.y, dn = a.dn, dv = a.dv, g = h0 / (a.H / a.G), ch = a.channels();
+    const StepShape sh(dn, dv);
+    const int c = threadIdx.x % sh.cols * 4, r0 = threadIdx.x / sh.cols, warp = threadIdx.x >> 5, stages = heads > 1 ? 2 : 1;
+    float4* stage = sm4 + threadIdx.x;                       // [stages][slots][ST]
+    float* X = reinterpret_cast<float*>(sm4 + stages * sh.slots * ST);   // [heads][dv]
+    float* B = X + heads * dv;                               // [dn]
     float* C = B + dn;                                       // [dn]
-    const bool on = r0 < parts;
+    float* O = C + dn;                                       // [2][partial][dv]
+    const bool on = r0 < sh.parts;
     // slots and positions, the state and the convolution's past are older than the kernel before this one
     const int pos = a.pos[b], slot = a.slots[b];
     const bool fresh = pos == 0;
-    float* S = a.state + ((long long)slot * a.H + h) * dn * dv;
-    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-    float4 s[NB];
-#pragma unroll
-    for (int i = 0; i < NB; ++i) {
-        const int r = r0 + i * parts;
-        s[i] = on && r < dn && !fresh ? *reinterpret_cast<const float4*>(S + (long long)r * dv + c) : zero;
-    }
+    float* S = a.state + ((long long)slot * a.H + h0) * dn * dv;
+    auto fetch = [&](int i) {                                // head h0 + i
+        if (i < heads && on && !fresh) {
+            const float* p = S + (long long)i * dn * dv;
+            for (int k = 0, r = r0; r < dn; ++k, r += sh.parts)
+                cp_async16(stage + ((i & (stages - 1)) * sh.slots + k) * ST, p + (long long)r * dv + c, true);
+        }
+        cp_async_commit();
+    };
+    fetch(0);
     T* tail = (T*)a.tail + (long long)slot * a.ring * ch;
-    const int back = min(a.taps - 1, pos);                   // inputs the convolution sees besides the token's own
-    float pre = 0.f;                                         // what they add up to for this thread's first channel
-    auto channel = [&](int i) { return i < dv ? h * dv + i : i < dv + dn ? a.H * dv + g * dn + i - dv : a.H * dv + (a.G + g) * dn + i - dv - dn; };
+    const int back = min(a.taps - 1, pos), own = heads * dv; // inputs the convolution sees besides the token's own
+    auto channel = [&](int i) { return i < own ? h0 * dv + i : i < own + dn ? a.H * dv + g * dn + i - own : a.H * dv + (a.G + g) * dn + i - own - dn; };
     auto older = [&](int k) {
         float v = a.conv_bias[k];
         for (int n = back; n > 0; --n) v += a.conv[(long long)(a.taps - 1 - n) * ch + k] * to_f(tail[(long long)((pos - n) % a.ring) * ch + k]);
         return v;
     };
-    const int numbers = dv + 2 * dn;
-    if (threadIdx.x < numbers) pre = older(channel(threadIdx.x));
-    const float a_exp = expf(a.a_log[h]), D = a.d[h], bias = a.dt_bias[h];
+    const int numbers = own + 2 * dn;
+    float pre[2];                                            // what they add up to for this thread's first channels
+    pre[0] = threadIdx.x < numbers ? older(channel(threadIdx.x)) : 0.f;
+    pre[1] = threadIdx.x + ST < numbers ? older(channel(threadIdx.x + ST)) : 0.f;
     pdl_trigger();
     asm volatile("griddepcontrol.wait;" ::: "memory");
     const T* z = (const T*)a.z + (long long)b * a.ldz;
-    for (int i = threadIdx.x; i < numbers; i += ST) {
+    for (int i = threadIdx.x, n = 0; i < numbers; i += ST, ++n) {
         const int k = channel(i);
         const T x = z[a.zx + k];
-        const float v = (i < ST ? pre : older(k)) + a.conv[(long long)(a.taps - 1) * ch + k] * to_f(x);
+        const float v = (n == 0 ? pre[0] : n == 1 ? pre[1] : older(k)) + a.conv[(long long)(a.taps - 1) * ch + k] * to_f(x);
         X[i] = to_f(from_f<T>(silu(v)));
         // a ring of `taps` rows: the place of this input is none that another CTA still reads
-        if (i < dv || h % (a.H / a.G) == 0) tail[(long long)(pos % a.ring) * ch + k] = x;
+        if (i < own || h0 % (a.H / a.G) == 0) tail[(long long)(pos % a.ring) * ch + k] = x;
     }
-    const float dt = softplus(to_f(z[a.zdt + h]) + bias), decay = expf(-a_exp * dt);
     __syncthreads();
-    float4 v = zero, o = zero;
-    if (on) v = load4(X + c);
-    v = make_float4(v.x * dt, v.y * dt, v.z * dt, v.w * dt);
-    for (int rb = r0; on && rb < dn; rb += NB * parts) {
-#pragma unroll
-        for (int i = 0; i < NB; ++i) {
-            const int r = rb + i * parts;
-            if (r < dn) {
-                const float k = B[r], q = C[r];
-                s[i].x = decay * s[i].x + k * v.x; s[i].y = decay * s[i].y + k * v.y;
-                s[i].z = decay * s[i].z + k * v.z; s[i].w = decay * s[i].w + k * v.w;
-                *reinterpret_cast<float4*>(S + (long long)r * dv + c) = s[i];
-                o.x += q * s[i].x; o.y += q * s[i].y; o.z += q * s[i].z; o.w += q * s[i].w;
+    for (int i = 0; i < heads; ++i) {
+        const int h = h0 + i;
+        if (stages > 1) fetch(i + 1);
+        const float dt = softplus(to_f(z[a.zdt + h]) + a.dt_bias[h]), decay = expf(-expf(a.a_log[h]) * dt);
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f), o = v;
+        if (on) v = load4(X + i * dv + c);
+        v = make_float4(v.x * dt, v.y * dt, v.z * dt, v.w * dt);
+        if (stages > 1) cp_async_wait<1>();
+        else cp_async_wait<0>();
+        if (on) {
+            const float4* from = stage + (i & (stages - 1)) * sh.slots * ST;
+            float* to = S + (long long)i * dn * dv + c;
+#pragma unroll 8
+            for (int k = 0; k < sh.slots; ++k) {
+                const int r = r0 + k * sh.parts;
+                if (r < dn) {
+                    float4 s = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : from[k * ST];
+                    const float in = B[r], q = C[r];
+                    s = make_float4(decay * s.x + in * v.x, decay * s.y + in * v.y, decay * s.z + in * v.z, decay * s.w + in * v.w);
+                    *reinterpret_cast<float4*>(to + (long long)r * dv) = s;
+                    o.x += q * s.x; o.y += q * s.y; o.z += q * s.z; o.w += q * s.w;
+                }
             }
         }
-#pragma unroll
-        for (int i = 0; i < NB; ++i) {
-            const int r = rb + (NB + i) * parts;
-            if (r < dn) s[i] = fresh ? zero : *reinterpret_cast<const float4*>(S + (long long)r * dv + c);
+        bool writes = on;
+        int at = r0;
+        if (sh.partial == SW && 32 % sh.cols == 0) {
+            for (int k = sh.cols; k < 32; k <<= 1) {
+                o.x += __shfl_xor_sync(0xffffffffu, o.x, k); o.y += __shfl_xor_sync(0xffffffffu, o.y, k);
+                o.z += __shfl_xor_sync(0xffffffffu, o.z, k); o.w += __shfl_xor_sync(0xffffffffu, o.w, k);
+            }
+            writes = (threadIdx.x & 31) < sh.cols;
+            at = warp;
         }
-    }
-    if (on) *reinterpret_cast<float4*>(O + r0 * dv + c) = o;
-    __syncthreads();
-    if (threadIdx.x < dv) {                                  // dv <= ST: a thread finishes one column
-        float y = D * X[threadIdx.x];
-        for (int r = 0; r < parts; ++r) y += O[r * dv + threadIdx.x];
-        ((float*)a.y)[b * a.ldy + h * dv + threadIdx.x] = y;
+        float* part = O + (i & 1) * sh.partial * dv;
+        if (writes) *reinterpret_cast<float4*>(part + at * dv + c) = o;
+        __syncthreads();
+        if (threadIdx.x < dv) {                              // dv <= ST: a thread finishes one column
+            float y = a.d[h] * X[i * dv + threadIdx.x];
+            for (int r = 0; r < sh.partial; ++r) y += part[r * dv + threadIdx.x];
+            ((float*)a.y)[b * a.ldy + h * dv + threadIdx.x] = y;
+        }
     }
 }
 
 template <typename T>
-static int launch_step(const Args& a, cudaStream_t st) {
-    const size_t smem = sizeof(float) * (a.dv + 2 * a.dn + ST / (a.dv / 4) * a.dv);
-    if (smem > 46 * 1024) return -2;
+static int launch_step(const Args& a, int sms, cudaStream_t st) {
+    const StepShape sh(a.dn, a.dv);
+    // several heads per CTA once there are more CTAs than fit the GPU at a time
+    int heads = 1;
+    const int each = a.H / a.G;
+    while (each % (2 * heads) == 0 && (long long)a.H * a.n >= 6LL * heads * sms && 2 * sh.stage() + sh.rest(a.dn, a.dv, 2 * heads) <= 74 * 1024) heads *= 2;
+    const int smem = (heads > 1 ? 2 : 1) * sh.stage() + sh.rest(a.dn, a.dv, heads);
+    if (smem > 220 * 1024) return -2;
+    cudaError_t e = cudaFuncSetAttribute(ssd_step_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return (int)e;
     cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3(a.H, a.n);
+    cfg.gridDim = dim3(a.H / heads, a.n);
     cfg.blockDim = dim3(ST);
     cfg.dynamicSmemBytes = smem;
     cfg.stream = st;
@@ -274,7 +310,7 @@ static int launch_step(const Args& a, cudaStream_t st) {
     attr[0].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
     cfg.numAttrs = 1;
-    return (int)cudaLaunchKernelEx(&cfg, ssd_step_kernel<T>, a);
+    return (int)cudaLaunchKernelEx(&cfg, ssd_step_kernel<T>, a, heads);
 }
 
 // ------------------------------------------------------------------------------------------------------------- gate and norm
@@ -390,12 +426,12 @@ LMOE_API int lmoe_ssd_scan(const ssd::Args* ap, int dt, cudaStream_t st) {
     return dt ? ssd::launch_scan<bf16>(a, st) : ssd::launch_scan<float>(a, st);
 }
 
-// One token per request, state and tail in place, y fp32: dv <= 256; rows with position 0 start from zero.  Slots and positions must have been
+// One token per request, state and tail in place, y fp32: dv <= 256, a state of up to 192 KB; rows with position 0 start from zero.  Slots and positions must have been
 // on the device before the kernel that precedes this one in the stream was launched.
-LMOE_API int lmoe_ssd_step(const ssd::Args* ap, int dt, cudaStream_t st) {
+LMOE_API int lmoe_ssd_step(const ssd::Args* ap, int dt, int sms, cudaStream_t st) {
     const ssd::Args& a = *ap;
-    if (!ssd::ok(a, dt) || a.n != a.rows || a.dv > 256 || a.state == nullptr || a.tail == nullptr || !a.y_f32) return -1;
-    return dt ? ssd::launch_step<bf16>(a, st) : ssd::launch_step<float>(a, st);
+    if (sms <= 0 || !ssd::ok(a, dt) || a.n != a.rows || a.dv > 256 || a.state == nullptr || a.tail == nullptr || !a.y_f32) return -1;
+    return dt ? ssd::launch_step<bf16>(a, sms, st) : ssd::launch_step<float>(a, sms, st);
 }
 
 // y, z -> out

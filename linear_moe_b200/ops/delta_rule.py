@@ -16,7 +16,7 @@ from typing import Optional
 import torch
 
 from ..ref import delta_rule as RD
-from .packed_attn import _fields, _no_grad, _ptr
+from .packed_attn import _fields, _no_grad
 from .retention import CHUNK
 from .row_batch import RowBatch, round_up
 
@@ -63,8 +63,17 @@ _P, _LL, _I, _F = ctypes.c_void_p, ctypes.c_longlong, ctypes.c_int, ctypes.c_flo
 
 
 class _Args(ctypes.Structure):
-    _fields_ = _fields(a=(_P, "z out w low w2 w0 a_bias norm state raw work pos slots groups"), b=(_LL, "ldz ldo ldw ldl"),
-                       c=(_I, "zr zk zv za zg zw H d nd rank rows n"), d=(_F, "eps"))
+    _fields_ = _fields(a=(_P, "z out w w0 a_bias norm state raw work pos slots groups"), b=(_LL, "ldz ldo ldw"),
+                       c=(_I, "zr zk zv za zg H d nd rows n"), d=(_F, "eps"))
+
+
+def decay_rows(z, lay: DeltaLayout, s: GeneralDeltaSpec, w2) -> torch.Tensor:
+    """What the decays are made of (``w0`` aside), ``[rows, heads * d]`` in fp32: the second projection of tanh of the first one's columns."""
+    from . import cuda as K
+    from . import linear_f32
+    ld, low = ctypes.c_longlong, torch.empty(z.shape[0], s.low, dtype=z.dtype, device=z.device)
+    K._check(K.lib().lmoe_delta_low(K._p(z[:, lay.w:]), ld(z.stride(0)), K._p(low), ld(s.low), z.shape[0], s.low, K._dt(z), K._st()), "delta_low")
+    return linear_f32(low, w2)
 
 
 def general_delta_rows(z, out, lay: DeltaLayout, s: GeneralDeltaSpec, w2, p: dict, eps: float, batch: RowBatch, cache: Optional[dict]):
@@ -73,28 +82,24 @@ def general_delta_rows(z, out, lay: DeltaLayout, s: GeneralDeltaSpec, w2, p: dic
     if not z.is_cuda:
         return RD.general_delta_rows(z, out, lay, s, w2, p, eps, batch, cache)
     from . import cuda as K
-    from . import linear_f32
     _no_grad(z)
     dev, dt, H, d, rows = z.device, K._dt(z), s.heads, s.d, z.shape[0]
     assert out.dtype == z.dtype == w2.dtype and z.stride(1) == out.stride(1) == w2.stride(1) == 1 and rows == out.shape[0] == batch.rows
     assert all(t.dtype == torch.float32 and t.is_contiguous() and t.shape == (H * d,) for t in p.values())
     a = _Args()
     a.z, a.out, a.ldz, a.ldo, a.rows = z.data_ptr(), out.data_ptr(), z.stride(0), out.stride(0), rows
-    a.w2, a.w0, a.a_bias, a.norm = w2.data_ptr(), *(p[n].data_ptr() for n in ("w0", "a_bias", "norm"))
+    a.w0, a.a_bias, a.norm = (p[n].data_ptr() for n in ("w0", "a_bias", "norm"))
     a.pos, a.slots = batch.pos.data_ptr(), batch.slot.data_ptr()
-    a.zr, a.zk, a.zv, a.za, a.zg, a.zw, a.H, a.d, a.nd, a.rank, a.eps = lay.r, lay.k, lay.v, lay.a, lay.g, lay.w, H, d, s.dim, s.low, eps
+    a.zr, a.zk, a.zv, a.za, a.zg, a.H, a.d, a.nd, a.eps = lay.r, lay.k, lay.v, lay.a, lay.g, H, d, s.dim, eps
     if cache is not None:
         assert cache["s"].is_contiguous() and cache["s"].shape[1:] == (H, d, d)
         a.state = cache["s"].data_ptr()
+    decay = decay_rows(z, lay, s, w2)
+    a.w, a.ldw = decay.data_ptr(), decay.stride(0)
     if batch.decode and d <= 256:
         a.n = rows
         K._check(K.lib().lmoe_delta_step(ctypes.byref(a), dt, K._st()), "delta_step")
         return
-    low = torch.empty(rows, s.low, dtype=z.dtype, device=dev)
-    a.low, a.ldl = low.data_ptr(), s.low
-    K._check(K.lib().lmoe_delta_low(ctypes.byref(a), dt, K._st()), "delta_low")
-    decay = linear_f32(low, w2)
-    a.w, a.ldw = decay.data_ptr(), decay.stride(0)
     if dt == 1 and not batch.decode and d <= 128:
         table, chunks = batch.recurrent_chunks(CHUNK)
         size = K.lib().lmoe_delta_tc_work

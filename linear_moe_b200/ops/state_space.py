@@ -16,9 +16,12 @@ from typing import Optional
 import torch
 
 from ..ref import state_space as RS
-from .packed_attn import _fields, _no_grad, _ptr
+from .packed_attn import _fields, _no_grad
 from .retention import CHUNK
 from .row_batch import RowBatch, round_up
+
+
+STEP_STATE = 40 * 1024         # numbers of a head's state that the one-token kernel keeps in shared memory
 
 
 @dataclass(frozen=True)
@@ -87,12 +90,24 @@ def ssd_rows(z, out, lay: SsdLayout, s: SsdSpec, w: dict, mul: float, eps: float
     the requests' states and the inputs of the convolution (row = position modulo taps)."""
     if not z.is_cuda:
         return RS.ssd_rows(z, out, lay, s, w, mul, eps, batch, cache)
+    steps, _ = launches(z, out, lay, s, w, mul, eps, batch, cache)
+    for step in steps:
+        launch(*step)
+
+
+def launch(name: str, a: _Args, n: int, *more):
+    from . import cuda as K
+    K._check(getattr(K.lib(), "lmoe_" + name)(ctypes.byref(a), *more, K._st()), name, n)
+
+
+def launches(z, out, lay: SsdLayout, s: SsdSpec, w: dict, mul: float, eps: float, batch: RowBatch, cache: Optional[dict]):
+    """What ``ssd_rows`` launches, as arguments of ``launch``, and the buffers that lie between the kernels."""
     from . import cuda as K
     _no_grad(z)
     dev, dt, H, dn, dv, rows = z.device, K._dt(z), s.heads, s.dn, s.dv, z.shape[0]
     assert out.dtype == z.dtype and z.stride(1) == out.stride(1) == 1 and rows == out.shape[0] == batch.rows
     assert all(t.dtype == torch.float32 and t.is_contiguous() for t in w.values())
-    a = _Args()
+    a, steps = _Args(), []
     a.z, a.out, a.ldz, a.ldo, a.rows = z.data_ptr(), out.data_ptr(), z.stride(0), out.stride(0), rows
     a.conv, a.conv_bias, a.dt_bias, a.a_log, a.d, a.norm = (w[n].data_ptr() for n in ("conv", "conv_bias", "dt_bias", "a_log", "d", "norm"))
     a.pos, a.slots = batch.pos.data_ptr(), batch.slot.data_ptr()
@@ -101,33 +116,38 @@ def ssd_rows(z, out, lay: SsdLayout, s: SsdSpec, w: dict, mul: float, eps: float
     if cache is not None:
         assert cache["s"].is_contiguous() and cache["s"].shape[1:] == (H, dn, dv) and cache["c"].is_contiguous() and cache["c"].dtype == z.dtype
         a.state, a.tail, a.ring = cache["s"].data_ptr(), cache["c"].data_ptr(), cache["c"].shape[1]
-    step = batch.decode and dv <= 256
     fast = dt == 1 and not batch.decode and dn <= 128 and dv <= 128
     y = torch.empty(rows, H * dv, dtype=torch.bfloat16 if fast else torch.float32, device=dev)
     a.y, a.ldy, a.y_f32 = y.data_ptr(), H * dv, int(not fast)
-    if step:
+    buffers = [y]
+    if batch.decode and dv <= 256 and dn * dv <= STEP_STATE:
         a.n = rows
-        K._check(K.lib().lmoe_ssd_step(ctypes.byref(a), dt, K._st()), "ssd_step")
+        steps.append(("ssd_step", a, 1, dt, K.num_sms()))
     else:
         xbc = torch.empty(rows, s.channels, dtype=z.dtype, device=dev)
-        steps = torch.empty(2, rows, H, dtype=torch.float32, device=dev)
-        a.xbc, a.ldx, a.dt, a.la = xbc.data_ptr(), s.channels, steps[0].data_ptr(), steps[1].data_ptr()
+        sizes = torch.empty(2, rows, H, dtype=torch.float32, device=dev)
+        buffers += [xbc, sizes]
+        a.xbc, a.ldx, a.dt, a.la = xbc.data_ptr(), s.channels, sizes[0].data_ptr(), sizes[1].data_ptr()
         if batch.decode:
             a.n = 0                                                  # one token each, positions only known on the device
         else:
             whole, _, _ = batch.recurrent_groups(max(batch.counts))
             a.groups, a.n = whole.data_ptr(), whole.shape[0]
-        K._check(K.lib().lmoe_ssd_conv(ctypes.byref(a), dt, K._st()), "ssd_conv", 2)
+        steps.append(("ssd_conv", a, 2, dt))
         if fast:
+            a = type(a).from_buffer_copy(a)
             groups, states, many = batch.recurrent_groups(group_tokens(batch.counts, H, K.num_sms()))
-            scratch = torch.empty(states, H, dn, dv, dtype=torch.float32, device=dev) if states else None
-            decay = torch.empty(states, H, dtype=torch.float32, device=dev) if states else None
-            a.groups, a.n, a.scratch, a.decay = groups.data_ptr(), groups.shape[0], _ptr(scratch), _ptr(decay)
+            if states:
+                scratch, decay = torch.empty(states, H, dn, dv, dtype=torch.float32, device=dev), torch.empty(states, H, dtype=torch.float32, device=dev)
+                a.scratch, a.decay = scratch.data_ptr(), decay.data_ptr()
+                buffers += [scratch, decay]
+            a.groups, a.n = groups.data_ptr(), groups.shape[0]
             a.requests, a.m = (0, 0) if many is None else (many.data_ptr(), many.shape[0])
-            K._check(K.lib().lmoe_ssd_tc(ctypes.byref(a), K._st()), "ssd_tc", 3 if states else 1)
+            steps.append(("ssd_tc", a, 3 if states else 1))
         else:
-            K._check(K.lib().lmoe_ssd_scan(ctypes.byref(a), dt, K._st()), "ssd_scan")
-    K._check(K.lib().lmoe_ssd_norm(ctypes.byref(a), dt, K._st()), "ssd_norm")
+            steps.append(("ssd_scan", a, 1, dt))
+    steps.append(("ssd_norm", a, 1, dt))
+    return steps, buffers
 
 
 def group_tokens(counts, heads: int, sms: int) -> int:
