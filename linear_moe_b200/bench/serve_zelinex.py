@@ -260,7 +260,10 @@ def kernels(size: str) -> list:
         zs, os_ = rnd(n, sl.width), torch.empty(n, r.inner, dtype=bf, device=dev)
         by = n * r.heads * r.dn * r.dv * 8
         sets = caches((LayerState(r.heads, r.dn, r.dv), LayerInputs(TAPS, r.channels)), by)
-        row(f"ssd_step + ssd_norm, batch {n}", "state decode", _graph_ms(lambda c_: SD.ssd_rows(zs, os_, sl, r, ws, 1.0, 1e-5, one_tok, c_), sets), bytes_=by)
+        plans = [(SD.launches(zs, os_, sl, r, ws, 1.0, 1e-5, one_tok, c_[0]),) for c_ in sets]
+        row(f"ssd_step, batch {n}", "state decode", _graph_ms(lambda p_: SD.launch(*p_[0][0]), plans), bytes_=by)
+        row(f"ssd_norm, batch {n}", "row kernel decode", _graph_ms(lambda p_: SD.launch(*p_[0][1]), plans * 4))
+        del plans
         del sets
         q, k, v = rnd(n, 1, r.heads // 2, 3 * 128).split([128, 128, 128], -1)
         by = n * (r.heads // 2) * 128 * 128 * 8
@@ -275,6 +278,8 @@ def kernels(size: str) -> list:
         row(f"the same and delta_step (norm, gate inside), batch {n}", "delta decode", _graph_ms(
             lambda c_: DR.general_delta_rows(zd, od, dlay, dl, w2, pd, 1e-5, one_tok, c_), sets), bytes_=by)
         q, k, v = rnd(n, 1, dl.heads, 3 * dl.d).split([dl.d] * 3, -1)
+        yg = rnd(n, 1, r.inner)
+        row(f"gated_rms_norm (mamba2), batch {n}", "row kernel decode", _graph_ms(lambda: ops.gated_rms_norm(yg, yg, gw, 1e-5, r.inner // r.norm_groups), [()] * 100))
         be, gs = torch.rand(n, 1, dl.heads, device=dev), -torch.rand(n, 1, dl.heads, device=dev)
         row(f"lsm_delta_step (hybrid), batch {n}", "delta decode", _graph_ms(lambda c_: ops.lsm_delta(q, k, v, be, gs, None, c_["s"]), sets), bytes_=by)
         del sets

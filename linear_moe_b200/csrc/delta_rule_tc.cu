@@ -5,7 +5,7 @@
 //     U_t = u e^{L_{t-1}},  B_t = a u e^{-L_t},  K_t = k e^{-L_t},  R_t = r e^{L_t}.
 // A log decay is at least -DECAY, so these stay far inside the range of bf16, and every product of two of them that is used decays.  What the
 // tokens read from the state along their keys, p_t = u_t^T S_{t-1}, obeys (I + tril(U B^T, -1)) P = U S + tril(U K^T, -1) V with the state S in
-// front of the chunk.  With M the inverse on the left, G = M U and H = M tril(U K^T, -1) V,
+// front of the chunk.  With M the inverse on the left, G = M U and H = M tril(U K^T, -1) V (found by substitution in blocks of 16),
 //     O  = Q S + N,     Q = R - tril(R B^T) G,    N = tril(R K^T) V - tril(R B^T) H
 //     S' = e^{L} S - E S + D,     E = e^{L} B^T G,    D = e^{L} (K^T V - B^T H)              (e^{L} of the whole chunk, row by row)
 //   delta_chunk_kernel   Q, N, E, D and e^{L} of every chunk, all in parallel
@@ -49,42 +49,56 @@ template <int D> struct Work {
 __device__ __forceinline__ float sigmoid(float x) { return 1.f / (1.f + __expf(-x)); }
 
 template <int D> struct Cfg {
-    static constexpr int LD = D + 8, LDA = CH + 1, SEGS = NT / D, SEG = CH / SEGS;       // segments of tokens a thread sums the log decays over
+    static constexpr int LD = D + 8, SEGS = NT / D, SEG = CH / SEGS;     // segments of tokens a thread sums the log decays over
     static constexpr int TILE = CH * LD * 2, PT = CH * PLD * 2;
-    static constexpr int XT = TILE > PT ? TILE : PT;
-    // one region: log decays, then tril(U B^T, -1) and its inverse in fp32, then the inverse in bf16, G and H
-    static constexpr int SUMS = CH * D * 4, PAIR = 2 * CH * LDA * 4, LAST = PT + 2 * TILE;
-    static constexpr int SOLVE = SUMS > PAIR ? (SUMS > LAST ? SUMS : LAST) : (PAIR > LAST ? PAIR : LAST);
-    static constexpr int SMEM = 5 * TILE + SOLVE + XT + 2 * PT;
+    static constexpr int SUMS = CH * D * 4 > 2 * TILE ? CH * D * 4 : 2 * TILE;           // log decays, then G and H
+    static constexpr int LDM = 24;                                       // row stride of the inverses of the diagonal blocks
+    static constexpr int SMEM = 5 * TILE + SUMS + 4 * PT + CH * 17 * 4 + CH * LDM * 2;
 };
+
+// acc (16 rows from m0) += A B with a lower triangular A (blocks of 16): B stored [k][n]
+template <int NTL>
+__device__ __forceinline__ void lower_gemm(float (&acc)[NTL][4], const bf16* A, int m0, const bf16* B, int ldb, int n0) {
+    for (int k0 = 0; k0 <= m0; k0 += 16) {
+        uint32_t p[4];
+        load_a(p, A, PLD, m0, k0);
+#pragma unroll
+        for (int t = 0; t < NTL; t += 2) {
+            uint32_t b[4];
+            load_b2_t(b, B, ldb, n0 + t * 8, k0);
+            mma16816(acc[t], p, b[0], b[1]);
+            mma16816(acc[t + 1], p, b[2], b[3]);
+        }
+    }
+}
 
 // grid (chunks, H)
 template <int D>
 __global__ void __launch_bounds__(NT, D == 64 ? 2 : 1) delta_chunk_kernel(Args a, int chunks) {
     using C = Cfg<D>;
-    constexpr int LD = C::LD, LDA = C::LDA, SEG = C::SEG, HT = D / 16;      // HT: n-tiles of a warp's half of D columns
+    constexpr int LD = C::LD, LDM = C::LDM, SEG = C::SEG, HT = D / 16;      // HT: n-tiles of a warp's half of D columns
     extern __shared__ __align__(16) unsigned char smem[];
     bf16* U = reinterpret_cast<bf16*>(smem);                 // [CH][LD] each
     bf16* B = U + CH * LD;
     bf16* K = B + CH * LD;
     bf16* R = K + CH * LD;
     bf16* V = R + CH * LD;
-    unsigned char* solve = smem + 5 * C::TILE;
-    float* Lw = reinterpret_cast<float*>(solve);             // [CH][D] log decays summed inside a segment
-    float* A = reinterpret_cast<float*>(solve);              // [CH][LDA] tril(U B^T, -1)
-    float* M = A + CH * LDA;                                 // [CH][LDA] its inverse (with I)
-    bf16* Mb = reinterpret_cast<bf16*>(solve);               // [CH][PLD]
-    bf16* G = Mb + CH * PLD;                                 // [CH][LD]
+    unsigned char* sums = smem + 5 * C::TILE;
+    float* Lw = reinterpret_cast<float*>(sums);              // [CH][D] log decays summed inside a segment
+    bf16* G = reinterpret_cast<bf16*>(sums);                 // [CH][LD]
     bf16* H = G + CH * LD;                                   // [CH][LD]
-    bf16* UK = reinterpret_cast<bf16*>(solve + C::SOLVE);    // [CH][PLD] tril(U K^T, -1), then
-    bf16* X = UK;                                            // [CH][LD] its product with V
-    bf16* RB = reinterpret_cast<bf16*>(solve + C::SOLVE + C::XT);     // [CH][PLD] tril(R B^T)
+    bf16* UB = reinterpret_cast<bf16*>(sums + C::SUMS);      // [CH][PLD] tril(U B^T, -1)
+    bf16* UK = UB + CH * PLD;                                // [CH][PLD] tril(U K^T, -1)
+    bf16* RB = UK + CH * PLD;                                // [CH][PLD] tril(R B^T)
     bf16* RK = RB + CH * PLD;                                // [CH][PLD] tril(R K^T)
+    float* A = reinterpret_cast<float*>(RK + CH * PLD);      // [CH][17] the diagonal blocks of tril(U B^T, -1)
+    bf16* M = reinterpret_cast<bf16*>(A + CH * 17);          // [CH][LDM] and the inverses of I plus them
     __shared__ float inv[CH], seg[C::SEGS][D], whole[D];
     const int* it = a.groups + blockIdx.x * G_INTS;
     const int h = blockIdx.y, row0 = it[G_ROW], n = it[G_N], d = a.d;
     const int w = threadIdx.x >> 5, l = threadIdx.x & 31, g = l >> 2, q = l & 3;
-    const int m0 = 16 * (w & 3), half = w >> 2, n0 = half * (D / 2);        // this warp's rows and columns of a D-wide product
+    // this warp's rows and columns of a D-wide product; the two warps of a scheduler share the work of triangular ones evenly
+    const int half = w >> 2, m0 = 16 * (half ? 3 - (w & 3) : w & 3), n0 = half * (D / 2);
     const bf16* z = (const bf16*)a.z + (long long)row0 * a.ldz + h * d;
     load_rows<D, LD>(K, z + a.zk, a.ldz, n, d);
     load_rows<D, LD>(R, z + a.zr, a.ldz, n, d);
@@ -145,87 +159,105 @@ __global__ void __launch_bounds__(NT, D == 64 ? 2 : 1) delta_chunk_kernel(Args a
         *reinterpret_cast<__nv_bfloat162*>(R + at) = __floats2bfloat162_rn(r.x * __expf(L.x), r.y * __expf(L.y));
     }
     __syncthreads();
-    {                                                        // scores: rows of U (warps 0 .. 3) or R against all rows of B and K
-        float s[8][4];
+    {                                                        // scores: rows of U (warps 0 .. 3) or R against the rows of B and K up to them
         const bf16* rows = half ? R : U;
 #pragma unroll
         for (int other = 0; other < 2; ++other) {
+            float s[8][4];
             zero_acc<8>(s);
-            warp_gemm<8, D, false, false>(s, rows, LD, m0, other ? K : B, LD, 0);
+#pragma unroll
+            for (int k0 = 0; k0 < D; k0 += 16) {
+                uint32_t p[4];
+                load_a(p, rows, LD, m0, k0);
+#pragma unroll
+                for (int t = 0; t < 8; t += 2)
+                    if (8 * t <= m0) {
+                        uint32_t b[4];
+                        load_b2(b, other ? K : B, LD, t * 8, k0);
+                        mma16816(s[t], p, b[0], b[1]);
+                        mma16816(s[t + 1], p, b[2], b[3]);
+                    }
+            }
+            bf16* to = half ? other ? RK : RB : other ? UK : UB;
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 const int i = m0 + g + 8 * e;
 #pragma unroll
-                for (int t = 0; t < 8; ++t) {
-                    const int j = 8 * t + 2 * q;
-                    const float x = (half ? i >= j : i > j) ? s[t][2 * e] : 0.f, y = (half ? i >= j + 1 : i > j + 1) ? s[t][2 * e + 1] : 0.f;
-                    if (!half && !other) A[i * LDA + j] = x, A[i * LDA + j + 1] = y;
-                    else *reinterpret_cast<__nv_bfloat162*>((half ? other ? RK : RB : UK) + i * PLD + j) = __floats2bfloat162_rn(x, y);
-                }
+                for (int t = 0; t < 8; ++t)
+                    if (8 * t <= m0 + 8) {
+                        const int j = 8 * t + 2 * q;
+                        const float x = (half ? i >= j : i > j) ? s[t][2 * e] : 0.f, y = (half ? i >= j + 1 : i > j + 1) ? s[t][2 * e + 1] : 0.f;
+                        *reinterpret_cast<__nv_bfloat162*>(to + i * PLD + j) = __floats2bfloat162_rn(x, y);
+                        if (!half && !other && j >= m0) A[i * 17 + j - m0] = x, A[i * 17 + j + 1 - m0] = y;
+                    }
             }
         }
     }
     __syncthreads();
-    {                                                        // X = UK V, kept until everyone has read UK
-        float x[HT][4];
-        zero_acc<HT>(x);
-        warp_gemm<HT, CH, false, true>(x, UK, PLD, m0, V, LD, n0);
-        // inverses of the diagonal blocks of 16, a thread per column
-        if (threadIdx.x < CH) {
-            const int b = threadIdx.x & ~15, c = threadIdx.x & 15;
-            float m[16];
+    if (threadIdx.x < CH) {                                  // inverses of the diagonal blocks of 16, a thread per column
+        const int b = threadIdx.x & ~15, c = threadIdx.x & 15;
+        float m[16];
 #pragma unroll
-            for (int i = 0; i < 16; ++i) {
-                float s = 0.f;
+        for (int i = 0; i < 16; ++i) {
+            float s0 = 0.f, s1 = 0.f;
 #pragma unroll
-                for (int k = 0; k < i; ++k) s += A[(b + i) * LDA + b + k] * m[k];
-                m[i] = i == c ? 1.f : -s;                    // (zero in front of the diagonal)
-            }
-#pragma unroll
-            for (int i = 0; i < 16; ++i) M[(b + i) * LDA + b + c] = m[i];
+            for (int k = 0; k < i; ++k) (k & 1 ? s1 : s0) += A[(b + i) * 17 + k] * m[k];
+            m[i] = i == c ? 1.f : -(s0 + s1);                // (zero in front of the diagonal)
         }
-        __syncthreads();
-        store_acc_bf16<HT>(x, X, LD, m0, n0);
-    }
-    // blocks below the diagonal: M21 = -M22 (A21 M11), with A21 M11 in the place above the diagonal
 #pragma unroll
-    for (int b = 16; b < CH; b *= 2) {
-        for (int i = threadIdx.x; i < CH / 2 * b; i += NT) {
-            const int o = i / (b * b) * 2 * b, r = i / b % b, c = i % b;
-            float s = 0.f;
-            for (int k = c; k < b; ++k) s += A[(o + b + r) * LDA + o + k] * M[(o + k) * LDA + o + c];
-            M[(o + r) * LDA + o + b + c] = s;
-        }
-        __syncthreads();
-        for (int i = threadIdx.x; i < CH / 2 * b; i += NT) {
-            const int o = i / (b * b) * 2 * b, r = i / b % b, c = i % b;
-            float s = 0.f;
-            for (int k = 0; k <= r; ++k) s += M[(o + b + r) * LDA + o + b + k] * M[(o + k) * LDA + o + b + c];
-            M[(o + b + r) * LDA + o + c] = -s;
-        }
-        __syncthreads();
-    }
-    for (int i = threadIdx.x; i < CH * CH; i += NT) {        // (A is not needed any more)
-        const int r = i / CH, c = i % CH;
-        Mb[r * PLD + c] = __float2bfloat16(c <= r ? M[r * LDA + c] : 0.f);
+        for (int i = 0; i < 16; ++i) M[(b + i) * LDM + c] = __float2bfloat16(m[i]);
     }
     __syncthreads();
-    {
-        float x[HT][4], y[HT][4];
-        zero_acc<HT>(x);
-        zero_acc<HT>(y);
-        warp_gemm<HT, CH, false, true>(x, Mb, PLD, m0, U, LD, n0);
-        warp_gemm<HT, CH, false, true>(y, Mb, PLD, m0, X, LD, n0);
-        // (M lies where G and H go; its copy has been made)
-        store_acc_bf16<HT>(x, G, LD, m0, n0);
-        store_acc_bf16<HT>(y, H, LD, m0, n0);
+    // G and H, 16 columns at a time from the first block of rows to the last: block i is M_ii times what is left of its right side when the
+    // blocks before it are known.  Warps 0 .. 3 have the columns of G, the others those of H (D = 128: two turns).
+    for (int strip = w & 3; strip < D / 16; strip += 4) {
+        bf16* X = half ? H : G;
+        const int c0 = strip * 16;
+        for (int i0 = 0; i0 < CH; i0 += 16) {
+            float x[2][4], y[2][4];
+            zero_acc<2>(x);
+            zero_acc<2>(y);
+            if (half) {
+                lower_gemm<2>(y, UK, i0, V, LD, c0);
+            } else {
+#pragma unroll
+                for (int t = 0; t < 2; ++t)
+#pragma unroll
+                    for (int e = 0; e < 2; ++e) {
+                        const float2 u = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(U + (i0 + g + 8 * e) * LD + c0 + 8 * t + 2 * q));
+                        y[t][2 * e] = u.x, y[t][2 * e + 1] = u.y;
+                    }
+            }
+            for (int k0 = 0; k0 < i0; k0 += 16) {
+                uint32_t p[4], b[4];
+                load_a(p, UB, PLD, i0, k0);
+                load_b2_t(b, X, LD, c0, k0);
+                mma16816(x[0], p, b[0], b[1]);
+                mma16816(x[1], p, b[2], b[3]);
+            }
+#pragma unroll
+            for (int t = 0; t < 2; ++t)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) y[t][e] -= x[t][e];
+            store_acc_bf16<2>(y, X, LD, i0, c0);
+            __syncwarp();
+            uint32_t p[4], b[4];
+            load_a(p, M, LDM, i0, 0);
+            load_b2_t(b, X, LD, c0, i0);
+            zero_acc<2>(x);
+            mma16816(x[0], p, b[0], b[1]);
+            mma16816(x[1], p, b[2], b[3]);
+            __syncwarp();
+            store_acc_bf16<2>(x, X, LD, i0, c0);
+            __syncwarp();
+        }
     }
     __syncthreads();
     const Work<D> out(a.work, (long long)chunks * a.H, (long long)blockIdx.x * a.H + h);
     {
         float x[HT][4];
         zero_acc<HT>(x);
-        warp_gemm<HT, CH, false, true>(x, RB, PLD, m0, G, LD, n0);
+        lower_gemm<HT>(x, RB, m0, G, LD, n0);
 #pragma unroll
         for (int t = 0; t < HT; ++t)
 #pragma unroll
@@ -237,8 +269,8 @@ __global__ void __launch_bounds__(NT, D == 64 ? 2 : 1) delta_chunk_kernel(Args a
         float y[HT][4];
         zero_acc<HT>(x);
         zero_acc<HT>(y);
-        warp_gemm<HT, CH, false, true>(x, RB, PLD, m0, H, LD, n0);
-        warp_gemm<HT, CH, false, true>(y, RK, PLD, m0, V, LD, n0);
+        lower_gemm<HT>(x, RB, m0, H, LD, n0);
+        lower_gemm<HT>(y, RK, m0, V, LD, n0);
 #pragma unroll
         for (int t = 0; t < HT; ++t)
 #pragma unroll
