@@ -183,7 +183,7 @@ __global__ void __launch_bounds__(256) moe_glu_kernel(const T* __restrict__ z, l
 #pragma unroll
         for (int e = 0; e < W; ++e) {
             const float t = g.get(e);
-            g.set(e, w * (t / (1.f + expf(-t))) * u.get(e));
+            g.set(e, w * (sizeof(T) == 2 ? __fdividef(t, 1.f + __expf(-t)) : t / (1.f + expf(-t))) * u.get(e));
         }
         g.store(out + row * ldo + c);
     }

@@ -12,7 +12,8 @@
 namespace lmoe {
 namespace ssd {
 
-__device__ __forceinline__ float silu(float x) { return x / (1.f + expf(-x)); }
+// as exactly as the model's type asks for
+template <typename T> __device__ __forceinline__ float silu(float x) { return sizeof(T) == 2 ? __fdividef(x, 1.f + __expf(-x)) : x / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
 // ------------------------------------------------------------------------------------------------------- prompts: convolution
@@ -72,7 +73,7 @@ __global__ void __launch_bounds__(CT) ssd_conv_kernel(Args a) {
 #pragma unroll
         for (int n = KEEP - 1; n > 0; --n) past[n] = past[n - 1];
         past[0] = x;
-        store4((T*)a.xbc + row * a.ldx + c, make_float4(silu(s.x), silu(s.y), silu(s.z), silu(s.w)));
+        store4((T*)a.xbc + row * a.ldx + c, make_float4(silu<T>(s.x), silu<T>(s.y), silu<T>(s.z), silu<T>(s.w)));
     }
 }
 
@@ -239,7 +240,7 @@ __global__ void __launch_bounds__(ST, 3) ssd_step_kernel(Args a, int heads) {
         const int k = channel(i);
         const T x = z[a.zx + k];
         const float v = (n == 0 ? pre[0] : n == 1 ? pre[1] : older(k)) + a.conv[(long long)(a.taps - 1) * ch + k] * to_f(x);
-        X[i] = to_f(from_f<T>(silu(v)));
+        X[i] = to_f(from_f<T>(silu<T>(v)));
         // a ring of `taps` rows: the place of this input is none that another CTA still reads
         if (i < own || h0 % (a.H / a.G) == 0) tail[(long long)(pos % a.ring) * ch + k] = x;
     }
@@ -344,7 +345,7 @@ __global__ void __launch_bounds__(NT) ssd_norm_kernel(Args a) {
                 f[0] = to_f(y[c]), q[0] = to_f(z[c]);
             }
 #pragma unroll
-            for (int e = 0; e < V; ++e) v[e] = f[e] * silu(q[e]);
+            for (int e = 0; e < V; ++e) v[e] = f[e] * silu<T>(q[e]);
         };
         float s = 0.f;
 #pragma unroll

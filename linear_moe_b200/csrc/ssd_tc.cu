@@ -18,8 +18,7 @@ using ssd::Args;
 template <int DK, int DV> struct Cfg : Shape<DK, DV> {
     using S = Shape<DK, DV>;
     static constexpr int STATE_SMEM = 2 * S::KV;
-    static constexpr int STAGE = S::KV + CH * S::LDK * 2;
-    static constexpr int OUT_SMEM = 2 * STAGE + DK * S::LDV * 2 + CH * PLD * 2 + CH * S::LDV * 2;
+    static constexpr int OUT_SMEM = 2 * S::KV + CH * S::LDK * 2 + DK * S::LDV * 2 + CH * PLD * 2 + CH * S::LDV * 2;
 };
 
 // a chunk's step sizes and the running sums of its log decays, two tokens per lane of one warp; tokens that are not there: 0
@@ -98,10 +97,11 @@ __global__ void __launch_bounds__(NT) ssd_combine_kernel(Args a) {
 
 // grid (groups, H)
 template <int DK, int DV>
-__global__ void __launch_bounds__(NT) ssd_out_kernel(Args a) {
+__global__ void __launch_bounds__(NT, Cfg<DK, DV>::OUT_SMEM <= 110 * 1024 ? 2 : 1) ssd_out_kernel(Args a) {
     using F = Cfg<DK, DV>;
     extern __shared__ __align__(16) unsigned char smem[];
-    bf16* Sb = reinterpret_cast<bf16*>(smem + 2 * F::STAGE); // [DK][LDV] the state in bf16
+    bf16* C = reinterpret_cast<bf16*>(smem + 2 * F::KV);     // [CH][LDK] (one stage: it is not needed for long)
+    bf16* Sb = C + CH * F::LDK;                              // [DK][LDV] the state in bf16
     bf16* P = Sb + DK * F::LDV;                              // [CH][PLD]
     bf16* Y = P + CH * PLD;                                  // [CH][LDV]
     __shared__ float dt[2][CH], L[2][CH];
@@ -115,18 +115,18 @@ __global__ void __launch_bounds__(NT) ssd_out_kernel(Args a) {
     const long long size = (long long)a.dn * a.dv;
     float* own = a.state == nullptr ? nullptr : a.state + ((long long)it[G_SLOT] * a.H + h) * size;
     const float D = a.d[h];
-    auto B = [&](int s) { return reinterpret_cast<bf16*>(smem + s * F::STAGE); };
+    auto B = [&](int s) { return reinterpret_cast<bf16*>(smem + s * F::KV); };
     auto X = [&](int s) { return B(s) + CH * F::LDK; };
-    auto C = [&](int s) { return X(s) + CH * F::LDV; };
+    auto load_c = [&](int t0) { load_rows<DK, F::LDK>(C, x + t0 * a.ldx + at_b + a.G * a.dn, a.ldx, n - t0, a.dn); };
     auto load = [&](int t0) {
         const int s = t0 / CH & 1;
         const bf16* p = x + t0 * a.ldx;
-        load_rows<DK, F::LDK>(C(s), p + at_b + a.G * a.dn, a.ldx, n - t0, a.dn);
         load_rows<DK, F::LDK>(B(s), p + at_b, a.ldx, n - t0, a.dn);
         load_rows<DV, F::LDV>(X(s), p + h * a.dv, a.ldx, n - t0, a.dv);
         if (threadIdx.x < 32) chunk_steps(a, row0 + t0, n - t0, h, dt[s], L[s]);
     };
     load(0);
+    load_c(0);
     cp_async_commit();
     State<DK, DV> S;
     S.load(from >= 0 ? a.scratch + ((long long)from * a.H + h) * size : (flags & 4) ? own : nullptr, a.dn, a.dv);
@@ -140,8 +140,8 @@ __global__ void __launch_bounds__(NT) ssd_out_kernel(Args a) {
         float o[F::O_NT][4], z[4][4];
         zero_acc<F::O_NT>(o);
         zero_acc<4>(z);
-        warp_gemm<F::O_NT, DK, false, true>(o, C(s), F::LDK, m0, Sb, F::LDV, o_n0);
-        if (a_n0 <= m0 + 15) warp_gemm<4, DK, false, false>(z, C(s), F::LDK, m0, B(s), F::LDK, a_n0);
+        warp_gemm<F::O_NT, DK, false, true>(o, C, F::LDK, m0, Sb, F::LDV, o_n0);
+        if (a_n0 <= m0 + 15) warp_gemm<4, DK, false, false>(z, C, F::LDK, m0, B(s), F::LDK, a_n0);
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
             const int i = m0 + g + 8 * e;
@@ -158,7 +158,9 @@ __global__ void __launch_bounds__(NT) ssd_out_kernel(Args a) {
         }
         const float last = L[s][CH - 1];
         S.advance(B(s), X(s), __expf(last), [&](int j) { return __expf(last - L[s][j]) * dt[s][j]; });
-        __syncthreads();                                     // P is complete, nobody reads Sb any more
+        __syncthreads();                                     // P is complete, nobody reads Sb and C any more
+        if (t0 + CH < n) load_c(t0 + CH);
+        cp_async_commit();
         for (int k0 = 0; k0 <= m0; k0 += 16) {               // tokens behind row m0 + 15 are hidden
             uint32_t p[4];
             load_a(p, P, PLD, m0, k0);
