@@ -1,14 +1,15 @@
 // Generalized delta rule over packed rows, head by head in fp32,
 //     S <- diag(w) S - (a u)(u^T S) + k v^T,    o = S^T r,    out = o / rms(o) * weight * sigmoid(gate)
 // with the unit key u, decays w = exp(-DECAY sigmoid(W2 tanh(.) + w0)) and rates a = sigmoid(. + bias) per channel:
-//   delta_low_kernel    tanh of the decay's inner activations (the second projection is a matrix product)
+//   delta_low_kernel    tanh of the decay's inner activations (the second projection is a matrix product), or for few rows in bf16
+//   delta_decay_kernel  both
 //   delta_rows_kernel   prompts of any size, bf16 or fp32, token by token (bf16 fast path: delta_rule_tc.cu), and
 //   delta_norm_kernel   the norm and gate behind it
 //   delta_step_kernel   one token per request, everything else in one pass over the state
 // With the old state S, p = S^T u and q = S^T (w r), the output is o = q - (r . a u) p + (r . k) v: one reduction over the rows of S.
 // Compiled without fast-math: the fp32 instantiations serve models in true 32-bit.
-#include "common.cuh"
 #include "delta_rule.cuh"
+#include "mma_utils.cuh"
 
 namespace lmoe {
 namespace dlt {
@@ -25,6 +26,53 @@ __global__ void __launch_bounds__(256) delta_low_kernel(const T* __restrict__ z,
         const float4 x = load4(z + row * ldz + c);
         store4(low + row * ldl + c, make_float4(tanhf(x.x), tanhf(x.y), tanhf(x.z), tanhf(x.w)));
     }
+}
+
+// Few rows, bf16: tanh and the second projection in one launch.  A CTA has 64 channels, a warp 16 of them; grid (channels / 64 rounded up).
+constexpr int DR = 64;                   // rows at most
+
+__global__ void __launch_bounds__(128) delta_decay_kernel(const bf16* __restrict__ z, long long ldz, const bf16* __restrict__ w2, float* __restrict__ out,
+                                                          int rows, int rank, int channels) {
+    extern __shared__ __align__(16) unsigned char smem[];
+    const int ld = rank + 8, c0 = blockIdx.x * 64, w = threadIdx.x >> 5, l = threadIdx.x & 31, g = l >> 2, q = l & 3;
+    bf16* W = reinterpret_cast<bf16*>(smem);                 // [64][ld]
+    bf16* L = W + 64 * ld;                                   // [rows up to the next 16][ld]
+    for (int i = threadIdx.x; i < 64 * (rank / 8); i += 128) {           // (weights do not change)
+        const int r = i / (rank / 8), c = i % (rank / 8) * 8;
+        cp_async16(W + r * ld + c, w2 + (c0 + r < channels ? (long long)(c0 + r) * rank + c : 0), c0 + r < channels);
+    }
+    cp_async_commit();
+    pdl_trigger();
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    const int tiles = (rows + 15) / 16;
+    for (int i = threadIdx.x; i < tiles * 16 * (rank / 4); i += 128) {
+        const int r = i / (rank / 4), c = i % (rank / 4) * 4;
+        const float4 x = r < rows ? load4(z + r * ldz + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        store4(L + r * ld + c, make_float4(tanhf(x.x), tanhf(x.y), tanhf(x.z), tanhf(x.w)));
+    }
+    cp_async_wait<0>();
+    __syncthreads();
+    float acc[DR / 8][4];
+    zero_acc<DR / 8>(acc);
+    for (int k0 = 0; k0 < rank; k0 += 16) {
+        uint32_t p[4];
+        load_a(p, W, ld, 16 * w, k0);
+#pragma unroll
+        for (int t = 0; t < DR / 16; ++t)
+            if (t < tiles) {
+                uint32_t b[4];
+                load_b2(b, L, ld, 16 * t, k0);
+                mma16816(acc[2 * t], p, b[0], b[1]);
+                mma16816(acc[2 * t + 1], p, b[2], b[3]);
+            }
+    }
+#pragma unroll
+    for (int t = 0; t < DR / 8; ++t)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int r = 8 * t + 2 * q + (e & 1), c = c0 + 16 * w + g + 8 * (e >> 1);
+            if (r < rows && c < channels) out[(long long)r * channels + c] = acc[t][e];
+        }
 }
 
 // ------------------------------------------------------------------------------------------------------------------ prompts
@@ -278,6 +326,26 @@ LMOE_API int lmoe_delta_low(const void* z, long long ldz, void* low, long long l
     if (dt) dlt::delta_low_kernel<bf16><<<grid, 256, 0, st>>>((const bf16*)z, ldz, (bf16*)low, ldl, rows, cols);
     else dlt::delta_low_kernel<float><<<grid, 256, 0, st>>>((const float*)z, ldz, (float*)low, ldl, rows, cols);
     return (int)cudaGetLastError();
+}
+
+// bf16: z [rows, ldz] (rank columns, a multiple of 32, up to 64 rows), w2 [channels, rank] -> out [rows, channels] fp32
+LMOE_API int lmoe_delta_decay(const void* z, long long ldz, const void* w2, float* out, int rows, int rank, int channels, cudaStream_t st) {
+    if (rows <= 0 || rows > dlt::DR || rank <= 0 || rank % 32 || channels <= 0 || ldz % 8 || !dlt::aligned(z) || !dlt::aligned(w2)) return -1;
+    const int smem = (64 + (rows + 15) / 16 * 16) * (rank + 8) * 2;
+    if (smem > 200 * 1024) return -2;
+    cudaError_t e = cudaFuncSetAttribute(dlt::delta_decay_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return (int)e;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3((channels + 63) / 64);
+    cfg.blockDim = dim3(128);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = st;
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = 1;
+    return (int)cudaLaunchKernelEx(&cfg, dlt::delta_decay_kernel, (const bf16*)z, ldz, (const bf16*)w2, out, rows, rank, channels);
 }
 
 // Groups that are whole requests (flags 3 or 7), or (a.groups null) one token per request; a.w, a.raw

@@ -63,6 +63,36 @@ __global__ void __launch_bounds__(THREADS) embed_norm_kernel(const long long* __
     float* xr = x + (long long)blockIdx.x * ldx;
     T* yr = y + (long long)blockIdx.x * ldy;
     float s = 0.f;
+    if (width % 4 == 0 && pad <= 4 * 4 * THREADS) {         // rows in registers, four numbers at a time
+        constexpr int NV = 4;
+        const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+        auto add = [](float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); };
+        float4 v[NV], e[NV], h[NV];
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int c = (threadIdx.x + i * THREADS) * 4;
+            v[i] = keep && c < pad ? load4(xr + c) : zero;
+            e[i] = er != nullptr && c < width ? load4(er + c) : zero;
+            h[i] = shift != nullptr && c < pad ? load4(shift + c) : zero;
+            if (pr != nullptr && c < width) e[i] = add(e[i], load4(pr + c));
+        }
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int c = (threadIdx.x + i * THREADS) * 4;
+            v[i] = add(add(v[i], e[i]), h[i]);
+            if (c < pad) store4(xr + c, v[i]);
+            s += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+        }
+        const float r = 1.f / sqrtf(block_sum(s, red) / width + eps);
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int c = (threadIdx.x + i * THREADS) * 4;
+            if (c >= pad) continue;
+            const float4 g = gain == nullptr ? make_float4(1.f, 1.f, 1.f, 1.f) : load4(gain + c);
+            store4(yr + c, make_float4(v[i].x * r * g.x, v[i].y * r * g.y, v[i].z * r * g.z, v[i].w * r * g.w));
+        }
+        return;
+    }
     for (int c = threadIdx.x; c < pad; c += THREADS) {
         float v = keep ? xr[c] : 0.f;
         if (c < width) v += (er == nullptr ? 0.f : to_f(er[c])) + (pr == nullptr ? 0.f : to_f(pr[c]));
@@ -149,7 +179,7 @@ LMOE_API int lmoe_stream_norm(const float* x, long long ldx, void* y, long long 
 LMOE_API int lmoe_embed_norm(const long long* ids, const int* pos, const void* emb, const void* ptab, float* x, long long ldx, void* y,
                              long long ldy, int rows, int width, int pad, int vocab, int npos, float eps, const float* gain,
                              const float* shift, int keep, int dt, cudaStream_t st) {
-    if (rows <= 0 || width <= 0 || pad < width || vocab <= 0 || (ptab != nullptr && npos <= 0)) return -1;
+    if (rows <= 0 || width <= 0 || pad < width || pad % 4 || ldx % 4 || ldy % 4 || vocab <= 0 || (ptab != nullptr && npos <= 0)) return -1;
     if (dt) pb::embed_norm_kernel<bf16><<<rows, pb::THREADS, 0, st>>>(ids, pos, (const bf16*)emb, (const bf16*)ptab, x, ldx, (bf16*)y,
                                                                       ldy, width, pad, vocab, npos, eps, gain, shift, keep);
     else pb::embed_norm_kernel<float><<<rows, pb::THREADS, 0, st>>>(ids, pos, (const float*)emb, (const float*)ptab, x, ldx, (float*)y,

@@ -20,6 +20,7 @@ from .packed_attn import _fields, _no_grad
 from .retention import CHUNK
 from .row_batch import RowBatch, round_up
 
+FEW_ROWS = 64                         # the decays of this few bf16 rows take one launch
 DECAY = math.exp(-0.5)                # a channel's log decay lies between -DECAY and 0
 
 
@@ -71,7 +72,13 @@ def decay_rows(z, lay: DeltaLayout, s: GeneralDeltaSpec, w2) -> torch.Tensor:
     """What the decays are made of (``w0`` aside), ``[rows, heads * d]`` in fp32: the second projection of tanh of the first one's columns."""
     from . import cuda as K
     from . import linear_f32
-    ld, low = ctypes.c_longlong, torch.empty(z.shape[0], s.low, dtype=z.dtype, device=z.device)
+    ld = ctypes.c_longlong
+    if z.dtype == torch.bfloat16 and z.shape[0] <= FEW_ROWS and s.low <= 512:
+        assert w2.is_contiguous() and w2.shape[1] == s.low
+        decay = torch.empty(z.shape[0], w2.shape[0], dtype=torch.float32, device=z.device)
+        K._check(K.lib().lmoe_delta_decay(K._p(z[:, lay.w:]), ld(z.stride(0)), K._p(w2), K._p(decay), z.shape[0], s.low, w2.shape[0], K._st()), "delta_decay")
+        return decay
+    low = torch.empty(z.shape[0], s.low, dtype=z.dtype, device=z.device)
     K._check(K.lib().lmoe_delta_low(K._p(z[:, lay.w:]), ld(z.stride(0)), K._p(low), ld(s.low), z.shape[0], s.low, K._dt(z), K._st()), "delta_low")
     return linear_f32(low, w2)
 

@@ -502,8 +502,9 @@ def test_scaled_residuals_with_another_row(where, top, ydt):
 
 
 @where
-def test_starting_again(where):
-    dev, dt, width, pad, eps = where[0], getattr(torch, where[1]), 50, 64, 1e-3
+@pytest.mark.parametrize("width", [50, 52, 64, 4100])
+def test_starting_again(where, width):
+    dev, dt, pad, eps = where[0], getattr(torch, where[1]), round_up(width, 32), 1e-3
     emb, ids, shift, gain = torch.randn(9, width).to(dt), torch.tensor([8, 0, 3, 3]), torch.zeros(pad), torch.zeros(pad)
     shift[:width], gain[:width] = torch.randn(width), torch.rand(width) + 0.5
     x, h = ops.embed_norm(ids.to(dev), torch.arange(4).int().to(dev), emb.to(dev), None, pad, eps, gain.to(dev), shift.to(dev))
